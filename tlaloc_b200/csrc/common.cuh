@@ -143,18 +143,25 @@ struct OncePerDevice {
   }
 };
 
-// Per-device kernel attribute set-up of each translation unit; called from tlaloc_b200_init and from the typed-FFI
-// handlers' INITIALIZE stage, so that no launch inside a CUDA graph capture has to change a function attribute.
-cudaError_t PreparePagedAttentionKernels();
-cudaError_t PrepareInt8GemmKernels();
+// Each translation unit with kernel attributes to set (per device) or a device-side status word registers them with one
+// static object.  tlaloc_b200_init and the typed-FFI handlers' INITIALIZE stage run every `prepare`, so that no launch
+// inside a CUDA graph capture has to change a function attribute; tlaloc_b200_device_status reads every `status`
+// (1 if a bounded device-side wait has timed out since the last read, 0 if not, -1 on a CUDA error; synchronous).
+struct KernelSetup {
+  cudaError_t (*prepare)();
+  int (*status)();
+  KernelSetup* next;
+  KernelSetup(cudaError_t (*prepare_fn)(), int (*status_fn)());
+};
+// The driver's cuTensorMapEncodeTiled, or null.
+void* TensorMapEncoder();
+
 cudaError_t PrepareInt8GemmTcKernels();
 
 // The tensor-core projection (int8_gemm_tc.cu): rows [0, m) of y = (x @ codes) * scales (+ residual), x bf16.
 cudaError_t LaunchInt8GemmTc(const __nv_bfloat16* x, const int8_t* codes, const float* scales, const float* residual,
                              void* y, int y_dtype, int m, int k, int n, cudaStream_t st, int* launches, bool weights_const,
                              bool swiglu = false);
-// 1 if a bounded device-side wait has timed out since the last call (synchronous read), 0 if not, -1 on a CUDA error.
-int ReadTcStatus();
 // The same projection with the codes fed to the tensor core as int8 and the activations as two int8 planes
 // (int8_gemm_i8.cu); m <= 128 rows per call.
 cudaError_t PrepareInt8GemmI8Kernels();
@@ -165,10 +172,7 @@ cudaError_t LaunchInt8GemmI8(const void* x, int x_dtype, const int8_t* codes, co
                              bool weights_const, bool swiglu, bool have_planes);
 // The quantizer alone: the planes of x [m, k] into `planes` (Int8GemmI8ScratchBytes(m, k) bytes).
 cudaError_t LaunchQuantizeRowsI8(const void* x, int x_dtype, void* planes, int m, int k, cudaStream_t st);
-int ReadI8Status();
 bool EncodeKvPoolMap(::CUtensorMap_st* map, const void* base, int head_dim, int kv_heads, unsigned long long positions, int elem_bytes);
-bool TensorMapEncoderReady();
-int ReadPaStatus();
 
 // The activation planes of the int8 tensor-core projection: row m of x as q = rint(x / s[m]) = 256 hi + lo with s[m] the
 // smallest power of two that keeps |q| <= 127 * 256.  Layout in the projection's scratch for an [m, k] activation:

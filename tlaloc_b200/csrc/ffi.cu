@@ -8,7 +8,6 @@
 //   3. any stage but EXECUTE: nothing to do;
 //   4. EXECUTE: validate operands/results/attrs, take XLA's stream, enqueue on it; never allocate or synchronise.
 // Handlers are thread-safe: they keep no state beyond the once-only kernel set-up, which is mutex-guarded.
-#include <atomic>
 #include <cstring>
 #include <string>
 
@@ -16,20 +15,6 @@
 #include "xla_abi.h"
 
 namespace tlaloc_b200 {
-
-char* ErrorBuffer()
-{
-  static thread_local char buf[kErrorBufferBytes] = {0};
-  return buf;
-}
-
-namespace {
-std::atomic<long long> g_launches{0};
-std::atomic<int> g_order_faithful{0};
-}  // namespace
-
-void CountLaunches(int n) { g_launches.fetch_add(n, std::memory_order_relaxed); }
-bool OrderFaithful() { return g_order_faithful.load(std::memory_order_relaxed) != 0; }
 
 namespace {
 
@@ -278,44 +263,6 @@ AbiFfiError* KvCacheWriteHandler(AbiFfiCallFrame* frame)
 }  // namespace tlaloc_b200
 
 using namespace tlaloc_b200;
-
-namespace tlaloc_b200 {
-bool PdlEnabled()
-{
-  static const bool on = [] {
-    const char* e = std::getenv("TLALOC_B200_PDL");
-    return e == nullptr || std::atoi(e) != 0;
-  }();
-  return on;
-}
-}  // namespace tlaloc_b200
-
-extern "C" int tlaloc_b200_abi_version(void) { return TLALOC_B200_ABI_VERSION; }
-
-extern "C" const char* tlaloc_b200_last_error(void) { return ErrorBuffer(); }
-
-extern "C" long long tlaloc_b200_launch_count(void) { return g_launches.load(std::memory_order_relaxed); }
-
-extern "C" int tlaloc_b200_device_status(void)
-{
-  const int a = ReadTcStatus(), b = ReadI8Status(), c = ReadPaStatus();
-  return a < 0 || b < 0 || c < 0 ? -1 : (a | b | c);
-}
-
-extern "C" int tlaloc_b200_set_order_faithful(int on)
-{
-  return g_order_faithful.exchange(on != 0 ? 1 : 0, std::memory_order_relaxed);
-}
-
-extern "C" int tlaloc_b200_init(void)
-{
-  cudaError_t e = PreparePagedAttentionKernels();
-  if (e == cudaSuccess) e = PrepareInt8GemmKernels();
-  if (e == cudaSuccess) e = PrepareInt8GemmTcKernels();
-  if (e == cudaSuccess) e = PrepareInt8GemmI8Kernels();
-  if (e != cudaSuccess) return CudaFail("kernel set-up", e);
-  return kOk;
-}
 
 // The handlers by name, for callers that register them one at a time (a JVM's registerExecuteHandler route,
 // runtime-pjrt/.../ffm/PjrtFfiRegistry.kt:168-182) and for tests that drive them with hand-built call frames.

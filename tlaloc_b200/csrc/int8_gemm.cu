@@ -425,6 +425,9 @@ cudaError_t PrepareInt8GemmKernels()
     return e;
   });
 }
+namespace {
+KernelSetup g_setup(PrepareInt8GemmKernels, nullptr);
+}
 
 }  // namespace tlaloc_b200
 

@@ -175,20 +175,6 @@ __device__ __forceinline__ void TcMmaI8(uint32_t d_tmem, uint64_t a_desc, uint64
       "l"(a_desc), "l"(b_desc), "r"(idesc), "r"(accumulate)
       : "memory");
 }
-__device__ __forceinline__ void MbarExpectTx(uint32_t bar, uint32_t bytes)
-{
-  asm volatile("mbarrier.arrive.expect_tx.shared::cta.b64 _, [%0], %1;\n" ::"r"(bar), "r"(bytes) : "memory");
-}
-// One box of a two-dimensional tensor map into shared memory; (x, y) = (innermost coordinate, row).  x times the element
-// size is always a multiple of 128 bytes here.
-__device__ __forceinline__ void TmaLoad2d(uint32_t dst, const CUtensorMap* map, int x, int y, uint32_t bar, uint64_t policy)
-{
-  asm volatile(
-      "cp.async.bulk.tensor.2d.shared::cluster.global.mbarrier::complete_tx::bytes.L2::cache_hint [%0], [%1, {%2, %3}], [%4], %5;\n" ::"r"(dst),
-      "l"(reinterpret_cast<uint64_t>(map)), "r"(x), "r"(y), "r"(bar), "l"(policy)
-      : "memory");
-}
-
 template <int MROWS, typename YT>
 __global__ void __launch_bounds__(kI8Threads, 1)
     Int8GemmI8Kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant__ CUtensorMap map_hi,
@@ -397,19 +383,7 @@ using EncodeTiledFn = CUresult (*)(CUtensorMap*, CUtensorMapDataType, cuuint32_t
                                    const cuuint32_t*, const cuuint32_t*, CUtensorMapInterleave, CUtensorMapSwizzle,
                                    CUtensorMapL2promotion, CUtensorMapFloatOOBfill);
 
-EncodeTiledFn EncodeTiled()
-{
-  static EncodeTiledFn fn = [] {
-    void* ptr = nullptr;
-    cudaDriverEntryPointQueryResult res;
-    if (cudaGetDriverEntryPoint("cuTensorMapEncodeTiled", &ptr, cudaEnableDefault, &res) != cudaSuccess || res != cudaDriverEntryPointSuccess) {
-      cudaGetLastError();
-      ptr = nullptr;
-    }
-    return reinterpret_cast<EncodeTiledFn>(ptr);
-  }();
-  return fn;
-}
+EncodeTiledFn EncodeTiled() { return reinterpret_cast<EncodeTiledFn>(TensorMapEncoder()); }
 
 // A [rows][inner] byte matrix with rows `pitch` bytes apart, read in boxes of 128 bytes x box_rows rows, 128-byte
 // swizzle, zeros outside.
@@ -525,9 +499,6 @@ cudaError_t LaunchI8Rows(const CUtensorMap& mw, const CUtensorMap& mh, const CUt
 
 }  // namespace
 
-// Resolves the driver's tensor-map encoder; called from kernel set-up so that no launch has to do it inside a capture.
-bool TensorMapEncoderReady() { return EncodeTiled() != nullptr; }
-
 // A [positions][kv_heads][head_dim] pool of 2-byte (bf16) or 1-byte (f8) elements, read in boxes of 16 positions of one
 // head: 64 bf16 channels under the 128-byte swizzle, or a whole row of D bytes under the swizzle of that width.
 bool EncodeKvPoolMap(::CUtensorMap_st* map, const void* base, int head_dim, int kv_heads, unsigned long long positions, int elem_bytes)
@@ -547,7 +518,7 @@ bool EncodeKvPoolMap(::CUtensorMap_st* map, const void* base, int head_dim, int 
 
 cudaError_t PrepareInt8GemmI8Kernels()
 {
-  EncodeTiled();  // resolves the driver entry point now rather than inside a later stream capture
+  TensorMapEncoder();  // resolves the driver entry point now rather than inside a later stream capture
   return PrepareI8();
 }
 
@@ -624,6 +595,9 @@ int ReadI8Status()
     cudaMemcpyToSymbol(g_i8_status, &zero, sizeof(int));
   }
   return v;
+}
+namespace {
+KernelSetup g_setup(PrepareInt8GemmI8Kernels, ReadI8Status);
 }
 
 }  // namespace tlaloc_b200

@@ -543,5 +543,8 @@ int ReadTcStatus()
   }
   return v;
 }
+namespace {
+KernelSetup g_setup(PrepareInt8GemmTcKernels, ReadTcStatus);
+}
 
 }  // namespace tlaloc_b200

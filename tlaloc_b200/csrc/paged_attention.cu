@@ -1518,7 +1518,7 @@ cudaError_t PreparePagedAttentionKernels()
 {
   static OncePerDevice once;
   return once.Run([](int) {
-    TensorMapEncoderReady();  // without it the bf16 kernel keeps its cp.async form
+    TensorMapEncoder();  // without it the bf16 kernel keeps its cp.async form
     cudaError_t e = PrepareMma<__nv_bfloat16, 64>();
     if (e == cudaSuccess) e = PrepareMma<__nv_bfloat16, 128>();
     if (e == cudaSuccess) e = PrepareMma<float, 64>();
@@ -1544,6 +1544,9 @@ int ReadPaStatus()
     cudaMemcpyToSymbol(g_pa_status, &zero, sizeof(int));
   }
   return v;
+}
+namespace {
+KernelSetup g_setup(PreparePagedAttentionKernels, ReadPaStatus);
 }
 
 }  // namespace tlaloc_b200

@@ -68,6 +68,20 @@ __device__ __forceinline__ uint64_t SmemDesc(uint32_t addr, uint32_t lbo_bytes, 
   return static_cast<uint64_t>((addr >> 4) & 0x3FFFu) | (static_cast<uint64_t>((lbo_bytes >> 4) & 0x3FFFu) << 16) |
          (static_cast<uint64_t>((sbo_bytes >> 4) & 0x3FFFu) << 32) | (1ull << 46) | (2ull << 61);
 }
+__device__ __forceinline__ void MbarExpectTx(uint32_t bar, uint32_t bytes)
+{
+  asm volatile("mbarrier.arrive.expect_tx.shared::cta.b64 _, [%0], %1;\n" ::"r"(bar), "r"(bytes) : "memory");
+}
+// One box of a two-dimensional tensor map into shared memory; (x, y) = (innermost coordinate, row).  x times the element
+// size must be a multiple of 16 bytes; every caller keeps it a multiple of 128.
+__device__ __forceinline__ void TmaLoad2d(uint32_t dst, const ::CUtensorMap_st* map, int x, int y, uint32_t bar, uint64_t policy)
+{
+  asm volatile(
+      "cp.async.bulk.tensor.2d.shared::cluster.global.mbarrier::complete_tx::bytes.L2::cache_hint [%0], [%1, {%2, %3}], [%4], %5;\n" ::"r"(dst),
+      "l"(reinterpret_cast<uint64_t>(map)), "r"(x), "r"(y), "r"(bar), "l"(policy)
+      : "memory");
+}
+
 __device__ __forceinline__ void TcCommit(uint32_t bar)
 {
   asm volatile("tcgen05.commit.cta_group::1.mbarrier::arrive::one.shared::cluster.b64 [%0];\n" ::"r"(bar) : "memory");
