@@ -294,6 +294,86 @@ int tlaloc_b200_swiglu(const float* gate, const float* up, int32_t ld, void* out
 /* Greedy NEXT_TOKEN (DxirInterpreter.kt:2414-2426; triton/kernels/sample.cu greedy arm): first index of the maximum. */
 int tlaloc_b200_argmax(const float* logits, int32_t* out, int32_t rows, int32_t n, void* stream);
 
+/* ------------------------------------------------------------------ unquantized projections */
+
+#define TLALOC_B200_ACT_NONE 0
+#define TLALOC_B200_ACT_RELU2 1 /* max(v, 0)^2 */
+
+/*
+ * One projection over weights kept in their own float type: per batch entry b,
+ *   y[m, n] = act(sum_k x[m, k] * w[n, k] + bias[n]) + residual[m, n]
+ * with w [batch][n][k] contiguous (a checkpoint's [out, in]).  x and y have row strides and batch strides of their own, so
+ * they may be column blocks of wider matrices (the heads of a projection, the halves of a concatenated input).
+ * Sums are f32.  bias (f32 [n]) and residual (f32, batch 1 only; may be y) may be NULL.
+ */
+typedef struct tlaloc_b200_dense_problem {
+  const void* x;
+  const void* w;
+  const float* bias;
+  const float* residual;
+  void* y;
+  int64_t ld_x, ld_res, ld_y;        /* row strides in elements */
+  int64_t batch_x, batch_w, batch_y; /* strides between batch entries in elements */
+  int32_t k, n, batch, act, y_dtype;
+} tlaloc_b200_dense_problem;
+
+/*
+ * `count` (1 or 2) projections of the same m rows in one launch where a tensor-core kernel takes them, else one launch
+ * each.  dtype: F32 or BF16, the type of x and w of every problem; y is F32 or BF16 per problem.  F32 runs in true f32 (FMA,
+ * no reduced-precision products).  flags: TLALOC_B200_GEMM_WEIGHTS_CONST.  Two problems of one call must not depend on
+ * each other's results.
+ */
+int tlaloc_b200_dense_gemm(const tlaloc_b200_dense_problem* problems, int32_t count, int32_t dtype, int32_t m, int32_t flags,
+                           void* stream);
+
+/* ------------------------------------------------------------------ latent attention */
+
+/*
+ * Two RMS norms of the same f32 row with different gains: out_a = x / sqrt(mean(x^2) + eps) * gain_a, out_b likewise
+ * with gain_b (out_b may be NULL).  Both outs have out_dtype F32 | BF16, [rows, n].
+ */
+int tlaloc_b200_rmsnorm_pair(const float* x, const float* gain_a, void* out_a, const float* gain_b, void* out_b, int32_t out_dtype,
+                             int32_t rows, int32_t n, float eps, void* stream);
+
+/*
+ * The step between the down- and up-projections of latent attention.  A row of `in` (f32, row stride ld) is
+ * [q_rank | kv_rank | rot_dim]: the query latent (RMS norm with q_gain into cq [T, q_rank]; q_rank 0 = no query latent),
+ * the key/value latent (RMS norm with kv_gain) and the key part that all heads share (its first rot_dims elements rotated by
+ * position, pairs (2i, 2i+1)).  Normalised latent and rotated key part go to the pool row slot_mapping[t] as
+ * [kv_rank | rot_dim]; a negative slot writes nothing there.  cos/sin f32 [max_pos, rot_dims / 2].  cq and the pool are F32 | BF16
+ * (`dtype`); pool rows are `pool_ld` elements apart.
+ */
+int tlaloc_b200_latent_kv_write(const float* in, int64_t ld, const float* q_gain, const float* kv_gain, float eps,
+                                const int32_t* positions, const float* cos_table, const float* sin_table,
+                                const int32_t* slot_mapping, void* cq, void* pool, int32_t dtype, int64_t pool_ld, int32_t num_tokens,
+                                int32_t q_rank, int32_t kv_rank, int32_t rot_dim, int32_t rot_dims, int32_t num_slots, int32_t max_pos,
+                                void* stream);
+
+/*
+ * Interleaved RoPE of `width` elements per (token, head), the first `rot_dims` of them rotated in pairs (2i, 2i+1), the rest
+ * copied: out[t, h, :] from in[t, h, :]; in and out may be the same.  Strides in elements.
+ */
+int tlaloc_b200_rope_interleaved(const void* in, int64_t in_ld_token, int64_t in_ld_head, void* out, int64_t out_ld_token,
+                                 int64_t out_ld_head, int32_t dtype, const int32_t* positions, const float* cos_table,
+                                 const float* sin_table, int32_t num_tokens, int32_t num_heads, int32_t width, int32_t rot_dims,
+                                 int32_t max_pos, void* stream);
+
+/*
+ * Attention of absorbed queries over a paged pool of latents, one pool row [kv_rank | rot_dim] per position shared by all heads:
+ *   out[t, h, :] = sum_j softmax_j(query[t, h, :] . pool[j, :] * scale) * pool[j, :kv_rank]
+ * over the positions j of the row's sequence with seq_lens[t] - window <= j < seq_lens[t] (window 0: all j < seq_lens[t]).
+ * query [T, H, kv_rank + rot_dim], out [T, H, kv_rank], pool rows pool_ld elements apart, all of `dtype`; block_tables i32
+ * [num_tables, max_blocks] of pages of block_size rows; row_tables i32 [T] names each row's table (NULL: row t uses table t).
+ * scratch: tlaloc_b200_latent_attention_scratch_bytes; scores, weights and sums are f32.
+ */
+size_t tlaloc_b200_latent_attention_scratch_bytes(int32_t num_tokens, int32_t num_heads, int32_t kv_rank, int32_t rot_dim,
+                                                  int32_t max_live);
+int tlaloc_b200_latent_attention(const void* query, const void* pool, int64_t pool_ld, int32_t dtype, const int32_t* block_tables,
+                                 const int32_t* row_tables, const int32_t* seq_lens, void* out, void* scratch, size_t scratch_bytes,
+                                 int32_t num_tokens, int32_t num_heads, int32_t kv_rank, int32_t rot_dim, int32_t num_blocks,
+                                 int32_t block_size, int32_t max_blocks, int32_t num_tables, int32_t window, int32_t max_live,
+                                 float scale, void* stream);
+
 /* ------------------------------------------------------------------ tensor parallelism: the sum over ranks */
 
 #define TLALOC_B200_MAX_PEERS 8

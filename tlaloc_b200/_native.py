@@ -14,9 +14,22 @@ F32, BF16, S8, S32, F8E4M3FN = 11, 16, 2, 4, 20
 OK, INVALID_ARGUMENT, UNSUPPORTED, INTERNAL = 0, -1, -2, -3
 GEMM_EXACT, GEMM_X_F32_EXACT, GEMM_WEIGHTS_CONST, GEMM_I8_MMA, GEMM_X_PLANES = 1, 2, 4, 8, 16
 
+ACT_NONE, ACT_RELU2 = 0, 1
+
 _lib = None
+_subset: str | None = None
 
 _vp, _i32, _f32, _sz = ctypes.c_void_p, ctypes.c_int32, ctypes.c_float, ctypes.c_size_t
+
+_i64 = ctypes.c_int64
+
+
+class DenseProblem(ctypes.Structure):
+    """tlaloc_b200_dense_problem"""
+    _fields_ = [("x", _vp), ("w", _vp), ("bias", _vp), ("residual", _vp), ("y", _vp),
+                ("ld_x", _i64), ("ld_res", _i64), ("ld_y", _i64), ("batch_x", _i64), ("batch_w", _i64), ("batch_y", _i64),
+                ("k", _i32), ("n", _i32), ("batch", _i32), ("act", _i32), ("y_dtype", _i32)]
+
 
 _SIGNATURES = {
     "tlaloc_b200_abi_version": (ctypes.c_int, []),
@@ -45,6 +58,12 @@ _SIGNATURES = {
     "tlaloc_b200_rope_kv_write": (ctypes.c_int, [_vp] * 8 + [_i32, _vp, _vp, _i32, _i32, _i32, _i32, _i32, _i32, _i32, _i32, _i32, _i32, _vp]),
     "tlaloc_b200_swiglu": (ctypes.c_int, [_vp, _vp, _i32, _vp, _i32, _i32, _i32, _vp]),
     "tlaloc_b200_argmax": (ctypes.c_int, [_vp, _vp, _i32, _i32, _vp]),
+    "tlaloc_b200_dense_gemm": (ctypes.c_int, [ctypes.POINTER(DenseProblem), _i32, _i32, _i32, _i32, _vp]),
+    "tlaloc_b200_rmsnorm_pair": (ctypes.c_int, [_vp, _vp, _vp, _vp, _vp, _i32, _i32, _i32, _f32, _vp]),
+    "tlaloc_b200_latent_kv_write": (ctypes.c_int, [_vp, _i64, _vp, _vp, _f32, _vp, _vp, _vp, _vp, _vp, _vp, _i32, _i64] + [_i32] * 7 + [_vp]),
+    "tlaloc_b200_rope_interleaved": (ctypes.c_int, [_vp, _i64, _i64, _vp, _i64, _i64, _i32, _vp, _vp, _vp] + [_i32] * 5 + [_vp]),
+    "tlaloc_b200_latent_attention_scratch_bytes": (_sz, [_i32] * 5),
+    "tlaloc_b200_latent_attention": (ctypes.c_int, [_vp, _vp, _i64, _i32, _vp, _vp, _vp, _vp, _vp, _sz] + [_i32] * 10 + [_f32, _vp]),
     "tlaloc_b200_peer_alloc": (ctypes.c_int, [_sz, ctypes.POINTER(_vp), ctypes.c_char_p]),
     "tlaloc_b200_peer_open": (ctypes.c_int, [ctypes.c_char_p, ctypes.POINTER(_vp)]),
     "tlaloc_b200_peer_close": (ctypes.c_int, [_vp]),
@@ -71,16 +90,26 @@ def declared_symbols() -> list[str]:
     return sorted(set(re.findall(r"\b(tlaloc_b200_\w+|TlalocRegisterKernels)\s*\(", text)))
 
 
+def select(subset: str | None) -> None:
+    """Before the library is first used: this process needs only the kernels of one of build.SUBSETS."""
+    global _subset
+    if _lib is None:
+        _subset = subset
+
+
 def lib() -> ctypes.CDLL:
     global _lib
     if _lib is None:
-        path = _build.build()
+        path = _build.build(subset=_subset)
         if not os.path.exists(path):
             raise RuntimeError(f"{path} is missing: the CUDA extension has not been built (python -m tlaloc_b200.build)")
-        _lib = ctypes.CDLL(path)
+        loaded = ctypes.CDLL(path)
         for name, (res, args) in _SIGNATURES.items():
-            fn = getattr(_lib, name)
+            if path != _build.LIB and not hasattr(loaded, name):
+                continue  # a kernel outside the subset
+            fn = getattr(loaded, name)
             fn.restype, fn.argtypes = res, args
+        _lib = loaded
     return _lib
 
 

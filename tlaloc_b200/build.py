@@ -6,6 +6,9 @@ Each .cu under csrc/ is compiled to an object in build/ (in parallel) and the ob
 tlaloc_b200/lib/libtlaloc_kernels.so, the name the reference's loaders look for
 (triton/backend/pjrt_runtime.cc:139-164).  A target newer than every source is left alone, so machines
 without nvcc (or without the sources' mtimes changing) just use the library that is there.
+
+A process that serves one model needs only that model's kernels: `build(subset="latent")` compiles the sources listed in
+SUBSETS (from the same objects) into a library of its own, unless the full library is there and current.
 """
 from __future__ import annotations
 
@@ -20,6 +23,7 @@ CSRC = os.path.join(HERE, "csrc")
 OBJ = os.path.join(HERE, "build")
 LIB_DIR = os.path.join(HERE, "lib")
 LIB = os.path.join(LIB_DIR, "libtlaloc_kernels.so")
+SUBSETS = {"latent": ("runtime", "decode_ops", "dense_gemm", "latent_ops", "latent_attention")}
 INCLUDE = os.path.join(os.path.dirname(HERE), "include")
 
 NVCC_FLAGS = [
@@ -28,37 +32,48 @@ NVCC_FLAGS = [
 ]
 
 
-def sources() -> list[str]:
-    return sorted(os.path.join(CSRC, f) for f in os.listdir(CSRC) if f.endswith(".cu"))
+def library(subset: str | None = None) -> str:
+    return LIB if subset is None else os.path.join(LIB_DIR, f"libtlaloc_{subset}.so")
 
 
-def _deps() -> list[str]:
+def sources(subset: str | None = None) -> list[str]:
+    names = sorted(f for f in os.listdir(CSRC) if f.endswith(".cu") and (subset is None or f[:-3] in SUBSETS[subset]))
+    return [os.path.join(CSRC, f) for f in names]
+
+
+def _deps(subset: str | None = None) -> list[str]:
     extra = [os.path.join(CSRC, f) for f in os.listdir(CSRC) if f.endswith((".cuh", ".h"))]
-    return sources() + extra + [os.path.join(INCLUDE, "tlaloc_b200.h")]
+    return sources(subset) + extra + [os.path.join(INCLUDE, "tlaloc_b200.h")]
 
 
-def up_to_date() -> bool:
-    if not os.path.exists(LIB):
+def up_to_date(subset: str | None = None) -> bool:
+    lib = library(subset)
+    if not os.path.exists(lib):
         return False
-    t = os.path.getmtime(LIB)
-    return all(os.path.getmtime(d) <= t for d in _deps())
+    t = os.path.getmtime(lib)
+    return all(os.path.getmtime(d) <= t for d in _deps(subset))
 
 
 def nvcc() -> str | None:
     return shutil.which("nvcc") or ("/usr/local/cuda/bin/nvcc" if os.path.exists("/usr/local/cuda/bin/nvcc") else None)
 
 
-def build(force: bool = False, verbose: bool = False) -> str:
-    if not force and up_to_date():
-        return LIB
+def build(force: bool = False, verbose: bool = False, subset: str | None = None) -> str:
+    """Path of an up-to-date library: the full one, or (subset given) one that holds at least the subset's kernels."""
+    lib = library(subset)
+    if not force:
+        for current in (None, subset):
+            if up_to_date(current) and (current == subset or subset is not None):
+                return library(current)
     cc = nvcc()
     if cc is None:
-        if os.path.exists(LIB):
-            return LIB
-        raise RuntimeError("nvcc not found and libtlaloc_kernels.so has not been built")
+        for there in (lib, LIB):
+            if os.path.exists(there):
+                return there
+        raise RuntimeError(f"nvcc not found and {os.path.basename(lib)} has not been built")
     os.makedirs(OBJ, exist_ok=True)
     os.makedirs(LIB_DIR, exist_ok=True)
-    hdr_time = max(os.path.getmtime(d) for d in _deps() if not d.endswith(".cu"))
+    hdr_time = max(os.path.getmtime(d) for d in _deps(subset) if not d.endswith(".cu"))
 
     def compile_one(src: str) -> str:
         obj = os.path.join(OBJ, os.path.basename(src)[:-3] + ".o")
@@ -73,13 +88,13 @@ def build(force: bool = False, verbose: bool = False) -> str:
         return obj
 
     with concurrent.futures.ThreadPoolExecutor(max_workers=8) as pool:
-        objs = list(pool.map(compile_one, sources()))
-    r = subprocess.run([cc, "-shared", "-o", LIB, *objs, "-gencode", "arch=compute_100a,code=sm_100a"],
+        objs = list(pool.map(compile_one, sources(subset)))
+    r = subprocess.run([cc, "-shared", "-o", lib, *objs, "-gencode", "arch=compute_100a,code=sm_100a"],
                        capture_output=True, text=True)
     if r.returncode != 0:
         sys.stderr.write(r.stdout + r.stderr)
         raise RuntimeError("link failed")
-    return LIB
+    return lib
 
 
 if __name__ == "__main__":

@@ -1,0 +1,25 @@
+// Shared by the kernels behind tlaloc_b200_dense_gemm.
+#pragma once
+
+#include "common.cuh"
+
+namespace tlaloc_b200 {
+
+// What happens to a finished sum before it is stored.
+__device__ __forceinline__ float DenseActivation(int act, float v)
+{
+  if (act == TLALOC_B200_ACT_RELU2) {
+    const float r = fmaxf(v, 0.f);
+    return r * r;
+  }
+  return v;
+}
+__device__ __forceinline__ float DenseEpilogue(const tlaloc_b200_dense_problem& p, float v, int m, int n)
+{
+  if (p.bias != nullptr) v += __ldg(p.bias + n);
+  v = DenseActivation(p.act, v);
+  if (p.residual != nullptr) v += p.residual[static_cast<size_t>(m) * p.ld_res + n];
+  return v;
+}
+
+}  // namespace tlaloc_b200

@@ -22,7 +22,10 @@ import numpy as np
 import torch
 
 from . import ops, sharding
+from .paging import RaggedStep
 from .peer import PeerBuffers
+from .rotary import rope_tables
+from .step_model import StepModel
 
 
 @dataclass
@@ -52,17 +55,7 @@ LLAMA3_70B = dict(num_layers=80, d_model=8192, num_heads=64, num_kv_heads=8, hea
 TINY = dict(num_layers=2, d_model=256, num_heads=4, num_kv_heads=2, head_dim=64, ffn=688, vocab=1024)
 
 
-def rope_tables(theta: float, head_dim: int, positions: int):
-    """HfDecoderGraph.ropeTables (:436-462): computed in double, narrowed to f32, both halves equal."""
-    half = head_dim // 2
-    inv = np.power(float(theta), -2.0 * np.arange(half, dtype=np.float64) / head_dim)
-    ang = np.arange(positions, dtype=np.float64)[:, None] * inv[None, :]
-    cos = np.concatenate([np.cos(ang), np.cos(ang)], axis=1).astype(np.float32)
-    sin = np.concatenate([np.sin(ang), np.sin(ang)], axis=1).astype(np.float32)
-    return cos, sin
-
-
-class Decoder:
+class Decoder(StepModel):
     """Weights, KV pools and step buffers of one rank; `step()` runs one decode step for `batch` sequences."""
 
     def __init__(self, cfg: DecoderConfig, batch: int, num_blocks: int, max_blocks_per_seq: int, *, device="cuda:0",
@@ -73,14 +66,14 @@ class Decoder:
         if not torch.cuda.is_available():
             raise RuntimeError("tlaloc_b200.Decoder needs a CUDA device: there is no CPU path")
         sharding.check_world(cfg.num_heads, cfg.num_kv_heads, cfg.ffn, cfg.vocab, world)
-        self.cfg, self.batch, self.device, self.rank, self.world, self.group = cfg, batch, torch.device(device), rank, world, group
+        super().__init__(batch, batch, num_blocks, max_blocks_per_seq, cfg.block_size, cfg.vocab, device)
+        self.cfg, self.batch, self.rank, self.world, self.group = cfg, batch, rank, world, group
         self.exact = bool(exact)
         # SwiGLU in the gate|up projection's epilogue: batches the tensor-core kernels take (17 rows and more) and FFN
         # widths that tile in blocks of 128 per rank; $TLALOC_B200_FUSE_SWIGLU=0 keeps the separate kernel
         self.fuse_swiglu = (not exact and batch >= 17 and (cfg.ffn // world) % 128 == 0
                             and os.environ.get("TLALOC_B200_FUSE_SWIGLU", "1") != "0")
         self.hq, self.hk, self.f = cfg.num_heads // world, cfg.num_kv_heads // world, cfg.ffn // world
-        self.num_blocks, self.max_blocks = num_blocks, max_blocks_per_seq
         dev, B, d, hd = self.device, batch, cfg.d_model, cfg.head_dim
         ops.init()
         self.layers: list[dict] = []
@@ -90,15 +83,8 @@ class Decoder:
         self.value_pools = [torch.zeros_like(p) for p in self.key_pools]
         cos, sin = rope_tables(cfg.rope_theta, hd, cfg.max_positions)
         self.cos, self.sin = torch.from_numpy(cos).to(dev), torch.from_numpy(sin).to(dev)
-        i32 = dict(dtype=torch.int32, device=dev)
         f32 = dict(dtype=torch.float32, device=dev)
         bf = dict(dtype=torch.bfloat16, device=dev)
-        # step inputs (static addresses: the CUDA graph reads them)
-        self.token_ids = torch.zeros((B,), **i32)
-        self.positions = torch.zeros((B,), **i32)
-        self.block_tables = torch.zeros((B, max_blocks_per_seq), **i32)
-        self.seq_lens = torch.ones((B,), **i32)
-        self.slot_mapping = torch.full((B,), -1, **i32)
         # step buffers
         nqkv = (self.hq + 2 * self.hk) * hd
         # Tensor parallelism, the sum over ranks after o_proj and down_proj.  $TLALOC_B200_TP_REDUCE:
@@ -153,12 +139,11 @@ class Decoder:
         self.rows_planes = (self.rows_residual and self.norm_planes and nqkv % 16 == 0 and (2 * self.f) % 16 == 0
                             and os.environ.get("TLALOC_B200_GEMM_I8", "1") != "0" and os.environ.get("TLALOC_B200_TP_PLANES", "1") != "0")
         self.logits = torch.empty((B, cfg.vocab // world), **f32)
-        self.next_ids = torch.zeros((B,), **i32)
+        self.next_ids = torch.zeros((B,), dtype=torch.int32, device=dev)
         self.best = torch.empty((B,), **f32)
         shape = ops.parse_paged_attention(self.q_rot, self.key_pools[0], self.value_pools[0], self.block_tables,
                                           self.seq_lens, scale=cfg.scale)
         self.att_scratch = ops.paged_attention_scratch(shape, dev)
-        self._graph = None
 
     # ------------------------------------------------------------------ weights
 
@@ -213,16 +198,6 @@ class Decoder:
 
     # ------------------------------------------------------------------ the step
 
-    def set_inputs(self, token_ids, positions, block_tables, seq_lens, slot_mapping) -> None:
-        """Host (NumPy or pinned torch) step inputs -> the device buffers the graph reads."""
-        for dst, src in ((self.token_ids, token_ids), (self.positions, positions), (self.block_tables, block_tables),
-                         (self.seq_lens, seq_lens), (self.slot_mapping, slot_mapping)):
-            if src is None:
-                continue
-            if isinstance(src, np.ndarray):
-                src = torch.from_numpy(np.ascontiguousarray(src, dtype=np.int32))
-            dst.copy_(src.reshape(dst.shape), non_blocking=True)
-
     def _all_reduce(self, x: torch.Tensor) -> None:
         if self.world == 1:
             return
@@ -231,7 +206,7 @@ class Decoder:
         else:
             torch.distributed.all_reduce(x, group=self.group)
 
-    def _run_step(self) -> None:
+    def _run_step(self, rows: int) -> None:
         if not self.exact:
             return self._launch_step()
         before = ops.set_order_faithful(True)
@@ -383,29 +358,14 @@ class Decoder:
         glob = ids.long() + (torch.arange(g, device=self.device) * vp)[:, None]
         self.next_ids.copy_(glob.gather(0, win[None, :])[0].to(torch.int32))
 
-    def capture(self) -> None:
-        """Capture the step into a CUDA graph (after one eager warm-up step on a side stream)."""
-        s = torch.cuda.Stream(device=self.device)
-        s.wait_stream(torch.cuda.current_stream(self.device))
-        with torch.cuda.stream(s):
-            self._run_step()
-        torch.cuda.current_stream(self.device).wait_stream(s)
-        torch.cuda.synchronize(self.device)
-        self._graph = torch.cuda.CUDAGraph()
-        with torch.cuda.graph(self._graph):
-            self._run_step()
-
     def exchange_status(self) -> int:
         """0, or the code a timed-out wait of the tensor-parallel sum left behind (see PeerBuffers.status)."""
         return self.peer.status() if self.peer is not None else 0
 
-    def step(self) -> torch.Tensor:
-        """One decode step over the current inputs; returns the device tensor of next token ids [batch]."""
-        if self._graph is not None:
-            self._graph.replay()
-        else:
-            self._run_step()
-        return self.next_ids
+    def run(self, step: RaggedStep, want) -> torch.Tensor:
+        self.set_inputs(*self._padded(step, self.batch))
+        self.step()
+        return self.logits[torch.as_tensor(want, dtype=torch.long, device=self.device)]
 
     # ------------------------------------------------------------------ traffic model
 

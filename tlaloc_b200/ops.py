@@ -243,3 +243,97 @@ def argmax(logits, out=None):
     _out("ARGMAX out", out, (rows,), torch.int32, logits)
     N.check(N.lib().tlaloc_b200_argmax(_ptr(logits), _ptr(out), rows, n, _stream(logits)))
     return out
+
+
+# ---------------------------------------------------------------------- unquantized projections, latent attention
+
+
+def dense(x, w, out, *, bias=None, residual=None, act=N.ACT_NONE) -> N.DenseProblem:
+    """One projection out = act(x @ w.T + bias) + residual for `dense_gemm`.  x [M, K], w [N, K], out [M, N]; or a batch
+    of them (the heads of a layer): x [B, M, K], w [B, N, K], out [B, M, N].  x, out and residual may be strided views whose
+    last dimension is dense; w is contiguous."""
+    batched = w.dim() == 3
+    for name, t in (("x", x), ("out", out)) + ((("residual", residual),) if residual is not None else ()):
+        if not t.is_cuda or t.stride(-1) != 1 or t.dim() != w.dim():
+            raise ValueError(f"DENSE_PROJ {name}: a CUDA tensor of rank {w.dim()} with a dense last dimension is needed")
+    _dev(w, bias)
+    b, n, k = w.shape if batched else (1, *w.shape)
+    m = x.shape[-2]
+    if x.shape[-1] != k or tuple(out.shape[-2:]) != (m, n) or (batched and (x.shape[0] != b or out.shape[0] != b)) or x.dtype != w.dtype:
+        raise ValueError(f"DENSE_PROJ: x {tuple(x.shape)} {x.dtype}, w {tuple(w.shape)} {w.dtype}, out {tuple(out.shape)} do not fit")
+    if (bias is not None and (bias.dtype != torch.float32 or tuple(bias.shape) != (n,))) or (
+            residual is not None and (residual.dtype != torch.float32 or tuple(residual.shape) != (m, n))):
+        raise ValueError(f"DENSE_PROJ: bias is f32 [{n}], residual f32 [{m}, {n}]")
+    p = N.DenseProblem(x=_ptr(x), w=_ptr(w), bias=_ptr(bias), residual=_ptr(residual), y=_ptr(out), ld_x=x.stride(-2),
+                       ld_res=residual.stride(-2) if residual is not None else 0, ld_y=out.stride(-2),
+                       batch_x=x.stride(0) if batched else 0, batch_w=n * k, batch_y=out.stride(0) if batched else 0,
+                       k=k, n=n, batch=b, act=act, y_dtype=_dt(out))
+    p.rows, p.like = m, x
+    return p
+
+
+def dense_gemm(*problems, weights_const=False) -> None:
+    """Runs one or two `dense` problems of the same rows and type."""
+    like, m = problems[0].like, problems[0].rows
+    if any(p.rows != m or p.like.dtype != like.dtype for p in problems):
+        raise ValueError("DENSE_PROJ: the problems of one call have the same rows and type")
+    N.check(N.lib().tlaloc_b200_dense_gemm((N.DenseProblem * len(problems))(*problems), len(problems), _dt(like), m,
+                                           N.GEMM_WEIGHTS_CONST if weights_const else 0, _stream(like)))
+
+
+def rmsnorm_pair(x, gain_a, out_a, eps, gain_b=None, out_b=None) -> None:
+    """out_a = x / sqrt(mean(x^2) + eps) * gain_a and, if given, the same with gain_b into out_b; x f32 [rows, n]."""
+    _dev(x, gain_a, gain_b)
+    rows, n = x.shape
+    _out("RMSNORM_PAIR out", out_a, (rows, n), (torch.float32, torch.bfloat16), x)
+    _out("RMSNORM_PAIR second out", out_b, (rows, n), out_a.dtype, x)
+    N.check(N.lib().tlaloc_b200_rmsnorm_pair(_ptr(x), _ptr(gain_a), _ptr(out_a), _ptr(gain_b), _ptr(out_b), _dt(out_a), rows, n, float(eps),
+                                             _stream(x)))
+
+
+def latent_kv_write(low, q_gain, kv_gain, eps, positions, cos, sin, slots, cq, pool, *, q_rank, kv_rank, rot_dim, rot_dims) -> None:
+    """low f32 [T, q_rank + kv_rank + rot_dim] -> cq [T, q_rank] (normed) and pool rows [kv_rank | rot_dim] (normed, rotated)."""
+    _dev(q_gain, kv_gain, positions, cos, sin, slots, cq, pool)
+    T = low.shape[0]
+    if low.dtype != torch.float32 or low.stride(1) != 1 or low.shape[1] != q_rank + kv_rank + rot_dim:
+        raise ValueError("LATENT_KV_WRITE: low is f32 [T, q_rank + kv_rank + rot_dim] with dense rows")
+    if pool.dim() != 3 or positions.shape[0] < T or slots.shape[0] < T or tuple(cos.shape) != (cos.shape[0], rot_dims // 2) or cos.shape != sin.shape:
+        raise ValueError("LATENT_KV_WRITE: pool [P, block, row], positions and slots [T], cos and sin [positions, rot_dims / 2]")
+    if q_rank:
+        _out("LATENT_KV_WRITE cq", cq, (T, q_rank), pool.dtype, low)
+    N.check(N.lib().tlaloc_b200_latent_kv_write(
+        _ptr(low), low.stride(0), _ptr(q_gain), _ptr(kv_gain), float(eps), _ptr(positions), _ptr(cos), _ptr(sin), _ptr(slots), _ptr(cq),
+        _ptr(pool), _dt(pool), pool.shape[2], T, q_rank, kv_rank, rot_dim, rot_dims, pool.shape[0] * pool.shape[1], cos.shape[0], _stream(low)))
+
+
+def rope_interleaved(x, out, positions, cos, sin, *, rot_dims) -> None:
+    """x, out [T, H, width] (strided views of the same type; may be the same): the first rot_dims elements rotated in pairs."""
+    T, H, width = x.shape
+    if x.shape != out.shape or x.dtype != out.dtype or x.stride(2) != 1 or out.stride(2) != 1 or not (x.is_cuda and out.is_cuda):
+        raise ValueError("ROPE_INTERLEAVED: x and out are CUDA tensors [T, H, width] of one type with dense rows")
+    _dev(positions, cos, sin)
+    N.check(N.lib().tlaloc_b200_rope_interleaved(_ptr(x), x.stride(0), x.stride(1), _ptr(out), out.stride(0), out.stride(1), _dt(x),
+                                                 _ptr(positions), _ptr(cos), _ptr(sin), T, H, width, rot_dims, cos.shape[0], _stream(x)))
+
+
+def latent_attention_scratch_bytes(rows, heads, kv_rank, rot_dim, max_live) -> int:
+    return int(N.lib().tlaloc_b200_latent_attention_scratch_bytes(rows, heads, kv_rank, rot_dim, max_live))
+
+
+def latent_attention(query, pool, block_tables, seq_lens, out, *, kv_rank, scale, window=0, row_tables=None, scratch=None, max_live=0) -> None:
+    """query [T, H, kv_rank + rot_dim] over pool [P, block, row] -> out [T, H, kv_rank]; see include/tlaloc_b200.h.
+    max_live: a bound on the live positions of any row (0: what the tables and the window allow)."""
+    _dev(query, pool, block_tables, seq_lens, out, row_tables, scratch)
+    T, H, row = query.shape
+    if query.dtype != pool.dtype or pool.dim() != 3:
+        raise ValueError("LATENT_ATTENTION: query and pool have one type; pool is [P, block, row]")
+    if any(t is not None and t.dtype != torch.int32 for t in (block_tables, seq_lens, row_tables)):
+        raise TypeError("LATENT_ATTENTION: tables and lengths are int32")
+    if seq_lens.shape[0] < T or (row_tables is not None and row_tables.shape[0] < T):
+        raise ValueError("LATENT_ATTENTION: one length and one table per row")
+    _out("LATENT_ATTENTION out", out, (T, H, kv_rank), query.dtype, query)
+    P, bs, ld = pool.shape
+    N.check(N.lib().tlaloc_b200_latent_attention(
+        _ptr(query), _ptr(pool), ld, _dt(query), _ptr(block_tables), _ptr(row_tables), _ptr(seq_lens), _ptr(out), _ptr(scratch),
+        0 if scratch is None else scratch.numel() * scratch.element_size(), T, H, kv_rank, row - kv_rank, P, bs, block_tables.shape[1],
+        block_tables.shape[0], int(window), int(max_live), float(scale), _stream(query)))

@@ -87,8 +87,17 @@ class Sequence:
         self.pages.extend(got)
         return True
 
+    def drop_before(self, pool: PagePool, position: int, block_size: int) -> int:
+        """Gives back the pages that hold only positions below `position` (a model whose every layer attends through a
+        sliding window never reads them again); their table entries become the padding page.  Returns how many."""
+        n = min(max(position, 0) // block_size, len(self.pages))
+        old = [p for p in self.pages[:n] if p != PADDING_PAGE]
+        pool.give(old)
+        self.pages[:n] = [PADDING_PAGE] * n
+        return len(old)
+
     def release(self, pool: PagePool) -> None:
-        pool.give(self.pages)
+        pool.give(p for p in self.pages if p != PADDING_PAGE)
         self.pages, self.length = [], 0
 
 
@@ -133,6 +142,42 @@ def stage_step(work, *, rows: int, width: int, max_blocks: int, block_size: int)
         tables[r, :k] = pages[:k]
         lens[r] = end
     return StepInputs(ids, pos, slots, tables, lens)
+
+
+@dataclass
+class RaggedStep:
+    """The integer operands of one step over a flat list of token rows, `len(starts) - 1` sequences one after the other."""
+
+    token_ids: np.ndarray     # i32 [tokens]
+    positions: np.ndarray     # i32 [tokens]
+    slot_mapping: np.ndarray  # i32 [tokens]
+    seq_lens: np.ndarray      # i32 [tokens]: position + 1
+    row_tables: np.ndarray    # i32 [tokens]: which row of block_tables
+    block_tables: np.ndarray  # i32 [sequences, max_blocks]
+    starts: np.ndarray        # i32 [sequences + 1]: first token row of each sequence
+
+
+def stage_ragged(work, *, max_blocks: int, block_size: int) -> RaggedStep:
+    """`work` = [(sequence, tokens)]: each sequence runs its tokens at positions sequence.length .. (its pages must already
+    cover them, see Sequence.reserve)."""
+    counts = [len(tokens) for _, tokens in work]
+    if not work or min(counts) < 1:
+        raise ValueError("a step needs at least one token of every sequence in it")
+    tables = np.full((len(work), max_blocks), PADDING_PAGE, np.int32)
+    pos, slots = [], []
+    for r, (seq, tokens) in enumerate(work):
+        end = seq.length + len(tokens)
+        if end > len(seq.pages) * block_size or len(seq.pages) > max_blocks:
+            raise ValueError(f"sequence {r}: positions up to {end - 1}, but {len(seq.pages)} pages of {block_size} in a table of {max_blocks}")
+        p = np.arange(seq.length, end, dtype=np.int64)
+        pages = np.asarray(seq.pages, np.int64)
+        pos.append(p)
+        slots.append(pages[p // block_size] * block_size + p % block_size)
+        tables[r, :len(seq.pages)] = pages
+    positions = np.concatenate(pos).astype(np.int32)
+    return RaggedStep(np.concatenate([np.asarray(t, np.int32) for _, t in work]), positions, np.concatenate(slots).astype(np.int32),
+                      positions + 1, np.repeat(np.arange(len(work), dtype=np.int32), counts), tables,
+                      np.concatenate([[0], np.cumsum(counts)]).astype(np.int32))
 
 
 def commit_step(work) -> None:

@@ -234,7 +234,7 @@ def write_staged(version_dir: str, w: DecoderWeights, model: dict, *, weight_dty
 # ---------------------------------------------------------------------------------------------- safetensors
 
 def read_safetensors(path: str) -> dict:
-    """name -> f32 array of a .safetensors file (F32, BF16 and F16 tensors; 8-byte little-endian header length, a JSON
+    """name -> array of a .safetensors file (F32, BF16 and F16 tensors widened to f32, I32 kept; 8-byte little-endian header length, a JSON
     header of dtype / shape / data_offsets, then the raw little-endian data)."""
     with open(path, "rb") as f:
         (n,) = struct.unpack("<Q", f.read(8))
@@ -254,6 +254,8 @@ def read_safetensors(path: str) -> dict:
                 a = bf16_to_f32(np.frombuffer(raw, dtype="<u2"))
             elif dt == "F16":
                 a = np.frombuffer(raw, dtype="<f2").astype(np.float32)
+            elif dt == "I32":
+                a = np.frombuffer(raw, dtype="<i4").astype(np.int32)
             else:
                 raise ValueError(f"{path}: tensor {name!r} has dtype {dt}, which this reader does not widen")
             out[name] = a.reshape(meta["shape"])
