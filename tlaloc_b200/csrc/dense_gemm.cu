@@ -87,7 +87,13 @@ extern "C" int tlaloc_b200_dense_gemm(const tlaloc_b200_dense_problem* problems,
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   int launches = 0;
   cudaError_t e = cudaSuccess;
-  for (int i = 0; i < count && e == cudaSuccess; ++i) {
+  bool tc = dtype == TLALOC_B200_BF16 && !OrderFaithful();
+  for (int i = 0; i < count; ++i) tc = tc && DenseGemmTcApplies(problems[i]);
+  if (tc) {
+    e = LaunchDenseGemmTc(problems, count, m, (flags & TLALOC_B200_GEMM_WEIGHTS_CONST) != 0, st);
+    launches = 1;
+  }
+  for (int i = 0; i < count && e == cudaSuccess && !tc; ++i) {
     e = dtype == TLALOC_B200_F32 ? LaunchTiled<float>(problems[i], m, st) : LaunchTiled<__nv_bfloat16>(problems[i], m, st);
     ++launches;
   }

@@ -22,4 +22,8 @@ __device__ __forceinline__ float DenseEpilogue(const tlaloc_b200_dense_problem& 
   return v;
 }
 
+// The tensor-core kernel (dense_gemm_tc.cu): bf16 x and w whose addresses, row and batch strides are multiples of 16 bytes.
+bool DenseGemmTcApplies(const tlaloc_b200_dense_problem& p);
+cudaError_t LaunchDenseGemmTc(const tlaloc_b200_dense_problem* problems, int count, int m, bool weights_const, cudaStream_t st);
+
 }  // namespace tlaloc_b200
