@@ -374,6 +374,28 @@ int tlaloc_b200_latent_attention(const void* query, const void* pool, int64_t po
                                  int32_t block_size, int32_t max_blocks, int32_t num_tables, int32_t window, int32_t max_live,
                                  float scale, void* stream);
 
+/*
+ * Rows [first, first + count) of one sequence out of a paged pool of latents: out[r, :row] = the pool row of position first + r
+ * under `table` (i32 [max_blocks]).  pool_ld and out_ld in elements, both a multiple of 16 bytes and at least `row` rounded up to it.
+ */
+int tlaloc_b200_latent_gather(const void* pool, int64_t pool_ld, int32_t dtype, const int32_t* table, void* out, int64_t out_ld,
+                              int32_t first, int32_t count, int32_t row, int32_t num_blocks, int32_t block_size, int32_t max_blocks,
+                              void* stream);
+
+/*
+ * Attention of a prompt portion over expanded keys and values, bf16: query i (row i of q [T, H, dim + rot_dim], rotated) is position
+ * first_query + i of the num_keys keys; it sees key j with 0 <= first_query + i - j < window (window 0: every j up to its own).
+ *   out[i, h, :] = sum_j softmax_j((q[i, h, :dim] . k[j, h, :] + q[i, h, dim:] . k_rot[j, :]) * scale) * v[j, h, :]
+ * k and v: rows kv_ld apart, heads kv_head_ld apart; k_rot rows rot_ld apart, shared by the heads; out rows out_ld apart, heads side
+ * by side.  All strides in elements and multiples of 16 bytes.  Scores, weights and sums are f32; the weights enter the product
+ * with v as bf16.  _applies: 1 if the kernel takes these sizes.
+ */
+int tlaloc_b200_window_attention_applies(int32_t dim, int32_t rot_dim, int32_t vdim);
+int tlaloc_b200_window_attention(const void* q, const void* k, const void* k_rot, int64_t rot_ld, const void* v, int64_t kv_ld,
+                                 int64_t kv_head_ld, void* out, int64_t out_ld, int32_t num_queries, int32_t num_keys,
+                                 int32_t first_query, int32_t num_heads, int32_t dim, int32_t rot_dim, int32_t vdim, int32_t window,
+                                 float scale, void* stream);
+
 /* ------------------------------------------------------------------ tensor parallelism: the sum over ranks */
 
 #define TLALOC_B200_MAX_PEERS 8

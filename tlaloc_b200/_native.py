@@ -64,6 +64,9 @@ _SIGNATURES = {
     "tlaloc_b200_rope_interleaved": (ctypes.c_int, [_vp, _i64, _i64, _vp, _i64, _i64, _i32, _vp, _vp, _vp] + [_i32] * 5 + [_vp]),
     "tlaloc_b200_latent_attention_scratch_bytes": (_sz, [_i32] * 5),
     "tlaloc_b200_latent_attention": (ctypes.c_int, [_vp, _vp, _i64, _i32, _vp, _vp, _vp, _vp, _vp, _sz] + [_i32] * 10 + [_f32, _vp]),
+    "tlaloc_b200_latent_gather": (ctypes.c_int, [_vp, _i64, _i32, _vp, _vp, _i64] + [_i32] * 6 + [_vp]),
+    "tlaloc_b200_window_attention_applies": (ctypes.c_int, [_i32] * 3),
+    "tlaloc_b200_window_attention": (ctypes.c_int, [_vp, _vp, _vp, _i64, _vp, _i64, _i64, _vp, _i64] + [_i32] * 8 + [_f32, _vp]),
     "tlaloc_b200_peer_alloc": (ctypes.c_int, [_sz, ctypes.POINTER(_vp), ctypes.c_char_p]),
     "tlaloc_b200_peer_open": (ctypes.c_int, [ctypes.c_char_p, ctypes.POINTER(_vp)]),
     "tlaloc_b200_peer_close": (ctypes.c_int, [_vp]),

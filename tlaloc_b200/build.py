@@ -23,7 +23,7 @@ CSRC = os.path.join(HERE, "csrc")
 OBJ = os.path.join(HERE, "build")
 LIB_DIR = os.path.join(HERE, "lib")
 LIB = os.path.join(LIB_DIR, "libtlaloc_kernels.so")
-SUBSETS = {"latent": ("runtime", "decode_ops", "dense_gemm", "dense_gemm_tc", "latent_ops", "latent_attention")}
+SUBSETS = {"latent": ("runtime", "decode_ops", "dense_gemm", "dense_gemm_tc", "latent_ops", "latent_attention", "latent_prefill")}
 INCLUDE = os.path.join(os.path.dirname(HERE), "include")
 
 NVCC_FLAGS = [

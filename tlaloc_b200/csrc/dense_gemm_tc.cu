@@ -36,7 +36,9 @@ struct Layout {
   static constexpr int kPipe = kStages * kStage;
   static constexpr int kTileStride = kBN + 4;  // the slice's partial tile [BT][kTileStride] f32, aliases the ring
   static_assert(kPipe >= BT * kTileStride * 4 || BT == 256, "the partial tile aliases the ring");
-  static constexpr int kBars = kPipe;
+  static constexpr int kRows = BT / 2 < 32 ? BT / 2 : 32;          // activation rows an epilogue group takes at a time
+  static constexpr int kOut = kPipe;                               // two groups' bf16 output rows [kRows][128]
+  static constexpr int kBars = kOut + 2 * kRows * kBN * 2;
   static constexpr int kSlot = kBars + 8 * (2 * kStages + 4);
   static constexpr int kBytes = kSlot + 8 + 1024;  // slack to align to 1024
 };
@@ -46,7 +48,7 @@ struct TcProblem {
   const float* residual;
   void* y;
   int64_t ld_res, ld_y, batch_y;
-  int k, n, act, y_f32, tiles_n, swap_x;  // swap_x: the activations' map has the batch before the rows
+  int k, n, act, y_f32, rows_bf16, tiles_n, swap_x;  // rows_bf16: y takes whole 16-byte words; swap_x: the activations' map has the batch before the rows
 };
 struct TcArgs {
   TcProblem p[2];
@@ -105,28 +107,60 @@ __device__ __forceinline__ Tile TileAt(const TcArgs& a, int id, int BT)
 }
 
 // One output column n of CH consecutive rows from m: bias, activation, residual, store.
+template <int CH, typename YT>
+__device__ __forceinline__ void StoreColumnAs(const TcProblem& p, YT* y, const float* res, int rows, const float* v, float bias)
+{
+  const int64_t ld = p.ld_y, ld_res = p.ld_res;
+  const int act = p.act;
+  float r[CH];
+#pragma unroll
+  for (int c = 0; c < CH; ++c) {
+    r[c] = 0.f;
+    if (res != nullptr && c < rows) {
+      r[c] = *res;
+      res += ld_res;
+    }
+  }
+#pragma unroll
+  for (int c = 0; c < CH; ++c) {
+    if (c < rows) *y = FromF32<YT>(DenseActivation(act, v[c] + bias) + r[c]);
+    y += ld;
+  }
+}
 template <int CH>
 __device__ __forceinline__ void StoreColumn(const TcProblem& p, const Tile& t, int n, int m, int M, const float* v, float bias)
 {
   const int rows = min(CH, M - m);
   if (n >= p.n || rows <= 0) return;
-  const bool has_res = p.residual != nullptr;
-  float r[CH];
-  const float* res = p.residual + static_cast<size_t>(m) * p.ld_res + n;
-#pragma unroll
-  for (int c = 0; c < CH; ++c) r[c] = has_res && c < rows ? res[c * p.ld_res] : 0.f;
+  const float* res = p.residual != nullptr ? p.residual + static_cast<size_t>(m) * p.ld_res + n : nullptr;
   const size_t at = t.b * p.batch_y + static_cast<size_t>(m) * p.ld_y + n;
-  if (p.y_f32) {
-    float* y = static_cast<float*>(p.y) + at;
+  if (p.y_f32) StoreColumnAs<CH>(p, static_cast<float*>(p.y) + at, res, rows, v, bias);
+  else StoreColumnAs<CH>(p, static_cast<__nv_bfloat16*>(p.y) + at, res, rows, v, bias);
+}
+
+// The same for a whole 128-column bf16 tile of a group of four warps: the rows meet in shared memory and leave as 16-byte words.
+template <int CH>
+__device__ __forceinline__ void StoreRowsBf16(const TcProblem& p, const Tile& t, int m, int M, const float* v, float bias, __nv_bfloat16* stage,
+                                              int tid, int group)
+{
+  const int col = tid & 127;
+  if (p.act == TLALOC_B200_ACT_RELU2) {
 #pragma unroll
-    for (int c = 0; c < CH; ++c)
-      if (c < rows) y[c * p.ld_y] = DenseActivation(p.act, v[c] + bias) + r[c];
+    for (int c = 0; c < CH; ++c) stage[c * kBN + col] = __float2bfloat16_rn(DenseActivation(TLALOC_B200_ACT_RELU2, v[c] + bias));
   } else {
-    __nv_bfloat16* y = static_cast<__nv_bfloat16*>(p.y) + at;
 #pragma unroll
-    for (int c = 0; c < CH; ++c)
-      if (c < rows) y[c * p.ld_y] = __float2bfloat16_rn(DenseActivation(p.act, v[c] + bias) + r[c]);
+    for (int c = 0; c < CH; ++c) stage[c * kBN + col] = __float2bfloat16_rn(v[c] + bias);
   }
+  asm volatile("bar.sync %0, 128;\n" ::"r"(1 + group) : "memory");
+  const int64_t ld = p.ld_y;
+  __nv_bfloat16* y = static_cast<__nv_bfloat16*>(p.y) + t.b * p.batch_y + static_cast<size_t>(m) * ld + t.n0 + (col & 15) * 8;
+  const uint4* src = reinterpret_cast<const uint4*>(stage) + (col & 15);
+#pragma unroll
+  for (int i = 0; i < CH / 8; ++i) {
+    const int r = i * 8 + (col >> 4);
+    if (m + r < M) *reinterpret_cast<uint4*>(y + r * ld) = src[r * 16];
+  }
+  asm volatile("bar.sync %0, 128;\n" ::"r"(1 + group) : "memory");
 }
 
 template <int BT, bool SPLIT>
@@ -281,7 +315,11 @@ __global__ void __launch_bounds__(kThreads, 1)
           float v[CH];
 #pragma unroll
           for (int e = 0; e < CH; ++e) v[e] = __uint_as_float(r[e]);
-          StoreColumn<CH>(p, t, n, t.m0 + c, a.M, v, bias);
+          if (p.rows_bf16 && t.n0 + kBN <= p.n) {
+            StoreRowsBf16<CH>(p, t, t.m0 + c, a.M, v, bias, reinterpret_cast<__nv_bfloat16*>(smem + L::kOut) + half * CH * kBN, tid, half);
+          } else {
+            StoreColumn<CH>(p, t, n, t.m0 + c, a.M, v, bias);
+          }
         }
       }
       asm volatile("tcgen05.fence::before_thread_sync;\n" ::: "memory");
@@ -475,6 +513,7 @@ cudaError_t LaunchDenseGemmTc(const tlaloc_b200_dense_problem* problems, int cou
     p.n = s.n;
     p.act = s.act;
     p.y_f32 = s.y_dtype == TLALOC_B200_F32 ? 1 : 0;
+    p.rows_bf16 = !p.y_f32 && !s.residual && s.ld_y % 8 == 0 && (s.batch == 1 || s.batch_y % 8 == 0) && Aligned16(s.y) ? 1 : 0;
     p.tiles_n = (s.n + kBN - 1) / kBN;
     a.tiles += p.tiles_n * a.tiles_m * s.batch;
     if (i == 0) a.tiles0 = a.tiles;

@@ -28,6 +28,9 @@ from .rotary import Rotation, YarnScaling, pair_tables
 from .step_model import StepModel
 
 
+EXPAND_FROM = 32  # tokens of a portion from which the expanded way of attending pays
+
+
 # ---------------------------------------------------------------------------------------------- configuration
 
 @dataclass(frozen=True)
@@ -171,7 +174,11 @@ class LatentDecoder(StepModel):
         max_live = min(self.max_positions, cfg.window or self.max_positions)
         self._att_scratch = torch.empty((max(ops.latent_attention_scratch_bytes(R, m.heads, m.kv_rank, m.rot_dim, max_live) for m in mixers)
                                          // 4 + 4,), **f32)
+        self._expanded = [dtype == torch.bfloat16 and ops.window_attention_applies(m.dim, m.rot_dim, m.vdim) and m.row % 8 == 0
+                          and (m.heads * m.vdim) % 8 == 0 and m.scale > 0 for m in mixers]
+        self._expand_space: dict[str, torch.Tensor] = {}  # gathered latents, keys and values of a portion's window; grown on demand
         self.hn = torch.empty((R, cfg.width), **ty)
+        self._decode_uses: dict[int, int] = {}
         self.logits = torch.empty((max_sequences, cfg.vocab), **f32)
         self.next_ids = torch.zeros((max_sequences,), dtype=torch.int32, device=dev)
 
@@ -208,6 +215,8 @@ class LatentDecoder(StepModel):
             lw = {"norm1": g(t[p + "norm1"]) + 1.0, "low": torch.cat([w(t[p + "mix.dq"]), w(t[p + "mix.dkv"])]),
                   "q_gain": g(t[p + "mix.dq.norm"]), "kv_gain": g(t[p + "mix.dkv.norm"]), "uq": w(t[p + "mix.uq"]),
                   "uk_t": uk.transpose(1, 2).contiguous(), "uv": uv}
+            if self._expanded[i]:
+                lw["ukv"] = torch.cat([uk, uv], dim=1).reshape(m.heads * (m.dim + m.vdim), m.kv_rank)
             out = w(t[p + "mix.o"])
             if l.mlp is not None:
                 pad = torch.zeros((self.cfg.width, self._o_width(l) - m.heads * m.vdim), dtype=self.dtype, device=dev)
@@ -235,13 +244,14 @@ class LatentDecoder(StepModel):
 
     def weight_bytes(self) -> int:
         """Bytes of weights one step reads (a shared layer is read each time it runs)."""
-        n = sum(v.numel() * v.element_size() for lw in self.layers for v in lw.values())
+        n = sum(v.numel() * v.element_size() for lw in self.layers for k, v in lw.items() if k != "ukv")
         return n + self.embed.numel() * self.embed.element_size() + 4 * self.final_norm.numel()
 
     # ------------------------------------------------------------------ the step
 
-    def _layer(self, i: int, n: int) -> None:
-        """One layer over rows [0, n): normed inputs h1 (and h2) -> residual stream x."""
+    def _layer(self, i: int, n: int, spans) -> None:
+        """One layer over rows [0, n): normed inputs h1 (and h2) -> residual stream x.  spans: [(first row, end row, table row,
+        position of the first)], the rows of each sequence; None: one row per sequence."""
         l, lw, eps = self.cfg.layers[i], self.layers[i], self.cfg.eps
         m, pool, (cos, sin) = l.mixer, self.pools[i], self._rot[i]
         x, h1, h2 = self.x[:n], self.h1[:n], self.h2[:n]
@@ -259,7 +269,15 @@ class LatentDecoder(StepModel):
                             q_rank=m.q_rank, kv_rank=m.kv_rank, rot_dim=m.rot_dim, rot_dims=m.rot.dims)
         q = self._q[:n * m.heads * m.q_dim].view(n, m.heads, m.q_dim)
         ops.dense_gemm(ops.dense(cq, lw["uq"], q.view(n, -1)), weights_const=True)
-        self._attend_absorbed(i, 0, n, q, cat)
+        lo = 0  # rows [lo, first) are waiting for one absorbed call
+        for first, end, table, pos in spans or ():
+            if self._expanded[i] and end - first >= EXPAND_FROM:
+                if first > lo:
+                    self._attend_absorbed(i, lo, first, q, cat)
+                self._attend_expanded(i, first, end, table, pos, q, cat)
+                lo = end
+        if lo < n:
+            self._attend_absorbed(i, lo, n, q, cat)
         ops.dense_gemm(ops.dense(cat, lw["out"], x, bias=lw.get("down_b"), residual=x), weights_const=True)
 
     def _attend_absorbed(self, i: int, lo: int, hi: int, q: torch.Tensor, cat: torch.Tensor) -> None:
@@ -276,18 +294,40 @@ class LatentDecoder(StepModel):
         o = cat[lo:hi, :m.heads * m.vdim].view(n, m.heads, m.vdim)
         ops.dense_gemm(ops.dense(olat.transpose(0, 1), lw["uv"], o.transpose(0, 1)), weights_const=True)
 
+    def _space(self, name: str, rows: int, cols: int) -> torch.Tensor:
+        flat = self._expand_space.get(name)
+        if flat is None or flat.numel() < rows * cols:
+            flat = self._expand_space[name] = torch.empty((rows * cols,), dtype=self.dtype, device=self.device)
+        return flat[:rows * cols].view(rows, cols)
+
+    def _attend_expanded(self, i: int, lo: int, hi: int, table: int, pos: int, q: torch.Tensor, cat: torch.Tensor) -> None:
+        """Rows [lo, hi) of one sequence, positions pos .., over the per-head keys and values of its window."""
+        m, lw, (cos, sin) = self.cfg.layers[i].mixer, self.layers[i], self._rot[i]
+        first = max(0, pos - m.window + 1) if m.window else 0
+        keys = pos + hi - lo - first
+        lat = self._space("latents", keys, m.row)
+        ops.latent_gather(self.pools[i], self.block_tables[table], lat, first=first)
+        kv = self._space("keys and values", keys, m.heads * (m.dim + m.vdim))
+        ops.dense_gemm(ops.dense(lat[:, :m.kv_rank], lw["ukv"], kv), weights_const=True)
+        if m.rot_dim:
+            rotated = q[lo:hi, :, m.dim:]
+            ops.rope_interleaved(rotated, rotated, self.positions[lo:hi], cos, sin, rot_dims=m.rot.dims)
+        kv = kv.view(keys, m.heads, m.dim + m.vdim)
+        ops.window_attention(q[lo:hi], kv[:, :, :m.dim], lat[:, m.kv_rank:], kv[:, :, m.dim:], cat[lo:hi, :m.heads * m.vdim],
+                             first_query=pos - first, scale=m.scale, window=m.window or 0)
+
     def _norms(self, i: int, n: int) -> None:
         """The norms in front of layer i's branches."""
         lw = self.layers[i]
         ops.rmsnorm_pair(self.x[:n], lw["norm1"], self.h1[:n], self.cfg.eps, lw.get("norm2"), self.h2[:n] if "norm2" in lw else None)
 
-    def _hidden(self, n: int, trace: list | None = None) -> None:
+    def _hidden(self, n: int, spans=None, trace: list | None = None) -> None:
         """Embedding and layers over rows [0, n) of the step inputs; the residual stream stays in x.  trace: receives a copy
         of it after every layer."""
         ops.embedding(self.embed, self.token_ids[:n], out=self.x[:n])
         for i in range(len(self.layers)):
             self._norms(i, n)
-            self._layer(i, n)
+            self._layer(i, n, spans)
             if trace is not None:
                 trace.append(self.x[:n].clone())
 
@@ -306,10 +346,10 @@ class LatentDecoder(StepModel):
         n, s = step.token_ids.shape[0], step.block_tables.shape[0]
         if n > self.max_tokens or s > self.max_sequences:
             raise ValueError(f"a step of {n} tokens of {s} sequences; this model takes {self.max_tokens} of {self.max_sequences}")
-        for dst, src in ((self.token_ids, step.token_ids), (self.positions, step.positions), (self.seq_lens, step.seq_lens),
-                         (self.slot_mapping, step.slot_mapping), (self.row_tables, step.row_tables), (self.block_tables, step.block_tables)):
-            self._put(dst[:src.shape[0]], src)
-        self._hidden(n, trace)
+        if n == s and trace is None:
+            return self._run_decode(step, want)
+        self._inputs(step)
+        self._hidden(n, [(int(a), int(b), r, int(step.positions[a])) for r, (a, b) in enumerate(zip(step.starts[:-1], step.starts[1:]))], trace)
         out = []
         for k in range(0, len(want), self.max_sequences):
             rows = torch.as_tensor(np.asarray(want[k:k + self.max_sequences], np.int32), device=self.device)
@@ -317,3 +357,29 @@ class LatentDecoder(StepModel):
             if len(want) > self.max_sequences:
                 out[-1] = out[-1].clone()
         return torch.cat(out) if len(out) > 1 else out[0] if out else self.logits[:0]
+
+    def _inputs(self, step: RaggedStep) -> None:
+        for dst, src in ((self.token_ids, step.token_ids), (self.positions, step.positions), (self.seq_lens, step.seq_lens),
+                         (self.slot_mapping, step.slot_mapping), (self.row_tables, step.row_tables), (self.block_tables, step.block_tables)):
+            self._put(dst[:src.shape[0]], src)
+
+    def _run_decode(self, step: RaggedStep, want) -> torch.Tensor:
+        """One token of every sequence: the batch is padded to a power of two, and a size that comes up again is captured into a
+        CUDA graph (padding rows write nothing and attend over the padding page)."""
+        n = step.token_ids.shape[0]
+        rows = min(1 << (n - 1).bit_length(), self.max_sequences)
+        self.set_decode_inputs(*self._padded(step, rows))
+        self._decode_uses[rows] = self._decode_uses.get(rows, 0) + 1
+        if self._decode_uses[rows] == 3 and rows not in self._graphs:
+            self.capture(rows)
+        self.step(rows)
+        if list(want) == list(range(n)):
+            return self.logits[:n]
+        return self.logits[torch.as_tensor(want, dtype=torch.long, device=self.device)]
+
+    def set_decode_inputs(self, token_ids, positions, block_tables, seq_lens, slot_mapping) -> None:
+        """Inputs of a step of one token per sequence, as many as there are ids; row r uses block table r."""
+        rows = token_ids.shape[0]
+        for dst, src in ((self.token_ids, token_ids), (self.positions, positions), (self.block_tables, block_tables),
+                         (self.seq_lens, seq_lens), (self.slot_mapping, slot_mapping), (self.row_tables, np.arange(rows, dtype=np.int32))):
+            self._put(dst[:rows], src)

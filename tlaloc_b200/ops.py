@@ -337,3 +337,33 @@ def latent_attention(query, pool, block_tables, seq_lens, out, *, kv_rank, scale
         _ptr(query), _ptr(pool), ld, _dt(query), _ptr(block_tables), _ptr(row_tables), _ptr(seq_lens), _ptr(out), _ptr(scratch),
         0 if scratch is None else scratch.numel() * scratch.element_size(), T, H, kv_rank, row - kv_rank, P, bs, block_tables.shape[1],
         block_tables.shape[0], int(window), int(max_live), float(scale), _stream(query)))
+
+
+def latent_gather(pool, table, out, *, first) -> None:
+    """out [count, row] = the pool rows of positions first .. of the sequence whose block table is `table` [max_blocks]."""
+    _dev(pool, table, out)
+    if table.dtype != torch.int32 or table.dim() != 1 or pool.dim() != 3 or out.dtype != pool.dtype:
+        raise ValueError("LATENT_GATHER: pool [P, block, row], table i32 [max_blocks], out [count, row] of the pool's type")
+    P, bs, ld = pool.shape
+    N.check(N.lib().tlaloc_b200_latent_gather(_ptr(pool), ld, _dt(pool), _ptr(table), _ptr(out), out.shape[1], int(first), out.shape[0],
+                                              out.shape[1], P, bs, table.shape[0], _stream(pool)))
+
+
+def window_attention_applies(dim, rot_dim, vdim) -> bool:
+    return bool(N.lib().tlaloc_b200_window_attention_applies(dim, rot_dim, vdim))
+
+
+def window_attention(q, k, k_rot, v, out, *, first_query, scale, window=0) -> None:
+    """q bf16 [T, H, dim + rot] (contiguous, rotated) over k [L, H, dim], k_rot [L, rot] and v [L, H, vdim] (strided views) -> out
+    [T, H * vdim] (a strided view); query i is key first_query + i.  See include/tlaloc_b200.h."""
+    _dev(q)
+    T, H, qd = q.shape
+    L, _, dim = k.shape
+    vdim = v.shape[2]
+    rot = qd - dim
+    if any(t.dtype != torch.bfloat16 or not t.is_cuda or t.stride(-1) != 1 for t in (q, k, k_rot, v, out)):
+        raise ValueError("WINDOW_ATTENTION: bf16 CUDA tensors with dense rows")
+    if k.shape[1] != H or v.shape[:2] != k.shape[:2] or tuple(k_rot.shape) != (L, rot) or tuple(out.shape) != (T, H * vdim) or v.stride()[:2] != k.stride()[:2]:
+        raise ValueError(f"WINDOW_ATTENTION: q {tuple(q.shape)}, k {tuple(k.shape)}, k_rot {tuple(k_rot.shape)}, v {tuple(v.shape)}, out {tuple(out.shape)} do not fit")
+    N.check(N.lib().tlaloc_b200_window_attention(_ptr(q), _ptr(k), _ptr(k_rot), k_rot.stride(0), _ptr(v), k.stride(0), k.stride(1), _ptr(out),
+                                                 out.stride(0), T, L, int(first_query), H, dim, rot, vdim, int(window), float(scale), _stream(q)))
