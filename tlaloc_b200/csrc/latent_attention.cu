@@ -6,9 +6,9 @@
 // LatentAttentionMma (bf16): all heads share a position's row, so a CTA takes 16 to 64 heads of one row and a slice of its
 // positions, and the row leaves HBM once for all of them.  Tiles of 64 positions arrive by 16-byte cp.async copies, two tiles in shared
 // memory; both products run on mma.sync m16n8k16 (heads are the M rows) with f32 accumulators:
-//   scores   the channels are split over four warps (and the positions over two), so that a warp's share of the query stays in
-//            registers for the whole slice; the four partial sums meet in shared memory, where the softmax adds them
-//   values   the latent channels are split over the eight warps; the tile is read again, transposed, as it lies
+//   scores   the channels are split over eight warps (and the positions over two), so that a warp's share of the query stays in
+//            registers for the whole slice; the eight partial sums meet in shared memory, where the softmax adds them
+//   values   the latent channels are split over the sixteen warps; the tile is read again, transposed, as it lies
 // Slices leave {max, sum, acc[kv_rank]} records in f32 that LatentCombine merges in slice order.
 #include <algorithm>
 
@@ -25,7 +25,7 @@ struct LatentParams {
   const int* seq_lens;
   void* out;
   int64_t pool_ld;
-  int T, H, kv_rank, row, num_blocks, block_size, max_blocks, num_tables, window;
+  int T, H, kv_rank, row, num_blocks, block_size, block_shift, max_blocks, num_tables, window;  // block_shift: log2 of block_size, or -1
   float scale;
 };
 
@@ -44,8 +44,9 @@ __device__ __forceinline__ const int* TableOf(const LatentParams& p, int t)
 }
 __device__ __forceinline__ size_t PoolRow(const LatentParams& p, const int* table, int pos)
 {
-  const int page = min(max(__ldg(table + pos / p.block_size), 0), p.num_blocks - 1);
-  return (static_cast<size_t>(page) * p.block_size + pos % p.block_size) * p.pool_ld;
+  const int block = p.block_shift >= 0 ? pos >> p.block_shift : pos / p.block_size;
+  const int page = min(max(__ldg(table + block), 0), p.num_blocks - 1);
+  return (static_cast<size_t>(page) * p.block_size + (pos - block * p.block_size)) * p.pool_ld;
 }
 
 template <typename T>
@@ -108,7 +109,7 @@ __global__ void __launch_bounds__(kGenericThreads) LatentAttentionGeneric(Latent
 }
 
 // ---- the tensor-core form ---------------------------------------------------------------------------------------------
-constexpr int kMmaTile = 64, kMmaThreads = 256, kPStride = kMmaTile + 8, kPartStride = kMmaTile + 2;
+constexpr int kMmaTile = 64, kMmaThreads = 512, kGroups = 8, kPStride = kMmaTile + 8, kPartStride = kMmaTile + 2;
 
 __device__ __forceinline__ uint32_t SmemAddr(const void* ptr) { return static_cast<uint32_t>(__cvta_generic_to_shared(ptr)); }
 __device__ __forceinline__ void CpAsync16(uint32_t dst, const void* src, int src_bytes)
@@ -147,17 +148,17 @@ struct SliceParams {
   int slices, slice_tiles, row_bytes;  // row_bytes: a tile row in shared memory, an odd number of 16-byte words
 };
 
-// MT: 16-head tiles of the CTA; KSG: 16-channel steps of the scores per warp; NP: 16-channel pairs of values per warp.
+// kGroups warps split the channels of the scores.  MT: 16-head tiles of the CTA; KSG: 16-channel steps of the scores per warp; NP: 16-channel pairs of values per warp.
 template <int MT, int KSG, int NP>
-__global__ void __launch_bounds__(kMmaThreads) LatentAttentionMma(LatentParams p, SliceParams sp)
+__global__ void __launch_bounds__(kMmaThreads, 1) LatentAttentionMma(LatentParams p, SliceParams sp)
 {
   constexpr int HT = MT * 16;
-  constexpr int kPerHead = HT <= 16 ? 16 : HT <= 32 ? 8 : 4, kPos = kMmaTile / kPerHead;  // softmax: threads of a head, positions of a thread
+  constexpr int kPerHead = HT <= 16 ? 32 : HT <= 32 ? 16 : 8, kPos = kMmaTile / kPerHead;  // softmax: threads of a head, positions of a thread
   GridDependencySync();
   extern __shared__ __align__(16) unsigned char smem[];
   const int tile_bytes = kMmaTile * sp.row_bytes;
-  float* part = reinterpret_cast<float*>(smem + 2 * tile_bytes);                        // [4][HT][kPartStride]
-  __nv_bfloat16* s_p = reinterpret_cast<__nv_bfloat16*>(part + 4 * HT * kPartStride);   // [HT][kPStride]
+  float* part = reinterpret_cast<float*>(smem + 2 * tile_bytes);                        // [kGroups][HT][kPartStride]
+  __nv_bfloat16* s_p = reinterpret_cast<__nv_bfloat16*>(part + kGroups * HT * kPartStride);   // [HT][kPStride]
   float* s_keep = reinterpret_cast<float*>(s_p + HT * kPStride);                        // [HT]
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, gid = lane >> 2, tig = lane & 3;
   const int t = blockIdx.z, h0 = blockIdx.y * HT, slice = blockIdx.x;
@@ -170,9 +171,9 @@ __global__ void __launch_bounds__(kMmaThreads) LatentAttentionMma(LatentParams p
   const int words = p.row >> 3;  // 16-byte words of a row
   const int steps = (p.row + 15) >> 4;
 
-  // Four threads copy a position's row; positions outside the live range become zeros.  The row's place is looked up a tile
+  // Eight threads copy a position's row; positions outside the live range become zeros.  The row's place is looked up a tile
   // ahead, so that its latency is not in front of the copies.
-  const int my_row = tid >> 2;
+  const int my_row = tid >> 3;
   auto place = [&](int tile) {
     const int pos = tile * kMmaTile + my_row;
     return pos >= live.x && pos < live.y ? pool + PoolRow(p, table, pos) : nullptr;
@@ -182,7 +183,7 @@ __global__ void __launch_bounds__(kMmaThreads) LatentAttentionMma(LatentParams p
     const int bytes = src != nullptr ? 16 : 0;
     if (src == nullptr) src = pool;
 #pragma unroll 4
-    for (int w = tid & 3; w < words; w += 4) CpAsync16(dst + w * 16, src + w * 8, bytes);
+    for (int w = tid & 7; w < words; w += 8) CpAsync16(dst + w * 16, src + w * 8, bytes);
     asm volatile("cp.async.commit_group;\n" ::: "memory");
   };
   const __nv_bfloat16* next_row = nullptr;
@@ -195,8 +196,8 @@ __global__ void __launch_bounds__(kMmaThreads) LatentAttentionMma(LatentParams p
       *reinterpret_cast<uint4*>(smem + (i / kMmaTile) * tile_bytes + (i % kMmaTile) * sp.row_bytes + words * 16) = make_uint4(0, 0, 0, 0);
     }
   }
-  // The warp's share of the query: steps kg, kg + 4, ... of the channels, as A fragments.
-  const int kg = warp & 3, ph = warp >> 2;
+  // The warp's share of the query: steps kg, kg + kGroups, ... of the channels, as A fragments.
+  const int kg = warp % kGroups, ph = warp / kGroups;
   uint32_t q[KSG][MT][4];
   const __nv_bfloat16* query = static_cast<const __nv_bfloat16*>(p.query) + static_cast<size_t>(t) * p.H * p.row;
 #pragma unroll
@@ -205,7 +206,7 @@ __global__ void __launch_bounds__(kMmaThreads) LatentAttentionMma(LatentParams p
     for (int m = 0; m < MT; ++m) {
 #pragma unroll
       for (int e = 0; e < 4; ++e) {
-        const int h = h0 + m * 16 + gid + (e & 1) * 8, k = (kg + 4 * i) * 16 + tig * 2 + (e >> 1) * 8;
+        const int h = h0 + m * 16 + gid + (e & 1) * 8, k = (kg + kGroups * i) * 16 + tig * 2 + (e >> 1) * 8;
         q[i][m][e] = h < p.H && k < p.row ? *reinterpret_cast<const uint32_t*>(query + static_cast<size_t>(h) * p.row + k) : 0u;
       }
     }
@@ -231,39 +232,37 @@ __global__ void __launch_bounds__(kMmaThreads) LatentAttentionMma(LatentParams p
       if (tile + 2 < tile_end) next_row = place(tile + 2);
     }
     const uint32_t tile_addr = SmemAddr(smem) + stage * tile_bytes;
-    {
-      float s[MT][4][4];
+    // B fragments: matrices (positions 0-7, channels 0-7), (0-7, 8-15), (8-15, 0-7), (8-15, 8-15) of a 16-position group
+    const uint32_t row_addr = tile_addr + (ph * 32 + (lane & 7) + ((lane >> 4) << 3)) * sp.row_bytes + ((lane >> 3) & 1) * 16;
+    float* dst = part + kg * HT * kPartStride + ph * 32 + tig * 2;
+#pragma unroll
+    for (int g = 0; g < 2; ++g) {
+      float s[MT][2][4];
 #pragma unroll
       for (int m = 0; m < MT; ++m)
 #pragma unroll
-        for (int n = 0; n < 4; ++n)
+        for (int n = 0; n < 2; ++n)
 #pragma unroll
           for (int e = 0; e < 4; ++e) s[m][n][e] = 0.f;
-      // B fragments: matrices (positions 0-7, channels 0-7), (0-7, 8-15), (8-15, 0-7), (8-15, 8-15) of a 16-position group
-      const uint32_t row_addr = tile_addr + (ph * 32 + (lane & 7) + ((lane >> 4) << 3)) * sp.row_bytes + ((lane >> 3) & 1) * 16;
 #pragma unroll
       for (int i = 0; i < KSG; ++i) {
-        const int step = kg + 4 * i;
+        const int step = kg + kGroups * i;
         if (step < steps) {
+          uint32_t b[4];
+          LdMatrixX4(b, row_addr + g * 16 * sp.row_bytes + step * 32);
 #pragma unroll
-          for (int g = 0; g < 2; ++g) {
-            uint32_t b[4];
-            LdMatrixX4(b, row_addr + g * 16 * sp.row_bytes + step * 32);
-#pragma unroll
-            for (int m = 0; m < MT; ++m) {
-              MmaBf16(s[m][2 * g], q[i][m], b[0], b[1]);
-              MmaBf16(s[m][2 * g + 1], q[i][m], b[2], b[3]);
-            }
+          for (int m = 0; m < MT; ++m) {
+            MmaBf16(s[m][0], q[i][m], b[0], b[1]);
+            MmaBf16(s[m][1], q[i][m], b[2], b[3]);
           }
         }
       }
-      float* dst = part + kg * HT * kPartStride + ph * 32 + tig * 2;
 #pragma unroll
       for (int m = 0; m < MT; ++m)
 #pragma unroll
-        for (int n = 0; n < 4; ++n) {
-          *reinterpret_cast<float2*>(dst + (m * 16 + gid) * kPartStride + n * 8) = make_float2(s[m][n][0], s[m][n][1]);
-          *reinterpret_cast<float2*>(dst + (m * 16 + gid + 8) * kPartStride + n * 8) = make_float2(s[m][n][2], s[m][n][3]);
+        for (int n = 0; n < 2; ++n) {
+          *reinterpret_cast<float2*>(dst + (m * 16 + gid) * kPartStride + g * 16 + n * 8) = make_float2(s[m][n][0], s[m][n][1]);
+          *reinterpret_cast<float2*>(dst + (m * 16 + gid + 8) * kPartStride + g * 16 + n * 8) = make_float2(s[m][n][2], s[m][n][3]);
         }
     }
     __syncthreads();
@@ -273,10 +272,15 @@ __global__ void __launch_bounds__(kMmaThreads) LatentAttentionMma(LatentParams p
       for (int e = 0; e < kPos; e += 2) {
         const int at = s0 + e * kPerHead, pos = tile * kMmaTile + at;
         const float* src = part + sh * kPartStride + at;
-        const float2 a = *reinterpret_cast<const float2*>(src), b = *reinterpret_cast<const float2*>(src + HT * kPartStride);
-        const float2 c = *reinterpret_cast<const float2*>(src + 2 * HT * kPartStride), d = *reinterpret_cast<const float2*>(src + 3 * HT * kPartStride);
-        v[e] = pos >= live.x && pos < live.y ? ((a.x + b.x) + (c.x + d.x)) * scale : -INFINITY;
-        v[e + 1] = pos + 1 >= live.x && pos + 1 < live.y ? ((a.y + b.y) + (c.y + d.y)) * scale : -INFINITY;
+        float2 d = *reinterpret_cast<const float2*>(src);
+#pragma unroll
+        for (int k = 1; k < kGroups; ++k) {
+          const float2 more = *reinterpret_cast<const float2*>(src + k * HT * kPartStride);
+          d.x += more.x;
+          d.y += more.y;
+        }
+        v[e] = pos >= live.x && pos < live.y ? d.x * scale : -INFINITY;
+        v[e + 1] = pos + 1 >= live.x && pos + 1 < live.y ? d.y * scale : -INFINITY;
         tile_top = fmaxf(tile_top, fmaxf(v[e], v[e + 1]));
       }
 #pragma unroll
@@ -295,7 +299,6 @@ __global__ void __launch_bounds__(kMmaThreads) LatentAttentionMma(LatentParams p
       if (tid % kPerHead == 0) s_keep[sh] = keep;
     }
     __syncthreads();
-    uint32_t pf[4][MT][4];
 #pragma unroll
     for (int m = 0; m < MT; ++m) {
       const float k0 = s_keep[m * 16 + gid], k1 = s_keep[m * 16 + gid + 8];
@@ -306,24 +309,23 @@ __global__ void __launch_bounds__(kMmaThreads) LatentAttentionMma(LatentParams p
           acc[m][n][2] *= k1; acc[m][n][3] *= k1;
         }
       }
-#pragma unroll
-      for (int k = 0; k < 4; ++k) {  // matrices (heads 0-7, positions 0-7), (8-15, 0-7), (0-7, 8-15), (8-15, 8-15)
-        LdMatrixX4(pf[k][m], SmemAddr(s_p + (m * 16 + (lane & 15)) * kPStride + k * 16 + (lane >> 4) * 8));
-      }
     }
     const uint32_t v_addr = tile_addr + (lane & 15) * sp.row_bytes + (lane >> 4) * 16;
 #pragma unroll
-    for (int i = 0; i < NP; ++i) {
-      const int pair = warp + 8 * i;
-      if (pair < pairs) {
+    for (int k = 0; k < 4; ++k) {
+      uint32_t pf[MT][4];  // matrices (heads 0-7, positions 0-7), (8-15, 0-7), (0-7, 8-15), (8-15, 8-15)
 #pragma unroll
-        for (int k = 0; k < 4; ++k) {
+      for (int m = 0; m < MT; ++m) LdMatrixX4(pf[m], SmemAddr(s_p + (m * 16 + (lane & 15)) * kPStride + k * 16 + (lane >> 4) * 8));
+#pragma unroll
+      for (int i = 0; i < NP; ++i) {
+        const int pair = warp + 16 * i;
+        if (pair < pairs) {
           uint32_t b[4];  // (positions 0-7, channels 0-7), (8-15, 0-7), (0-7, 8-15), (8-15, 8-15), transposed
           LdMatrixX4Trans(b, v_addr + k * 16 * sp.row_bytes + pair * 32);
 #pragma unroll
           for (int m = 0; m < MT; ++m) {
-            MmaBf16(acc[m][2 * i], pf[k][m], b[0], b[1]);
-            MmaBf16(acc[m][2 * i + 1], pf[k][m], b[2], b[3]);
+            MmaBf16(acc[m][2 * i], pf[m], b[0], b[1]);
+            MmaBf16(acc[m][2 * i + 1], pf[m], b[2], b[3]);
           }
         }
       }
@@ -351,7 +353,7 @@ __global__ void __launch_bounds__(kMmaThreads) LatentAttentionMma(LatentParams p
       const float total = s_keep[m * 16 + gid + half * 8], inv = total > 0.f ? 1.f / total : 0.f;
 #pragma unroll
       for (int n = 0; n < 2 * NP; ++n) {
-        const int c = (warp + 8 * (n >> 1)) * 16 + (n & 1) * 8 + tig * 2;
+        const int c = (warp + 16 * (n >> 1)) * 16 + (n & 1) * 8 + tig * 2;
         if (c >= p.kv_rank) continue;
         const float a = acc[m][n][2 * half], b = acc[m][n][2 * half + 1];
         if (sp.records != nullptr) {
@@ -396,7 +398,7 @@ __global__ void __launch_bounds__(128) LatentCombine(LatentParams p, SliceParams
 int RowBytes(int row) { return ((2 * ((row + 15) / 16)) | 1) * 16; }
 size_t MmaSmem(int mt, int row)
 {
-  return 2 * static_cast<size_t>(kMmaTile) * RowBytes(row) + mt * 16 * (4 * kPartStride * sizeof(float) + kPStride * 2 + sizeof(float));
+  return 2 * static_cast<size_t>(kMmaTile) * RowBytes(row) + mt * 16 * (kGroups * kPartStride * sizeof(float) + kPStride * 2 + sizeof(float));
 }
 constexpr size_t kMmaMaxSmem = 227 * 1024;
 
@@ -448,7 +450,7 @@ cudaError_t LaunchMma(const LatentParams& p, const SliceParams& sp, cudaStream_t
 }
 
 #define TLALOC_LATENT_FORMS(X) \
-  X(1, 3, 1) X(2, 3, 1) X(3, 3, 1) X(4, 3, 1) X(1, 5, 2) X(2, 5, 2) X(3, 5, 2) X(4, 5, 2) X(1, 9, 4) X(2, 9, 4)
+  X(1, 3, 1) X(2, 3, 1) X(3, 3, 1) X(4, 3, 1) X(1, 5, 2) X(2, 5, 2)
 
 cudaError_t PrepareLatentAttention()
 {
@@ -466,7 +468,7 @@ KernelSetup g_setup(PrepareLatentAttention, nullptr);
 
 cudaError_t LaunchMmaForm(const LatentParams& p, const SliceParams& sp, cudaStream_t st)
 {
-  const int mt = HeadTiles(p.H, p.kv_rank), ksg = ((p.row + 15) / 16 + 3) / 4, np = ((p.kv_rank + 15) / 16 + 7) / 8;
+  const int mt = HeadTiles(p.H, p.kv_rank), ksg = ((p.row + 15) / 16 + kGroups - 1) / kGroups, np = ((p.kv_rank + 15) / 16 + 15) / 16;
 #define TLALOC_TRY(MT, KSG, NP) \
   if (mt == MT && ksg <= KSG && np <= NP) return LaunchMma<MT, KSG, NP>(p, sp, st);
   TLALOC_LATENT_FORMS(TLALOC_TRY)
@@ -536,6 +538,9 @@ extern "C" int tlaloc_b200_latent_attention(const void* query, const void* pool,
   p.row = kv_rank + rot_dim;
   p.num_blocks = num_blocks;
   p.block_size = block_size;
+  p.block_shift = -1;
+  for (int k = 0; k < 31; ++k)
+    if (block_size == 1 << k) p.block_shift = k;
   p.max_blocks = max_blocks;
   p.num_tables = num_tables;
   p.window = window;

@@ -109,7 +109,8 @@ __global__ void __launch_bounds__(kThreads, 1)
   volatile uint32_t* slot = slot_store;
   volatile uint32_t* abort_word = slot_store + 1;
   const uint32_t sk = a.qk_atoms * kAtom, sv = sk + a.k_stages * kAtom;  // offsets of the K and V rings, behind Q
-  const int v_tile = a.v_atoms * kAtom;
+  const int qk_atoms = a.qk_atoms, dim_atoms = a.dim_atoms, v_atoms = a.v_atoms, k_stages = a.k_stages, v_stages = a.v_stages;
+  const int v_tile = v_atoms * kAtom;
   const int m0 = blockIdx.x * kQ, head = blockIdx.y;
   const int q_last = min(m0 + kQ, a.T) - 1;
   const int tile_lo = a.window > 0 ? max(0, a.q0 + m0 - a.window + 1) / kKeys : 0;
@@ -143,35 +144,46 @@ __global__ void __launch_bounds__(kThreads, 1)
 
   if (warp == kSoftmaxWarps) {
     if (lane == 0) {
-      int kit = 0;
+      // Ring positions and phases are counted along: a division per box would take longer than the box.
+      int ks = 0, vs = 0;
+      uint32_t kphase = 1, vphase = 1;  // a fresh barrier passes a wait for the phase before its first
       auto load_k = [&](int j) {
-        for (int c = 0; c < a.qk_atoms; ++c, ++kit) {
-          const int s = kit % a.k_stages;
-          if (kit >= a.k_stages) ok = MbarWait(kempty + 8 * s, ((kit / a.k_stages) - 1) & 1, abort_word) && ok;
-          MbarExpectTx(kfull + 8 * s, kAtom);
-          const int key = (tile_lo + j) * kKeys;
-          if (c < a.dim_atoms) TmaBox(base + sk + s * kAtom, &map_k, c * 64, head, key, kfull + 8 * s);
-          else TmaBox(base + sk + s * kAtom, &map_rot, (c - a.dim_atoms) * 64, 0, key, kfull + 8 * s);
+        const int key = (tile_lo + j) * kKeys;
+        for (int c = 0; c < qk_atoms; ++c) {
+          const uint32_t bar = kfull + 8 * ks, dst = base + sk + ks * kAtom;
+          ok = MbarWait(kempty + 8 * ks, kphase, abort_word) && ok;
+          MbarExpectTx(bar, kAtom);
+          if (c < dim_atoms) TmaBox(dst, &map_k, c * 64, head, key, bar);
+          else TmaBox(dst, &map_rot, (c - dim_atoms) * 64, 0, key, bar);
+          if (++ks == k_stages) {
+            ks = 0;
+            kphase ^= 1;
+          }
         }
       };
-      MbarExpectTx(qfull, a.qk_atoms * kAtom);
-      for (int c = 0; c < a.qk_atoms; ++c) {
-        TmaBox(base + c * kAtom, &map_q, c < a.dim_atoms ? c * 64 : a.dim + (c - a.dim_atoms) * 64, head, m0, qfull);
+      MbarExpectTx(qfull, qk_atoms * kAtom);
+      for (int c = 0; c < qk_atoms; ++c) {
+        TmaBox(base + c * kAtom, &map_q, c < dim_atoms ? c * 64 : a.dim + (c - dim_atoms) * 64, head, m0, qfull);
       }
       load_k(0);
       for (int j = 0; j < tiles; ++j) {
         if (j + 1 < tiles) load_k(j + 1);
-        const int s = j % a.v_stages;
-        if (j >= a.v_stages) ok = MbarWait(vempty + 8 * s, ((j / a.v_stages) - 1) & 1, abort_word) && ok;
-        MbarExpectTx(vfull + 8 * s, v_tile);
-        for (int c = 0; c < a.v_atoms; ++c) TmaBox(base + sv + s * v_tile + c * kAtom, &map_v, c * 64, head, (tile_lo + j) * kKeys, vfull + 8 * s);
+        const uint32_t bar = vfull + 8 * vs;
+        ok = MbarWait(vempty + 8 * vs, vphase, abort_word) && ok;
+        MbarExpectTx(bar, v_tile);
+        for (int c = 0; c < v_atoms; ++c) TmaBox(base + sv + vs * v_tile + c * kAtom, &map_v, c * 64, head, (tile_lo + j) * kKeys, bar);
+        if (++vs == v_stages) {
+          vs = 0;
+          vphase ^= 1;
+        }
       }
       if (!ok) {  // given up: let the copies in flight land before the CTA's shared memory goes away
         volatile uint32_t never = 0;
-        for (int s = 0; s < a.k_stages; ++s)
-          if (kit > s) MbarWait(kfull + 8 * s, ((kit - 1 - s) / a.k_stages) & 1, &never);
-        for (int s = 0; s < a.v_stages; ++s)
-          if (tiles > s) MbarWait(vfull + 8 * s, ((tiles - 1 - s) / a.v_stages) & 1, &never);
+        const int k_boxes = tiles * qk_atoms;
+        for (int s = 0; s < k_stages; ++s)
+          if (k_boxes > s) MbarWait(kfull + 8 * s, ((k_boxes - 1 - s) / k_stages) & 1, &never);
+        for (int s = 0; s < v_stages; ++s)
+          if (tiles > s) MbarWait(vfull + 8 * s, ((tiles - 1 - s) / v_stages) & 1, &never);
       }
     }
     __syncwarp();
@@ -180,38 +192,51 @@ __global__ void __launch_bounds__(kThreads, 1)
       const uint32_t s_idesc = InstrDesc(kKeys, false), o_idesc = InstrDesc((a.vdim + 15) / 16 * 16, true);
       const uint64_t qd = SmemDesc(base, 16, 1024), kd = SmemDesc(base + sk, 16, 1024);
       const uint64_t vd = SmemDesc(base + sv, kAtom, 1024);
-      int kit = 0;
       ok = MbarWait(qfull, 0, abort_word) && ok;
+      int ks = 0, vs = 0;
+      uint32_t kphase = 0, vphase = 0;
       auto scores = [&](int j) {
-        const int b = j & 1;
+        const uint32_t b = j & 1, acc = tmem + b * 128;
         // The buffer held P(j - 2), whose product is in front of these MMAs in the same queue.
-        for (int c = 0; c < a.qk_atoms; ++c, ++kit) {
-          const int s = kit % a.k_stages;
-          ok = MbarWait(kfull + 8 * s, (kit / a.k_stages) & 1, abort_word) && ok;
+        uint64_t qa = qd;
+        for (int c = 0; c < qk_atoms; ++c, qa += kAtom >> 4) {
+          const int width = c < dim_atoms ? a.dim - 64 * c : a.rot - 64 * (c - dim_atoms);
+          const uint64_t ka = kd + static_cast<uint64_t>((ks * kAtom) >> 4);
+          ok = MbarWait(kfull + 8 * ks, kphase, abort_word) && ok;
           asm volatile("tcgen05.fence::after_thread_sync;\n" ::: "memory");
-          const int width = c < a.dim_atoms ? a.dim - 64 * c : a.rot - 64 * (c - a.dim_atoms);
-          const int steps = min(4, (width + 15) / 16);
-          const uint64_t qa = qd + ((c * kAtom) >> 4), ka = kd + ((s * kAtom) >> 4);
-          for (int k = 0; k < steps; ++k) Mma(tmem + b * 128, qa + 2 * k, ka + 2 * k, s_idesc, (c > 0 || k > 0) ? 1u : 0u);
-          TcCommit(kempty + 8 * s);
+          Mma(acc, qa, ka, s_idesc, c > 0 ? 1u : 0u);
+          if (width > 48) {
+#pragma unroll
+            for (int k = 1; k < 4; ++k) Mma(acc, qa + 2 * k, ka + 2 * k, s_idesc, 1u);
+          } else {
+            for (int k = 1; 16 * k < width; ++k) Mma(acc, qa + 2 * k, ka + 2 * k, s_idesc, 1u);
+          }
+          TcCommit(kempty + 8 * ks);
+          if (++ks == k_stages) {
+            ks = 0;
+            kphase ^= 1;
+          }
         }
         TcCommit(sfull + 8 * b);
       };
       scores(0);
       for (int j = 0; j < tiles; ++j) {
         if (j + 1 < tiles) scores(j + 1);
-        const int s = j % a.v_stages;
-        ok = MbarWait(vfull + 8 * s, (j / a.v_stages) & 1, abort_word) && ok;
+        const uint64_t va = vd + static_cast<uint64_t>((vs * v_tile) >> 4);
+        const uint32_t pa = tmem + (j & 1) * 128;
+        ok = MbarWait(vfull + 8 * vs, vphase, abort_word) && ok;
         ok = MbarWait(pfull, j & 1, abort_word) && ok;
         asm volatile("tcgen05.fence::after_thread_sync;\n" ::: "memory");
-        const uint64_t va = vd + ((s * v_tile) >> 4);
+        // P: eight columns per 16 keys; V: keys are its rows, 16 of them per step
+        MmaTmemA(tmem_o, pa, va, o_idesc, j > 0 ? 1u : 0u);
 #pragma unroll
-        for (int k = 0; k < kKeys / 16; ++k) {
-          // P: eight columns per 16 keys; V: keys are its rows, 16 of them per step
-          MmaTmemA(tmem_o, tmem + (j & 1) * 128 + 8 * k, va + ((k * 16 * 128) >> 4), o_idesc, (j > 0 || k > 0) ? 1u : 0u);
-        }
-        TcCommit(vempty + 8 * s);
+        for (int k = 1; k < kKeys / 16; ++k) MmaTmemA(tmem_o, pa + 8 * k, va + ((k * 16 * 128) >> 4), o_idesc, 1u);
+        TcCommit(vempty + 8 * vs);
         TcCommit(odone + 8 * (j & 1));
+        if (++vs == v_stages) {
+          vs = 0;
+          vphase ^= 1;
+        }
       }
     }
     __syncwarp();

@@ -71,8 +71,8 @@ class Scheduler:
         while self.waiting and rows > 0 and len(self.running) < self.max_sequences:
             r = self.waiting[0]
             n = self._fitting(r, rows)
-            if n < 1:
-                break
+            if n < 1 or (self.running and self._room(r) < r.pending):
+                break  # beside running requests one is admitted only if all of its tokens fit: it would soon be sent back
             r.seq.reserve(self.pool, n, self.block_size)
             self.waiting.popleft()
             self.running.append(r)
@@ -84,8 +84,10 @@ class Scheduler:
 
     def _fitting(self, r: Request, rows: int) -> int:
         """How many of the request's pending tokens the rows and the free pages take."""
-        room = (len(r.seq.pages) + self.pool.free_count) * self.block_size - r.seq.length
-        return min(r.pending, rows, room)
+        return min(r.pending, rows, self._room(r))
+
+    def _room(self, r: Request) -> int:
+        return (len(r.seq.pages) + self.pool.free_count) * self.block_size - r.seq.length
 
     def _preempt(self, r: Request) -> None:
         r.seq.release(self.pool)
