@@ -5,6 +5,7 @@ cache, on N B200s of one box (tensor parallel), plus the HBM roofline of its ker
     python -m torch.distributed.run --nnodes=1 --nproc-per-node N ... bench.py --gpus N ...
     python bench.py --impl reference --gpus 1 --steps 3 --warmup 1                  # the CPU restatement of the reference
     python bench.py --workload llama8b | paged_attn | int8_proj | peer_sum          # one configuration / operator alone
+    python bench.py --workload marotar                                              # the latent-attention decoder beside Llama
     python bench.py --timeline                                                      # per-kernel times inside one step
 
 One JSON line on stdout (rank 0).  A step is one decode step: one new token for every sequence of the batch.
@@ -45,6 +46,17 @@ WORKLOADS = {
                 64, (128, 4096), "llama3-8b-shape decode, int8 per-channel weights, bf16 paged KV block 16, batch 64, "
                                  "contexts U[128,4096]"),
 }
+# The latent-attention decoder at sizes of real models' layers, each beside a Llama of the same width, heads and feed-forward
+# parameters (the gated feed-forward has three matrices for this one's two), eight layers of each.
+MAROTAR = {
+    "width 4096": (dict(width=4096, heads=32, dim=128, rot_dim=64, vdim=128, q_rank=1536, kv_rank=512, ff=21504),
+                   dict(d_model=4096, num_heads=32, num_kv_heads=8, head_dim=128, ffn=14336)),
+    "width 2560": (dict(width=2560, heads=40, dim=64, rot_dim=32, vdim=64, q_rank=768, kv_rank=256, ff=9600),
+                   dict(d_model=2560, num_heads=20, num_kv_heads=5, head_dim=128, ffn=6400)),
+    "width 2048": (dict(width=2048, heads=16, dim=128, rot_dim=64, vdim=128, q_rank=768, kv_rank=512, ff=8256),
+                   dict(d_model=2048, num_heads=16, num_kv_heads=4, head_dim=128, ffn=5504)),
+}
+MAROTAR_LAYERS, MAROTAR_VOCAB, MAROTAR_WINDOW, MAROTAR_BATCH, MAROTAR_PROMPT = 8, 32768, 4096, 64, 8192
 METRIC, UNIT = "decode_tokens_per_s", "tokens/s"
 BS = 16  # KV block size
 
@@ -757,6 +769,209 @@ def operator_int8_projection(torch, dev, pk, only="") -> dict:
     return {"rows": rows, "hbm_gbs": pk["hbm_gbs"], "bf16_tflops": pk["bf16_tflops"], "peak_kind": pk["kind"]}
 
 
+def marotar_config(sizes: dict, layers: int = MAROTAR_LAYERS) -> dict:
+    """A config.json of the design at one of the bench's sizes."""
+    mixer = {k: sizes[k] for k in ("heads", "dim", "rot_dim", "vdim", "q_rank", "kv_rank")}
+    mixer.update(scale=(sizes["dim"] + sizes["rot_dim"]) ** -0.5, mask={"size": MAROTAR_WINDOW},
+                 rot={"base": 10000.0, "dims": sizes["rot_dim"], "scaling": {"factor": 4.0, "original": 4096, "fast": 32.0, "slow": 1.0}})
+    layer = {"type": "latent_attention", "mixer": mixer, "mlp": {"kind": "dense", "ff": sizes["ff"]}}
+    return {"architecture": "Marotar", "width": sizes["width"], "vocab": MAROTAR_VOCAB, "norm": {"eps": 1e-5}, "layers": [layer] * layers}
+
+
+def _stepped(torch, model, step_inputs, steps, warm=3):
+    """ms per step of CUDA-graph decode steps over fixed inputs."""
+    for _ in range(warm):
+        model.step(step_inputs)
+    a, b = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+    torch.cuda.synchronize()
+    a.record()
+    for _ in range(steps):
+        model.step(step_inputs)
+    b.record()
+    torch.cuda.synchronize()
+    return a.elapsed_time(b) / steps
+
+
+def _prefill(torch, model, tokens, portion):
+    """(ms of the whole prompt, ms of its last portion) through the engine's step function, portions of `portion` tokens."""
+    from tlaloc_b200.engine import Engine
+    from tlaloc_b200.paging import Sequence, stage_ragged
+
+    eng, best = Engine(model), None
+    for _ in range(3):
+        seq, events = Sequence(), []
+        for lo in range(0, len(tokens), portion):
+            part = tokens[lo:lo + portion]
+            assert seq.reserve(eng.pool, len(part), model.block_size)
+            step = stage_ragged([(seq, part)], max_blocks=model.max_blocks, block_size=model.block_size)
+            ev = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+            ev[0].record()
+            model.run(step, [len(part) - 1])
+            ev[1].record()
+            events.append(ev)
+            eng.scheduler.advance(seq, len(part))
+        torch.cuda.synchronize()
+        seq.release(eng.pool)
+        t = events[0][0].elapsed_time(events[-1][1]), events[-1][0].elapsed_time(events[-1][1])
+        best = t if best is None or t[0] < best[0] else best
+    return best
+
+
+def marotar_case(torch, dev, pk, sizes, llama, steps, local) -> dict:
+    """Decode (batch 64, contexts U[1024, 8192], window 4096) and prefill (one prompt of 8192) of both models, and the kernels of each
+    alone against their rooflines: HBM for a decode step's kernels, the bf16 rate for a portion's products and attention."""
+    from tlaloc_b200 import _native as N
+    from tlaloc_b200 import decoder as D
+    from tlaloc_b200 import ops, sharding
+    from tlaloc_b200.attrs import parse_paged_attention
+    from tlaloc_b200.latent_decoder import LatentDecoder, LatentDecoderConfig
+
+    rng = np.random.default_rng(11)
+    B, L = MAROTAR_BATCH, MAROTAR_LAYERS
+    lens = rng.integers(1024, 8193, size=B).astype(np.int64)
+    tokens = rng.integers(0, MAROTAR_VOCAB, size=MAROTAR_PROMPT).tolist()
+    max_len = 8192 + 64
+    out = {"sizes": dict(sizes, layers=L, vocab=MAROTAR_VOCAB, window=MAROTAR_WINDOW), "llama_sizes": dict(llama, layers=L, vocab=MAROTAR_VOCAB)}
+
+    def tables(block):
+        M = -(-max_len // block)
+        return (1 + np.random.default_rng(3).permutation(B * M)).reshape(B, M).astype(np.int32), 1 + B * M
+
+    # ---- the latent-attention decoder
+    cfg = LatentDecoderConfig.from_config(marotar_config(sizes))
+    tab, blocks = tables(cfg.block_size)
+    m = LatentDecoder(cfg, num_blocks=blocks, max_len=max_len, max_tokens=2048, max_sequences=B, device=dev)
+    m.init_random_weights(0)
+    for p in m.pools:
+        p.normal_()
+    x = cfg.layers[0].mixer
+    pos = lens.astype(np.int32)
+    m.set_decode_inputs(rng.integers(0, MAROTAR_VOCAB, size=B).astype(np.int32), pos, tab, pos + 1, sharding.slot_mapping(tab, pos, cfg.block_size))
+    m.capture(B)
+    with ClockSampler(local) as clocks:
+        ms = _stepped(torch, m, B, steps)
+    live = int(np.minimum(lens + 1, MAROTAR_WINDOW).sum())
+    step_bytes = m.weight_bytes() + 2 * live * x.row * L
+    out["decode"] = {"tokens_per_s": B / ms * 1e3, "ms_per_step": ms, "step_hbm_frac": step_bytes / ms / 1e6 / pk["hbm_gbs"], "clocks": clocks.summary()}
+    kernels = []
+
+    def time_kernel(name, calls, bytes_, flops, bound):
+        _, med = _time_graph(torch, lambda: [c() for c in calls], 10)
+        us = med / len(calls) * 1e3
+        frac = bytes_ / us / 1e3 / pk["hbm_gbs"] if bound == "hbm" else flops / us / 1e6 / pk["bf16_tflops"]
+        kernels.append({"kernel": name, "us": us, "bound": bound, "gbs": bytes_ / us / 1e3, "tflops": flops / us / 1e6, "frac": frac})
+
+    def copies(lws, key):
+        """That weight of every layer, repeated until the set is well past L2."""
+        ws = [lw[key] for lw in lws]
+        while sum(w.numel() * w.element_size() for w in ws) < 4e8:
+            ws = ws + [w.clone() for w in ws[:max(1, len(lws))]]
+        return ws
+
+    def project(name, key, rows, x_, y_, bound, **kw):
+        ws = copies(m.layers, key)
+        n = ws[0].numel()
+        byts = 2 * n + x_.numel() * 2 + y_.numel() * y_.element_size() * (2 if kw.get("residual") is not None else 1)
+        time_kernel(name, [lambda w=w: ops.dense_gemm(ops.dense(x_, w, y_, **kw), weights_const=True) for w in ws], byts, 2.0 * rows * n, bound)
+
+    def kernels_at(rows, bound):
+        lw, ow = m.layers[0], x.heads * x.vdim
+        bf = lambda *s: torch.randn(s, device=dev, dtype=torch.bfloat16)
+        h, low, cat = bf(rows, cfg.width), torch.empty((rows, x.q_rank + x.row), device=dev), bf(rows, ow + sizes["ff"])
+        q, qlat, olat, res = bf(rows, x.heads, x.q_dim), bf(rows, x.heads, x.row), bf(rows, x.heads, x.kv_rank), torch.randn((rows, cfg.width), device=dev)
+        ups, lows = copies(m.layers, "up"), copies(m.layers, "low")
+        n = ups[0].numel() + lows[0].numel()
+        time_kernel("down-projections + feed-forward up, one launch",
+                    [lambda a=a, b=b: ops.dense_gemm(ops.dense(h, a, low), ops.dense(h, b, cat[:, ow:], bias=lw["up_b"], act=N.ACT_RELU2), weights_const=True)
+                     for a, b in zip(lows, ups)], 2 * n + 4 * h.numel() + 4 * low.numel() + 2 * rows * sizes["ff"], 2.0 * rows * n, bound)
+        project("query up-projection", "uq", rows, bf(rows, x.q_rank), q.view(rows, -1), bound)
+        project("output + feed-forward down + residual", "out", rows, cat, res, bound, bias=lw["down_b"], residual=res)
+        if bound == "hbm":
+            project("query into latent space", "uk_t", rows, q[:, :, :x.dim].transpose(0, 1), qlat[:, :, :x.kv_rank].transpose(0, 1), bound)
+            project("value up-projection", "uv", rows, olat.transpose(0, 1), bf(rows, x.heads, x.vdim).transpose(0, 1), bound)
+            sl = torch.from_numpy(np.minimum(lens + 1, max_len).astype(np.int32)).to(dev)
+            time_kernel("latent attention over pages", [lambda p=p: ops.latent_attention(qlat, p, m.block_tables[:rows], sl, olat, kv_rank=x.kv_rank, scale=x.scale,
+                                                                                        window=MAROTAR_WINDOW, scratch=m._att_scratch) for p in m.pools],
+                        2 * live * x.row + 2 * (qlat.numel() + olat.numel()), 2.0 * live * x.heads * (x.row + x.kv_rank), bound)
+        else:
+            keys = rows + MAROTAR_WINDOW - 1
+            lat, kv = bf(keys, x.row), bf(keys, x.heads, x.dim + x.vdim)
+            ukv = copies(m.layers, "ukv")
+            time_kernel("keys and values of the window", [lambda w=w: ops.dense_gemm(ops.dense(lat[:, :x.kv_rank], w, kv.view(keys, -1)), weights_const=True) for w in ukv],
+                        2 * (ukv[0].numel() + lat.numel() + kv.numel()), 2.0 * keys * ukv[0].numel(), bound)
+            o = cat[:, :ow]
+            time_kernel("attention of the portion", [lambda: ops.window_attention(q, kv[:, :, :x.dim], lat[:, x.kv_rank:], kv[:, :, x.dim:], o, first_query=MAROTAR_WINDOW - 1,
+                                                                                scale=x.scale, window=MAROTAR_WINDOW)] * 4,
+                        2 * (q.numel() + kv.numel() + o.numel()), 2.0 * rows * MAROTAR_WINDOW * x.heads * (x.q_dim + x.vdim), bound)
+
+    kernels_at(B, "hbm")
+    out["decode"]["kernels"], kernels = kernels, []
+    whole, last = _prefill(torch, m, tokens, 2048)
+    out["prefill"] = {"tokens_per_s": MAROTAR_PROMPT / whole * 1e3, "ms": whole, "portion": 2048, "ms_last_portion": last,
+                      "tokens_per_s_last_portion": 2048 / last * 1e3}
+    kernels_at(2048, "tensor")
+    out["prefill"]["kernels"], kernels = kernels, []
+    out["device_status"] = N.lib().tlaloc_b200_device_status()
+    del m
+    gc.collect()
+    torch.cuda.empty_cache()
+
+    # ---- the closest model the framework had
+    lc = D.DecoderConfig(**llama, num_layers=L, vocab=MAROTAR_VOCAB, head_quant=True, max_positions=max_len)
+    tab, blocks = tables(lc.block_size)
+    d = D.Decoder(lc, B, blocks, tab.shape[1], device=dev)
+    d.init_random_weights(0)
+    for p in d.key_pools + d.value_pools:
+        p.normal_()
+    d.set_inputs(rng.integers(0, MAROTAR_VOCAB, size=B).astype(np.int32), pos, tab, pos + 1, sharding.slot_mapping(tab, pos, lc.block_size))
+    d.capture()
+    ms = _stepped(torch, d, B, steps)
+    sb = d.step_bytes(lens + 1)
+    out["llama_decode"] = {"tokens_per_s": B / ms * 1e3, "ms_per_step": ms, "step_hbm_frac": (sb["weights"] + sb["kv"]) / ms / 1e6 / pk["hbm_gbs"]}
+    for key, x_ in (("qkv", d.hn), ("o", d.att.view(B, -1)), ("gate_up", d.hn), ("down", d.act)):
+        ws = [lw[key] for lw in d.layers]
+        while sum(w[0].numel() for w in ws) < 4e8:
+            ws = ws + [tuple(t.clone() for t in w) for w in ws[:L]]
+        k_, n_ = ws[0][0].shape
+        y_ = torch.empty((B, n_), device=dev)
+        time_kernel(f"int8 projection {key}", [lambda w=w: ops.int8_gemm(x_, *w, out=y_, weights_const=True, scratch=d.proj_scratch, i8_mma=d.i8_mma) for w in ws],
+                    k_ * n_ + 4 * n_ + 2 * B * k_ + 4 * B * n_, 2.0 * B * k_ * n_, "hbm")
+    time_kernel("paged attention", [lambda l=l: ops.paged_attention(d.q_rot, d.key_pools[l], d.value_pools[l], d.block_tables, d.seq_lens, scale=lc.scale, out=d.att,
+                                                                     scratch=d.att_scratch) for l in range(L)],
+                sb["kv"] // L, 4.0 * int(lens.sum()) * lc.num_heads * lc.head_dim, "hbm")
+    out["llama_decode"]["kernels"], kernels = kernels, []
+    del d
+    gc.collect()
+    torch.cuda.empty_cache()
+    # Prefill there is the decode step with consecutive rows of one sequence, 128 at a time.
+    d = D.Decoder(lc, 128, 1 + tab.shape[1], tab.shape[1], device=dev)
+    d.init_random_weights(0)
+    d.capture()
+    whole, last = _prefill(torch, d, tokens, 128)
+    out["llama_prefill"] = {"tokens_per_s": MAROTAR_PROMPT / whole * 1e3, "ms": whole, "portion": 128, "ms_last_portion": last}
+    del d
+    gc.collect()
+    torch.cuda.empty_cache()
+    return out
+
+
+def run_marotar(args) -> dict:
+    import torch
+
+    local = int(os.environ.get("LOCAL_RANK", "0"))
+    dev = torch.device("cuda", local)
+    torch.cuda.set_device(dev)
+    pk = peaks()
+    names = [n for n in MAROTAR if not args.only or args.only in n]
+    cases = {n: marotar_case(torch, dev, pk, *MAROTAR[n], max(args.steps, 5), local) for n in names}
+    head = cases[names[0]]
+    return {"metric": "marotar_decode_tokens_per_s", "value": head["decode"]["tokens_per_s"], "unit": UNIT, "n_gpus": 1, "steps": max(args.steps, 5),
+            "warmup": 3, "ms_per_step": head["decode"]["ms_per_step"], "higher_is_better": True, "data": "synthetic", "dtype": "bf16",
+            "config": {"workload": f"{MAROTAR_LAYERS} layers of the latent-attention decoder at real models' layer sizes (random weights), batch {MAROTAR_BATCH}, "
+                                   f"contexts U[1024,8192], window {MAROTAR_WINDOW}; prefill of {MAROTAR_PROMPT} tokens; beside a Llama of equal size; weights "
+                                   "and pools of a timed set exceed L2", "peaks": pk, "cases": cases}}
+
+
 def run_operator(args) -> dict:
     """The two operators alone (single GPU)."""
     import torch
@@ -959,9 +1174,9 @@ def main() -> None:
     ap.add_argument("--steps", type=int, default=20)
     ap.add_argument("--warmup", type=int, default=3)
     ap.add_argument("--impl", default="ours", choices=["ours", "reference"])
-    ap.add_argument("--workload", default="llama70b", choices=sorted(WORKLOADS) + ["paged_attn", "int8_proj", "peer_sum"])
+    ap.add_argument("--workload", default="llama70b", choices=sorted(WORKLOADS) + ["paged_attn", "int8_proj", "peer_sum", "marotar"])
     ap.add_argument("--layers", type=int, default=0, help="override the layer count (debugging only; not a bench value)")
-    ap.add_argument("--only", default="", help="int8_proj: a single shape NxKxM")
+    ap.add_argument("--only", default="", help="int8_proj: a single shape NxKxM; marotar: a single size, e.g. 4096")
     ap.add_argument("--no-cpu", action="store_true", help="skip the CPU baseline leg")
     ap.add_argument("--lean", action="store_true", help="skip the projection roofline, the operator sweeps and the 8B-shape block")
     ap.add_argument("--timeline", action="store_true", help="per-kernel durations inside one graph replay of the step")
@@ -976,6 +1191,8 @@ def main() -> None:
         line = run_operator(args)
     elif args.workload == "peer_sum":
         line = run_peer_sum(args)
+    elif args.workload == "marotar":
+        line = run_marotar(args)
     else:
         line = run_ours(args)
     if line:

@@ -78,10 +78,6 @@ __device__ __forceinline__ void TmaBox3d(uint32_t dst, const CUtensorMap* map, i
       "l"(reinterpret_cast<uint64_t>(map)), "r"(x), "r"(y), "r"(z), "r"(bar), "l"(policy)
       : "memory");
 }
-__device__ __forceinline__ void MbarArrive(uint32_t bar)
-{
-  asm volatile("mbarrier.arrive.shared::cta.b64 _, [%0];\n" ::"r"(bar) : "memory");
-}
 __device__ __forceinline__ void TcLd16(uint32_t taddr, uint32_t* r)
 {
   asm volatile(

@@ -3,16 +3,24 @@
 // LatentAttentionGeneric: any sizes, f32 or bf16, plain FMA.  A CTA serves one (row, head): tiles of 128 positions, a warp
 // per position for the scores (lanes over the channels), an online softmax in f32, then a thread per latent channel.
 //
-// LatentAttentionMma (bf16): all heads share a position's row, so a CTA takes 16 to 64 heads of one row and a slice of its
-// positions, and the row leaves HBM once for all of them.  Tiles of 64 positions arrive by 16-byte cp.async copies, two tiles in shared
-// memory; both products run on mma.sync m16n8k16 (heads are the M rows) with f32 accumulators:
-//   scores   the channels are split over eight warps (and the positions over two), so that a warp's share of the query stays in
-//            registers for the whole slice; the eight partial sums meet in shared memory, where the softmax adds them
-//   values   the latent channels are split over the sixteen warps; the tile is read again, transposed, as it lies
-// Slices leave {max, sum, acc[kv_rank]} records in f32 that LatentCombine merges in slice order.
+// LatentAttentionTc (bf16, pages of a multiple of 64 positions): all heads share a position's row, so a CTA takes 16 to 64 heads of one
+// row of the batch and a slice of its positions, and the cached row leaves HBM once for all of them.  Tiles of 64 positions arrive as boxes of a
+// tensor map over the pool (atoms of 64 positions x 64 channels, 128-byte swizzle) in a ring of two to four stages.
+//   producer lane   boxes of the tiles
+//   MMA lane        scores: tcgen05.mma with the query as A out of TMEM (heads are its lanes, put there once) and the tile as B,
+//                   into one of two accumulators of 64 columns
+//   1 - 2 warps     softmax: a thread owns a head's row of 64 scores; the weights go to shared memory as bf16.  The running maximum is
+//                   raised lazily (the exponentials stay below 2^8), so the values' accumulators are rarely rescaled
+//   sixteen warps   values: mma.sync m16n8k16 over the tile as it lies, the latent channels split over the warps, accumulators
+//                   in registers (a TMEM accumulator of 512 channels would leave no room for the query)
+// Each of the four works on a tile of its own.  Slices leave {max, sum, acc[kv_rank]} records in f32 that LatentCombine merges in slice
+// order.  Every mbarrier wait is bounded.
+#include <cuda.h>
+
 #include <algorithm>
 
 #include "common.cuh"
+#include "tc_common.cuh"
 
 namespace tlaloc_b200 {
 namespace {
@@ -109,13 +117,13 @@ __global__ void __launch_bounds__(kGenericThreads) LatentAttentionGeneric(Latent
 }
 
 // ---- the tensor-core form ---------------------------------------------------------------------------------------------
-constexpr int kMmaTile = 64, kMmaThreads = 512, kGroups = 8, kPStride = kMmaTile + 8, kPartStride = kMmaTile + 2;
+using namespace tc;
 
-__device__ __forceinline__ uint32_t SmemAddr(const void* ptr) { return static_cast<uint32_t>(__cvta_generic_to_shared(ptr)); }
-__device__ __forceinline__ void CpAsync16(uint32_t dst, const void* src, int src_bytes)
-{
-  asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;\n" ::"r"(dst), "l"(src), "r"(src_bytes) : "memory");
-}
+constexpr int kAtomBytes = 64 * 128;
+constexpr int kMmaTile = 64, kValueWarps = 16, kSoftmaxWarps = 2;
+constexpr int kMmaThreads = (kValueWarps + kSoftmaxWarps + 2) * 32;
+constexpr int kPStride = kMmaTile + 8, kMaxStages = 4;
+
 __device__ __forceinline__ void LdMatrixX4(uint32_t (&r)[4], uint32_t addr)
 {
   asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];\n"
@@ -131,8 +139,7 @@ __device__ __forceinline__ void LdMatrixX4Trans(uint32_t (&r)[4], uint32_t addr)
 // Not volatile: the next fragments' loads may move ahead of it.
 __device__ __forceinline__ void MmaBf16(float (&c)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1)
 {
-  asm(
-      "mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};\n"
+  asm("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};\n"
       : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
       : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
 }
@@ -142,228 +149,310 @@ __device__ __forceinline__ float Exp2(float x)
   asm("ex2.approx.ftz.f32 %0, %1;\n" : "=f"(y) : "f"(x));
   return y;
 }
+__device__ __forceinline__ uint32_t Pack(float a, float b)
+{
+  const __nv_bfloat162 v = __floats2bfloat162_rn(a, b);
+  return *reinterpret_cast<const uint32_t*>(&v);
+}
 
 struct SliceParams {
   float* records;  // [slices][T][H][kv_rank + 2], or null: one slice, straight to out
-  int slices, slice_tiles, row_bytes;  // row_bytes: a tile row in shared memory, an odd number of 16-byte words
+  int slices, slice_tiles, atoms, stages;  // atoms: 64-channel atoms of a tile
 };
 
-// kGroups warps split the channels of the scores.  MT: 16-head tiles of the CTA; KSG: 16-channel steps of the scores per warp; NP: 16-channel pairs of values per warp.
-template <int MT, int KSG, int NP>
-__global__ void __launch_bounds__(kMmaThreads, 1) LatentAttentionMma(LatentParams p, SliceParams sp)
+__device__ int g_latent_status = 0;  // nonzero after a wait timed out (sticky until read)
+
+// A 16-byte word of a tile: 128-byte rows, the words of a row permuted by the row's place in its group of eight.
+__device__ __forceinline__ uint32_t TileWord(int position, int word)
+{
+  return (word >> 3) * kAtomBytes + position * 128 + (((word & 7) ^ (position & 7)) << 4);
+}
+constexpr float kLazy = 8.f;  // how far (log2) a head's maximum may grow past the reference in use
+
+// MT: 16-head tiles of the CTA; NP: 16-channel pairs of values per warp.
+template <int MT, int NP>
+__global__ void __launch_bounds__(kMmaThreads, 1)
+    LatentAttentionTc(const __grid_constant__ CUtensorMap map, const __grid_constant__ LatentParams p, const __grid_constant__ SliceParams sp)
 {
   constexpr int HT = MT * 16;
-  constexpr int kPerHead = HT <= 16 ? 32 : HT <= 32 ? 16 : 8, kPos = kMmaTile / kPerHead;  // softmax: threads of a head, positions of a thread
   GridDependencySync();
-  extern __shared__ __align__(16) unsigned char smem[];
-  const int tile_bytes = kMmaTile * sp.row_bytes;
-  float* part = reinterpret_cast<float*>(smem + 2 * tile_bytes);                        // [kGroups][HT][kPartStride]
-  __nv_bfloat16* s_p = reinterpret_cast<__nv_bfloat16*>(part + kGroups * HT * kPartStride);   // [HT][kPStride]
-  float* s_keep = reinterpret_cast<float*>(s_p + HT * kPStride);                        // [HT]
-  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, gid = lane >> 2, tig = lane & 3;
+  extern __shared__ unsigned char smem_raw[];
+  __shared__ alignas(8) uint64_t bars[2 * kMaxStages + 9];
+  __shared__ uint32_t slot_store[2];
+  __shared__ float s_keep[2][HT], s_total[HT];
+  __shared__ alignas(16) __nv_bfloat16 s_p[2][HT * kPStride];
+  const uint32_t base = (SmemAddr(smem_raw) + 1023u) & ~1023u;  // the swizzle is a function of address bits 4..9
+  unsigned char* smem = smem_raw + (base - SmemAddr(smem_raw));
+  const int tile_bytes = sp.atoms * kAtomBytes, stages = sp.stages;
+  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
   const int t = blockIdx.z, h0 = blockIdx.y * HT, slice = blockIdx.x;
   const int2 live = LiveRange(p, t);
   const int tile0 = live.x / kMmaTile + slice * sp.slice_tiles;
-  const int tile_end = min((live.y + kMmaTile - 1) / kMmaTile, tile0 + sp.slice_tiles);
-  if (tile0 >= tile_end && !(slice == 0 && sp.records == nullptr)) return;  // an empty slice writes nothing; an empty row writes zeros
-  const int* table = TableOf(p, t);
-  const __nv_bfloat16* pool = static_cast<const __nv_bfloat16*>(p.pool);
-  const int words = p.row >> 3;  // 16-byte words of a row
-  const int steps = (p.row + 15) >> 4;
-
-  // Eight threads copy a position's row; positions outside the live range become zeros.  The row's place is looked up a tile
-  // ahead, so that its latency is not in front of the copies.
-  const int my_row = tid >> 3;
-  auto place = [&](int tile) {
-    const int pos = tile * kMmaTile + my_row;
-    return pos >= live.x && pos < live.y ? pool + PoolRow(p, table, pos) : nullptr;
-  };
-  auto load = [&](const __nv_bfloat16* src, int stage) {
-    const uint32_t dst = SmemAddr(smem) + stage * tile_bytes + my_row * sp.row_bytes;
-    const int bytes = src != nullptr ? 16 : 0;
-    if (src == nullptr) src = pool;
-#pragma unroll 4
-    for (int w = tid & 7; w < words; w += 8) CpAsync16(dst + w * 16, src + w * 8, bytes);
-    asm volatile("cp.async.commit_group;\n" ::: "memory");
-  };
-  const __nv_bfloat16* next_row = nullptr;
-  if (tile0 < tile_end) {
-    load(place(tile0), 0);
-    if (tile0 + 1 < tile_end) next_row = place(tile0 + 1);
-  }
-  if (p.row & 8) {  // the last step's upper channels
-    for (int i = tid; i < 2 * kMmaTile; i += kMmaThreads) {
-      *reinterpret_cast<uint4*>(smem + (i / kMmaTile) * tile_bytes + (i % kMmaTile) * sp.row_bytes + words * 16) = make_uint4(0, 0, 0, 0);
+  const int n = min((live.y + kMmaTile - 1) / kMmaTile, tile0 + sp.slice_tiles) - tile0;  // tiles of this CTA
+  if (n <= 0) {  // an empty slice writes nothing; an empty row writes zeros
+    if (slice == 0 && sp.records == nullptr) {
+      __nv_bfloat16* out = static_cast<__nv_bfloat16*>(p.out) + (static_cast<size_t>(t) * p.H + h0) * p.kv_rank;
+      for (int i = tid; i < min(HT, p.H - h0) * p.kv_rank; i += kMmaThreads) out[i] = __float2bfloat16_rn(0.f);
     }
+    return;
   }
-  // The warp's share of the query: steps kg, kg + kGroups, ... of the channels, as A fragments.
-  const int kg = warp % kGroups, ph = warp / kGroups;
-  uint32_t q[KSG][MT][4];
-  const __nv_bfloat16* query = static_cast<const __nv_bfloat16*>(p.query) + static_cast<size_t>(t) * p.H * p.row;
-#pragma unroll
-  for (int i = 0; i < KSG; ++i) {
-#pragma unroll
-    for (int m = 0; m < MT; ++m) {
-#pragma unroll
-      for (int e = 0; e < 4; ++e) {
-        const int h = h0 + m * 16 + gid + (e & 1) * 8, k = (kg + kGroups * i) * 16 + tig * 2 + (e >> 1) * 8;
-        q[i][m][e] = h < p.H && k < p.row ? *reinterpret_cast<const uint32_t*>(query + static_cast<size_t>(h) * p.row + k) : 0u;
+  const uint32_t full = SmemAddr(bars), free0 = full + 8 * kMaxStages, sfull = free0 + 8 * kMaxStages, sempty = sfull + 16;
+  const uint32_t pfull = sempty + 16, pempty = pfull + 16, qready = pempty + 16;
+  volatile uint32_t* abort_word = slot_store + 1;
+  if (tid == 0) {
+    slot_store[1] = 0u;
+    for (int i = 0; i < kMaxStages; ++i) {
+      MbarInit(full + 8 * i, 1);
+      MbarInit(free0 + 8 * i, kValueWarps);
+    }
+    for (int i = 0; i < 2; ++i) {
+      MbarInit(sfull + 8 * i, 1);
+      MbarInit(sempty + 8 * i, (HT + 31) / 32);
+      MbarInit(pfull + 8 * i, (HT + 31) / 32);
+      MbarInit(pempty + 8 * i, kValueWarps);
+    }
+    MbarInit(qready, 4);
+    asm volatile("fence.mbarrier_init.release.cluster;\n" ::: "memory");
+  }
+  if (warp == 0) {
+    asm volatile("tcgen05.alloc.cta_group::1.sync.aligned.shared::cta.b32 [%0], %1;\n" ::"r"(SmemAddr(slot_store)), "r"(512u) : "memory");
+    asm volatile("tcgen05.relinquish_alloc_permit.cta_group::1.sync.aligned;\n" ::: "memory");
+  }
+  asm volatile("tcgen05.fence::before_thread_sync;\n" ::: "memory");
+  __syncthreads();
+  asm volatile("tcgen05.fence::after_thread_sync;\n" ::: "memory");
+  const uint32_t tmem = *static_cast<volatile uint32_t*>(slot_store), tmem_q = tmem + 2 * kMmaTile;  // two score accumulators, then the query
+  bool ok = true;
+
+  if (warp == kValueWarps + kSoftmaxWarps) {
+    if (lane == 0) {
+      const int* table = TableOf(p, t);
+      int stage = 0;
+      uint32_t phase = 1;  // a fresh barrier passes a wait for the phase before its first
+      for (int j = 0; j < n; ++j) {
+        const int pos = (tile0 + j) * kMmaTile, block = pos >> p.block_shift;  // the tile's 64 rows lie in one page
+        const int row = min(max(__ldg(table + block), 0), p.num_blocks - 1) * p.block_size + (pos - (block << p.block_shift));
+        const uint32_t bar = full + 8 * stage, dst = base + stage * tile_bytes;
+        ok = MbarWait(free0 + 8 * stage, phase, abort_word) && ok;
+        MbarExpectTx(bar, tile_bytes);
+        for (int c = 0; c < sp.atoms; ++c) {  // x = 64 c elements: a multiple of 128 bytes
+          asm volatile("cp.async.bulk.tensor.2d.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1, {%2, %3}], [%4];\n" ::"r"(dst + c * kAtomBytes),
+                       "l"(reinterpret_cast<uint64_t>(&map)), "r"(c * 64), "r"(row), "r"(bar)
+                       : "memory");
+        }
+        if (++stage == stages) {
+          stage = 0;
+          phase ^= 1;
+        }
+      }
+      if (!ok) {  // given up: let the copies in flight land before the CTA's shared memory goes away
+        volatile uint32_t never = 0;
+        for (int s = 0; s < stages; ++s)
+          if (n > s) MbarWait(full + 8 * s, ((n - 1 - s) / stages) & 1, &never);
       }
     }
-  }
-  float acc[MT][2 * NP][4];
+    __syncwarp();
+  } else if (warp == kValueWarps + kSoftmaxWarps + 1) {
+    if (lane == 0) {
+      // f32 accumulator, bf16, both K-major, M = 128 (the lanes past the heads hold zeros), N = 64
+      constexpr uint32_t idesc = (1u << 4) | (1u << 7) | (1u << 10) | (static_cast<uint32_t>(kMmaTile >> 3) << 17) | (8u << 24);
+      const uint64_t d0 = SmemDesc(base, 16, 1024);
+      const int steps = (p.row + 15) >> 4;
+      ok = MbarWait(qready, 0, abort_word) && ok;
+      int stage = 0;
+      uint32_t phase = 0;
+      for (int j = 0; j < n; ++j) {
+        const uint32_t b = j & 1, acc = tmem + b * kMmaTile;
+        ok = MbarWait(full + 8 * stage, phase, abort_word) && ok;
+        ok = MbarWait(sempty + 8 * b, ((j >> 1) & 1) ^ 1, abort_word) && ok;
+        asm volatile("tcgen05.fence::after_thread_sync;\n" ::: "memory");
+        uint64_t d = d0 + static_cast<uint64_t>((stage * tile_bytes) >> 4);
+        uint32_t q = tmem_q;
+        for (int c = 0; c < sp.atoms; ++c, d += kAtomBytes >> 4, q += 32) {
 #pragma unroll
-  for (int m = 0; m < MT; ++m)
-#pragma unroll
-    for (int n = 0; n < 2 * NP; ++n)
-#pragma unroll
-      for (int e = 0; e < 4; ++e) acc[m][n][e] = 0.f;
-  const int sh = tid / kPerHead, s0 = (tid % kPerHead) * 2;  // softmax: this thread's head and first pair of positions
-  const float scale = p.scale * 1.4426950408889634f;
-  float top = -INFINITY, sum = 0.f;
-  const int pairs = (p.kv_rank + 15) >> 4;
-
-  for (int tile = tile0; tile < tile_end; ++tile) {
-    const int stage = (tile - tile0) & 1;
-    asm volatile("cp.async.wait_group 0;\n" ::: "memory");
-    __syncthreads();  // the tile has landed and the tile before it has been read
-    if (tile + 1 < tile_end) {
-      load(next_row, stage ^ 1);
-      if (tile + 2 < tile_end) next_row = place(tile + 2);
+          for (int k = 0; k < 4; ++k)
+            if (4 * c + k < steps) TcMmaTmemA(acc, q + 8 * k, d + 2 * k, idesc, c > 0 || k > 0 ? 1u : 0u);
+        }
+        TcCommit(sfull + 8 * b);
+        if (++stage == stages) {
+          stage = 0;
+          phase ^= 1;
+        }
+      }
     }
-    const uint32_t tile_addr = SmemAddr(smem) + stage * tile_bytes;
-    // B fragments: matrices (positions 0-7, channels 0-7), (0-7, 8-15), (8-15, 0-7), (8-15, 8-15) of a 16-position group
-    const uint32_t row_addr = tile_addr + (ph * 32 + (lane & 7) + ((lane >> 4) << 3)) * sp.row_bytes + ((lane >> 3) & 1) * 16;
-    float* dst = part + kg * HT * kPartStride + ph * 32 + tig * 2;
+    __syncwarp();
+  } else if (warp >= kValueWarps) {
+    const int quad = warp - kValueWarps, head = quad * 32 + lane;  // TMEM lane; kValueWarps is a multiple of 4
+    const uint32_t lanes = static_cast<uint32_t>(quad * 32) << 16;
+    if (quad * 32 < HT) {
+      const float scale = p.scale * 1.4426950408889634f;
+      float top = -INFINITY, sum = 0.f;
+      for (int j = 0; j < n; ++j) {
+        const int b = j & 1, pos = (tile0 + j) * kMmaTile;
+        ok = MbarWaitWarp(sfull + 8 * b, (j >> 1) & 1, lane, abort_word) && ok;
+        asm volatile("tcgen05.fence::after_thread_sync;\n" ::: "memory");
+        uint32_t s[kMmaTile];
+        TcLd32(tmem + lanes + b * kMmaTile, s);
+        TcLd32(tmem + lanes + b * kMmaTile + 32, s + 32);
+        asm volatile("tcgen05.wait::ld.sync.aligned;\n" ::: "memory");
+        asm volatile("tcgen05.fence::before_thread_sync;\n" ::: "memory");
+        __syncwarp();
+        if (lane == 0) MbarArrive(sempty + 8 * b);
+        float t4[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
+        const bool edge = pos < live.x || pos + kMmaTile > live.y;
 #pragma unroll
-    for (int g = 0; g < 2; ++g) {
-      float s[MT][2][4];
+        for (int e = 0; e < kMmaTile; ++e) {
+          float v = __uint_as_float(s[e]) * scale;
+          if (edge && (pos + e < live.x || pos + e >= live.y)) v = -INFINITY;
+          s[e] = __float_as_uint(v);
+          t4[e & 3] = fmaxf(t4[e & 3], v);
+        }
+        const float tile_top = fmaxf(fmaxf(t4[0], t4[1]), fmaxf(t4[2], t4[3]));  // finite: a tile holds at least one live position
+        float keep = 1.f;
+        if (tile_top > top + kLazy || top == -INFINITY) {
+          const float next = fmaxf(top, tile_top);
+          keep = Exp2(top - next);
+          sum *= keep;
+          top = next;
+        }
+        float add[2] = {0.f, 0.f};
 #pragma unroll
-      for (int m = 0; m < MT; ++m)
+        for (int e = 0; e < kMmaTile; e += 2) {
+          const float p0 = Exp2(__uint_as_float(s[e]) - top), p1 = Exp2(__uint_as_float(s[e + 1]) - top);
+          add[0] += p0;
+          add[1] += p1;
+          s[e / 2] = Pack(p0, p1);
+        }
+        sum += add[0] + add[1];
+        ok = MbarWaitWarp(pempty + 8 * b, ((j >> 1) & 1) ^ 1, lane, abort_word) && ok;
+        if (head < HT) {
+          uint4* dst = reinterpret_cast<uint4*>(s_p[b] + head * kPStride);
 #pragma unroll
-        for (int n = 0; n < 2; ++n)
+          for (int c = 0; c < 8; ++c) dst[c] = make_uint4(s[4 * c], s[4 * c + 1], s[4 * c + 2], s[4 * c + 3]);
+          s_keep[b][head] = keep;
+          if (j == n - 1) {
+            s_total[head] = sum;
+            if (sp.records != nullptr && h0 + head < p.H) {
+              float* rec = sp.records + ((static_cast<size_t>(slice) * p.T + t) * p.H + h0 + head) * (p.kv_rank + 2);
+              rec[0] = top;
+              rec[1] = sum;
+            }
+          }
+        }
+        __syncwarp();
+        if (lane == 0) MbarArrive(pfull + 8 * b);
+      }
+    }
+  } else {
+    if (warp < 4) {  // the query into TMEM, zeros in the lanes past the heads
+      const int head = warp * 32 + lane;
+      const bool there = head < HT && h0 + head < p.H;
+      const uint32_t* q = reinterpret_cast<const uint32_t*>(static_cast<const __nv_bfloat16*>(p.query) + (static_cast<size_t>(t) * p.H + h0 + head) * p.row);
+      for (int c = 0; c < sp.atoms; ++c) {
+        uint32_t w[32];
 #pragma unroll
-          for (int e = 0; e < 4; ++e) s[m][n][e] = 0.f;
+        for (int e = 0; e < 32; ++e) w[e] = there && c * 64 + 2 * e < p.row ? __ldg(q + c * 32 + e) : 0u;
+        TcSt32(tmem_q + (static_cast<uint32_t>(warp * 32) << 16) + c * 32, w);
+      }
+      asm volatile("tcgen05.wait::st.sync.aligned;\n" ::: "memory");
+      asm volatile("tcgen05.fence::before_thread_sync;\n" ::: "memory");
+      __syncwarp();
+      if (lane == 0) MbarArrive(qready);
+    }
+    const int gid = lane >> 2, tig = lane & 3;
+    const int pairs = (p.kv_rank + 15) >> 4;
+    float acc[MT][2 * NP][4];
 #pragma unroll
-      for (int i = 0; i < KSG; ++i) {
-        const int step = kg + kGroups * i;
-        if (step < steps) {
-          uint32_t b[4];
-          LdMatrixX4(b, row_addr + g * 16 * sp.row_bytes + step * 32);
+    for (int m = 0; m < MT; ++m)
 #pragma unroll
-          for (int m = 0; m < MT; ++m) {
-            MmaBf16(s[m][0], q[i][m], b[0], b[1]);
-            MmaBf16(s[m][1], q[i][m], b[2], b[3]);
+      for (int c = 0; c < 2 * NP; ++c)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) acc[m][c][e] = 0.f;
+    int stage = 0;
+    uint32_t phase = 0;
+    for (int j = 0; j < n; ++j) {
+      const int b = j & 1, pos = (tile0 + j) * kMmaTile;
+      ok = MbarWaitWarp(full + 8 * stage, phase, lane, abort_word) && ok;
+      ok = MbarWaitWarp(pfull + 8 * b, (j >> 1) & 1, lane, abort_word) && ok;
+      const uint32_t tile_addr = base + stage * tile_bytes;
+      // Rows of the page outside the live range may hold anything: 0 times it must stay 0.
+      const int live_lo = live.x - pos, live_hi = live.y - pos;
+      if (live_lo > 0 || live_hi < kMmaTile) {
+        for (int i = tid; i < kMmaTile * sp.atoms * 8; i += kValueWarps * 32) {
+          const int r = i & (kMmaTile - 1);
+          if (r < live_lo || r >= live_hi) *reinterpret_cast<uint4*>(smem + stage * tile_bytes + TileWord(r, i / kMmaTile)) = make_uint4(0, 0, 0, 0);
+        }
+        asm volatile("fence.proxy.async.shared::cta;\n" ::: "memory");  // before the stage is fetched into again
+        asm volatile("bar.sync 1, %0;\n" ::"n"(kValueWarps * 32) : "memory");
+      }
+#pragma unroll
+      for (int m = 0; m < MT; ++m) {
+        const float k0 = s_keep[b][m * 16 + gid], k1 = s_keep[b][m * 16 + gid + 8];
+        if (__any_sync(0xffffffffu, k0 != 1.f || k1 != 1.f)) {
+#pragma unroll
+          for (int c = 0; c < 2 * NP; ++c) {
+            acc[m][c][0] *= k0; acc[m][c][1] *= k0;
+            acc[m][c][2] *= k1; acc[m][c][3] *= k1;
           }
         }
       }
 #pragma unroll
-      for (int m = 0; m < MT; ++m)
+      for (int k = 0; k < 4; ++k) {
+        uint32_t pf[MT][4];  // matrices (heads 0-7, positions 0-7), (8-15, 0-7), (0-7, 8-15), (8-15, 8-15)
 #pragma unroll
-        for (int n = 0; n < 2; ++n) {
-          *reinterpret_cast<float2*>(dst + (m * 16 + gid) * kPartStride + g * 16 + n * 8) = make_float2(s[m][n][0], s[m][n][1]);
-          *reinterpret_cast<float2*>(dst + (m * 16 + gid + 8) * kPartStride + g * 16 + n * 8) = make_float2(s[m][n][2], s[m][n][3]);
+        for (int m = 0; m < MT; ++m) LdMatrixX4(pf[m], SmemAddr(s_p[b] + (m * 16 + (lane & 15)) * kPStride + k * 16 + (lane >> 4) * 8));
+#pragma unroll
+        for (int i = 0; i < NP; ++i) {
+          const int pair = warp + kValueWarps * i;
+          if (pair < pairs) {
+            uint32_t v[4];  // (positions 0-7, channels 0-7), (8-15, 0-7), (0-7, 8-15), (8-15, 8-15), transposed
+            LdMatrixX4Trans(v, tile_addr + TileWord(k * 16 + (lane & 15), 2 * pair + (lane >> 4)));
+#pragma unroll
+            for (int m = 0; m < MT; ++m) {
+              MmaBf16(acc[m][2 * i], pf[m], v[0], v[1]);
+              MmaBf16(acc[m][2 * i + 1], pf[m], v[2], v[3]);
+            }
+          }
         }
-    }
-    __syncthreads();
-    if (sh < HT) {  // whole warps
-      float v[kPos], tile_top = -INFINITY;  // positions s0, s0 + 1, s0 + 2 kPerHead, ...
-#pragma unroll
-      for (int e = 0; e < kPos; e += 2) {
-        const int at = s0 + e * kPerHead, pos = tile * kMmaTile + at;
-        const float* src = part + sh * kPartStride + at;
-        float2 d = *reinterpret_cast<const float2*>(src);
-#pragma unroll
-        for (int k = 1; k < kGroups; ++k) {
-          const float2 more = *reinterpret_cast<const float2*>(src + k * HT * kPartStride);
-          d.x += more.x;
-          d.y += more.y;
-        }
-        v[e] = pos >= live.x && pos < live.y ? d.x * scale : -INFINITY;
-        v[e + 1] = pos + 1 >= live.x && pos + 1 < live.y ? d.y * scale : -INFINITY;
-        tile_top = fmaxf(tile_top, fmaxf(v[e], v[e + 1]));
       }
-#pragma unroll
-      for (int o = kPerHead / 2; o > 0; o >>= 1) tile_top = fmaxf(tile_top, __shfl_xor_sync(0xffffffffu, tile_top, o));
-      const float next = fmaxf(top, tile_top);  // finite: a tile holds at least one live position
-      const float keep = Exp2(top - next);
-      float add = 0.f;
-#pragma unroll
-      for (int e = 0; e < kPos; e += 2) {
-        const float p0 = Exp2(v[e] - next), p1 = Exp2(v[e + 1] - next);
-        add += p0 + p1;
-        *reinterpret_cast<__nv_bfloat162*>(s_p + sh * kPStride + s0 + e * kPerHead) = __floats2bfloat162_rn(p0, p1);
+      __syncwarp();
+      if (lane == 0) {
+        MbarArrive(pempty + 8 * b);
+        MbarArrive(free0 + 8 * stage);
       }
-      sum = sum * keep + add;
-      top = next;
-      if (tid % kPerHead == 0) s_keep[sh] = keep;
+      if (++stage == stages) {
+        stage = 0;
+        phase ^= 1;
+      }
     }
-    __syncthreads();
 #pragma unroll
     for (int m = 0; m < MT; ++m) {
-      const float k0 = s_keep[m * 16 + gid], k1 = s_keep[m * 16 + gid + 8];
-      if (__any_sync(0xffffffffu, k0 != 1.f || k1 != 1.f)) {
 #pragma unroll
-        for (int n = 0; n < 2 * NP; ++n) {
-          acc[m][n][0] *= k0; acc[m][n][1] *= k0;
-          acc[m][n][2] *= k1; acc[m][n][3] *= k1;
-        }
-      }
-    }
-    const uint32_t v_addr = tile_addr + (lane & 15) * sp.row_bytes + (lane >> 4) * 16;
+      for (int half = 0; half < 2; ++half) {
+        const int hl = m * 16 + gid + half * 8, h = h0 + hl;
+        if (h >= p.H) continue;
+        const float total = s_total[hl], inv = total > 0.f ? 1.f / total : 0.f;
 #pragma unroll
-    for (int k = 0; k < 4; ++k) {
-      uint32_t pf[MT][4];  // matrices (heads 0-7, positions 0-7), (8-15, 0-7), (0-7, 8-15), (8-15, 8-15)
-#pragma unroll
-      for (int m = 0; m < MT; ++m) LdMatrixX4(pf[m], SmemAddr(s_p + (m * 16 + (lane & 15)) * kPStride + k * 16 + (lane >> 4) * 8));
-#pragma unroll
-      for (int i = 0; i < NP; ++i) {
-        const int pair = warp + 16 * i;
-        if (pair < pairs) {
-          uint32_t b[4];  // (positions 0-7, channels 0-7), (8-15, 0-7), (0-7, 8-15), (8-15, 8-15), transposed
-          LdMatrixX4Trans(b, v_addr + k * 16 * sp.row_bytes + pair * 32);
-#pragma unroll
-          for (int m = 0; m < MT; ++m) {
-            MmaBf16(acc[m][2 * i], pf[m], b[0], b[1]);
-            MmaBf16(acc[m][2 * i + 1], pf[m], b[2], b[3]);
+        for (int c2 = 0; c2 < 2 * NP; ++c2) {
+          const int c = (warp + kValueWarps * (c2 >> 1)) * 16 + (c2 & 1) * 8 + tig * 2;
+          if (c >= p.kv_rank) continue;
+          const float x = acc[m][c2][2 * half], y = acc[m][c2][2 * half + 1];
+          if (sp.records != nullptr) {
+            *reinterpret_cast<float2*>(sp.records + ((static_cast<size_t>(slice) * p.T + t) * p.H + h) * (p.kv_rank + 2) + 2 + c) = make_float2(x, y);
+          } else {
+            *reinterpret_cast<__nv_bfloat162*>(static_cast<__nv_bfloat16*>(p.out) + (static_cast<size_t>(t) * p.H + h) * p.kv_rank + c) =
+                __floats2bfloat162_rn(x * inv, y * inv);
           }
         }
       }
     }
   }
-  // Sums of a head's threads, and its maximum, to everybody.
-#pragma unroll
-  for (int o = kPerHead / 2; o > 0; o >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, o);
+  if (!ok) atomicExch(&g_latent_status, 1);
+  asm volatile("tcgen05.fence::before_thread_sync;\n" ::: "memory");
   __syncthreads();
-  if (sh < HT && tid % kPerHead == 0) {
-    s_keep[sh] = sum;
-    if (sp.records != nullptr && h0 + sh < p.H) {
-      float* rec = sp.records + ((static_cast<size_t>(slice) * p.T + t) * p.H + h0 + sh) * (p.kv_rank + 2);
-      rec[0] = top;
-      rec[1] = sum;
-    }
-  }
-  __syncthreads();
-#pragma unroll
-  for (int m = 0; m < MT; ++m) {
-#pragma unroll
-    for (int half = 0; half < 2; ++half) {
-      const int h = h0 + m * 16 + gid + half * 8;
-      if (h >= p.H) continue;
-      const float total = s_keep[m * 16 + gid + half * 8], inv = total > 0.f ? 1.f / total : 0.f;
-#pragma unroll
-      for (int n = 0; n < 2 * NP; ++n) {
-        const int c = (warp + 16 * (n >> 1)) * 16 + (n & 1) * 8 + tig * 2;
-        if (c >= p.kv_rank) continue;
-        const float a = acc[m][n][2 * half], b = acc[m][n][2 * half + 1];
-        if (sp.records != nullptr) {
-          *reinterpret_cast<float2*>(sp.records + ((static_cast<size_t>(slice) * p.T + t) * p.H + h) * (p.kv_rank + 2) + 2 + c) = make_float2(a, b);
-        } else {
-          *reinterpret_cast<__nv_bfloat162*>(static_cast<__nv_bfloat16*>(p.out) + (static_cast<size_t>(t) * p.H + h) * p.kv_rank + c) =
-              __floats2bfloat162_rn(a * inv, b * inv);
-        }
-      }
-    }
+  if (warp == 0) {
+    asm volatile("tcgen05.fence::after_thread_sync;\n" ::: "memory");
+    asm volatile("tcgen05.dealloc.cta_group::1.sync.aligned.b32 %0, %1;\n" ::"r"(tmem), "r"(512u) : "memory");
   }
 }
 
@@ -395,12 +484,12 @@ __global__ void __launch_bounds__(128) LatentCombine(LatentParams p, SliceParams
   }
 }
 
-int RowBytes(int row) { return ((2 * ((row + 15) / 16)) | 1) * 16; }
-size_t MmaSmem(int mt, int row)
-{
-  return 2 * static_cast<size_t>(kMmaTile) * RowBytes(row) + mt * 16 * (kGroups * kPartStride * sizeof(float) + kPStride * 2 + sizeof(float));
-}
-constexpr size_t kMmaMaxSmem = 227 * 1024;
+constexpr int kMmaMaxSmem = 227 * 1024;
+
+int Atoms(int row) { return (row + 63) / 64; }
+// Stages beside the static shared memory (weights of up to 64 heads, barriers: under 20 KB).
+int Stages(int row) { return std::min(kMaxStages, (kMmaMaxSmem - 1024 - (Atoms(row) > 8 ? 10 : 20) * 1024) / (Atoms(row) * kAtomBytes)); }
+size_t MmaSmem(int row) { return 1024 + static_cast<size_t>(Stages(row)) * Atoms(row) * kAtomBytes; }
 
 // 16-head tiles of a CTA: enough for all heads where registers allow (two for latents wider than 256 channels, four up to that),
 // else the count that leaves the fewest absent heads.
@@ -417,16 +506,17 @@ int HeadTiles(int heads, int kv_rank)
 
 bool MmaApplies(int kv_rank, int rot_dim)
 {
-  return kv_rank % 8 == 0 && rot_dim % 8 == 0 && kv_rank <= 512 && (kv_rank + rot_dim + 15) / 16 <= 36 && (kv_rank > 256 || kv_rank + rot_dim <= 320);
+  const int row = kv_rank + rot_dim;
+  return kv_rank % 8 == 0 && rot_dim % 8 == 0 && kv_rank <= 512 && Atoms(row) * 32 + 2 * kMmaTile <= 512 && Stages(row) >= 2;
 }
 
 // Slices of the positions: the fewest waves of CTAs times the tiles a CTA walks, for the longest live range a row may have.
-int ChooseLatentSlices(int rows, int heads, int kv_rank, int row, int max_live, int* slice_tiles)
+int ChooseLatentSlices(int rows, int heads, int kv_rank, int max_live, int* slice_tiles)
 {
   const int tiles = (max_live + kMmaTile - 1) / kMmaTile + 1;
   const int mt = HeadTiles(heads, kv_rank);
   const int ctas = rows * ((heads + 16 * mt - 1) / (16 * mt));
-  const int slots = 148 * std::max(1, std::min<int>(4, static_cast<int>(kMmaMaxSmem / MmaSmem(mt, row))));
+  const int slots = 148;  // a CTA's TMEM and shared memory fill its SM
   int best = 1;
   double best_cost = 1e30;
   for (int s = 1; s <= std::min(tiles, 32); ++s) {
@@ -442,35 +532,63 @@ int ChooseLatentSlices(int rows, int heads, int kv_rank, int row, int max_live, 
   return (tiles + *slice_tiles - 1) / *slice_tiles;
 }
 
-template <int MT, int KSG, int NP>
-cudaError_t LaunchMma(const LatentParams& p, const SliceParams& sp, cudaStream_t st)
+using EncodeTiledFn = CUresult (*)(CUtensorMap*, CUtensorMapDataType, cuuint32_t, void*, const cuuint64_t*, const cuuint64_t*,
+                                   const cuuint32_t*, const cuuint32_t*, CUtensorMapInterleave, CUtensorMapSwizzle,
+                                   CUtensorMapL2promotion, CUtensorMapFloatOOBfill);
+
+// The pool as rows of `row` bf16 channels, boxes of 64 channels x 64 rows; channels past the row arrive as zeros.
+bool EncodePool(CUtensorMap* map, const LatentParams& p)
 {
-  const dim3 grid(sp.slices, (p.H + 16 * MT - 1) / (16 * MT), p.T);
-  return LaunchChained(LatentAttentionMma<MT, KSG, NP>, grid, kMmaThreads, MmaSmem(MT, p.row), st, p, sp);
+  auto encode = reinterpret_cast<EncodeTiledFn>(TensorMapEncoder());
+  if (encode == nullptr || p.block_shift < 6) return false;
+  const cuuint64_t dims[2] = {static_cast<cuuint64_t>(p.row), static_cast<cuuint64_t>(p.num_blocks) * p.block_size};
+  const cuuint64_t strides[1] = {static_cast<cuuint64_t>(p.pool_ld) * 2};
+  const cuuint32_t box[2] = {64, kMmaTile};
+  const cuuint32_t elem[2] = {1, 1};
+  return encode(map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, const_cast<void*>(p.pool), dims, strides, box, elem, CU_TENSOR_MAP_INTERLEAVE_NONE,
+                CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE) == CUDA_SUCCESS;
 }
 
-#define TLALOC_LATENT_FORMS(X) \
-  X(1, 3, 1) X(2, 3, 1) X(3, 3, 1) X(4, 3, 1) X(1, 5, 2) X(2, 5, 2)
+template <int MT, int NP>
+cudaError_t LaunchTc(const CUtensorMap& map, const LatentParams& p, const SliceParams& sp, cudaStream_t st)
+{
+  const dim3 grid(sp.slices, (p.H + 16 * MT - 1) / (16 * MT), p.T);
+  return LaunchChained(LatentAttentionTc<MT, NP>, grid, kMmaThreads, MmaSmem(p.row), st, map, p, sp);
+}
+
+#define TLALOC_LATENT_FORMS(X) X(1, 1) X(2, 1) X(3, 1) X(4, 1) X(1, 2) X(2, 2)
 
 cudaError_t PrepareLatentAttention()
 {
   static OncePerDevice once;
   return once.Run([](int) {
+    TensorMapEncoder();
     cudaError_t e = cudaSuccess;
-#define TLALOC_OPT_IN(MT, KSG, NP) \
-  if (e == cudaSuccess) e = cudaFuncSetAttribute(LatentAttentionMma<MT, KSG, NP>, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(kMmaMaxSmem));
+    const int most = static_cast<int>(std::max({MmaSmem(640), MmaSmem(576), MmaSmem(512), MmaSmem(448), MmaSmem(384), MmaSmem(320), MmaSmem(256), MmaSmem(192)}));
+#define TLALOC_OPT_IN(MT, NP) \
+  if (e == cudaSuccess) e = cudaFuncSetAttribute(LatentAttentionTc<MT, NP>, cudaFuncAttributeMaxDynamicSharedMemorySize, std::min(most, kMmaMaxSmem - (MT > 2 ? 20 : 10) * 1024));
     TLALOC_LATENT_FORMS(TLALOC_OPT_IN)
 #undef TLALOC_OPT_IN
     return e;
   });
 }
-KernelSetup g_setup(PrepareLatentAttention, nullptr);
-
-cudaError_t LaunchMmaForm(const LatentParams& p, const SliceParams& sp, cudaStream_t st)
+int ReadLatentStatus()
 {
-  const int mt = HeadTiles(p.H, p.kv_rank), ksg = ((p.row + 15) / 16 + kGroups - 1) / kGroups, np = ((p.kv_rank + 15) / 16 + 15) / 16;
-#define TLALOC_TRY(MT, KSG, NP) \
-  if (mt == MT && ksg <= KSG && np <= NP) return LaunchMma<MT, KSG, NP>(p, sp, st);
+  int v = 0;
+  if (cudaMemcpyFromSymbol(&v, g_latent_status, sizeof(int)) != cudaSuccess) return -1;
+  if (v != 0) {
+    const int zero = 0;
+    cudaMemcpyToSymbol(g_latent_status, &zero, sizeof(int));
+  }
+  return v;
+}
+KernelSetup g_setup(PrepareLatentAttention, ReadLatentStatus);
+
+cudaError_t LaunchTcForm(const CUtensorMap& map, const LatentParams& p, const SliceParams& sp, cudaStream_t st)
+{
+  const int mt = HeadTiles(p.H, p.kv_rank), np = ((p.kv_rank + 15) / 16 + kValueWarps - 1) / kValueWarps;
+#define TLALOC_TRY(MT, NP) \
+  if (mt == MT && np <= NP) return LaunchTc<MT, NP>(map, p, sp, st);
   TLALOC_LATENT_FORMS(TLALOC_TRY)
 #undef TLALOC_TRY
   return cudaErrorInvalidValue;
@@ -497,7 +615,7 @@ extern "C" size_t tlaloc_b200_latent_attention_scratch_bytes(int32_t num_tokens,
   size_t most = 0;
   for (int rows = 1;; rows = std::min(2 * rows, num_tokens)) {
     int tiles = 0;
-    const int s = ChooseLatentSlices(rows, num_heads, kv_rank, kv_rank + rot_dim, max_live, &tiles);
+    const int s = ChooseLatentSlices(rows, num_heads, kv_rank, max_live, &tiles);
     if (s > 1) most = std::max(most, static_cast<size_t>(s) * std::min(2 * rows, num_tokens) * num_heads * (kv_rank + 2) * sizeof(float));
     if (rows == num_tokens) break;
   }
@@ -546,13 +664,14 @@ extern "C" int tlaloc_b200_latent_attention(const void* query, const void* pool,
   p.window = window;
   p.scale = scale;
   cudaStream_t st = static_cast<cudaStream_t>(stream);
+  CUtensorMap map;
   if (dtype == TLALOC_B200_BF16 && !OrderFaithful() && MmaApplies(kv_rank, rot_dim) && pool_ld % 8 == 0 && Aligned16(query) && Aligned16(pool) &&
-      Aligned16(out) && (scratch == nullptr || Aligned16(scratch))) {
+      Aligned16(out) && (scratch == nullptr || Aligned16(scratch)) && EncodePool(&map, p)) {
     cudaError_t e = PrepareLatentAttention();
     if (e != cudaSuccess) return CudaFail("LATENT_ATTENTION set-up", e);
     SliceParams sp;
     const int live = MaxLive(max_live, window, static_cast<int64_t>(max_blocks) * block_size);
-    sp.slices = ChooseLatentSlices(num_tokens, num_heads, kv_rank, p.row, live, &sp.slice_tiles);
+    sp.slices = ChooseLatentSlices(num_tokens, num_heads, kv_rank, live, &sp.slice_tiles);
     const size_t need = static_cast<size_t>(sp.slices) * num_tokens * num_heads * (kv_rank + 2) * sizeof(float);
     if (sp.slices > 1 && (scratch == nullptr || scratch_bytes < need)) {
       sp.slices = 1;
@@ -560,8 +679,9 @@ extern "C" int tlaloc_b200_latent_attention(const void* query, const void* pool,
     }
     if (sp.slices == 1) sp.slice_tiles = 0x3fffffff;
     sp.records = sp.slices > 1 ? static_cast<float*>(scratch) : nullptr;
-    sp.row_bytes = RowBytes(p.row);
-    e = LaunchMmaForm(p, sp, st);
+    sp.atoms = Atoms(p.row);
+    sp.stages = Stages(p.row);
+    e = LaunchTcForm(map, p, sp, st);
     if (e == cudaSuccess && sp.slices > 1) e = LaunchChained(LatentCombine, dim3(num_heads, num_tokens), 128, 0, st, p, sp);
     if (e != cudaSuccess) return CudaFail("LATENT_ATTENTION launch", e);
     CountLaunches(sp.slices > 1 ? 2 : 1);
