@@ -208,7 +208,7 @@ __global__ void __launch_bounds__(kThreads, 1)
   bool ok = true;
 
   if (warp == kEpiWarps) {
-    if (lane == 0) {
+    if (ElectOne()) {
       uint64_t w_policy, x_policy;
       if (a.tiles_m == 1) asm volatile("createpolicy.fractional.L2::evict_first.b64 %0, 1.0;\n" : "=l"(w_policy));
       else asm volatile("createpolicy.fractional.L2::evict_normal.b64 %0, 1.0;\n" : "=l"(w_policy));
@@ -255,7 +255,7 @@ __global__ void __launch_bounds__(kThreads, 1)
     __syncwarp();
   } else if (warp == kEpiWarps + 1) {
     GridDependencySync();  // nothing to read, but the time limit of its waits then starts with the work
-    if (lane == 0) {
+    if (ElectOne()) {
       constexpr uint32_t idesc = InstrDescBf16(BT);
       const uint64_t wd0 = SmemDesc(base, 16, 1024), xd0 = SmemDesc(base + kWBytes, 16, 1024);
       int it = 0, lt = 0;

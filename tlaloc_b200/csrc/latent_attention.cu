@@ -225,7 +225,7 @@ __global__ void __launch_bounds__(kMmaThreads, 1)
   bool ok = true;
 
   if (warp == kValueWarps + kSoftmaxWarps) {
-    if (lane == 0) {
+    if (ElectOne()) {
       const int* table = TableOf(p, t);
       int stage = 0;
       uint32_t phase = 1;  // a fresh barrier passes a wait for the phase before its first
@@ -253,7 +253,7 @@ __global__ void __launch_bounds__(kMmaThreads, 1)
     }
     __syncwarp();
   } else if (warp == kValueWarps + kSoftmaxWarps + 1) {
-    if (lane == 0) {
+    if (ElectOne()) {
       // f32 accumulator, bf16, both K-major, M = 128 (the lanes past the heads hold zeros), N = 64
       constexpr uint32_t idesc = (1u << 4) | (1u << 7) | (1u << 10) | (static_cast<uint32_t>(kMmaTile >> 3) << 17) | (8u << 24);
       const uint64_t d0 = SmemDesc(base, 16, 1024);

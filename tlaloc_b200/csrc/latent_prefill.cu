@@ -26,7 +26,6 @@ constexpr int kQ = 128, kKeys = 128;           // queries of a CTA, keys of a ti
 constexpr int kAtom = kQ * 64 * 2;             // 128 rows x 64 channels
 constexpr int kSoftmaxWarps = 8;
 constexpr int kThreads = kSoftmaxWarps * 32 + 64;
-constexpr int kMaxKStages = 8;
 constexpr int kMaxSmem = 227 * 1024;
 
 struct WindowArgs {
@@ -77,32 +76,29 @@ __global__ void __launch_bounds__(kThreads, 1)
                       const __grid_constant__ CUtensorMap map_rot, const __grid_constant__ CUtensorMap map_v, const __grid_constant__ WindowArgs a)
 {
   extern __shared__ unsigned char smem_raw[];
-  __shared__ alignas(8) uint64_t bars[2 * kMaxKStages + 4 + 1 + 2 + 1 + 2];
+  __shared__ alignas(8) uint64_t bars[2 + 2 + 1 + 2 + 1 + 2];
   __shared__ uint32_t slot_store[2];
   __shared__ float s_row[2][2][kQ];  // [tile parity][half of the keys][query]
   const uint32_t base = (SmemAddr(smem_raw) + 1023u) & ~1023u;
   unsigned char* smem = smem_raw + (base - SmemAddr(smem_raw));
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
-  const uint32_t kfull = SmemAddr(bars), kempty = kfull + 8 * kMaxKStages, vfull = kempty + 8 * kMaxKStages, vempty = vfull + 16;
-  const uint32_t qfull = vempty + 16, sfull = qfull + 8, pfull = sfull + 16, odone = pfull + 8;
+  // Of the tiles in the rings: kfull, vfull "landed"; a K stage is free again when the scores of its tile are there (sfull), a V stage
+  // when its product is (odone).
+  const uint32_t kfull = SmemAddr(bars), vfull = kfull + 16, qfull = vfull + 16, sfull = qfull + 8, pfull = sfull + 16, odone = pfull + 8;
   volatile uint32_t* slot = slot_store;
   volatile uint32_t* abort_word = slot_store + 1;
-  const uint32_t sk = a.qk_atoms * kAtom, sv = sk + a.k_stages * kAtom;  // offsets of the K and V rings, behind Q
+  const uint32_t sk = a.qk_atoms * kAtom, sv = sk + a.k_stages * a.qk_atoms * kAtom;  // offsets of the K and V rings, behind Q
   const int qk_atoms = a.qk_atoms, dim_atoms = a.dim_atoms, v_atoms = a.v_atoms, k_stages = a.k_stages, v_stages = a.v_stages;
-  const int v_tile = v_atoms * kAtom;
+  const int v_tile = v_atoms * kAtom, k_tile = qk_atoms * kAtom;
   const int m0 = blockIdx.x * kQ, head = blockIdx.y;
   const int q_last = min(m0 + kQ, a.T) - 1;
   const int tile_lo = a.window > 0 ? max(0, a.q0 + m0 - a.window + 1) / kKeys : 0;
   const int tiles = min(a.q0 + q_last, a.L - 1) / kKeys - tile_lo + 1;
   if (tid == 0) {
     *abort_word = 0u;
-    for (int i = 0; i < kMaxKStages; ++i) {
-      MbarInit(kfull + 8 * i, 1);
-      MbarInit(kempty + 8 * i, 1);
-    }
     for (int i = 0; i < 2; ++i) {
+      MbarInit(kfull + 8 * i, 1);
       MbarInit(vfull + 8 * i, 1);
-      MbarInit(vempty + 8 * i, 1);
       MbarInit(sfull + 8 * i, 1);
       MbarInit(odone + 8 * i, 1);
     }
@@ -122,23 +118,16 @@ __global__ void __launch_bounds__(kThreads, 1)
   bool ok = true;
 
   if (warp == kSoftmaxWarps) {
-    if (lane == 0) {
-      // Ring positions and phases are counted along: a division per box would take longer than the box.
-      int ks = 0, vs = 0;
-      uint32_t kphase = 1, vphase = 1;  // a fresh barrier passes a wait for the phase before its first
+    if (ElectOne()) {
+      // Stages are one or two per ring; everything is counted along (a division per box would take longer than the box).
       auto load_k = [&](int j) {
-        const int key = (tile_lo + j) * kKeys;
-        for (int c = 0; c < qk_atoms; ++c) {
-          const uint32_t bar = kfull + 8 * ks, dst = base + sk + ks * kAtom;
-          ok = MbarWait(kempty + 8 * ks, kphase, abort_word) && ok;
-          MbarExpectTx(bar, kAtom);
-          if (c < dim_atoms) TmaBox(dst, &map_k, c * 64, head, key, bar);
-          else TmaBox(dst, &map_rot, (c - dim_atoms) * 64, 0, key, bar);
-          if (++ks == k_stages) {
-            ks = 0;
-            kphase ^= 1;
-          }
-        }
+        const int key = (tile_lo + j) * kKeys, stage = k_stages == 2 ? j & 1 : 0, before = j - k_stages;
+        const uint32_t bar = kfull + 8 * stage;
+        uint32_t dst = base + sk + stage * k_tile;
+        if (before >= 0) ok = MbarWait(sfull + 8 * (before & 1), (before >> 1) & 1, abort_word) && ok;
+        MbarExpectTx(bar, k_tile);
+        for (int c = 0; c < dim_atoms; ++c, dst += kAtom) TmaBox(dst, &map_k, c * 64, head, key, bar);
+        for (int c = dim_atoms; c < qk_atoms; ++c, dst += kAtom) TmaBox(dst, &map_rot, (c - dim_atoms) * 64, 0, key, bar);
       };
       MbarExpectTx(qfull, qk_atoms * kAtom);
       for (int c = 0; c < qk_atoms; ++c) {
@@ -147,53 +136,41 @@ __global__ void __launch_bounds__(kThreads, 1)
       load_k(0);
       for (int j = 0; j < tiles; ++j) {
         if (j + 1 < tiles) load_k(j + 1);
-        const uint32_t bar = vfull + 8 * vs;
-        ok = MbarWait(vempty + 8 * vs, vphase, abort_word) && ok;
+        const int stage = v_stages == 2 ? j & 1 : 0, before = j - v_stages;
+        const uint32_t bar = vfull + 8 * stage;
+        if (before >= 0) ok = MbarWait(odone + 8 * (before & 1), (before >> 1) & 1, abort_word) && ok;
         MbarExpectTx(bar, v_tile);
-        for (int c = 0; c < v_atoms; ++c) TmaBox(base + sv + vs * v_tile + c * kAtom, &map_v, c * 64, head, (tile_lo + j) * kKeys, bar);
-        if (++vs == v_stages) {
-          vs = 0;
-          vphase ^= 1;
-        }
+        for (int c = 0; c < v_atoms; ++c) TmaBox(base + sv + stage * v_tile + c * kAtom, &map_v, c * 64, head, (tile_lo + j) * kKeys, bar);
       }
       if (!ok) {  // given up: let the copies in flight land before the CTA's shared memory goes away
         volatile uint32_t never = 0;
-        const int k_boxes = tiles * qk_atoms;
         for (int s = 0; s < k_stages; ++s)
-          if (k_boxes > s) MbarWait(kfull + 8 * s, ((k_boxes - 1 - s) / k_stages) & 1, &never);
+          if (tiles > s) MbarWait(kfull + 8 * s, ((tiles - 1 - s) / k_stages) & 1, &never);
         for (int s = 0; s < v_stages; ++s)
           if (tiles > s) MbarWait(vfull + 8 * s, ((tiles - 1 - s) / v_stages) & 1, &never);
       }
     }
     __syncwarp();
   } else if (warp == kSoftmaxWarps + 1) {
-    if (lane == 0) {
+    if (ElectOne()) {
       const uint32_t s_idesc = InstrDesc(kKeys, false), o_idesc = InstrDesc((a.vdim + 15) / 16 * 16, true);
       const uint64_t qd = SmemDesc(base, 16, 1024), kd = SmemDesc(base + sk, 16, 1024);
       const uint64_t vd = SmemDesc(base + sv, kAtom, 1024);
       ok = MbarWait(qfull, 0, abort_word) && ok;
-      int ks = 0, vs = 0;
-      uint32_t kphase = 0, vphase = 0;
       auto scores = [&](int j) {
         const uint32_t b = j & 1, acc = tmem + b * 128;
         // The buffer held P(j - 2), whose product is in front of these MMAs in the same queue.
-        uint64_t qa = qd;
-        for (int c = 0; c < qk_atoms; ++c, qa += kAtom >> 4) {
+        const int stage = k_stages == 2 ? j & 1 : 0;
+        uint64_t qa = qd, ka = kd + static_cast<uint64_t>((stage * k_tile) >> 4);
+        ok = MbarWait(kfull + 8 * stage, (k_stages == 2 ? j >> 1 : j) & 1, abort_word) && ok;
+        asm volatile("tcgen05.fence::after_thread_sync;\n" ::: "memory");
+        for (int c = 0; c < qk_atoms; ++c, qa += kAtom >> 4, ka += kAtom >> 4) {
           const int width = c < dim_atoms ? a.dim - 64 * c : a.rot - 64 * (c - dim_atoms);
-          const uint64_t ka = kd + static_cast<uint64_t>((ks * kAtom) >> 4);
-          ok = MbarWait(kfull + 8 * ks, kphase, abort_word) && ok;
-          asm volatile("tcgen05.fence::after_thread_sync;\n" ::: "memory");
-          Mma(acc, qa, ka, s_idesc, c > 0 ? 1u : 0u);
           if (width > 48) {
 #pragma unroll
-            for (int k = 1; k < 4; ++k) Mma(acc, qa + 2 * k, ka + 2 * k, s_idesc, 1u);
+            for (int k = 0; k < 4; ++k) Mma(acc, qa + 2 * k, ka + 2 * k, s_idesc, c > 0 || k > 0 ? 1u : 0u);
           } else {
-            for (int k = 1; 16 * k < width; ++k) Mma(acc, qa + 2 * k, ka + 2 * k, s_idesc, 1u);
-          }
-          TcCommit(kempty + 8 * ks);
-          if (++ks == k_stages) {
-            ks = 0;
-            kphase ^= 1;
+            for (int k = 0; 16 * k < width; ++k) Mma(acc, qa + 2 * k, ka + 2 * k, s_idesc, c > 0 || k > 0 ? 1u : 0u);
           }
         }
         TcCommit(sfull + 8 * b);
@@ -201,21 +178,17 @@ __global__ void __launch_bounds__(kThreads, 1)
       scores(0);
       for (int j = 0; j < tiles; ++j) {
         if (j + 1 < tiles) scores(j + 1);
-        const uint64_t va = vd + static_cast<uint64_t>((vs * v_tile) >> 4);
+        const int stage = v_stages == 2 ? j & 1 : 0;
+        const uint64_t va = vd + static_cast<uint64_t>((stage * v_tile) >> 4);
         const uint32_t pa = tmem + (j & 1) * 128;
-        ok = MbarWait(vfull + 8 * vs, vphase, abort_word) && ok;
+        ok = MbarWait(vfull + 8 * stage, (v_stages == 2 ? j >> 1 : j) & 1, abort_word) && ok;
         ok = MbarWait(pfull, j & 1, abort_word) && ok;
         asm volatile("tcgen05.fence::after_thread_sync;\n" ::: "memory");
         // P: eight columns per 16 keys; V: keys are its rows, 16 of them per step
         TcMmaTmemA(tmem_o, pa, va, o_idesc, j > 0 ? 1u : 0u);
 #pragma unroll
         for (int k = 1; k < kKeys / 16; ++k) TcMmaTmemA(tmem_o, pa + 8 * k, va + ((k * 16 * 128) >> 4), o_idesc, 1u);
-        TcCommit(vempty + 8 * vs);
         TcCommit(odone + 8 * (j & 1));
-        if (++vs == v_stages) {
-          vs = 0;
-          vphase ^= 1;
-        }
       }
     }
     __syncwarp();
@@ -379,9 +352,9 @@ bool Rings(int dim, int rot, int vdim, WindowArgs* a)
   a->qk_atoms = a->dim_atoms + (rot + 63) / 64;
   a->v_atoms = (vdim + 63) / 64;
   const int atoms = (kMaxSmem - 4096) / kAtom - a->qk_atoms;  // static shared memory and the alignment slack aside
-  a->v_stages = atoms - 2 * a->v_atoms >= a->qk_atoms + 1 ? 2 : 1;
-  a->k_stages = min(kMaxKStages, atoms - a->v_stages * a->v_atoms);
-  return vdim <= 256 && a->k_stages >= 2;
+  a->k_stages = atoms >= 2 * a->qk_atoms + a->v_atoms ? 2 : 1;
+  a->v_stages = atoms - a->k_stages * a->qk_atoms >= 2 * a->v_atoms ? 2 : 1;
+  return vdim <= 256 && atoms >= a->qk_atoms + a->v_atoms;
 }
 
 }  // namespace
@@ -457,7 +430,7 @@ extern "C" int tlaloc_b200_window_attention(const void* q, const void* k, const 
     return Fail(kInternal, "%s: the tensor maps could not be encoded", op);
   }
   if (rot_dim == 0) mr = mk;
-  const size_t smem = static_cast<size_t>(a.qk_atoms + a.k_stages + a.v_stages * a.v_atoms) * kAtom + 1024;
+  const size_t smem = static_cast<size_t>(a.qk_atoms + a.k_stages * a.qk_atoms + a.v_stages * a.v_atoms) * kAtom + 1024;
   const dim3 grid((num_queries + kQ - 1) / kQ, num_heads);
   e = LaunchChained(WindowAttentionTc, grid, kThreads, smem, static_cast<cudaStream_t>(stream), mq, mk, mr, mv, a);
   if (e != cudaSuccess) return CudaFail("WINDOW_ATTENTION launch", e);
