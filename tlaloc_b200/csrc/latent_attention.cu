@@ -6,11 +6,12 @@
 // LatentAttentionTc (bf16, pages of a multiple of 64 positions): all heads share a position's row, so a CTA takes 16 to 64 heads of one
 // row of the batch and a slice of its positions, and the cached row leaves HBM once for all of them.  Tiles of 64 positions arrive as boxes of a
 // tensor map over the pool (atoms of 64 positions x 64 channels, 128-byte swizzle) in a ring of two to four stages.
-//   producer lane   boxes of the tiles
+//   producer lane   boxes of the tiles, and an L2 prefetch two tiles ahead of them: the ring is full of tiles at work, so the way from
+//                   HBM is hidden in front of it
 //   MMA lane        scores: tcgen05.mma with the query as A out of TMEM (heads are its lanes, put there once) and the tile as B,
 //                   into one of two accumulators of 64 columns
-//   1 - 2 warps     softmax: a thread owns a head's row of 64 scores; the weights go to shared memory as bf16.  The running maximum is
-//                   raised lazily (the exponentials stay below 2^8), so the values' accumulators are rarely rescaled
+//   2 - 4 warps     softmax: two threads own a head's row of 64 scores and exchange its maximum; the weights go to shared memory as
+//                   bf16.  The running maximum is raised lazily (the exponentials stay below 2^8), so the values' accumulators are rarely rescaled
 //   sixteen warps   values: mma.sync m16n8k16 over the tile as it lies, the latent channels split over the warps, accumulators
 //                   in registers (a TMEM accumulator of 512 channels would leave no room for the query)
 // Each of the four works on a tile of its own.  Slices leave {max, sum, acc[kv_rank]} records in f32 that LatentCombine merges in slice
@@ -120,8 +121,9 @@ __global__ void __launch_bounds__(kGenericThreads) LatentAttentionGeneric(Latent
 using namespace tc;
 
 constexpr int kAtomBytes = 64 * 128;
-constexpr int kMmaTile = 64, kValueWarps = 16, kSoftmaxWarps = 2;
-constexpr int kMmaThreads = (kValueWarps + kSoftmaxWarps + 2) * 32;
+constexpr int kMmaTile = 64, kValueWarps = 16, kProducerWarp = 18, kMmaWarp = 19;
+// Warps 16, 17 and 20, 21 are the softmax: a warp reads the TMEM lanes of its number modulo 4, so both of a pair see the same heads.
+constexpr int kMmaThreads = 22 * 32;
 constexpr int kPStride = kMmaTile + 8, kMaxStages = 4;
 
 __device__ __forceinline__ void LdMatrixX4(uint32_t (&r)[4], uint32_t addr)
@@ -179,7 +181,7 @@ __global__ void __launch_bounds__(kMmaThreads, 1)
   extern __shared__ unsigned char smem_raw[];
   __shared__ alignas(8) uint64_t bars[2 * kMaxStages + 9];
   __shared__ uint32_t slot_store[2];
-  __shared__ float s_keep[2][HT], s_total[HT];
+  __shared__ float s_keep[2][HT], s_row[2][2][(HT + 31) / 32 * 32];  // s_row: [tile parity][half of the positions][head]
   __shared__ alignas(16) __nv_bfloat16 s_p[2][HT * kPStride];
   const uint32_t base = (SmemAddr(smem_raw) + 1023u) & ~1023u;  // the swizzle is a function of address bits 4..9
   unsigned char* smem = smem_raw + (base - SmemAddr(smem_raw));
@@ -207,8 +209,8 @@ __global__ void __launch_bounds__(kMmaThreads, 1)
     }
     for (int i = 0; i < 2; ++i) {
       MbarInit(sfull + 8 * i, 1);
-      MbarInit(sempty + 8 * i, (HT + 31) / 32);
-      MbarInit(pfull + 8 * i, (HT + 31) / 32);
+      MbarInit(sempty + 8 * i, 2 * ((HT + 31) / 32));
+      MbarInit(pfull + 8 * i, 2 * ((HT + 31) / 32));
       MbarInit(pempty + 8 * i, kValueWarps);
     }
     MbarInit(qready, 4);
@@ -224,14 +226,23 @@ __global__ void __launch_bounds__(kMmaThreads, 1)
   const uint32_t tmem = *static_cast<volatile uint32_t*>(slot_store), tmem_q = tmem + 2 * kMmaTile;  // two score accumulators, then the query
   bool ok = true;
 
-  if (warp == kValueWarps + kSoftmaxWarps) {
+  if (warp == kProducerWarp) {
     if (ElectOne()) {
       const int* table = TableOf(p, t);
       int stage = 0;
       uint32_t phase = 1;  // a fresh barrier passes a wait for the phase before its first
-      for (int j = 0; j < n; ++j) {
+      auto pool_row = [&](int j) {
         const int pos = (tile0 + j) * kMmaTile, block = pos >> p.block_shift;  // the tile's 64 rows lie in one page
-        const int row = min(max(__ldg(table + block), 0), p.num_blocks - 1) * p.block_size + (pos - (block << p.block_shift));
+        return min(max(__ldg(table + block), 0), p.num_blocks - 1) * p.block_size + (pos - (block << p.block_shift));
+      };
+      int row = pool_row(0), row1 = n > 1 ? pool_row(1) : 0, row2 = n > 2 ? pool_row(2) : 0;
+      for (int j = 0; j < n; ++j) {
+        const int row3 = j + 3 < n ? pool_row(j + 3) : 0;
+        if (j + 2 < n && j + 2 >= stages) {
+          for (int c = 0; c < sp.atoms; ++c) {
+            asm volatile("cp.async.bulk.prefetch.tensor.2d.L2.global [%0, {%1, %2}];\n" ::"l"(reinterpret_cast<uint64_t>(&map)), "r"(c * 64), "r"(row2) : "memory");
+          }
+        }
         const uint32_t bar = full + 8 * stage, dst = base + stage * tile_bytes;
         ok = MbarWait(free0 + 8 * stage, phase, abort_word) && ok;
         MbarExpectTx(bar, tile_bytes);
@@ -240,6 +251,9 @@ __global__ void __launch_bounds__(kMmaThreads, 1)
                        "l"(reinterpret_cast<uint64_t>(&map)), "r"(c * 64), "r"(row), "r"(bar)
                        : "memory");
         }
+        row = row1;
+        row1 = row2;
+        row2 = row3;
         if (++stage == stages) {
           stage = 0;
           phase ^= 1;
@@ -252,7 +266,7 @@ __global__ void __launch_bounds__(kMmaThreads, 1)
       }
     }
     __syncwarp();
-  } else if (warp == kValueWarps + kSoftmaxWarps + 1) {
+  } else if (warp == kMmaWarp) {
     if (ElectOne()) {
       // f32 accumulator, bf16, both K-major, M = 128 (the lanes past the heads hold zeros), N = 64
       constexpr uint32_t idesc = (1u << 4) | (1u << 7) | (1u << 10) | (static_cast<uint32_t>(kMmaTile >> 3) << 17) | (8u << 24);
@@ -281,33 +295,40 @@ __global__ void __launch_bounds__(kMmaThreads, 1)
       }
     }
     __syncwarp();
-  } else if (warp >= kValueWarps) {
-    const int quad = warp - kValueWarps, head = quad * 32 + lane;  // TMEM lane; kValueWarps is a multiple of 4
+  } else if (warp >= kValueWarps) {  // softmax
+    const int quad = warp & 3, half = warp >= kMmaWarp ? 1 : 0, head = quad * 32 + lane;  // TMEM lane; positions [32 half, 32 half + 32)
     const uint32_t lanes = static_cast<uint32_t>(quad * 32) << 16;
+    constexpr int kHalf = kMmaTile / 2;
+    // The other half of the row: the two warps of a quad meet at a named barrier of 64 threads.
+    auto other = [&](int b, float mine) {
+      s_row[b][half][head] = mine;
+      asm volatile("bar.sync %0, 64;\n" ::"r"(2 + quad) : "memory");
+      return s_row[b][half ^ 1][head];
+    };
     if (quad * 32 < HT) {
       const float scale = p.scale * 1.4426950408889634f;
       float top = -INFINITY, sum = 0.f;
       for (int j = 0; j < n; ++j) {
-        const int b = j & 1, pos = (tile0 + j) * kMmaTile;
+        const int b = j & 1, tile_pos = (tile0 + j) * kMmaTile, pos = tile_pos + half * kHalf;
         ok = MbarWaitWarp(sfull + 8 * b, (j >> 1) & 1, lane, abort_word) && ok;
         asm volatile("tcgen05.fence::after_thread_sync;\n" ::: "memory");
-        uint32_t s[kMmaTile];
-        TcLd32(tmem + lanes + b * kMmaTile, s);
-        TcLd32(tmem + lanes + b * kMmaTile + 32, s + 32);
+        uint32_t s[kHalf];
+        TcLd32(tmem + lanes + b * kMmaTile + half * kHalf, s);
         asm volatile("tcgen05.wait::ld.sync.aligned;\n" ::: "memory");
         asm volatile("tcgen05.fence::before_thread_sync;\n" ::: "memory");
         __syncwarp();
         if (lane == 0) MbarArrive(sempty + 8 * b);
         float t4[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
-        const bool edge = pos < live.x || pos + kMmaTile > live.y;
+        const bool edge = tile_pos < live.x || tile_pos + kMmaTile > live.y;
 #pragma unroll
-        for (int e = 0; e < kMmaTile; ++e) {
+        for (int e = 0; e < kHalf; ++e) {
           float v = __uint_as_float(s[e]) * scale;
           if (edge && (pos + e < live.x || pos + e >= live.y)) v = -INFINITY;
           s[e] = __float_as_uint(v);
           t4[e & 3] = fmaxf(t4[e & 3], v);
         }
-        const float tile_top = fmaxf(fmaxf(t4[0], t4[1]), fmaxf(t4[2], t4[3]));  // finite: a tile holds at least one live position
+        const float mine = fmaxf(fmaxf(t4[0], t4[1]), fmaxf(t4[2], t4[3]));
+        const float tile_top = fmaxf(mine, other(b, mine));  // finite: a tile holds at least one live position
         float keep = 1.f;
         if (tile_top > top + kLazy || top == -INFINITY) {
           const float next = fmaxf(top, tile_top);
@@ -317,25 +338,28 @@ __global__ void __launch_bounds__(kMmaThreads, 1)
         }
         float add[2] = {0.f, 0.f};
 #pragma unroll
-        for (int e = 0; e < kMmaTile; e += 2) {
+        for (int e = 0; e < kHalf; e += 2) {
           const float p0 = Exp2(__uint_as_float(s[e]) - top), p1 = Exp2(__uint_as_float(s[e + 1]) - top);
           add[0] += p0;
           add[1] += p1;
           s[e / 2] = Pack(p0, p1);
         }
         sum += add[0] + add[1];
+        const float total = j == n - 1 ? sum + other(b ^ 1, sum) : 0.f;
         ok = MbarWaitWarp(pempty + 8 * b, ((j >> 1) & 1) ^ 1, lane, abort_word) && ok;
         if (head < HT) {
-          uint4* dst = reinterpret_cast<uint4*>(s_p[b] + head * kPStride);
+          uint4* dst = reinterpret_cast<uint4*>(s_p[b] + head * kPStride + half * kHalf);
 #pragma unroll
-          for (int c = 0; c < 8; ++c) dst[c] = make_uint4(s[4 * c], s[4 * c + 1], s[4 * c + 2], s[4 * c + 3]);
-          s_keep[b][head] = keep;
-          if (j == n - 1) {
-            s_total[head] = sum;
-            if (sp.records != nullptr && h0 + head < p.H) {
-              float* rec = sp.records + ((static_cast<size_t>(slice) * p.T + t) * p.H + h0 + head) * (p.kv_rank + 2);
-              rec[0] = top;
-              rec[1] = sum;
+          for (int c = 0; c < 4; ++c) dst[c] = make_uint4(s[4 * c], s[4 * c + 1], s[4 * c + 2], s[4 * c + 3]);
+          if (half == 0) {
+            s_keep[b][head] = keep;
+            if (j == n - 1) {
+              s_row[b][0][head] = total;  // both maxima of this tile have been read
+              if (sp.records != nullptr && h0 + head < p.H) {
+                float* rec = sp.records + ((static_cast<size_t>(slice) * p.T + t) * p.H + h0 + head) * (p.kv_rank + 2);
+                rec[0] = top;
+                rec[1] = total;
+              }
             }
           }
         }
@@ -431,7 +455,7 @@ __global__ void __launch_bounds__(kMmaThreads, 1)
       for (int half = 0; half < 2; ++half) {
         const int hl = m * 16 + gid + half * 8, h = h0 + hl;
         if (h >= p.H) continue;
-        const float total = s_total[hl], inv = total > 0.f ? 1.f / total : 0.f;
+        const float total = s_row[(n - 1) & 1][0][hl], inv = total > 0.f ? 1.f / total : 0.f;
 #pragma unroll
         for (int c2 = 0; c2 < 2 * NP; ++c2) {
           const int c = (warp + kValueWarps * (c2 >> 1)) * 16 + (c2 & 1) * 8 + tig * 2;
