@@ -213,7 +213,7 @@ __global__ void __launch_bounds__(kMmaThreads, 1)
       MbarInit(pfull + 8 * i, 2 * ((HT + 31) / 32));
       MbarInit(pempty + 8 * i, kValueWarps);
     }
-    MbarInit(qready, 4);
+    MbarInit(qready, kValueWarps);
     asm volatile("fence.mbarrier_init.release.cluster;\n" ::: "memory");
   }
   if (warp == 0) {
@@ -368,15 +368,19 @@ __global__ void __launch_bounds__(kMmaThreads, 1)
       }
     }
   } else {
-    if (warp < 4) {  // the query into TMEM, zeros in the lanes past the heads
-      const int head = warp * 32 + lane;
+    {  // the query into TMEM, zeros in the lanes past the heads: a warp takes the lanes of its quadrant and every fourth atom
+      const int quad = warp & 3, head = quad * 32 + lane;
       const bool there = head < HT && h0 + head < p.H;
-      const uint32_t* q = reinterpret_cast<const uint32_t*>(static_cast<const __nv_bfloat16*>(p.query) + (static_cast<size_t>(t) * p.H + h0 + head) * p.row);
-      for (int c = 0; c < sp.atoms; ++c) {
+      const uint4* q = reinterpret_cast<const uint4*>(static_cast<const __nv_bfloat16*>(p.query) + (static_cast<size_t>(t) * p.H + h0 + head) * p.row);
+      const int words = p.row >> 3;
+      for (int c = warp >> 2; c < sp.atoms; c += kValueWarps / 4) {
         uint32_t w[32];
 #pragma unroll
-        for (int e = 0; e < 32; ++e) w[e] = there && c * 64 + 2 * e < p.row ? __ldg(q + c * 32 + e) : 0u;
-        TcSt32(tmem_q + (static_cast<uint32_t>(warp * 32) << 16) + c * 32, w);
+        for (int e = 0; e < 8; ++e) {
+          const uint4 v = there && c * 8 + e < words ? __ldg(q + c * 8 + e) : make_uint4(0, 0, 0, 0);
+          w[4 * e] = v.x; w[4 * e + 1] = v.y; w[4 * e + 2] = v.z; w[4 * e + 3] = v.w;
+        }
+        TcSt32(tmem_q + (static_cast<uint32_t>(quad * 32) << 16) + c * 32, w);
       }
       asm volatile("tcgen05.wait::st.sync.aligned;\n" ::: "memory");
       asm volatile("tcgen05.fence::before_thread_sync;\n" ::: "memory");
@@ -396,8 +400,8 @@ __global__ void __launch_bounds__(kMmaThreads, 1)
     uint32_t phase = 0;
     for (int j = 0; j < n; ++j) {
       const int b = j & 1, pos = (tile0 + j) * kMmaTile;
-      ok = MbarWaitWarp(full + 8 * stage, phase, lane, abort_word) && ok;
-      ok = MbarWaitWarp(pfull + 8 * b, (j >> 1) & 1, lane, abort_word) && ok;
+      if (lane == 0) ok = MbarWait(pfull + 8 * b, (j >> 1) & 1, abort_word) && MbarWait(full + 8 * stage, phase, abort_word) && ok;
+      __syncwarp();
       const uint32_t tile_addr = base + stage * tile_bytes;
       // Rows of the page outside the live range may hold anything: 0 times it must stay 0.
       const int live_lo = live.x - pos, live_hi = live.y - pos;
