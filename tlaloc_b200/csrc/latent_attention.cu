@@ -179,7 +179,7 @@ __global__ void __launch_bounds__(kMmaThreads, 1)
   constexpr int HT = MT * 16;
   GridDependencySync();
   extern __shared__ unsigned char smem_raw[];
-  __shared__ alignas(8) uint64_t bars[2 * kMaxStages + 9];
+  __shared__ alignas(8) uint64_t bars[2 * kMaxStages + 5];
   __shared__ uint32_t slot_store[2];
   __shared__ float s_keep[2][HT], s_row[2][2][(HT + 31) / 32 * 32];  // s_row: [tile parity][half of the positions][head]
   __shared__ alignas(16) __nv_bfloat16 s_p[2][HT * kPStride];
@@ -199,7 +199,10 @@ __global__ void __launch_bounds__(kMmaThreads, 1)
     return;
   }
   const uint32_t full = SmemAddr(bars), free0 = full + 8 * kMaxStages, sfull = free0 + 8 * kMaxStages, sempty = sfull + 16;
-  const uint32_t pfull = sempty + 16, pempty = pfull + 16, qready = pempty + 16;
+  const uint32_t qready = sempty + 16;
+  // The weights change hands at named barriers (4, 5: there; 6, 7: read), where a waiting warp costs no issue slots: sixteen warps
+  // polling an mbarrier slowed the softmax down.  Trip counts are fixed, so every arrival has its wait.
+  constexpr int kHandOver = (kValueWarps + 2 * ((HT + 31) / 32)) * 32;
   volatile uint32_t* abort_word = slot_store + 1;
   if (tid == 0) {
     slot_store[1] = 0u;
@@ -210,8 +213,6 @@ __global__ void __launch_bounds__(kMmaThreads, 1)
     for (int i = 0; i < 2; ++i) {
       MbarInit(sfull + 8 * i, 1);
       MbarInit(sempty + 8 * i, 2 * ((HT + 31) / 32));
-      MbarInit(pfull + 8 * i, 2 * ((HT + 31) / 32));
-      MbarInit(pempty + 8 * i, kValueWarps);
     }
     MbarInit(qready, kValueWarps);
     asm volatile("fence.mbarrier_init.release.cluster;\n" ::: "memory");
@@ -346,7 +347,7 @@ __global__ void __launch_bounds__(kMmaThreads, 1)
         }
         sum += add[0] + add[1];
         const float total = j == n - 1 ? sum + other(b ^ 1, sum) : 0.f;
-        ok = MbarWaitWarp(pempty + 8 * b, ((j >> 1) & 1) ^ 1, lane, abort_word) && ok;
+        if (j >= 2) asm volatile("bar.sync %0, %1;\n" ::"r"(6 + b), "n"(kHandOver) : "memory");
         if (head < HT) {
           uint4* dst = reinterpret_cast<uint4*>(s_p[b] + head * kPStride + half * kHalf);
 #pragma unroll
@@ -363,8 +364,7 @@ __global__ void __launch_bounds__(kMmaThreads, 1)
             }
           }
         }
-        __syncwarp();
-        if (lane == 0) MbarArrive(pfull + 8 * b);
+        asm volatile("bar.arrive %0, %1;\n" ::"r"(4 + b), "n"(kHandOver) : "memory");
       }
     }
   } else {
@@ -400,7 +400,8 @@ __global__ void __launch_bounds__(kMmaThreads, 1)
     uint32_t phase = 0;
     for (int j = 0; j < n; ++j) {
       const int b = j & 1, pos = (tile0 + j) * kMmaTile;
-      if (lane == 0) ok = MbarWait(pfull + 8 * b, (j >> 1) & 1, abort_word) && MbarWait(full + 8 * stage, phase, abort_word) && ok;
+      asm volatile("bar.sync %0, %1;\n" ::"r"(4 + b), "n"(kHandOver) : "memory");
+      if (lane == 0) ok = MbarWait(full + 8 * stage, phase, abort_word) && ok;  // the scores are there, so the tile is
       __syncwarp();
       const uint32_t tile_addr = base + stage * tile_bytes;
       // Rows of the page outside the live range may hold anything: 0 times it must stay 0.
@@ -443,11 +444,9 @@ __global__ void __launch_bounds__(kMmaThreads, 1)
           }
         }
       }
+      if (j + 2 < n) asm volatile("bar.arrive %0, %1;\n" ::"r"(6 + b), "n"(kHandOver) : "memory");
       __syncwarp();
-      if (lane == 0) {
-        MbarArrive(pempty + 8 * b);
-        MbarArrive(free0 + 8 * stage);
-      }
+      if (lane == 0) MbarArrive(free0 + 8 * stage);
       if (++stage == stages) {
         stage = 0;
         phase ^= 1;
