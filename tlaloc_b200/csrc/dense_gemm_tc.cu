@@ -61,15 +61,6 @@ __host__ __device__ constexpr uint32_t InstrDescBf16(int n)  // f32 accumulator,
 {
   return (1u << 4) | (1u << 7) | (1u << 10) | (static_cast<uint32_t>(n >> 3) << 17) | (8u << 24);
 }
-__device__ __forceinline__ void TcMmaBf16(uint32_t d_tmem, uint64_t a_desc, uint64_t b_desc, uint32_t idesc, uint32_t accumulate)
-{
-  asm volatile(
-      "{\n\t.reg .pred p;\n\t"
-      "setp.ne.b32 p, %4, 0;\n\t"
-      "tcgen05.mma.cta_group::1.kind::f16 [%0], %1, %2, %3, p;\n\t}\n" ::"r"(d_tmem),
-      "l"(a_desc), "l"(b_desc), "r"(idesc), "r"(accumulate)
-      : "memory");
-}
 // x (the k coordinate) is a multiple of 64 elements: always a 16-byte boundary.
 __device__ __forceinline__ void TmaBox3d(uint32_t dst, const CUtensorMap* map, int x, int y, int z, uint32_t bar, uint64_t policy)
 {

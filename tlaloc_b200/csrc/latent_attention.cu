@@ -8,13 +8,13 @@
 // tensor map over the pool (atoms of 64 positions x 64 channels, 128-byte swizzle) in a ring of two to four stages.
 //   producer lane   boxes of the tiles, and an L2 prefetch two tiles ahead of them: the ring is full of tiles at work, so the way from
 //                   HBM is hidden in front of it
-//   MMA lane        scores: tcgen05.mma with the query as A out of TMEM (heads are its lanes, put there once) and the tile as B,
-//                   into one of two accumulators of 64 columns
+//   MMA lane        scores S = Q C^T: the query is the A operand out of TMEM (heads are its lanes, put there once), the tile is B;
+//                   then O^T += C^T P^T: the same tile, its channels now the M rows (an MN-major A operand, 128 channels at a time), the
+//                   weights B, accumulators of 128 channel lanes x heads in TMEM
 //   2 - 4 warps     softmax: two threads own a head's row of 64 scores and exchange its maximum; the weights go to shared memory as
-//                   bf16.  The running maximum is raised lazily (the exponentials stay below 2^8), so the values' accumulators are rarely rescaled
-//   sixteen warps   values: mma.sync m16n8k16 over the tile as it lies, the latent channels split over the warps, accumulators
-//                   in registers (a TMEM accumulator of 512 channels would leave no room for the query)
-// Each of the four works on a tile of its own.  Slices leave {max, sum, acc[kv_rank]} records in f32 that LatentCombine merges in slice
+//                   bf16.  The running maximum is raised lazily (the exponentials stay below 2^8), so O is rarely rescaled
+//   four warps      rescale O when a maximum was raised, blank the dead rows of the edge tiles, and write the result
+// Slices leave {max, sum, acc[kv_rank]} records in f32 that LatentCombine merges in slice
 // order.  Every mbarrier wait is bounded.
 #include <cuda.h>
 
@@ -121,30 +121,11 @@ __global__ void __launch_bounds__(kGenericThreads) LatentAttentionGeneric(Latent
 using namespace tc;
 
 constexpr int kAtomBytes = 64 * 128;
-constexpr int kMmaTile = 64, kValueWarps = 16, kProducerWarp = 18, kMmaWarp = 19;
-// Warps 16, 17 and 20, 21 are the softmax: a warp reads the TMEM lanes of its number modulo 4, so both of a pair see the same heads.
-constexpr int kMmaThreads = 22 * 32;
-constexpr int kPStride = kMmaTile + 8, kMaxStages = 4;
+constexpr int kMmaTile = 64, kMaxStages = 4;
+// Warps 0 - 3 write the output; 4, 5 and 8, 9 are the softmax: a warp reads the TMEM lanes of its number modulo 4, so both of a pair
+// see the same heads.
+constexpr int kOutWarps = 4, kProducerWarp = 6, kMmaWarp = 7, kMmaThreads = 10 * 32;
 
-__device__ __forceinline__ void LdMatrixX4(uint32_t (&r)[4], uint32_t addr)
-{
-  asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];\n"
-               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3])
-               : "r"(addr));
-}
-__device__ __forceinline__ void LdMatrixX4Trans(uint32_t (&r)[4], uint32_t addr)
-{
-  asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];\n"
-               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3])
-               : "r"(addr));
-}
-// Not volatile: the next fragments' loads may move ahead of it.
-__device__ __forceinline__ void MmaBf16(float (&c)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1)
-{
-  asm("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};\n"
-      : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
-      : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
-}
 __device__ __forceinline__ float Exp2(float x)
 {
   float y;
@@ -159,7 +140,7 @@ __device__ __forceinline__ uint32_t Pack(float a, float b)
 
 struct SliceParams {
   float* records;  // [slices][T][H][kv_rank + 2], or null: one slice, straight to out
-  int slices, slice_tiles, atoms, stages;  // atoms: 64-channel atoms of a tile
+  int slices, slice_tiles, atoms, stages, score_buffers;  // atoms: 64-channel atoms of a tile
 };
 
 __device__ int g_latent_status = 0;  // nonzero after a wait timed out (sticky until read)
@@ -171,21 +152,24 @@ __device__ __forceinline__ uint32_t TileWord(int position, int word)
 }
 constexpr float kLazy = 8.f;  // how far (log2) a head's maximum may grow past the reference in use
 
-// MT: 16-head tiles of the CTA; NP: 16-channel pairs of values per warp.
-template <int MT, int NP>
+// HT: heads of the CTA, a multiple of 16.
+template <int HT>
 __global__ void __launch_bounds__(kMmaThreads, 1)
     LatentAttentionTc(const __grid_constant__ CUtensorMap map, const __grid_constant__ LatentParams p, const __grid_constant__ SliceParams sp)
 {
-  constexpr int HT = MT * 16;
+  constexpr int kQuads = (HT + 31) / 32;   // TMEM lane quadrants with heads in them
+  constexpr int kOCols = kQuads * 32;      // columns of one O^T accumulator
+  constexpr int kPBytes = HT * 128;        // one tile's weights: [heads][64 positions] bf16, 128-byte swizzle
+  constexpr int kHandOver = (kOutWarps + 2 * kQuads) * 32;
   GridDependencySync();
   extern __shared__ unsigned char smem_raw[];
-  __shared__ alignas(8) uint64_t bars[2 * kMaxStages + 5];
+  __shared__ alignas(8) uint64_t bars[2 * kMaxStages + 9];
   __shared__ uint32_t slot_store[2];
-  __shared__ float s_keep[2][HT], s_row[2][2][(HT + 31) / 32 * 32];  // s_row: [tile parity][half of the positions][head]
-  __shared__ alignas(16) __nv_bfloat16 s_p[2][HT * kPStride];
+  __shared__ float s_keep[2][kOCols], s_row[2][2][kOCols];  // s_row: [tile parity][half of the positions][head]
   const uint32_t base = (SmemAddr(smem_raw) + 1023u) & ~1023u;  // the swizzle is a function of address bits 4..9
   unsigned char* smem = smem_raw + (base - SmemAddr(smem_raw));
   const int tile_bytes = sp.atoms * kAtomBytes, stages = sp.stages;
+  const uint32_t ring = base + 2 * kPBytes;
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
   const int t = blockIdx.z, h0 = blockIdx.y * HT, slice = blockIdx.x;
   const int2 live = LiveRange(p, t);
@@ -198,23 +182,24 @@ __global__ void __launch_bounds__(kMmaThreads, 1)
     }
     return;
   }
+  // full: a tile has landed; free: its products are done; sfull, sempty: scores there, read; pready: weights there and O in their
+  // scale; odone: O has the tile in it.
   const uint32_t full = SmemAddr(bars), free0 = full + 8 * kMaxStages, sfull = free0 + 8 * kMaxStages, sempty = sfull + 16;
-  const uint32_t qready = sempty + 16;
-  // The weights change hands at named barriers (4, 5: there; 6, 7: read), where a waiting warp costs no issue slots: sixteen warps
-  // polling an mbarrier slowed the softmax down.  Trip counts are fixed, so every arrival has its wait.
-  constexpr int kHandOver = (kValueWarps + 2 * ((HT + 31) / 32)) * 32;
+  const uint32_t pready = sempty + 16, odone = pready + 16, qready = odone + 16;
   volatile uint32_t* abort_word = slot_store + 1;
   if (tid == 0) {
     slot_store[1] = 0u;
     for (int i = 0; i < kMaxStages; ++i) {
       MbarInit(full + 8 * i, 1);
-      MbarInit(free0 + 8 * i, kValueWarps);
+      MbarInit(free0 + 8 * i, 1);
     }
     for (int i = 0; i < 2; ++i) {
       MbarInit(sfull + 8 * i, 1);
-      MbarInit(sempty + 8 * i, 2 * ((HT + 31) / 32));
+      MbarInit(sempty + 8 * i, 2 * kQuads);
+      MbarInit(pready + 8 * i, kOutWarps);
+      MbarInit(odone + 8 * i, 1);
     }
-    MbarInit(qready, kValueWarps);
+    MbarInit(qready, 8);
     asm volatile("fence.mbarrier_init.release.cluster;\n" ::: "memory");
   }
   if (warp == 0) {
@@ -224,8 +209,31 @@ __global__ void __launch_bounds__(kMmaThreads, 1)
   asm volatile("tcgen05.fence::before_thread_sync;\n" ::: "memory");
   __syncthreads();
   asm volatile("tcgen05.fence::after_thread_sync;\n" ::: "memory");
-  const uint32_t tmem = *static_cast<volatile uint32_t*>(slot_store), tmem_q = tmem + 2 * kMmaTile;  // two score accumulators, then the query
+  const uint32_t tmem = *static_cast<volatile uint32_t*>(slot_store);
+  const int o_tiles = (p.kv_rank + 127) >> 7;
+  const uint32_t tmem_q = tmem + sp.score_buffers * kMmaTile, tmem_o = tmem_q + sp.atoms * 32;
   bool ok = true;
+
+  if (warp != kProducerWarp && warp != kMmaWarp) {
+    // The query into TMEM, zeros in the lanes past the heads; the warps of a quadrant share its atoms.
+    const int quad = warp & 3, head = quad * 32 + lane;
+    const bool there = head < HT && h0 + head < p.H;
+    const uint4* q = reinterpret_cast<const uint4*>(static_cast<const __nv_bfloat16*>(p.query) + (static_cast<size_t>(t) * p.H + h0 + head) * p.row);
+    const int words = p.row >> 3;
+    for (int c = warp >> 2; c < sp.atoms; c += quad < 2 ? 3 : 1) {
+      uint32_t w[32];
+#pragma unroll
+      for (int e = 0; e < 8; ++e) {
+        const uint4 v = there && c * 8 + e < words ? __ldg(q + c * 8 + e) : make_uint4(0, 0, 0, 0);
+        w[4 * e] = v.x; w[4 * e + 1] = v.y; w[4 * e + 2] = v.z; w[4 * e + 3] = v.w;
+      }
+      TcSt32(tmem_q + (static_cast<uint32_t>(quad * 32) << 16) + c * 32, w);
+    }
+    asm volatile("tcgen05.wait::st.sync.aligned;\n" ::: "memory");
+    asm volatile("tcgen05.fence::before_thread_sync;\n" ::: "memory");
+    __syncwarp();
+    if (lane == 0) MbarArrive(qready);
+  }
 
   if (warp == kProducerWarp) {
     if (ElectOne()) {
@@ -244,7 +252,7 @@ __global__ void __launch_bounds__(kMmaThreads, 1)
             asm volatile("cp.async.bulk.prefetch.tensor.2d.L2.global [%0, {%1, %2}];\n" ::"l"(reinterpret_cast<uint64_t>(&map)), "r"(c * 64), "r"(row2) : "memory");
           }
         }
-        const uint32_t bar = full + 8 * stage, dst = base + stage * tile_bytes;
+        const uint32_t bar = full + 8 * stage, dst = ring + stage * tile_bytes;
         ok = MbarWait(free0 + 8 * stage, phase, abort_word) && ok;
         MbarExpectTx(bar, tile_bytes);
         for (int c = 0; c < sp.atoms; ++c) {  // x = 64 c elements: a multiple of 128 bytes
@@ -269,35 +277,56 @@ __global__ void __launch_bounds__(kMmaThreads, 1)
     __syncwarp();
   } else if (warp == kMmaWarp) {
     if (ElectOne()) {
-      // f32 accumulator, bf16, both K-major, M = 128 (the lanes past the heads hold zeros), N = 64
-      constexpr uint32_t idesc = (1u << 4) | (1u << 7) | (1u << 10) | (static_cast<uint32_t>(kMmaTile >> 3) << 17) | (8u << 24);
-      const uint64_t d0 = SmemDesc(base, 16, 1024);
-      const int steps = (p.row + 15) >> 4;
+      // f32 accumulators, bf16, M = 128.  Scores: both K-major (the lanes past the heads hold zeros), N = 64 positions.  Output: the
+      // tile's channels MN-major, N = heads.
+      constexpr uint32_t s_idesc = (1u << 4) | (1u << 7) | (1u << 10) | (static_cast<uint32_t>(kMmaTile >> 3) << 17) | (8u << 24);
+      constexpr uint32_t o_idesc = (1u << 4) | (1u << 7) | (1u << 10) | (1u << 15) | (static_cast<uint32_t>(HT >> 3) << 17) | (8u << 24);
+      const uint64_t sd = SmemDesc(ring, 16, 1024), cd = SmemDesc(ring, kAtomBytes, 1024), pd = SmemDesc(base, 16, 1024);
+      const int steps = (p.row + 15) >> 4, buffers = sp.score_buffers;
       ok = MbarWait(qready, 0, abort_word) && ok;
-      int stage = 0;
-      uint32_t phase = 0;
-      for (int j = 0; j < n; ++j) {
-        const uint32_t b = j & 1, acc = tmem + b * kMmaTile;
-        ok = MbarWait(full + 8 * stage, phase, abort_word) && ok;
-        ok = MbarWait(sempty + 8 * b, ((j >> 1) & 1) ^ 1, abort_word) && ok;
+      int s_stage = 0;
+      uint32_t s_phase = 0;
+      auto scores = [&](int j) {
+        const uint32_t acc = tmem + (buffers == 2 ? (j & 1) * kMmaTile : 0);
+        const int read = j - buffers;  // the scores whose place these take
+        ok = MbarWait(full + 8 * s_stage, s_phase, abort_word) && ok;
+        if (read >= 0) ok = MbarWait(sempty + 8 * (read & 1), (read >> 1) & 1, abort_word) && ok;
         asm volatile("tcgen05.fence::after_thread_sync;\n" ::: "memory");
-        uint64_t d = d0 + static_cast<uint64_t>((stage * tile_bytes) >> 4);
+        uint64_t d = sd + static_cast<uint64_t>((s_stage * tile_bytes) >> 4);
         uint32_t q = tmem_q;
         for (int c = 0; c < sp.atoms; ++c, d += kAtomBytes >> 4, q += 32) {
 #pragma unroll
           for (int k = 0; k < 4; ++k)
-            if (4 * c + k < steps) TcMmaTmemA(acc, q + 8 * k, d + 2 * k, idesc, c > 0 || k > 0 ? 1u : 0u);
+            if (4 * c + k < steps) TcMmaTmemA(acc, q + 8 * k, d + 2 * k, s_idesc, c > 0 || k > 0 ? 1u : 0u);
         }
-        TcCommit(sfull + 8 * b);
-        if (++stage == stages) {
-          stage = 0;
-          phase ^= 1;
+        TcCommit(sfull + 8 * (j & 1));
+        if (++s_stage == stages) {
+          s_stage = 0;
+          s_phase ^= 1;
         }
+      };
+      scores(0);
+      int stage = 0;
+      for (int j = 0; j < n; ++j) {
+        if (j + 1 < n) scores(j + 1);
+        const int b = j & 1;
+        ok = MbarWait(pready + 8 * b, (j >> 1) & 1, abort_word) && ok;
+        asm volatile("tcgen05.fence::after_thread_sync;\n" ::: "memory");
+        uint64_t d = cd + static_cast<uint64_t>((stage * tile_bytes) >> 4);
+        const uint64_t w = pd + static_cast<uint64_t>((b * kPBytes) >> 4);
+        uint32_t acc = tmem_o;
+        for (int i = 0; i < o_tiles; ++i, d += (2 * kAtomBytes) >> 4, acc += kOCols) {
+#pragma unroll
+          for (int k = 0; k < 4; ++k) TcMmaBf16(acc, d + ((k * 16 * 128) >> 4), w + 2 * k, o_idesc, j > 0 || k > 0 ? 1u : 0u);
+        }
+        TcCommit(free0 + 8 * stage);
+        TcCommit(odone + 8 * b);
+        if (++stage == stages) stage = 0;
       }
     }
     __syncwarp();
-  } else if (warp >= kValueWarps) {  // softmax
-    const int quad = warp & 3, half = warp >= kMmaWarp ? 1 : 0, head = quad * 32 + lane;  // TMEM lane; positions [32 half, 32 half + 32)
+  } else if (warp >= kOutWarps) {  // softmax
+    const int quad = warp & 3, half = warp >= 8 ? 1 : 0, head = quad * 32 + lane;  // TMEM lane; positions [32 half, 32 half + 32)
     const uint32_t lanes = static_cast<uint32_t>(quad * 32) << 16;
     constexpr int kHalf = kMmaTile / 2;
     // The other half of the row: the two warps of a quad meet at a named barrier of 64 threads.
@@ -306,7 +335,7 @@ __global__ void __launch_bounds__(kMmaThreads, 1)
       asm volatile("bar.sync %0, 64;\n" ::"r"(2 + quad) : "memory");
       return s_row[b][half ^ 1][head];
     };
-    if (quad * 32 < HT) {
+    if (quad < kQuads) {
       const float scale = p.scale * 1.4426950408889634f;
       float top = -INFINITY, sum = 0.f;
       for (int j = 0; j < n; ++j) {
@@ -314,7 +343,7 @@ __global__ void __launch_bounds__(kMmaThreads, 1)
         ok = MbarWaitWarp(sfull + 8 * b, (j >> 1) & 1, lane, abort_word) && ok;
         asm volatile("tcgen05.fence::after_thread_sync;\n" ::: "memory");
         uint32_t s[kHalf];
-        TcLd32(tmem + lanes + b * kMmaTile + half * kHalf, s);
+        TcLd32(tmem + lanes + (sp.score_buffers == 2 ? b * kMmaTile : 0) + half * kHalf, s);
         asm volatile("tcgen05.wait::ld.sync.aligned;\n" ::: "memory");
         asm volatile("tcgen05.fence::before_thread_sync;\n" ::: "memory");
         __syncwarp();
@@ -347,135 +376,97 @@ __global__ void __launch_bounds__(kMmaThreads, 1)
         }
         sum += add[0] + add[1];
         const float total = j == n - 1 ? sum + other(b ^ 1, sum) : 0.f;
-        if (j >= 2) asm volatile("bar.sync %0, %1;\n" ::"r"(6 + b), "n"(kHandOver) : "memory");
+        if (j >= 2) ok = MbarWaitWarp(odone + 8 * b, ((j >> 1) - 1) & 1, lane, abort_word) && ok;  // the weights of tile j - 2 have been read
         if (head < HT) {
-          uint4* dst = reinterpret_cast<uint4*>(s_p[b] + head * kPStride + half * kHalf);
+          unsigned char* dst = smem + b * kPBytes + head * 128;
 #pragma unroll
-          for (int c = 0; c < 4; ++c) dst[c] = make_uint4(s[4 * c], s[4 * c + 1], s[4 * c + 2], s[4 * c + 3]);
-          if (half == 0) {
-            s_keep[b][head] = keep;
-            if (j == n - 1) {
-              s_row[b][0][head] = total;  // both maxima of this tile have been read
-              if (sp.records != nullptr && h0 + head < p.H) {
-                float* rec = sp.records + ((static_cast<size_t>(slice) * p.T + t) * p.H + h0 + head) * (p.kv_rank + 2);
-                rec[0] = top;
-                rec[1] = total;
-              }
+          for (int c = 0; c < 4; ++c) {
+            *reinterpret_cast<uint4*>(dst + (((half * 4 + c) ^ (head & 7)) << 4)) = make_uint4(s[4 * c], s[4 * c + 1], s[4 * c + 2], s[4 * c + 3]);
+          }
+        }
+        if (half == 0) {
+          s_keep[b][head] = keep;
+          if (j == n - 1) {
+            s_row[b][0][head] = total;  // both maxima of this tile have been read
+            if (sp.records != nullptr && head < HT && h0 + head < p.H) {
+              float* rec = sp.records + ((static_cast<size_t>(slice) * p.T + t) * p.H + h0 + head) * (p.kv_rank + 2);
+              rec[0] = top;
+              rec[1] = total;
             }
           }
         }
+        asm volatile("fence.proxy.async.shared::cta;\n" ::: "memory");
+        __syncwarp();
+        // A named barrier: waiting there costs no issue slots.  Trip counts are fixed, so every arrival has its wait.
         asm volatile("bar.arrive %0, %1;\n" ::"r"(4 + b), "n"(kHandOver) : "memory");
       }
     }
-  } else {
-    {  // the query into TMEM, zeros in the lanes past the heads: a warp takes the lanes of its quadrant and every fourth atom
-      const int quad = warp & 3, head = quad * 32 + lane;
-      const bool there = head < HT && h0 + head < p.H;
-      const uint4* q = reinterpret_cast<const uint4*>(static_cast<const __nv_bfloat16*>(p.query) + (static_cast<size_t>(t) * p.H + h0 + head) * p.row);
-      const int words = p.row >> 3;
-      for (int c = warp >> 2; c < sp.atoms; c += kValueWarps / 4) {
-        uint32_t w[32];
-#pragma unroll
-        for (int e = 0; e < 8; ++e) {
-          const uint4 v = there && c * 8 + e < words ? __ldg(q + c * 8 + e) : make_uint4(0, 0, 0, 0);
-          w[4 * e] = v.x; w[4 * e + 1] = v.y; w[4 * e + 2] = v.z; w[4 * e + 3] = v.w;
-        }
-        TcSt32(tmem_q + (static_cast<uint32_t>(quad * 32) << 16) + c * 32, w);
-      }
-      asm volatile("tcgen05.wait::st.sync.aligned;\n" ::: "memory");
-      asm volatile("tcgen05.fence::before_thread_sync;\n" ::: "memory");
-      __syncwarp();
-      if (lane == 0) MbarArrive(qready);
-    }
-    const int gid = lane >> 2, tig = lane & 3;
-    const int pairs = (p.kv_rank + 15) >> 4;
-    float acc[MT][2 * NP][4];
-#pragma unroll
-    for (int m = 0; m < MT; ++m)
-#pragma unroll
-      for (int c = 0; c < 2 * NP; ++c)
-#pragma unroll
-        for (int e = 0; e < 4; ++e) acc[m][c][e] = 0.f;
+  } else {  // output: this thread's TMEM lane is channel 128 i + tid of accumulator i
+    const uint32_t lanes = static_cast<uint32_t>(warp * 32) << 16;
     int stage = 0;
-    uint32_t phase = 0;
     for (int j = 0; j < n; ++j) {
       const int b = j & 1, pos = (tile0 + j) * kMmaTile;
       asm volatile("bar.sync %0, %1;\n" ::"r"(4 + b), "n"(kHandOver) : "memory");
-      if (lane == 0) ok = MbarWait(full + 8 * stage, phase, abort_word) && ok;  // the scores are there, so the tile is
-      __syncwarp();
-      const uint32_t tile_addr = base + stage * tile_bytes;
       // Rows of the page outside the live range may hold anything: 0 times it must stay 0.
       const int live_lo = live.x - pos, live_hi = live.y - pos;
       if (live_lo > 0 || live_hi < kMmaTile) {
-        for (int i = tid; i < kMmaTile * sp.atoms * 8; i += kValueWarps * 32) {
+        for (int i = tid; i < kMmaTile * sp.atoms * 8; i += kOutWarps * 32) {
           const int r = i & (kMmaTile - 1);
-          if (r < live_lo || r >= live_hi) *reinterpret_cast<uint4*>(smem + stage * tile_bytes + TileWord(r, i / kMmaTile)) = make_uint4(0, 0, 0, 0);
+          if (r < live_lo || r >= live_hi) *reinterpret_cast<uint4*>(smem + 2 * kPBytes + stage * tile_bytes + TileWord(r, i / kMmaTile)) = make_uint4(0, 0, 0, 0);
         }
-        asm volatile("fence.proxy.async.shared::cta;\n" ::: "memory");  // before the stage is fetched into again
-        asm volatile("bar.sync 1, %0;\n" ::"n"(kValueWarps * 32) : "memory");
+        asm volatile("fence.proxy.async.shared::cta;\n" ::: "memory");
       }
+      if (j > 0) {
+        bool raised = false;
 #pragma unroll
-      for (int m = 0; m < MT; ++m) {
-        const float k0 = s_keep[b][m * 16 + gid], k1 = s_keep[b][m * 16 + gid + 8];
-        if (__any_sync(0xffffffffu, k0 != 1.f || k1 != 1.f)) {
+        for (int k = 0; k < kQuads; ++k) raised = raised || s_keep[b][k * 32 + lane] != 1.f;
+        if (__any_sync(0xffffffffu, raised)) {
+          ok = MbarWaitWarp(odone + 8 * (b ^ 1), ((j - 1) >> 1) & 1, lane, abort_word) && ok;
+          asm volatile("tcgen05.fence::after_thread_sync;\n" ::: "memory");
+          for (int c = 0; c < o_tiles * kOCols; c += 32) {
+            uint32_t o[32];
+            TcLd32(tmem_o + lanes + c, o);
+            asm volatile("tcgen05.wait::ld.sync.aligned;\n" ::: "memory");
+            const float* keep = s_keep[b] + c % kOCols;
 #pragma unroll
-          for (int c = 0; c < 2 * NP; ++c) {
-            acc[m][c][0] *= k0; acc[m][c][1] *= k0;
-            acc[m][c][2] *= k1; acc[m][c][3] *= k1;
+            for (int e = 0; e < 32; ++e) o[e] = __float_as_uint(__uint_as_float(o[e]) * keep[e]);
+            TcSt32(tmem_o + lanes + c, o);
           }
+          asm volatile("tcgen05.wait::st.sync.aligned;\n" ::: "memory");
         }
       }
+      asm volatile("tcgen05.fence::before_thread_sync;\n" ::: "memory");
+      __syncwarp();
+      if (lane == 0) MbarArrive(pready + 8 * b);
+      if (++stage == stages) stage = 0;
+    }
+    ok = MbarWaitWarp(odone + 8 * ((n - 1) & 1), ((n - 1) >> 1) & 1, lane, abort_word) && ok;
+    asm volatile("tcgen05.fence::after_thread_sync;\n" ::: "memory");
+    const float* totals = s_row[(n - 1) & 1][0];
+    for (int i = 0; i < o_tiles; ++i) {
+      const int channel = i * 128 + tid;
+      for (int g = 0; g < kQuads; ++g) {
+        uint32_t o[32];
+        TcLd32(tmem_o + lanes + i * kOCols + g * 32, o);
+        asm volatile("tcgen05.wait::ld.sync.aligned;\n" ::: "memory");
+        if (channel < p.kv_rank) {
 #pragma unroll
-      for (int k = 0; k < 4; ++k) {
-        uint32_t pf[MT][4];  // matrices (heads 0-7, positions 0-7), (8-15, 0-7), (0-7, 8-15), (8-15, 8-15)
-#pragma unroll
-        for (int m = 0; m < MT; ++m) LdMatrixX4(pf[m], SmemAddr(s_p[b] + (m * 16 + (lane & 15)) * kPStride + k * 16 + (lane >> 4) * 8));
-#pragma unroll
-        for (int i = 0; i < NP; ++i) {
-          const int pair = warp + kValueWarps * i;
-          if (pair < pairs) {
-            uint32_t v[4];  // (positions 0-7, channels 0-7), (8-15, 0-7), (0-7, 8-15), (8-15, 8-15), transposed
-            LdMatrixX4Trans(v, tile_addr + TileWord(k * 16 + (lane & 15), 2 * pair + (lane >> 4)));
-#pragma unroll
-            for (int m = 0; m < MT; ++m) {
-              MmaBf16(acc[m][2 * i], pf[m], v[0], v[1]);
-              MmaBf16(acc[m][2 * i + 1], pf[m], v[2], v[3]);
+          for (int e = 0; e < 32; ++e) {
+            const int hl = g * 32 + e, h = h0 + hl;
+            if (hl >= HT || h >= p.H) break;
+            const float v = __uint_as_float(o[e]);
+            if (sp.records != nullptr) {
+              sp.records[((static_cast<size_t>(slice) * p.T + t) * p.H + h) * (p.kv_rank + 2) + 2 + channel] = v;
+            } else {
+              static_cast<__nv_bfloat16*>(p.out)[(static_cast<size_t>(t) * p.H + h) * p.kv_rank + channel] = __float2bfloat16_rn(v / totals[hl]);
             }
           }
         }
       }
-      if (j + 2 < n) asm volatile("bar.arrive %0, %1;\n" ::"r"(6 + b), "n"(kHandOver) : "memory");
-      __syncwarp();
-      if (lane == 0) MbarArrive(free0 + 8 * stage);
-      if (++stage == stages) {
-        stage = 0;
-        phase ^= 1;
-      }
     }
-#pragma unroll
-    for (int m = 0; m < MT; ++m) {
-#pragma unroll
-      for (int half = 0; half < 2; ++half) {
-        const int hl = m * 16 + gid + half * 8, h = h0 + hl;
-        if (h >= p.H) continue;
-        const float total = s_row[(n - 1) & 1][0][hl], inv = total > 0.f ? 1.f / total : 0.f;
-#pragma unroll
-        for (int c2 = 0; c2 < 2 * NP; ++c2) {
-          const int c = (warp + kValueWarps * (c2 >> 1)) * 16 + (c2 & 1) * 8 + tig * 2;
-          if (c >= p.kv_rank) continue;
-          const float x = acc[m][c2][2 * half], y = acc[m][c2][2 * half + 1];
-          if (sp.records != nullptr) {
-            *reinterpret_cast<float2*>(sp.records + ((static_cast<size_t>(slice) * p.T + t) * p.H + h) * (p.kv_rank + 2) + 2 + c) = make_float2(x, y);
-          } else {
-            *reinterpret_cast<__nv_bfloat162*>(static_cast<__nv_bfloat16*>(p.out) + (static_cast<size_t>(t) * p.H + h) * p.kv_rank + c) =
-                __floats2bfloat162_rn(x * inv, y * inv);
-          }
-        }
-      }
-    }
+    asm volatile("tcgen05.fence::before_thread_sync;\n" ::: "memory");
   }
   if (!ok) atomicExch(&g_latent_status, 1);
-  asm volatile("tcgen05.fence::before_thread_sync;\n" ::: "memory");
   __syncthreads();
   if (warp == 0) {
     asm volatile("tcgen05.fence::after_thread_sync;\n" ::: "memory");
@@ -511,15 +502,11 @@ __global__ void __launch_bounds__(128) LatentCombine(LatentParams p, SliceParams
   }
 }
 
-constexpr int kMmaMaxSmem = 227 * 1024;
+constexpr int kMmaMaxSmem = 227 * 1024, kStaticSmem = 2048;
 
 int Atoms(int row) { return (row + 63) / 64; }
-// Stages beside the static shared memory (weights of up to 64 heads, barriers: under 20 KB).
-int Stages(int row) { return std::min(kMaxStages, (kMmaMaxSmem - 1024 - (Atoms(row) > 8 ? 10 : 20) * 1024) / (Atoms(row) * kAtomBytes)); }
-size_t MmaSmem(int row) { return 1024 + static_cast<size_t>(Stages(row)) * Atoms(row) * kAtomBytes; }
-
-// 16-head tiles of a CTA: enough for all heads where registers allow (two for latents wider than 256 channels, four up to that),
-// else the count that leaves the fewest absent heads.
+// 16-head tiles of a CTA: enough for all heads where TMEM allows (two for latents wider than 256 channels, four up to that), else
+// the count that leaves the fewest absent heads.
 int HeadTiles(int heads, int kv_rank)
 {
   const int most = kv_rank > 256 ? 2 : 4, need = (heads + 15) / 16;
@@ -530,11 +517,22 @@ int HeadTiles(int heads, int kv_rank)
   }
   return best;
 }
-
-bool MmaApplies(int kv_rank, int rot_dim)
+// TMEM columns beside the scores: the query, and O^T in accumulators of 128 channels.
+int FixedColumns(int mt, int kv_rank, int row) { return Atoms(row) * 32 + (kv_rank + 127) / 128 * ((mt + 1) / 2 * 32); }
+// What the last 128-channel operand of a tile may reach past its atoms.
+int Slack(int kv_rank, int row) { return std::max(0, (kv_rank + 127) / 128 * 2 - Atoms(row)) * kAtomBytes; }
+int Stages(int mt, int kv_rank, int row)
 {
-  const int row = kv_rank + rot_dim;
-  return kv_rank % 8 == 0 && rot_dim % 8 == 0 && kv_rank <= 512 && Atoms(row) * 32 + 2 * kMmaTile <= 512 && Stages(row) >= 2;
+  return std::min(kMaxStages, (kMmaMaxSmem - kStaticSmem - 1024 - 2 * mt * 16 * 128 - Slack(kv_rank, row)) / (Atoms(row) * kAtomBytes));
+}
+size_t MmaSmem(int mt, int kv_rank, int row)
+{
+  return 1024 + 2 * mt * 16 * 128 + static_cast<size_t>(Stages(mt, kv_rank, row)) * Atoms(row) * kAtomBytes + Slack(kv_rank, row);
+}
+bool MmaApplies(int heads, int kv_rank, int rot_dim)
+{
+  const int row = kv_rank + rot_dim, mt = HeadTiles(heads, kv_rank);
+  return kv_rank % 8 == 0 && rot_dim % 8 == 0 && kv_rank <= 512 && FixedColumns(mt, kv_rank, row) + kMmaTile <= 512 && Stages(mt, kv_rank, row) >= 2;
 }
 
 // Slices of the positions: the fewest waves of CTAs times the tiles a CTA walks, for the longest live range a row may have.
@@ -576,14 +574,12 @@ bool EncodePool(CUtensorMap* map, const LatentParams& p)
                 CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE) == CUDA_SUCCESS;
 }
 
-template <int MT, int NP>
+template <int MT>
 cudaError_t LaunchTc(const CUtensorMap& map, const LatentParams& p, const SliceParams& sp, cudaStream_t st)
 {
   const dim3 grid(sp.slices, (p.H + 16 * MT - 1) / (16 * MT), p.T);
-  return LaunchChained(LatentAttentionTc<MT, NP>, grid, kMmaThreads, MmaSmem(p.row), st, map, p, sp);
+  return LaunchChained(LatentAttentionTc<16 * MT>, grid, kMmaThreads, MmaSmem(MT, p.kv_rank, p.row), st, map, p, sp);
 }
-
-#define TLALOC_LATENT_FORMS(X) X(1, 1) X(2, 1) X(3, 1) X(4, 1) X(1, 2) X(2, 2)
 
 cudaError_t PrepareLatentAttention()
 {
@@ -591,10 +587,12 @@ cudaError_t PrepareLatentAttention()
   return once.Run([](int) {
     TensorMapEncoder();
     cudaError_t e = cudaSuccess;
-    const int most = static_cast<int>(std::max({MmaSmem(640), MmaSmem(576), MmaSmem(512), MmaSmem(448), MmaSmem(384), MmaSmem(320), MmaSmem(256), MmaSmem(192)}));
-#define TLALOC_OPT_IN(MT, NP) \
-  if (e == cudaSuccess) e = cudaFuncSetAttribute(LatentAttentionTc<MT, NP>, cudaFuncAttributeMaxDynamicSharedMemorySize, std::min(most, kMmaMaxSmem - (MT > 2 ? 20 : 10) * 1024));
-    TLALOC_LATENT_FORMS(TLALOC_OPT_IN)
+#define TLALOC_OPT_IN(MT) \
+  if (e == cudaSuccess) e = cudaFuncSetAttribute(LatentAttentionTc<16 * MT>, cudaFuncAttributeMaxDynamicSharedMemorySize, kMmaMaxSmem - kStaticSmem)
+    TLALOC_OPT_IN(1);
+    TLALOC_OPT_IN(2);
+    TLALOC_OPT_IN(3);
+    TLALOC_OPT_IN(4);
 #undef TLALOC_OPT_IN
     return e;
   });
@@ -611,14 +609,18 @@ int ReadLatentStatus()
 }
 KernelSetup g_setup(PrepareLatentAttention, ReadLatentStatus);
 
-cudaError_t LaunchTcForm(const CUtensorMap& map, const LatentParams& p, const SliceParams& sp, cudaStream_t st)
+cudaError_t LaunchTcForm(const CUtensorMap& map, const LatentParams& p, SliceParams sp, cudaStream_t st)
 {
-  const int mt = HeadTiles(p.H, p.kv_rank), np = ((p.kv_rank + 15) / 16 + kValueWarps - 1) / kValueWarps;
-#define TLALOC_TRY(MT, NP) \
-  if (mt == MT && np <= NP) return LaunchTc<MT, NP>(map, p, sp, st);
-  TLALOC_LATENT_FORMS(TLALOC_TRY)
-#undef TLALOC_TRY
-  return cudaErrorInvalidValue;
+  const int mt = HeadTiles(p.H, p.kv_rank);
+  sp.atoms = Atoms(p.row);
+  sp.stages = Stages(mt, p.kv_rank, p.row);
+  sp.score_buffers = FixedColumns(mt, p.kv_rank, p.row) + 2 * kMmaTile <= 512 ? 2 : 1;
+  switch (mt) {
+    case 1: return LaunchTc<1>(map, p, sp, st);
+    case 2: return LaunchTc<2>(map, p, sp, st);
+    case 3: return LaunchTc<3>(map, p, sp, st);
+    default: return LaunchTc<4>(map, p, sp, st);
+  }
 }
 
 int MaxLive(int max_live, int window, int64_t table_positions)
@@ -637,7 +639,7 @@ using namespace tlaloc_b200;
 extern "C" size_t tlaloc_b200_latent_attention_scratch_bytes(int32_t num_tokens, int32_t num_heads, int32_t kv_rank, int32_t rot_dim,
                                                              int32_t max_live)
 {
-  if (num_tokens < 1 || num_heads < 1 || max_live < 1 || !MmaApplies(kv_rank, rot_dim)) return 0;
+  if (num_tokens < 1 || num_heads < 1 || max_live < 1 || !MmaApplies(num_heads, kv_rank, rot_dim)) return 0;
   // fewer rows may take more slices: the largest need over the row counts up to num_tokens
   size_t most = 0;
   for (int rows = 1;; rows = std::min(2 * rows, num_tokens)) {
@@ -692,7 +694,7 @@ extern "C" int tlaloc_b200_latent_attention(const void* query, const void* pool,
   p.scale = scale;
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   CUtensorMap map;
-  if (dtype == TLALOC_B200_BF16 && !OrderFaithful() && MmaApplies(kv_rank, rot_dim) && pool_ld % 8 == 0 && Aligned16(query) && Aligned16(pool) &&
+  if (dtype == TLALOC_B200_BF16 && !OrderFaithful() && MmaApplies(num_heads, kv_rank, rot_dim) && pool_ld % 8 == 0 && Aligned16(query) && Aligned16(pool) &&
       Aligned16(out) && (scratch == nullptr || Aligned16(scratch)) && EncodePool(&map, p)) {
     cudaError_t e = PrepareLatentAttention();
     if (e != cudaSuccess) return CudaFail("LATENT_ATTENTION set-up", e);
@@ -706,8 +708,6 @@ extern "C" int tlaloc_b200_latent_attention(const void* query, const void* pool,
     }
     if (sp.slices == 1) sp.slice_tiles = 0x3fffffff;
     sp.records = sp.slices > 1 ? static_cast<float*>(scratch) : nullptr;
-    sp.atoms = Atoms(p.row);
-    sp.stages = Stages(p.row);
     e = LaunchTcForm(map, p, sp, st);
     if (e == cudaSuccess && sp.slices > 1) e = LaunchChained(LatentCombine, dim3(num_heads, num_tokens), 128, 0, st, p, sp);
     if (e != cudaSuccess) return CudaFail("LATENT_ATTENTION launch", e);

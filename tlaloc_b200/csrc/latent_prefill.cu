@@ -43,15 +43,6 @@ __host__ __device__ constexpr uint32_t InstrDesc(int n, bool b_mn_major)  // f32
 {
   return (1u << 4) | (1u << 7) | (1u << 10) | (b_mn_major ? 1u << 16 : 0u) | (static_cast<uint32_t>(n >> 3) << 17) | (8u << 24);
 }
-__device__ __forceinline__ void Mma(uint32_t d_tmem, uint64_t a_desc, uint64_t b_desc, uint32_t idesc, uint32_t accumulate)
-{
-  asm volatile(
-      "{\n\t.reg .pred p;\n\t"
-      "setp.ne.b32 p, %4, 0;\n\t"
-      "tcgen05.mma.cta_group::1.kind::f16 [%0], %1, %2, %3, p;\n\t}\n" ::"r"(d_tmem),
-      "l"(a_desc), "l"(b_desc), "r"(idesc), "r"(accumulate)
-      : "memory");
-}
 __device__ __forceinline__ void TmaBox(uint32_t dst, const CUtensorMap* map, int x, int y, int z, uint32_t bar)
 {
   asm volatile("cp.async.bulk.tensor.3d.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1, {%2, %3, %4}], [%5];\n" ::"r"(dst),
@@ -168,9 +159,9 @@ __global__ void __launch_bounds__(kThreads, 1)
           const int width = c < dim_atoms ? a.dim - 64 * c : a.rot - 64 * (c - dim_atoms);
           if (width > 48) {
 #pragma unroll
-            for (int k = 0; k < 4; ++k) Mma(acc, qa + 2 * k, ka + 2 * k, s_idesc, c > 0 || k > 0 ? 1u : 0u);
+            for (int k = 0; k < 4; ++k) TcMmaBf16(acc, qa + 2 * k, ka + 2 * k, s_idesc, c > 0 || k > 0 ? 1u : 0u);
           } else {
-            for (int k = 0; 16 * k < width; ++k) Mma(acc, qa + 2 * k, ka + 2 * k, s_idesc, c > 0 || k > 0 ? 1u : 0u);
+            for (int k = 0; 16 * k < width; ++k) TcMmaBf16(acc, qa + 2 * k, ka + 2 * k, s_idesc, c > 0 || k > 0 ? 1u : 0u);
           }
         }
         TcCommit(sfull + 8 * b);
