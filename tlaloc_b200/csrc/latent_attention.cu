@@ -11,7 +11,7 @@
 //   MMA lane        scores S = Q C^T: the query is the A operand out of TMEM (heads are its lanes, put there once), the tile is B;
 //                   then O^T += C^T P^T: the same tile, its channels now the M rows (an MN-major A operand, 128 channels at a time), the
 //                   weights B, accumulators of 128 channel lanes x heads in TMEM
-//   2 - 4 warps     softmax: two threads own a head's row of 64 scores and exchange its maximum; the weights go to shared memory as
+//   4 - 8 warps     softmax: four threads own a head's row of 64 scores and exchange its maximum; the weights go to shared memory as
 //                   bf16.  The running maximum is raised lazily (the exponentials stay below 2^8), so O is rarely rescaled
 //   four warps      rescale O when a maximum was raised, blank the dead rows of the edge tiles, and write the result
 // Slices leave {max, sum, acc[kv_rank]} records in f32 that LatentCombine merges in slice
@@ -122,9 +122,9 @@ using namespace tc;
 
 constexpr int kAtomBytes = 64 * 128;
 constexpr int kMmaTile = 64, kMaxStages = 4;
-// Warps 0 - 3 write the output; 4, 5 and 8, 9 are the softmax: a warp reads the TMEM lanes of its number modulo 4, so both of a pair
-// see the same heads.
-constexpr int kOutWarps = 4, kProducerWarp = 6, kMmaWarp = 7, kMmaThreads = 10 * 32;
+// Warps 0 - 3 write the output; 4, 8, 12, 16 (heads 0 - 31) and 5, 9, 13, 17 (32 - 63) are the softmax: a warp reads the TMEM lanes of
+// its number modulo 4.  10, 11, 14, 15 have no work.
+constexpr int kOutWarps = 4, kProducerWarp = 6, kMmaWarp = 7, kParts = 4, kMmaThreads = 18 * 32;
 
 __device__ __forceinline__ float Exp2(float x)
 {
@@ -160,12 +160,12 @@ __global__ void __launch_bounds__(kMmaThreads, 1)
   constexpr int kQuads = (HT + 31) / 32;   // TMEM lane quadrants with heads in them
   constexpr int kOCols = kQuads * 32;      // columns of one O^T accumulator
   constexpr int kPBytes = HT * 128;        // one tile's weights: [heads][64 positions] bf16, 128-byte swizzle
-  constexpr int kHandOver = (kOutWarps + 2 * kQuads) * 32;
+  constexpr int kHandOver = (kOutWarps + kParts * kQuads) * 32;
   GridDependencySync();
   extern __shared__ unsigned char smem_raw[];
   __shared__ alignas(8) uint64_t bars[2 * kMaxStages + 9];
   __shared__ uint32_t slot_store[2];
-  __shared__ float s_keep[2][kOCols], s_row[2][2][kOCols];  // s_row: [tile parity][half of the positions][head]
+  __shared__ float s_keep[2][kOCols], s_row[2][kParts][kOCols];  // s_row: [tile parity][quarter of the positions][head]
   const uint32_t base = (SmemAddr(smem_raw) + 1023u) & ~1023u;  // the swizzle is a function of address bits 4..9
   unsigned char* smem = smem_raw + (base - SmemAddr(smem_raw));
   const int tile_bytes = sp.atoms * kAtomBytes, stages = sp.stages;
@@ -195,11 +195,11 @@ __global__ void __launch_bounds__(kMmaThreads, 1)
     }
     for (int i = 0; i < 2; ++i) {
       MbarInit(sfull + 8 * i, 1);
-      MbarInit(sempty + 8 * i, 2 * kQuads);
+      MbarInit(sempty + 8 * i, kParts * kQuads);
       MbarInit(pready + 8 * i, kOutWarps);
       MbarInit(odone + 8 * i, 1);
     }
-    MbarInit(qready, 8);
+    MbarInit(qready, 12);
     asm volatile("fence.mbarrier_init.release.cluster;\n" ::: "memory");
   }
   if (warp == 0) {
@@ -214,13 +214,13 @@ __global__ void __launch_bounds__(kMmaThreads, 1)
   const uint32_t tmem_q = tmem + sp.score_buffers * kMmaTile, tmem_o = tmem_q + sp.atoms * 32;
   bool ok = true;
 
-  if (warp != kProducerWarp && warp != kMmaWarp) {
+  if ((warp & 3) < 2 ? warp < 18 : warp < kOutWarps) {
     // The query into TMEM, zeros in the lanes past the heads; the warps of a quadrant share its atoms.
     const int quad = warp & 3, head = quad * 32 + lane;
     const bool there = head < HT && h0 + head < p.H;
     const uint4* q = reinterpret_cast<const uint4*>(static_cast<const __nv_bfloat16*>(p.query) + (static_cast<size_t>(t) * p.H + h0 + head) * p.row);
     const int words = p.row >> 3;
-    for (int c = warp >> 2; c < sp.atoms; c += quad < 2 ? 3 : 1) {
+    for (int c = warp >> 2; c < sp.atoms; c += quad < 2 ? 5 : 1) {
       uint32_t w[32];
 #pragma unroll
       for (int e = 0; e < 8; ++e) {
@@ -325,25 +325,25 @@ __global__ void __launch_bounds__(kMmaThreads, 1)
       }
     }
     __syncwarp();
-  } else if (warp >= kOutWarps) {  // softmax
-    const int quad = warp & 3, half = warp >= 8 ? 1 : 0, head = quad * 32 + lane;  // TMEM lane; positions [32 half, 32 half + 32)
+  } else if (warp >= kOutWarps) {  // softmax, or nothing
+    const int quad = warp & 3, part = (warp >> 2) - 1, head = quad * 32 + lane;  // TMEM lane; positions [16 part, 16 part + 16)
     const uint32_t lanes = static_cast<uint32_t>(quad * 32) << 16;
-    constexpr int kHalf = kMmaTile / 2;
-    // The other half of the row: the two warps of a quad meet at a named barrier of 64 threads.
-    auto other = [&](int b, float mine) {
-      s_row[b][half][head] = mine;
-      asm volatile("bar.sync %0, 64;\n" ::"r"(2 + quad) : "memory");
-      return s_row[b][half ^ 1][head];
+    constexpr int kPart = kMmaTile / kParts;
+    // Every part's value: the four warps of a quad meet at a named barrier of 128 threads.
+    auto share = [&](int b, float mine) {
+      s_row[b][part][head] = mine;
+      asm volatile("bar.sync %0, 128;\n" ::"r"(2 + quad) : "memory");
+      return make_float4(s_row[b][0][head], s_row[b][1][head], s_row[b][2][head], s_row[b][3][head]);
     };
     if (quad < kQuads) {
       const float scale = p.scale * 1.4426950408889634f;
       float top = -INFINITY, sum = 0.f;
       for (int j = 0; j < n; ++j) {
-        const int b = j & 1, tile_pos = (tile0 + j) * kMmaTile, pos = tile_pos + half * kHalf;
+        const int b = j & 1, tile_pos = (tile0 + j) * kMmaTile, pos = tile_pos + part * kPart;
         ok = MbarWaitWarp(sfull + 8 * b, (j >> 1) & 1, lane, abort_word) && ok;
         asm volatile("tcgen05.fence::after_thread_sync;\n" ::: "memory");
-        uint32_t s[kHalf];
-        TcLd32(tmem + lanes + (sp.score_buffers == 2 ? b * kMmaTile : 0) + half * kHalf, s);
+        uint32_t s[kPart];
+        TcLd16(tmem + lanes + (sp.score_buffers == 2 ? b * kMmaTile : 0) + part * kPart, s);
         asm volatile("tcgen05.wait::ld.sync.aligned;\n" ::: "memory");
         asm volatile("tcgen05.fence::before_thread_sync;\n" ::: "memory");
         __syncwarp();
@@ -351,14 +351,14 @@ __global__ void __launch_bounds__(kMmaThreads, 1)
         float t4[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
         const bool edge = tile_pos < live.x || tile_pos + kMmaTile > live.y;
 #pragma unroll
-        for (int e = 0; e < kHalf; ++e) {
+        for (int e = 0; e < kPart; ++e) {
           float v = __uint_as_float(s[e]) * scale;
           if (edge && (pos + e < live.x || pos + e >= live.y)) v = -INFINITY;
           s[e] = __float_as_uint(v);
           t4[e & 3] = fmaxf(t4[e & 3], v);
         }
-        const float mine = fmaxf(fmaxf(t4[0], t4[1]), fmaxf(t4[2], t4[3]));
-        const float tile_top = fmaxf(mine, other(b, mine));  // finite: a tile holds at least one live position
+        const float4 tops = share(b, fmaxf(fmaxf(t4[0], t4[1]), fmaxf(t4[2], t4[3])));
+        const float tile_top = fmaxf(fmaxf(tops.x, tops.y), fmaxf(tops.z, tops.w));  // finite: a tile holds at least one live position
         float keep = 1.f;
         if (tile_top > top + kLazy || top == -INFINITY) {
           const float next = fmaxf(top, tile_top);
@@ -368,26 +368,30 @@ __global__ void __launch_bounds__(kMmaThreads, 1)
         }
         float add[2] = {0.f, 0.f};
 #pragma unroll
-        for (int e = 0; e < kHalf; e += 2) {
+        for (int e = 0; e < kPart; e += 2) {
           const float p0 = Exp2(__uint_as_float(s[e]) - top), p1 = Exp2(__uint_as_float(s[e + 1]) - top);
           add[0] += p0;
           add[1] += p1;
           s[e / 2] = Pack(p0, p1);
         }
         sum += add[0] + add[1];
-        const float total = j == n - 1 ? sum + other(b ^ 1, sum) : 0.f;
+        float total = 0.f;
+        if (j == n - 1) {
+          const float4 sums = share(b ^ 1, sum);
+          total = (sums.x + sums.y) + (sums.z + sums.w);
+        }
         if (j >= 2) ok = MbarWaitWarp(odone + 8 * b, ((j >> 1) - 1) & 1, lane, abort_word) && ok;  // the weights of tile j - 2 have been read
         if (head < HT) {
           unsigned char* dst = smem + b * kPBytes + head * 128;
 #pragma unroll
-          for (int c = 0; c < 4; ++c) {
-            *reinterpret_cast<uint4*>(dst + (((half * 4 + c) ^ (head & 7)) << 4)) = make_uint4(s[4 * c], s[4 * c + 1], s[4 * c + 2], s[4 * c + 3]);
+          for (int c = 0; c < 2; ++c) {
+            *reinterpret_cast<uint4*>(dst + (((part * 2 + c) ^ (head & 7)) << 4)) = make_uint4(s[4 * c], s[4 * c + 1], s[4 * c + 2], s[4 * c + 3]);
           }
         }
-        if (half == 0) {
+        if (part == 0) {
           s_keep[b][head] = keep;
           if (j == n - 1) {
-            s_row[b][0][head] = total;  // both maxima of this tile have been read
+            s_row[b][0][head] = total;  // every maximum of this tile has been read
             if (sp.records != nullptr && head < HT && h0 + head < p.H) {
               float* rec = sp.records + ((static_cast<size_t>(slice) * p.T + t) * p.H + h0 + head) * (p.kv_rank + 2);
               rec[0] = top;
@@ -445,21 +449,21 @@ __global__ void __launch_bounds__(kMmaThreads, 1)
     const float* totals = s_row[(n - 1) & 1][0];
     for (int i = 0; i < o_tiles; ++i) {
       const int channel = i * 128 + tid;
-      for (int g = 0; g < kQuads; ++g) {
-        uint32_t o[32];
-        TcLd32(tmem_o + lanes + i * kOCols + g * 32, o);
+#pragma unroll 1
+      for (int g = 0; g < HT; g += 16) {
+        uint32_t o[16];
+        TcLd16(tmem_o + lanes + i * kOCols + g, o);
         asm volatile("tcgen05.wait::ld.sync.aligned;\n" ::: "memory");
         if (channel < p.kv_rank) {
+          const size_t at = static_cast<size_t>(t) * p.H + h0 + g;
+          float* rec = sp.records + (static_cast<size_t>(slice) * p.T * p.H + at) * (p.kv_rank + 2) + 2 + channel;
+          __nv_bfloat16* out = static_cast<__nv_bfloat16*>(p.out) + at * p.kv_rank + channel;
+          const int heads = p.H - h0 - g;
 #pragma unroll
-          for (int e = 0; e < 32; ++e) {
-            const int hl = g * 32 + e, h = h0 + hl;
-            if (hl >= HT || h >= p.H) break;
-            const float v = __uint_as_float(o[e]);
-            if (sp.records != nullptr) {
-              sp.records[((static_cast<size_t>(slice) * p.T + t) * p.H + h) * (p.kv_rank + 2) + 2 + channel] = v;
-            } else {
-              static_cast<__nv_bfloat16*>(p.out)[(static_cast<size_t>(t) * p.H + h) * p.kv_rank + channel] = __float2bfloat16_rn(v / totals[hl]);
-            }
+          for (int e = 0; e < 16; ++e) {
+            if (e >= heads) break;
+            if (sp.records != nullptr) rec[e * (p.kv_rank + 2)] = __uint_as_float(o[e]);
+            else out[e * p.kv_rank] = __float2bfloat16_rn(__uint_as_float(o[e]) / totals[g + e]);
           }
         }
       }
@@ -502,7 +506,8 @@ __global__ void __launch_bounds__(128) LatentCombine(LatentParams p, SliceParams
   }
 }
 
-constexpr int kMmaMaxSmem = 227 * 1024, kStaticSmem = 2048;
+constexpr int kMmaMaxSmem = 227 * 1024;
+constexpr int StaticSmem(int mt) { return mt > 2 ? 3072 : 2048; }  // at least what the kernel declares
 
 int Atoms(int row) { return (row + 63) / 64; }
 // 16-head tiles of a CTA: enough for all heads where TMEM allows (two for latents wider than 256 channels, four up to that), else
@@ -523,7 +528,7 @@ int FixedColumns(int mt, int kv_rank, int row) { return Atoms(row) * 32 + (kv_ra
 int Slack(int kv_rank, int row) { return std::max(0, (kv_rank + 127) / 128 * 2 - Atoms(row)) * kAtomBytes; }
 int Stages(int mt, int kv_rank, int row)
 {
-  return std::min(kMaxStages, (kMmaMaxSmem - kStaticSmem - 1024 - 2 * mt * 16 * 128 - Slack(kv_rank, row)) / (Atoms(row) * kAtomBytes));
+  return std::min(kMaxStages, (kMmaMaxSmem - StaticSmem(mt) - 1024 - 2 * mt * 16 * 128 - Slack(kv_rank, row)) / (Atoms(row) * kAtomBytes));
 }
 size_t MmaSmem(int mt, int kv_rank, int row)
 {
@@ -588,7 +593,7 @@ cudaError_t PrepareLatentAttention()
     TensorMapEncoder();
     cudaError_t e = cudaSuccess;
 #define TLALOC_OPT_IN(MT) \
-  if (e == cudaSuccess) e = cudaFuncSetAttribute(LatentAttentionTc<16 * MT>, cudaFuncAttributeMaxDynamicSharedMemorySize, kMmaMaxSmem - kStaticSmem)
+  if (e == cudaSuccess) e = cudaFuncSetAttribute(LatentAttentionTc<16 * MT>, cudaFuncAttributeMaxDynamicSharedMemorySize, kMmaMaxSmem - StaticSmem(MT))
     TLALOC_OPT_IN(1);
     TLALOC_OPT_IN(2);
     TLALOC_OPT_IN(3);
