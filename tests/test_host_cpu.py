@@ -31,6 +31,37 @@ def test_library_loads_and_exports_every_declared_symbol():
     assert seen == [b""]
 
 
+def test_a_subset_of_the_kernels_is_a_library_of_its_own():
+    path = B.build(subset="latent", own=True)
+    assert os.path.basename(path) == "libtlaloc_latent.so"
+    lib = ctypes.CDLL(path)  # every symbol it needs is in it
+    for name in ("init", "device_status", "embedding", "argmax", "dense_gemm", "rmsnorm_pair", "latent_kv_write", "rope_interleaved",
+                 "latent_attention", "latent_attention_scratch_bytes", "latent_gather", "window_attention", "window_attention_applies"):
+        assert hasattr(lib, "tlaloc_b200_" + name), name
+    assert not hasattr(lib, "tlaloc_b200_int8_gemm")
+
+
+def test_dense_and_latent_refusals_need_no_gpu():
+    lib = N.lib()
+    one, i = ctypes.c_void_p(16), N.INVALID_ARGUMENT
+    p = N.DenseProblem(x=16, w=16, y=16, ld_x=8, ld_y=8, k=8, n=8, batch=1, act=0, y_dtype=N.F32)
+    call = lambda count=1, dtype=N.BF16, m=1: lib.tlaloc_b200_dense_gemm((N.DenseProblem * 2)(p, p), count, dtype, m, 0, None)
+    assert call(count=3) == i and call(dtype=N.S8) == i and call(m=-1) == i and call(m=0) == N.OK
+    for field, bad in (("k", 0), ("ld_x", 4), ("ld_y", 4), ("act", 7), ("y_dtype", N.S8), ("x", None), ("batch", 0)):
+        was = getattr(p, field)
+        setattr(p, field, bad)
+        assert call() == i, field
+        setattr(p, field, was)
+    att = lambda **kw: lib.tlaloc_b200_latent_attention(one, one, kw.get("ld", 56), N.BF16, one, None, one, one, None, 0, kw.get("rows", 1), 3, 48, 8, 9,
+                                                        64, 4, kw.get("tables", 1), kw.get("window", 0), 0, 0.1, None)
+    assert att(ld=40) == i and att(rows=2) == i and att(window=-1) == i and att(rows=0) == N.OK
+    assert lib.tlaloc_b200_window_attention_applies(128, 64, 128) == 1 and lib.tlaloc_b200_window_attention_applies(12, 4, 10) == 0
+    win = lambda **kw: lib.tlaloc_b200_window_attention(one, one, one, 8, one, 96, 48, one, 48, kw.get("q", 2), kw.get("k", 2), 0, 2, 24, 8, 24, 0,
+                                                        kw.get("scale", 0.1), None)
+    assert win(q=3) == i and win(scale=-1.0) == N.UNSUPPORTED and win(q=0) == N.OK
+    assert lib.tlaloc_b200_latent_gather(one, 56, N.BF16, one, one, 56, 200, 100, 56, 9, 64, 4, None) == i
+
+
 def test_argument_refusals_need_no_gpu():
     lib = N.lib()
     # a null pointer, a bad dtype and a bad shape are refused before any CUDA call

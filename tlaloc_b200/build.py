@@ -23,7 +23,7 @@ CSRC = os.path.join(HERE, "csrc")
 OBJ = os.path.join(HERE, "build")
 LIB_DIR = os.path.join(HERE, "lib")
 LIB = os.path.join(LIB_DIR, "libtlaloc_kernels.so")
-SUBSETS = {"latent": ("runtime", "decode_ops", "dense_gemm", "dense_gemm_tc", "latent_ops", "latent_attention", "latent_prefill")}
+SUBSETS = {"latent": ("runtime", "token_ops", "dense_gemm", "dense_gemm_tc", "latent_ops", "latent_attention", "latent_prefill")}
 INCLUDE = os.path.join(os.path.dirname(HERE), "include")
 
 NVCC_FLAGS = [
@@ -58,11 +58,12 @@ def nvcc() -> str | None:
     return shutil.which("nvcc") or ("/usr/local/cuda/bin/nvcc" if os.path.exists("/usr/local/cuda/bin/nvcc") else None)
 
 
-def build(force: bool = False, verbose: bool = False, subset: str | None = None) -> str:
-    """Path of an up-to-date library: the full one, or (subset given) one that holds at least the subset's kernels."""
+def build(force: bool = False, verbose: bool = False, subset: str | None = None, own: bool = False) -> str:
+    """Path of an up-to-date library: the full one, or (subset given) one that holds at least the subset's kernels.  own: the
+    subset's own library even where the full one would do."""
     lib = library(subset)
     if not force:
-        for current in (None, subset):
+        for current in (subset,) if own else (None, subset):
             if up_to_date(current) and (current == subset or subset is not None):
                 return library(current)
     cc = nvcc()
@@ -89,7 +90,7 @@ def build(force: bool = False, verbose: bool = False, subset: str | None = None)
 
     with concurrent.futures.ThreadPoolExecutor(max_workers=8) as pool:
         objs = list(pool.map(compile_one, sources(subset)))
-    r = subprocess.run([cc, "-shared", "-o", lib, *objs, "-gencode", "arch=compute_100a,code=sm_100a"],
+    r = subprocess.run([cc, "-shared", "-Xlinker", "--no-undefined", "-o", lib, *objs, "-gencode", "arch=compute_100a,code=sm_100a"],
                        capture_output=True, text=True)
     if r.returncode != 0:
         sys.stderr.write(r.stdout + r.stderr)
