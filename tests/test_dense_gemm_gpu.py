@@ -8,6 +8,16 @@ pytestmark = pytest.mark.gpu
 DEV = "cuda:0"
 
 
+@pytest.fixture(autouse=True)
+def no_wait_runs_out():
+    """Every device-side wait is bounded; one that runs out leaves a status word (and a wrong result)."""
+    yield
+    from tlaloc_b200 import _native
+
+    torch.cuda.synchronize()
+    assert _native.lib().tlaloc_b200_device_status() == 0
+
+
 def reference(x, w, bias=None, residual=None, relu2=False):
     y = x.double() @ w.double().transpose(-1, -2)
     if bias is not None:
@@ -116,10 +126,3 @@ def test_bad_arguments_are_refused():
                 lambda: ops.dense(x, w, y, residual=torch.zeros((4, 8), device=DEV, dtype=torch.bfloat16))):
         with pytest.raises(ValueError):
             bad()
-
-
-def test_no_wait_ran_out():
-    from tlaloc_b200 import _native
-
-    torch.cuda.synchronize()
-    assert _native.lib().tlaloc_b200_device_status() == 0

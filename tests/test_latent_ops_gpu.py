@@ -14,6 +14,16 @@ DEV = "cuda:0"
 TYPES = [torch.float32, torch.bfloat16]
 
 
+@pytest.fixture(autouse=True)
+def no_wait_runs_out():
+    """Every device-side wait is bounded; one that runs out leaves a status word (and a wrong result)."""
+    yield
+    from tlaloc_b200 import _native
+
+    torch.cuda.synchronize()
+    assert _native.lib().tlaloc_b200_device_status() == 0
+
+
 def gen(seed):
     g = torch.Generator(device=DEV)
     g.manual_seed(seed)
@@ -206,7 +216,7 @@ def window_reference(q, k, k_rot, v, first, scale, window):
 @pytest.mark.parametrize("heads,dim,rot,vdim", [(3, 24, 8, 40), (2, 128, 64, 128), (2, 64, 32, 64), (1, 72, 16, 136), (2, 192, 64, 256), (2, 64, 0, 96)])
 @pytest.mark.parametrize("T,first,window", [(1, 0, 0), (2, 5, 3), (128, 0, 0), (129, 0, 1), (100, 28, 128), (300, 400, 129), (260, 127, 50), (130, 1000, 0)])
 def test_expanded_attention(heads, dim, rot, vdim, T, first, window):
-    from tlaloc_b200 import _native, ops
+    from tlaloc_b200 import ops
 
     L = first + T
     q = 2 * randn(T, heads, dim + rot, seed=1)
@@ -219,7 +229,6 @@ def test_expanded_attention(heads, dim, rot, vdim, T, first, window):
     want = window_reference(q, kv[:, :, :dim], lat[:, 16:], kv[:, :, dim:], first, scale, window)
     assert float((out[:, :heads * vdim].double() - want).abs().max()) <= 2.5e-2
     assert bool((out[:, heads * vdim:] == 5).all())
-    assert _native.lib().tlaloc_b200_device_status() == 0
 
 
 @pytest.mark.parametrize("window", [64, 127, 128, 129, 300])
@@ -242,6 +251,29 @@ def test_expanded_attention_needle_at_the_window_edge(window):
             assert abs(got - 3.0) < 0.05 if distance < window else abs(got) < 0.2, (i, distance, got)
             want = window_reference(q, kv[:, :, :dim], k_rot, kv[:, :, dim:], first, 0.2, window)
             assert float((out.double() - want).abs().max()) <= 2e-2
+
+
+def test_the_same_launches_many_times_over():
+    """A whole GPU of CTAs whose loads contend: every repetition gives the same bits, prompt portions and decoding alike."""
+    from tlaloc_b200 import ops
+
+    T, L, heads = 1024, 3072, 32
+    q, kv, lat = randn(T, heads, 192, dtype=torch.bfloat16), randn(L, heads, 256, seed=1, dtype=torch.bfloat16), randn(L, 64, seed=2, dtype=torch.bfloat16)
+    first = None
+    for _ in range(150):
+        out = torch.empty((T, heads * 128), device=DEV, dtype=torch.bfloat16)
+        ops.window_attention(q, kv[:, :, :128], lat, kv[:, :, 128:], out, first_query=L - T, scale=0.07, window=2048)
+        first = out if first is None else first
+        assert torch.equal(out, first)
+    pool = randn(48 * 33 + 1, 64, 576, dtype=torch.bfloat16)
+    table = (1 + torch.randperm(48 * 33, device=DEV)).int().view(48, 33)
+    ends, ql = torch.full((48,), 2100, dtype=torch.int32, device=DEV), randn(48, heads, 576, seed=3, dtype=torch.bfloat16)
+    scratch, first = torch.empty((1 << 24,), device=DEV), None
+    for _ in range(150):
+        out = torch.empty((48, heads, 512), device=DEV, dtype=torch.bfloat16)
+        ops.latent_attention(ql, pool, table, ends, out, kv_rank=512, scale=0.04, window=2000, scratch=scratch)
+        first = out if first is None else first
+        assert torch.equal(out, first)
 
 
 @pytest.mark.parametrize("dtype", TYPES)

@@ -17,6 +17,16 @@ ROOT = os.path.dirname(os.path.dirname(os.path.abspath(__file__)))
 F32, BF16 = torch.float32, torch.bfloat16
 
 
+@pytest.fixture(autouse=True)
+def no_wait_runs_out():
+    """Every device-side wait is bounded; one that runs out leaves a status word (and a wrong result)."""
+    yield
+    from tlaloc_b200 import _native
+
+    torch.cuda.synchronize()
+    assert _native.lib().tlaloc_b200_device_status() == 0
+
+
 def build(config, weights, dtype=F32, max_len=512, blocks=64, **kw):
     from tlaloc_b200.engine import Engine
     from tlaloc_b200.latent_decoder import LatentDecoder, LatentDecoderConfig

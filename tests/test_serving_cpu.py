@@ -49,6 +49,11 @@ class HistoryModel(StepModel):
     def greedy(self, logits):
         return logits.argmax(-1)
 
+    status = 0
+
+    def device_status(self):
+        return self.status
+
 
 def expected(prompt, n, vocab=97, window=None, stop=()):
     h = list(prompt)
@@ -108,6 +113,15 @@ def test_feeding_in_portions(cut):
     assert got.argmax(-1).tolist() == [HistoryModel.answer(texts["a"], 97, None)]
     with pytest.raises(RuntimeError):
         eng.feed([("d", list(range(25)), [])])
+
+
+def test_a_wait_that_ran_out_is_an_error():
+    model = HistoryModel()
+    model.status = 1
+    with pytest.raises(RuntimeError):
+        Engine(model).feed([("a", [1, 2], [1])])
+    with pytest.raises(RuntimeError):
+        Engine(model).generate([[1, 2]], 2)
 
 
 def test_pages_behind_the_window_go_back_once():

@@ -161,7 +161,6 @@ __global__ void __launch_bounds__(kMmaThreads, 1)
   constexpr int kOCols = kQuads * 32;      // columns of one O^T accumulator
   constexpr int kPBytes = HT * 128;        // one tile's weights: [heads][64 positions] bf16, 128-byte swizzle
   constexpr int kHandOver = (kOutWarps + kParts * kQuads) * 32;
-  GridDependencySync();
   extern __shared__ unsigned char smem_raw[];
   __shared__ alignas(8) uint64_t bars[2 * kMaxStages + 9];
   __shared__ uint32_t slot_store[2];
@@ -171,17 +170,6 @@ __global__ void __launch_bounds__(kMmaThreads, 1)
   const int tile_bytes = sp.atoms * kAtomBytes, stages = sp.stages;
   const uint32_t ring = base + 2 * kPBytes;
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
-  const int t = blockIdx.z, h0 = blockIdx.y * HT, slice = blockIdx.x;
-  const int2 live = LiveRange(p, t);
-  const int tile0 = live.x / kMmaTile + slice * sp.slice_tiles;
-  const int n = min((live.y + kMmaTile - 1) / kMmaTile, tile0 + sp.slice_tiles) - tile0;  // tiles of this CTA
-  if (n <= 0) {  // an empty slice writes nothing; an empty row writes zeros
-    if (slice == 0 && sp.records == nullptr) {
-      __nv_bfloat16* out = static_cast<__nv_bfloat16*>(p.out) + (static_cast<size_t>(t) * p.H + h0) * p.kv_rank;
-      for (int i = tid; i < min(HT, p.H - h0) * p.kv_rank; i += kMmaThreads) out[i] = __float2bfloat16_rn(0.f);
-    }
-    return;
-  }
   // full: a tile has landed; free: its products are done; sfull, sempty: scores there, read; pready: weights there and O in their
   // scale; odone: O has the tile in it.
   const uint32_t full = SmemAddr(bars), free0 = full + 8 * kMaxStages, sfull = free0 + 8 * kMaxStages, sempty = sfull + 16;
@@ -210,6 +198,21 @@ __global__ void __launch_bounds__(kMmaThreads, 1)
   __syncthreads();
   asm volatile("tcgen05.fence::after_thread_sync;\n" ::: "memory");
   const uint32_t tmem = *static_cast<volatile uint32_t*>(slot_store);
+  // Only with its TMEM in hand may the CTA let the next kernel's start (which may want some of it and waits for this one).
+  GridDependencySync();
+  const int t = blockIdx.z, h0 = blockIdx.y * HT, slice = blockIdx.x;
+  const int2 live = LiveRange(p, t);
+  const int tile0 = live.x / kMmaTile + slice * sp.slice_tiles;
+  const int n = min((live.y + kMmaTile - 1) / kMmaTile, tile0 + sp.slice_tiles) - tile0;  // tiles of this CTA
+  if (n <= 0) {  // an empty slice writes nothing; an empty row writes zeros
+    if (slice == 0 && sp.records == nullptr) {
+      __nv_bfloat16* out = static_cast<__nv_bfloat16*>(p.out) + (static_cast<size_t>(t) * p.H + h0) * p.kv_rank;
+      for (int i = tid; i < min(HT, p.H - h0) * p.kv_rank; i += kMmaThreads) out[i] = __float2bfloat16_rn(0.f);
+    }
+    __syncthreads();
+    if (warp == 0) asm volatile("tcgen05.dealloc.cta_group::1.sync.aligned.b32 %0, %1;\n" ::"r"(tmem), "r"(512u) : "memory");
+    return;
+  }
   const int o_tiles = (p.kv_rank + 127) >> 7;
   const uint32_t tmem_q = tmem + sp.score_buffers * kMmaTile, tmem_o = tmem_q + sp.atoms * 32;
   bool ok = true;

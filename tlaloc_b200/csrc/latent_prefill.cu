@@ -67,15 +67,16 @@ __global__ void __launch_bounds__(kThreads, 1)
                       const __grid_constant__ CUtensorMap map_rot, const __grid_constant__ CUtensorMap map_v, const __grid_constant__ WindowArgs a)
 {
   extern __shared__ unsigned char smem_raw[];
-  __shared__ alignas(8) uint64_t bars[2 + 2 + 1 + 2 + 1 + 2];
+  __shared__ alignas(8) uint64_t bars[2 + 2 + 1 + 2 + 2 + 2];
   __shared__ uint32_t slot_store[2];
   __shared__ float s_row[2][2][kQ];  // [tile parity][half of the keys][query]
   const uint32_t base = (SmemAddr(smem_raw) + 1023u) & ~1023u;
   unsigned char* smem = smem_raw + (base - SmemAddr(smem_raw));
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
   // Of the tiles in the rings: kfull, vfull "landed"; a K stage is free again when the scores of its tile are there (sfull), a V stage
-  // when its product is (odone).
-  const uint32_t kfull = SmemAddr(bars), vfull = kfull + 16, qfull = vfull + 16, sfull = qfull + 8, pfull = sfull + 16, odone = pfull + 8;
+  // when its product is (odone).  pfull: the weights are there; two barriers, because the softmax may be a tile ahead of the product (one
+  // that is two phases ahead of a wait looks like one that has not come).
+  const uint32_t kfull = SmemAddr(bars), vfull = kfull + 16, qfull = vfull + 16, sfull = qfull + 8, pfull = sfull + 16, odone = pfull + 16;
   volatile uint32_t* slot = slot_store;
   volatile uint32_t* abort_word = slot_store + 1;
   const uint32_t sk = a.qk_atoms * kAtom, sv = sk + a.k_stages * a.qk_atoms * kAtom;  // offsets of the K and V rings, behind Q
@@ -91,10 +92,10 @@ __global__ void __launch_bounds__(kThreads, 1)
       MbarInit(kfull + 8 * i, 1);
       MbarInit(vfull + 8 * i, 1);
       MbarInit(sfull + 8 * i, 1);
+      MbarInit(pfull + 8 * i, kSoftmaxWarps);
       MbarInit(odone + 8 * i, 1);
     }
     MbarInit(qfull, 1);
-    MbarInit(pfull, kSoftmaxWarps);
     asm volatile("fence.mbarrier_init.release.cluster;\n" ::: "memory");
   }
   if (warp == 0) {
@@ -173,7 +174,7 @@ __global__ void __launch_bounds__(kThreads, 1)
         const uint64_t va = vd + static_cast<uint64_t>((stage * v_tile) >> 4);
         const uint32_t pa = tmem + (j & 1) * 128;
         ok = MbarWait(vfull + 8 * stage, (v_stages == 2 ? j >> 1 : j) & 1, abort_word) && ok;
-        ok = MbarWait(pfull, j & 1, abort_word) && ok;
+        ok = MbarWait(pfull + 8 * (j & 1), (j >> 1) & 1, abort_word) && ok;
         asm volatile("tcgen05.fence::after_thread_sync;\n" ::: "memory");
         // P: eight columns per 16 keys; V: keys are its rows, 16 of them per step
         TcMmaTmemA(tmem_o, pa, va, o_idesc, j > 0 ? 1u : 0u);
@@ -255,7 +256,7 @@ __global__ void __launch_bounds__(kThreads, 1)
       asm volatile("tcgen05.wait::st.sync.aligned;\n" ::: "memory");
       asm volatile("tcgen05.fence::before_thread_sync;\n" ::: "memory");
       __syncwarp();
-      if (lane == 0) MbarArrive(pfull);
+      if (lane == 0) MbarArrive(pfull + 8 * b);
     }
     sum += other(tiles & 1, sum);
     ok = MbarWaitWarp(odone + 8 * ((tiles - 1) & 1), ((tiles - 1) >> 1) & 1, lane, abort_word) && ok;

@@ -33,7 +33,7 @@ class Engine:
         """entries [(id, tokens, want)]: the next tokens of each sequence (a new id opens one) and the places among them whose
         logits are asked for.  Returns one f32 tensor [len(want), vocab] on the host per entry.  More tokens than a step takes run in
         several steps."""
-        out = []
+        out = []  # (reading the logits waits for the step, so the status read below costs no wait of its own)
         for key, tokens, want in entries:
             seq = self.sequences.setdefault(key, Sequence())
             rows = []
@@ -43,7 +43,12 @@ class Engine:
                     raise RuntimeError(f"sequence {key!r}: no pages left for {len(part)} more tokens")
                 rows.append(self._run([(seq, part)], [w - lo for w in want if lo <= w < lo + len(part)]).cpu())
             out.append(torch.cat(rows) if rows else torch.empty((0, self.model.vocab)))
+        self._check()
         return out
+
+    def _check(self) -> None:
+        if self.model.device_status() != 0:
+            raise RuntimeError("a wait inside a kernel ran out: the results of this step are not valid")
 
     def close(self, key) -> None:
         """The sequence is finished; its pages go back."""
@@ -83,4 +88,5 @@ class Engine:
                 self.scheduler.add(r)
         while not self.scheduler.idle:
             self.step()
+        self._check()
         return [r.output for r in requests]

@@ -10,6 +10,7 @@ from __future__ import annotations
 import numpy as np
 import torch
 
+from . import _native as N
 from . import ops
 from .paging import PADDING_LENGTH, PADDING_PAGE, PADDING_SLOT, RaggedStep
 
@@ -79,6 +80,10 @@ class StepModel:
         """Runs the step's tokens; returns the f32 logits [len(want), vocab] of the rows named in `want` (device tensor,
         valid until the next step)."""
         raise NotImplementedError
+
+    def device_status(self) -> int:
+        """Nonzero if a bounded wait inside a kernel ran out since the last read: results since then are not valid."""
+        return N.lib().tlaloc_b200_device_status()
 
     def greedy(self, logits: torch.Tensor) -> torch.Tensor:
         """First maximum of every row of logits, int32 on the device."""
