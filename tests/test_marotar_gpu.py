@@ -56,6 +56,7 @@ CONFIGS = {
     "two layers": oracle.model(oracle.layer(), oracle.layer(heads=5, dim=16, rot_dim=16, vdim=24, q_rank=40, kv_rank=72, window=33, ff=120)),
     "shared weights": oracle.model(oracle.layer(window=9), oracle.layer(window=40, ff=0), oracle.layer(window=9, weights_of=0),
                                    oracle.layer(window=40, ff=0, weights_of=1), oracle.layer(window=9, weights_of=2)),
+    "weights of a later layer": oracle.model(oracle.layer(window=12, weights_of=1), oracle.layer(window=12)),
     "no feed-forward, no scaling": oracle.model(oracle.layer(ff=0, scaling=False, window=15), eps=1e-3),
     "part of the key part rotated": oracle.model(oracle.layer(rot_dim=24, rot_dims=16, window=50), oracle.layer(window=0, scaling=False)),
     "one head, one pair": oracle.model(oracle.layer(heads=1, dim=8, rot_dim=2, vdim=8, q_rank=8, kv_rank=8, window=1, ff=8), width=40, vocab=33),

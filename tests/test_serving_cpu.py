@@ -198,8 +198,11 @@ def test_configuration_is_read_whole():
     assert cfg.layers[0].mixer.heads == 3 and cfg.layers[1].mixer.heads == 7 and cfg.eps == 1e-5
     assert {k: tuple(v.shape) for k, v in oracle.make_weights(c).items()} == cfg.tensor_shapes()
     assert LatentDecoderConfig.from_config(oracle.model(oracle.layer(window=7), oracle.layer(window=30))).window == 30
+    borrowed = oracle.model(oracle.layer(weights_of=2), oracle.layer(ff=0), oracle.layer())  # a layer may also use a later one's weights
+    assert [l.weights for l in LatentDecoderConfig.from_config(borrowed).layers] == [2, 1, 2]
     for change in (lambda d: d["layers"][0].update(type="other"), lambda d: d["layers"][0]["mlp"].update(kind="gated"),
-                   lambda d: d["layers"][2].update(weights_of=2), lambda d: d["layers"][0]["mixer"]["rot"].update(dims=64)):
+                   lambda d: d["layers"][2].update(weights_of=2), lambda d: d["layers"][0].update(weights_of=3),
+                   lambda d: d["layers"][0]["mixer"]["rot"].update(dims=64)):
         bad = json.loads(json.dumps(c))
         change(bad)
         with pytest.raises(ValueError):

@@ -101,11 +101,12 @@ class LatentDecoderConfig:
             mlp = e.get("mlp")
             if mlp is not None and mlp["kind"] != "dense":
                 raise ValueError(f"layer {i}: feed-forward kind {mlp['kind']!r} is not built")
-            source = i
+            source, passed = i, {i}
             while c["layers"][source].get("weights_of") is not None:
                 nxt = int(c["layers"][source]["weights_of"])
-                if not 0 <= nxt < source:
-                    raise ValueError(f"layer {source}: weights_of {nxt} must name an earlier layer")
+                if not 0 <= nxt < len(c["layers"]) or nxt in passed:
+                    raise ValueError(f"layer {source}: weights_of {nxt} leads to no layer with weights")
+                passed.add(nxt)
                 source = nxt
             layers.append(Layer(mixer, FeedForward(int(mlp["ff"])) if mlp is not None else None, source))
         return cls(width=int(c["width"]), vocab=int(c["vocab"]), eps=float(c["norm"]["eps"]), layers=tuple(layers))
@@ -194,7 +195,8 @@ class LatentDecoder(StepModel):
         zero) in the layout the step wants: query and key/value down-projection stacked, the two output projections side by side, the
         key up-projection also transposed per head."""
         shapes = self.cfg.tensor_shapes()
-        missing, extra = sorted(set(shapes) - set(t)), sorted(set(t) - set(shapes))
+        unused = {f"l{i}.norm2" for i, l in enumerate(self.cfg.layers) if l.mlp is None}  # the norm of a branch that is absent
+        missing, extra = sorted(set(shapes) - set(t)), sorted(set(t) - set(shapes) - unused)
         if missing or extra:
             raise ValueError(f"the checkpoint does not fit its configuration: missing {missing[:5]}, unknown {extra[:5]}")
         for name, shape in shapes.items():
