@@ -15,9 +15,9 @@ from .step_model import StepModel
 class Engine:
     def __init__(self, model: StepModel):
         self.model = model
-        self.pool = PagePool(model.num_blocks)
+        self.pool = PagePool(model.num_blocks, model.num_states)
         self.scheduler = Scheduler(self.pool, block_size=model.block_size, max_tokens=model.max_tokens, max_sequences=model.max_sequences,
-                                   window=model.window)
+                                   window=model.window, keep_first=model.keep_first)
         self.sequences: dict[object, Sequence] = {}
 
     # ------------------------------------------------------------------ token by token
@@ -40,7 +40,7 @@ class Engine:
             for lo in range(0, len(tokens), self.model.max_tokens):
                 part = tokens[lo:lo + self.model.max_tokens]
                 if not seq.reserve(self.pool, len(part), self.model.block_size):
-                    raise RuntimeError(f"sequence {key!r}: no pages left for {len(part)} more tokens")
+                    raise RuntimeError(f"sequence {key!r}: no pages (or no state slot) left for {len(part)} more tokens")
                 rows.append(self._run([(seq, part)], [w - lo for w in want if lo <= w < lo + len(part)]).cpu())
             out.append(torch.cat(rows) if rows else torch.empty((0, self.model.vocab)))
         self._check()
@@ -51,7 +51,7 @@ class Engine:
             raise RuntimeError("a wait inside a kernel ran out: the results of this step are not valid")
 
     def close(self, key) -> None:
-        """The sequence is finished; its pages go back."""
+        """The sequence is finished; its pages and its state slot go back."""
         self.sequences.pop(key).release(self.pool)
 
     # ------------------------------------------------------------------ generation

@@ -23,9 +23,8 @@ import torch
 
 from . import _native as N
 from . import ops
-from .paging import RaggedStep
 from .rotary import Rotation, YarnScaling, pair_tables
-from .step_model import StepModel
+from .step_model import RaggedModel
 
 
 EXPAND_FROM = 32  # tokens of a portion from which the expanded way of attending pays
@@ -136,24 +135,17 @@ class LatentDecoderConfig:
 
 # ---------------------------------------------------------------------------------------------- the model
 
-class LatentDecoder(StepModel):
+class LatentDecoder(RaggedModel):
     """Weights, latent pools and step buffers; `run` takes a ragged step, `step(rows)` one token of `rows` sequences."""
 
     def __init__(self, cfg: LatentDecoderConfig, *, num_blocks: int, max_len: int, max_tokens: int = 2048, max_sequences: int = 64,
                  dtype: torch.dtype = torch.bfloat16, device="cuda:0"):
-        if not torch.cuda.is_available():
-            raise RuntimeError("tlaloc_b200.LatentDecoder needs a CUDA device: there is no CPU path")
-        if dtype not in (torch.bfloat16, torch.float32):
-            raise ValueError(f"LatentDecoder runs in bfloat16 or float32, not {dtype}")
-        max_blocks = -(-max_len // cfg.block_size)
-        super().__init__(max(max_tokens, max_sequences), max_sequences, num_blocks, max_blocks, cfg.block_size, cfg.vocab, device)
-        self.cfg, self.dtype, self.window = cfg, dtype, cfg.window
-        self.max_positions = max_blocks * cfg.block_size
-        ops.init()
+        super().__init__(width=cfg.width, dtype=dtype, max_tokens=max_tokens, max_sequences=max_sequences, num_blocks=num_blocks, max_len=max_len,
+                         block_size=cfg.block_size, vocab=cfg.vocab, device=device)
+        self.cfg, self.window = cfg, cfg.window
         dev, R = self.device, self.rows
         ty, f32 = dict(dtype=dtype, device=dev), dict(dtype=torch.float32, device=dev)
         mixers = [l.mixer for l in cfg.layers]
-        self.row_tables = torch.zeros((R,), dtype=torch.int32, device=dev)
         self.pools = [torch.zeros((num_blocks, cfg.block_size, -(-m.row // 8) * 8), **ty) for m in mixers]
         tables: dict[Rotation, tuple] = {}
         for m in mixers:
@@ -164,7 +156,6 @@ class LatentDecoder(StepModel):
         self.embed = self.final_norm = None
         # step buffers, shared by the layers: flat, viewed in each layer's own shape
         big = lambda f: max(f(l) for l in cfg.layers)
-        self.x = torch.empty((R, cfg.width), **f32)
         self.h1, self.h2 = torch.empty((R, cfg.width), **ty), torch.empty((R, cfg.width), **ty)
         self._low = torch.empty((R * big(lambda l: l.mixer.q_rank + l.mixer.row),), **f32)
         self._cq = torch.empty((R * big(lambda l: l.mixer.q_rank),), **ty)
@@ -178,10 +169,6 @@ class LatentDecoder(StepModel):
         self._expanded = [dtype == torch.bfloat16 and ops.window_attention_applies(m.dim, m.rot_dim, m.vdim) and m.row % 8 == 0
                           and (m.heads * m.vdim) % 8 == 0 and m.scale > 0 for m in mixers]
         self._expand_space: dict[str, torch.Tensor] = {}  # gathered latents, keys and values of a portion's window; grown on demand
-        self.hn = torch.empty((R, cfg.width), **ty)
-        self._decode_uses: dict[int, int] = {}
-        self.logits = torch.empty((max_sequences, cfg.vocab), **f32)
-        self.next_ids = torch.zeros((max_sequences,), dtype=torch.int32, device=dev)
 
     @staticmethod
     def _o_width(l: Layer) -> int:
@@ -324,8 +311,6 @@ class LatentDecoder(StepModel):
         ops.rmsnorm_pair(self.x[:n], lw["norm1"], self.h1[:n], self.cfg.eps, lw.get("norm2"), self.h2[:n] if "norm2" in lw else None)
 
     def _hidden(self, n: int, spans=None, trace: list | None = None) -> None:
-        """Embedding and layers over rows [0, n) of the step inputs; the residual stream stays in x.  trace: receives a copy
-        of it after every layer."""
         ops.embedding(self.embed, self.token_ids[:n], out=self.x[:n])
         for i in range(len(self.layers)):
             self._norms(i, n)
@@ -338,50 +323,3 @@ class LatentDecoder(StepModel):
         ops.rmsnorm_pair(x, self.final_norm, self.hn[:k], self.cfg.eps)
         ops.dense_gemm(ops.dense(self.hn[:k], self.embed, self.logits[:k]), weights_const=True)
         return self.logits[:k]
-
-    def _run_step(self, rows: int) -> None:
-        """One token of `rows` sequences: row r uses block table r."""
-        self._hidden(rows)
-        ops.argmax(self._head(self.x[:rows]), out=self.next_ids[:rows])
-
-    def run(self, step: RaggedStep, want, trace: list | None = None) -> torch.Tensor:
-        n, s = step.token_ids.shape[0], step.block_tables.shape[0]
-        if n > self.max_tokens or s > self.max_sequences:
-            raise ValueError(f"a step of {n} tokens of {s} sequences; this model takes {self.max_tokens} of {self.max_sequences}")
-        if n == s and trace is None:
-            return self._run_decode(step, want)
-        self._inputs(step)
-        self._hidden(n, [(int(a), int(b), r, int(step.positions[a])) for r, (a, b) in enumerate(zip(step.starts[:-1], step.starts[1:]))], trace)
-        out = []
-        for k in range(0, len(want), self.max_sequences):
-            rows = torch.as_tensor(np.asarray(want[k:k + self.max_sequences], np.int32), device=self.device)
-            out.append(self._head(ops.embedding(self.x[:n], rows)))
-            if len(want) > self.max_sequences:
-                out[-1] = out[-1].clone()
-        return torch.cat(out) if len(out) > 1 else out[0] if out else self.logits[:0]
-
-    def _inputs(self, step: RaggedStep) -> None:
-        for dst, src in ((self.token_ids, step.token_ids), (self.positions, step.positions), (self.seq_lens, step.seq_lens),
-                         (self.slot_mapping, step.slot_mapping), (self.row_tables, step.row_tables), (self.block_tables, step.block_tables)):
-            self._put(dst[:src.shape[0]], src)
-
-    def _run_decode(self, step: RaggedStep, want) -> torch.Tensor:
-        """One token of every sequence: the batch is padded to a power of two, and a size that comes up again is captured into a
-        CUDA graph (padding rows write nothing and attend over the padding page)."""
-        n = step.token_ids.shape[0]
-        rows = min(1 << (n - 1).bit_length(), self.max_sequences)
-        self.set_decode_inputs(*self._padded(step, rows))
-        self._decode_uses[rows] = self._decode_uses.get(rows, 0) + 1
-        if self._decode_uses[rows] == 3 and rows not in self._graphs:
-            self.capture(rows)
-        self.step(rows)
-        if list(want) == list(range(n)):
-            return self.logits[:n]
-        return self.logits[torch.as_tensor(want, dtype=torch.long, device=self.device)]
-
-    def set_decode_inputs(self, token_ids, positions, block_tables, seq_lens, slot_mapping) -> None:
-        """Inputs of a step of one token per sequence, as many as there are ids; row r uses block table r."""
-        rows = token_ids.shape[0]
-        for dst, src in ((self.token_ids, token_ids), (self.positions, positions), (self.block_tables, block_tables),
-                         (self.seq_lens, seq_lens), (self.slot_mapping, slot_mapping), (self.row_tables, np.arange(rows, dtype=np.int32))):
-            self._put(dst[:rows], src)

@@ -1,4 +1,5 @@
-"""The caller's side of the paged KV cache: which physical page holds which positions, and the integer inputs of a step.
+"""The caller's side of what a sequence holds on the device: which physical page of the paged KV cache holds which positions, which
+slot its recurrent state lives in, and the integer inputs of a step.
 
 Mirrors the behaviour of the reference's serving backend, not its code: the page pool of one model instance
 (triton/backend/sequence_mode.h:315-336: page 0 is never handed out, it is where the block tables of padding rows
@@ -17,15 +18,19 @@ import numpy as np
 PADDING_PAGE = 0
 PADDING_SLOT = -1
 PADDING_LENGTH = 1
+PADDING_STATE = 0
 
 
 class PagePool:
-    """The physical pages 1 .. num_blocks - 1 of one KV pool."""
+    """The physical pages 1 .. num_blocks - 1 of one KV pool and, for a model with recurrent layers, the state slots 1 .. num_states
+    (slot 0 is where padding rows point)."""
 
-    def __init__(self, num_blocks: int):
+    def __init__(self, num_blocks: int, num_states: int = 0):
         if num_blocks < 2:
             raise ValueError("a pool needs page 0 (padding) and at least one page to hand out")
         self.capacity = num_blocks - 1
+        self.num_states = num_states
+        self._free_states = set(range(1, num_states + 1))
         self._free = set(range(1, num_blocks))
         self._extra_holders: dict[int, int] = {}
 
@@ -42,6 +47,24 @@ class PagePool:
         pages = sorted(self._free)[:n]
         self._free.difference_update(pages)
         return pages
+
+    @property
+    def has_state(self) -> bool:
+        """Whether one more sequence can be opened."""
+        return self.num_states == 0 or bool(self._free_states)
+
+    def take_state(self) -> int | None:
+        """The lowest free state slot, None when all are held."""
+        if not self._free_states:
+            return None
+        s = min(self._free_states)
+        self._free_states.remove(s)
+        return s
+
+    def give_state(self, s: int) -> None:
+        if not 1 <= s <= self.num_states or s in self._free_states:
+            raise ValueError(f"state slot {s} is not held")
+        self._free_states.add(s)
 
     def share(self, pages) -> None:
         """One more holder of each page (a cached prefix, or a sequence that starts from one)."""
@@ -71,34 +94,45 @@ class PagePool:
 
 @dataclass
 class Sequence:
-    """One sequence's pages (logical block b lives on pages[b]) and how many tokens have their KV in the pool."""
+    """One sequence's pages (logical block b lives on pages[b]), its state slot, and how many tokens are in the cache and the state."""
 
     pages: list[int] = field(default_factory=list)
     length: int = 0
+    state: int = PADDING_STATE
 
     def reserve(self, pool: PagePool, tokens: int, block_size: int) -> bool:
-        """Makes room for `tokens` more tokens; False (and nothing taken) if the pool cannot supply the pages."""
-        need = -(-(self.length + tokens) // block_size) - len(self.pages)
-        if need <= 0:
-            return True
-        got = pool.take(need)
-        if got is None:
+        """Makes room for `tokens` more tokens; False (and nothing taken) if the pool cannot supply the pages or, to a sequence
+        that starts, a state slot.  A slot is handed out as it was left: a state begins at zero because position 0 says so."""
+        if self.state == PADDING_STATE and not pool.has_state:
             return False
-        self.pages.extend(got)
+        need = -(-(self.length + tokens) // block_size) - len(self.pages)
+        if need > 0:
+            got = pool.take(need)
+            if got is None:
+                return False
+            self.pages.extend(got)
+        if self.state == PADDING_STATE and pool.num_states:
+            self.state = pool.take_state()
         return True
 
-    def drop_before(self, pool: PagePool, position: int, block_size: int) -> int:
-        """Gives back the pages that hold only positions below `position` (a model whose every layer attends through a
-        sliding window never reads them again); their table entries become the padding page.  Returns how many."""
+    def drop_before(self, pool: PagePool, position: int, block_size: int, keep_first: int = 0) -> int:
+        """Gives back the pages that hold only positions in [keep_first, position) (a model whose every layer attends through a
+        sliding window, and perhaps to the first tokens, never reads them again); their table entries become the padding page.
+        Returns how many."""
+        lo = -(-keep_first // block_size)
         n = min(max(position, 0) // block_size, len(self.pages))
-        old = [p for p in self.pages[:n] if p != PADDING_PAGE]
+        if n <= lo:
+            return 0
+        old = [p for p in self.pages[lo:n] if p != PADDING_PAGE]
         pool.give(old)
-        self.pages[:n] = [PADDING_PAGE] * n
+        self.pages[lo:n] = [PADDING_PAGE] * (n - lo)
         return len(old)
 
     def release(self, pool: PagePool) -> None:
         pool.give(p for p in self.pages if p != PADDING_PAGE)
-        self.pages, self.length = [], 0
+        if self.state != PADDING_STATE:
+            pool.give_state(self.state)
+        self.pages, self.length, self.state = [], 0, PADDING_STATE
 
 
 @dataclass
@@ -155,6 +189,7 @@ class RaggedStep:
     row_tables: np.ndarray    # i32 [tokens]: which row of block_tables
     block_tables: np.ndarray  # i32 [sequences, max_blocks]
     starts: np.ndarray        # i32 [sequences + 1]: first token row of each sequence
+    row_states: np.ndarray    # i32 [tokens]: the state slot of the row's sequence (0: the model keeps no state)
 
 
 def stage_ragged(work, *, max_blocks: int, block_size: int) -> RaggedStep:
@@ -177,7 +212,8 @@ def stage_ragged(work, *, max_blocks: int, block_size: int) -> RaggedStep:
     positions = np.concatenate(pos).astype(np.int32)
     return RaggedStep(np.concatenate([np.asarray(t, np.int32) for _, t in work]), positions, np.concatenate(slots).astype(np.int32),
                       positions + 1, np.repeat(np.arange(len(work), dtype=np.int32), counts), tables,
-                      np.concatenate([[0], np.cumsum(counts)]).astype(np.int32))
+                      np.concatenate([[0], np.cumsum(counts)]).astype(np.int32),
+                      np.repeat(np.asarray([seq.state for seq, _ in work], np.int32), counts))
 
 
 def commit_step(work) -> None:

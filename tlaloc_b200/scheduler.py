@@ -35,8 +35,8 @@ class Scheduler:
     those whose prompt is not all in; then admits waiting ones while rows, sequences and pages are left.  When a running
     request cannot get a page, the youngest one gives its pages back and waits to be read again."""
 
-    def __init__(self, pool: PagePool, *, block_size: int, max_tokens: int, max_sequences: int, window: int | None = None):
-        self.pool, self.block_size, self.window = pool, block_size, window
+    def __init__(self, pool: PagePool, *, block_size: int, max_tokens: int, max_sequences: int, window: int | None = None, keep_first: int = 0):
+        self.pool, self.block_size, self.window, self.keep_first = pool, block_size, window, keep_first
         self.max_tokens, self.max_sequences = max_tokens, max_sequences
         self.waiting: deque[Request] = deque()
         self.running: list[Request] = []
@@ -87,6 +87,8 @@ class Scheduler:
         return min(r.pending, rows, self._room(r))
 
     def _room(self, r: Request) -> int:
+        if r.seq.length == 0 and not r.seq.pages and not self.pool.has_state:
+            return 0
         return (len(r.seq.pages) + self.pool.free_count) * self.block_size - r.seq.length
 
     def _preempt(self, r: Request) -> None:
@@ -95,10 +97,10 @@ class Scheduler:
         self.waiting.appendleft(r)
 
     def advance(self, seq: Sequence, n: int) -> None:
-        """The cache now holds n more tokens; pages no window reaches any more go back."""
+        """The cache now holds n more tokens; pages no window reaches any more go back (those of the kept first tokens stay)."""
         seq.length += n
         if self.window is not None:
-            seq.drop_before(self.pool, seq.length - self.window + 1, self.block_size)
+            seq.drop_before(self.pool, seq.length - self.window + 1, self.block_size, self.keep_first)
 
     def finish(self, r: Request) -> None:
         r.seq.release(self.pool)

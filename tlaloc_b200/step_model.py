@@ -12,7 +12,7 @@ import torch
 
 from . import _native as N
 from . import ops
-from .paging import PADDING_LENGTH, PADDING_PAGE, PADDING_SLOT, RaggedStep
+from .paging import PADDING_LENGTH, PADDING_PAGE, PADDING_SLOT, PADDING_STATE, RaggedStep
 
 
 class StepModel:
@@ -20,6 +20,8 @@ class StepModel:
     and `next_ids[:rows]`."""
 
     window: int | None = None  # no row attends further back than this many positions (itself included); None: unbounded
+    keep_first: int = 0        # ... except to this many first positions
+    num_states: int = 0        # state slots of a model with recurrent layers: sequences it can hold at a time
 
     def __init__(self, rows: int, tables: int, num_blocks: int, max_blocks_per_seq: int, block_size: int, vocab: int, device):
         self.rows, self.device, self.vocab = rows, torch.device(device), vocab
@@ -104,3 +106,91 @@ class StepModel:
         tables[:n] = step.block_tables[step.row_tables]
         return (pad(step.token_ids, 0), pad(step.positions, 0), tables, pad(step.seq_lens, PADDING_LENGTH),
                 pad(step.slot_mapping, PADDING_SLOT))
+
+
+class RaggedModel(StepModel):
+    """A model whose step takes ragged rows: every row names its block table and its state slot.  A subclass computes the residual
+    stream of rows [0, n) in `x` (`_hidden`) and the logits of rows of it (`_head`, into `logits`)."""
+
+    def __init__(self, *, width: int, dtype: torch.dtype, max_tokens: int, max_sequences: int, num_blocks: int, max_len: int,
+                 block_size: int, vocab: int, device):
+        if not torch.cuda.is_available():
+            raise RuntimeError(f"tlaloc_b200.{type(self).__name__} needs a CUDA device: there is no CPU path")
+        if dtype not in (torch.bfloat16, torch.float32):
+            raise ValueError(f"{type(self).__name__} runs in bfloat16 or float32, not {dtype}")
+        max_blocks = -(-max_len // block_size)
+        super().__init__(max(max_tokens, max_sequences), max_sequences, num_blocks, max_blocks, block_size, vocab, device)
+        self.dtype, self.max_positions = dtype, max_blocks * block_size
+        ops.init()
+        dev, i32 = self.device, dict(dtype=torch.int32, device=self.device)
+        self.row_tables = torch.zeros((self.rows,), **i32)
+        self.row_states = torch.zeros((self.rows,), **i32)
+        self.x = torch.empty((self.rows, width), dtype=torch.float32, device=dev)
+        self.hn = torch.empty((self.rows, width), dtype=dtype, device=dev)
+        self.logits = torch.empty((max_sequences, vocab), dtype=torch.float32, device=dev)
+        self.next_ids = torch.zeros((max_sequences,), **i32)
+        self._decode_uses: dict[int, int] = {}
+
+    def _hidden(self, n: int, spans=None, trace: list | None = None) -> None:
+        """Embedding and layers over rows [0, n) of the step inputs; the residual stream stays in x.  spans: [(first row, end row,
+        table row, position of the first)], the rows of each sequence; None: one row per sequence.  trace: receives a copy of
+        the residual stream after every layer."""
+        raise NotImplementedError
+
+    def _head(self, x: torch.Tensor) -> torch.Tensor:
+        """Logits of rows of the residual stream: a view of `logits`."""
+        raise NotImplementedError
+
+    def _run_step(self, rows: int) -> None:
+        """One token of `rows` sequences: row r uses block table r."""
+        self._hidden(rows)
+        ops.argmax(self._head(self.x[:rows]), out=self.next_ids[:rows])
+
+    def run(self, step: RaggedStep, want, trace: list | None = None) -> torch.Tensor:
+        n, s = step.token_ids.shape[0], step.block_tables.shape[0]
+        if n > self.max_tokens or s > self.max_sequences:
+            raise ValueError(f"a step of {n} tokens of {s} sequences; this model takes {self.max_tokens} of {self.max_sequences}")
+        if n == s and trace is None:
+            return self._run_decode(step, want)
+        self._inputs(step)
+        self._hidden(n, [(int(a), int(b), r, int(step.positions[a])) for r, (a, b) in enumerate(zip(step.starts[:-1], step.starts[1:]))], trace)
+        out = []
+        for k in range(0, len(want), self.max_sequences):
+            rows = torch.as_tensor(np.asarray(want[k:k + self.max_sequences], np.int32), device=self.device)
+            out.append(self._head(ops.embedding(self.x[:n], rows)))
+            if len(want) > self.max_sequences:
+                out[-1] = out[-1].clone()
+        return torch.cat(out) if len(out) > 1 else out[0] if out else self.logits[:0]
+
+    def _inputs(self, step: RaggedStep) -> None:
+        for dst, src in ((self.token_ids, step.token_ids), (self.positions, step.positions), (self.seq_lens, step.seq_lens),
+                         (self.slot_mapping, step.slot_mapping), (self.row_tables, step.row_tables), (self.row_states, step.row_states),
+                         (self.block_tables, step.block_tables)):
+            self._put(dst[:src.shape[0]], src)
+
+    def _run_decode(self, step: RaggedStep, want) -> torch.Tensor:
+        """One token of every sequence: the batch is padded to a power of two, and a size that comes up again is captured into a
+        CUDA graph (padding rows write nothing a sequence reads and attend over the padding page)."""
+        n = step.token_ids.shape[0]
+        rows = min(1 << (n - 1).bit_length(), self.max_sequences)
+        self._decode_uses[rows] = self._decode_uses.get(rows, 0) + 1
+        if self._decode_uses[rows] == 3 and rows not in self._graphs:
+            zeros = np.zeros((rows,), np.int32)  # the warm-up step of a capture must not touch any sequence's state: padding rows alone
+            self.set_decode_inputs(zeros, zeros, np.full((rows, self.max_blocks), PADDING_PAGE, np.int32), zeros + PADDING_LENGTH,
+                                   zeros + PADDING_SLOT, zeros + PADDING_STATE)
+            self.capture(rows)
+        states = np.full((rows,), PADDING_STATE, np.int32)
+        states[:n] = step.row_states
+        self.set_decode_inputs(*self._padded(step, rows), states)
+        self.step(rows)
+        if list(want) == list(range(n)):
+            return self.logits[:n]
+        return self.logits[torch.as_tensor(want, dtype=torch.long, device=self.device)]
+
+    def set_decode_inputs(self, token_ids, positions, block_tables, seq_lens, slot_mapping, row_states=None) -> None:
+        """Inputs of a step of one token per sequence, as many as there are ids; row r uses block table r."""
+        rows = token_ids.shape[0]
+        for dst, src in ((self.token_ids, token_ids), (self.positions, positions), (self.block_tables, block_tables),
+                         (self.seq_lens, seq_lens), (self.slot_mapping, slot_mapping), (self.row_tables, np.arange(rows, dtype=np.int32)),
+                         (self.row_states, row_states)):
+            self._put(dst[:rows], src)
