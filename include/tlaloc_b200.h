@@ -298,6 +298,10 @@ int tlaloc_b200_argmax(const float* logits, int32_t* out, int32_t rows, int32_t 
 
 #define TLALOC_B200_ACT_NONE 0
 #define TLALOC_B200_ACT_RELU2 1 /* max(v, 0)^2 */
+/* Gated: the rows of w come in blocks of 32, 16 of the gate and the 16 of the other factor that belong to them, and y has n / 2
+ * columns act(gate) * other.  No bias, no residual. */
+#define TLALOC_B200_ACT_SILU_MUL 2      /* act(z) = z / (1 + exp(-z)) */
+#define TLALOC_B200_ACT_GELU_TANH_MUL 3 /* act(z) = z (1 + tanh(sqrt(2/pi) (z + 0.044715 z^3))) / 2 */
 
 /*
  * One projection over weights kept in their own float type: per batch entry b,
@@ -305,6 +309,8 @@ int tlaloc_b200_argmax(const float* logits, int32_t* out, int32_t rows, int32_t 
  * with w [batch][n][k] contiguous (a checkpoint's [out, in]).  x and y have row strides and batch strides of their own, so
  * they may be column blocks of wider matrices (the heads of a projection, the halves of a concatenated input).
  * Sums are f32.  bias (f32 [n]) and residual (f32, batch 1 only; may be y) may be NULL.
+ * Grouped (row_offsets given): x and y are one matrix of `rows` rows, and weight b applies to the rows [row_offsets[b],
+ * row_offsets[b + 1]) alone (the tokens of an expert, sorted by expert); batch_x and batch_y are not used, batch is at most 1024.
  */
 typedef struct tlaloc_b200_dense_problem {
   const void* x;
@@ -315,10 +321,12 @@ typedef struct tlaloc_b200_dense_problem {
   int64_t ld_x, ld_res, ld_y;        /* row strides in elements */
   int64_t batch_x, batch_w, batch_y; /* strides between batch entries in elements */
   int32_t k, n, batch, act, y_dtype;
+  int32_t rows;               /* rows of x and y where they are not the call's m (0: they are) */
+  const int32_t* row_offsets; /* NULL, or i32 [batch + 1] in device memory: GROUPED, see below */
 } tlaloc_b200_dense_problem;
 
 /*
- * `count` (1 or 2) projections of the same m rows in one launch where a tensor-core kernel takes them, else one launch
+ * `count` (1 or 2) projections of the same m rows (or of `rows` of their own) in one launch where a tensor-core kernel takes them, else one launch
  * each.  dtype: F32 or BF16, the type of x and w of every problem; y is F32 or BF16 per problem.  F32 runs in true f32 (FMA,
  * no reduced-precision products).  flags: TLALOC_B200_GEMM_WEIGHTS_CONST.  Two problems of one call must not depend on
  * each other's results.
@@ -375,26 +383,116 @@ int tlaloc_b200_latent_attention(const void* query, const void* pool, int64_t po
                                  float scale, void* stream);
 
 /*
- * Rows [first, first + count) of one sequence out of a paged pool of latents: out[r, :row] = the pool row of position first + r
- * under `table` (i32 [max_blocks]).  pool_ld and out_ld in elements, both a multiple of 16 bytes and at least `row` rounded up to it.
+ * The first `keep` rows and the rows [first, first + count - keep) of one sequence out of a paged pool: out[r, :row] = the pool row of
+ * position r (r < keep) or first + r - keep under `table` (i32 [max_blocks]); first >= keep.  pool_ld and out_ld in elements, both a multiple of 16 bytes and at least `row` rounded up to it.
  */
 int tlaloc_b200_latent_gather(const void* pool, int64_t pool_ld, int32_t dtype, const int32_t* table, void* out, int64_t out_ld,
-                              int32_t first, int32_t count, int32_t row, int32_t num_blocks, int32_t block_size, int32_t max_blocks,
-                              void* stream);
+                              int32_t first, int32_t keep, int32_t count, int32_t row, int32_t num_blocks, int32_t block_size,
+                              int32_t max_blocks, void* stream);
 
 /*
  * Attention of a prompt portion over expanded keys and values, bf16: query i (row i of q [T, H, dim + rot_dim], rotated) is position
- * first_query + i of the num_keys keys; it sees key j with 0 <= first_query + i - j < window (window 0: every j up to its own).
- *   out[i, h, :] = sum_j softmax_j((q[i, h, :dim] . k[j, h, :] + q[i, h, dim:] . k_rot[j, :]) * scale) * v[j, h, :]
- * k and v: rows kv_ld apart, heads kv_head_ld apart; k_rot rows rot_ld apart, shared by the heads; out rows out_ld apart, heads side
- * by side.  All strides in elements and multiples of 16 bytes.  Scores, weights and sums are f32; the weights enter the product
- * with v as bf16.  _applies: 1 if the kernel takes these sizes.
+ * first_query + i of the num_keys keys; it sees key j <= first_query + i with first_query + i - j < window (window 0: every one)
+ * or j < keep_first.
+ *   out[i, h, :] = sum_j softmax_j((q[i, h, :dim] . k[j, kh, :] + q[i, h, dim:] . k_rot[j, :]) * scale) * v[j, vh, :]
+ * The H query heads are v_heads groups of equal size, a group's heads each with `maps` consecutive ones: vh = h / (H / v_heads),
+ * kh = vh * maps + h % maps of v_heads * maps key heads (maps 1 and v_heads H: every head has keys and values of its own).
+ * k and v: rows kv_ld apart, heads k_head_ld and v_head_ld apart; k_rot rows rot_ld apart, shared by the heads; out (F32 | BF16)
+ * rows out_ld apart, heads side by side.  All strides in elements and multiples of 16 bytes.  Scores, weights and sums are f32; the
+ * weights enter the product with v as bf16.  _applies: 1 if the kernel takes these sizes.
  */
 int tlaloc_b200_window_attention_applies(int32_t dim, int32_t rot_dim, int32_t vdim);
-int tlaloc_b200_window_attention(const void* q, const void* k, const void* k_rot, int64_t rot_ld, const void* v, int64_t kv_ld,
-                                 int64_t kv_head_ld, void* out, int64_t out_ld, int32_t num_queries, int32_t num_keys,
-                                 int32_t first_query, int32_t num_heads, int32_t dim, int32_t rot_dim, int32_t vdim, int32_t window,
-                                 float scale, void* stream);
+int tlaloc_b200_window_attention(const void* q, const void* k, int64_t k_head_ld, const void* k_rot, int64_t rot_ld, const void* v,
+                                 int64_t v_head_ld, int64_t kv_ld, void* out, int64_t out_ld, int32_t out_dtype, int32_t num_queries,
+                                 int32_t num_keys, int32_t first_query, int32_t num_heads, int32_t v_heads, int32_t maps, int32_t dim,
+                                 int32_t rot_dim, int32_t vdim, int32_t window, int32_t keep_first, float scale, void* stream);
+
+/* ------------------------------------------------------------------ mixers of several kinds */
+
+/*
+ * The end of a branch and the beginning of the next one, per row of n values: the branch's output y is normalised (RMS, gain_post)
+ * and added to the residual stream x, and `out` (NULL: not wanted) is the RMS norm of the new x with gain_next, as `dtype`.
+ *   y = sigmoid(gate) * y + sum_k part_weights[row, k] * parts[part_rows[row, k], :]     (k < top)
+ * y: f32 [rows, n] or NULL; gate: one logit per row, gate_ld apart, or NULL (1); parts: rows of n values of `dtype` (the experts'
+ * outputs) or NULL with top 0.
+ */
+int tlaloc_b200_residual_norm(const float* y, const float* gate, int64_t gate_ld, const void* parts, const int32_t* part_rows,
+                              const float* part_weights, int32_t top, float* x, const float* gain_post, const float* gain_next, void* out,
+                              int32_t dtype, int32_t rows, int32_t n, float eps, void* stream);
+
+/*
+ * Parts of projected rows (f32, row stride ld) with rotary positions: part i's `heads` heads of `dim` values start at column `first`; the
+ * first rot_dims values of each are rotated if `rotate` (value c together with value c + rot_dims / 2), all are multiplied by
+ * `scale` and go, widened to `padded` values with zeros, to out + r * out_ld + head * out_head_ld, r the token or (by_slot) its slot;
+ * a slot below 0 writes nothing.  out has `dtype`; cos/sin f32 [max_pos, rot_dims / 2].
+ */
+typedef struct tlaloc_b200_rotate_part {
+  void* out;
+  int64_t out_ld, out_head_ld;
+  int32_t first, heads, dim, padded, rotate, by_slot;
+  float scale;
+} tlaloc_b200_rotate_part;
+int tlaloc_b200_rotate_rows(const float* in, int64_t ld, const tlaloc_b200_rotate_part* parts, int32_t count, int32_t dtype,
+                            const int32_t* positions, const float* cos_table, const float* sin_table, const int32_t* slot_mapping,
+                            int32_t num_tokens, int32_t rot_dims, int32_t num_slots, int32_t max_pos, void* stream);
+
+/*
+ * Attention of single tokens over a paged pool whose rows hold v_heads * maps key heads of `dim` values and, from column v_first, v_heads
+ * value heads of `vdim` values.  q [T, H, dim], heads as tlaloc_b200_window_attention has them.  Row t sees position j < seq_lens[t]
+ * with j >= seq_lens[t] - window (window 0: every one) or j < keep_first.  The result are records for tlaloc_b200_map_difference:
+ * f32 [slices][T][H][2 + vdim] = {largest score (times scale, log2), sum of weights, weighted sum of values}, slices as
+ * tlaloc_b200_grouped_attention_slices says (max_live: the most positions a row sees).  q and the pool have `dtype`; pool_ld in
+ * elements; in bf16 dim and vdim are multiples of 16 and the pool's strides multiples of 8.
+ */
+int tlaloc_b200_grouped_attention_slices(int32_t num_tokens, int32_t num_heads, int32_t v_heads, int32_t maps, int32_t dim, int32_t vdim,
+                                         int32_t dtype, int32_t max_live);
+int tlaloc_b200_grouped_attention(const void* q, const void* pool, int64_t pool_ld, int32_t dtype, const int32_t* block_tables,
+                                  const int32_t* row_tables, const int32_t* seq_lens, float* records, int32_t slices, int32_t num_tokens,
+                                  int32_t num_heads, int32_t v_heads, int32_t maps, int32_t dim, int32_t vdim, int32_t v_first,
+                                  int32_t num_blocks, int32_t block_size, int32_t max_blocks, int32_t num_tables, int32_t window,
+                                  int32_t keep_first, float scale, void* stream);
+
+/*
+ * Differential attention's end: per row and head out = rms_norm(a1 - lambda * a2) * keep * sigmoid(gate[row, head]) over the head's vdim
+ * values, no gain.  in: records of `slices` slices, the heads' two maps side by side ([slices][rows][heads][2][2 + in_ld]), or
+ * (slices 0) the maps' outputs themselves, f32 [rows][heads][2][in_ld].  gate: logits, rows gate_ld apart, or NULL; out: `dtype`.
+ */
+int tlaloc_b200_map_difference(const float* in, int32_t slices, const float* gate, int64_t gate_ld, void* out, int64_t out_ld, int32_t dtype,
+                               int32_t rows, int32_t heads, int32_t vdim, int32_t in_ld, float lambda, float keep, float eps, void* stream);
+
+/* A recurrence's end: per row and head out = in / rms(in) * silu(gate) over the head's vdim values; in f32 [rows][heads][vdim], gate
+ * f32 with rows gate_ld apart, out `dtype`. */
+int tlaloc_b200_head_norm_gate(const float* in, const float* gate, int64_t gate_ld, void* out, int64_t out_ld, int32_t dtype, int32_t rows,
+                               int32_t heads, int32_t vdim, float eps, void* stream);
+
+/*
+ * Retention: per head S <- decay * S + k v^T, o = S^T q, S [dim][vdim rounded up to a multiple of 4] in f32, one state per slot
+ * ([num_slots][heads][dim][..]); a row at position 0 starts from zero, whatever the slot holds.
+ * _step: one token per row, with everything around it: a row of `in` (f32, row stride ld) is [q heads x dim | k heads x dim |
+ * v heads x vdim | gate heads x vdim]; the first rot_dims values of q and k are rotated (halves), k is multiplied by k_scale, and
+ * out = o / rms(o) * silu(gate) as `dtype`.  row_states i32 [rows]; decay f32 [heads].
+ * _scan: the `tokens` tokens of ONE sequence in order, q and k [tokens][heads][dim_ld] (rotated, scaled) and v [tokens][heads][v_ld] of
+ * `dtype`; o f32 [tokens][heads][vdim].  row_states and positions are those of its first token.
+ */
+int tlaloc_b200_retention_step(const float* in, int64_t ld, const int32_t* positions, const float* cos_table, const float* sin_table,
+                               const float* decay, const int32_t* row_states, float* state, void* out, int64_t out_ld, int32_t dtype,
+                               int32_t rows, int32_t heads, int32_t dim, int32_t vdim, int32_t rot_dims, int32_t num_slots, int32_t max_pos,
+                               float k_scale, float eps, void* stream);
+int tlaloc_b200_retention_scan(const void* q, const void* k, int32_t dim_ld, const void* v, int32_t v_ld, int32_t dtype,
+                               const int32_t* positions, const float* decay, const int32_t* row_states, float* state, float* o, int32_t tokens,
+                               int32_t heads, int32_t dim, int32_t vdim, int32_t num_slots, void* stream);
+
+/* ------------------------------------------------------------------ mixture of experts */
+
+/*
+ * Per token the `top` experts with the largest of `experts` logits (f32, rows ld apart; the first of equals) and the softmax over those
+ * (ids, weights [tokens][top], largest first); then the entries (token, k) sorted by expert: expert e has the rows [offsets[e],
+ * offsets[e + 1]) (i32 [experts + 1]), entry i is row entry_rows[i], row r belongs to token row_tokens[r].  At most 1024 experts.
+ */
+int tlaloc_b200_moe_route(const float* logits, int64_t ld, int32_t* ids, float* weights, int32_t* offsets, int32_t* entry_rows,
+                          int32_t* row_tokens, int32_t tokens, int32_t experts, int32_t top, void* stream);
+/* out[r, :] = in[rows[r], :], rows of row_bytes (even) bytes. */
+int tlaloc_b200_gather_rows(const void* in, const int32_t* rows, void* out, int32_t count, int64_t row_bytes, void* stream);
 
 /* ------------------------------------------------------------------ tensor parallelism: the sum over ranks */
 

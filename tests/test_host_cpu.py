@@ -39,6 +39,10 @@ def test_a_subset_of_the_kernels_is_a_library_of_its_own():
                  "latent_attention", "latent_attention_scratch_bytes", "latent_gather", "window_attention", "window_attention_applies"):
         assert hasattr(lib, "tlaloc_b200_" + name), name
     assert not hasattr(lib, "tlaloc_b200_int8_gemm")
+    lib = ctypes.CDLL(B.build(subset="mixed", own=True))
+    for name in ("init", "device_status", "embedding", "argmax", "dense_gemm", "rmsnorm_pair", "latent_gather", "window_attention", "residual_norm", "rotate_rows",
+                 "grouped_attention", "map_difference", "retention_step", "retention_scan", "head_norm_gate", "moe_route", "gather_rows"):
+        assert hasattr(lib, "tlaloc_b200_" + name), name
 
 
 def test_dense_and_latent_refusals_need_no_gpu():
@@ -56,10 +60,46 @@ def test_dense_and_latent_refusals_need_no_gpu():
                                                         64, 4, kw.get("tables", 1), kw.get("window", 0), 0, 0.1, None)
     assert att(ld=40) == i and att(rows=2) == i and att(window=-1) == i and att(rows=0) == N.OK
     assert lib.tlaloc_b200_window_attention_applies(128, 64, 128) == 1 and lib.tlaloc_b200_window_attention_applies(12, 4, 10) == 0
-    win = lambda **kw: lib.tlaloc_b200_window_attention(one, one, one, 8, one, 96, 48, one, 48, kw.get("q", 2), kw.get("k", 2), 0, 2, 24, 8, 24, 0,
-                                                        kw.get("scale", 0.1), None)
+    win = lambda **kw: lib.tlaloc_b200_window_attention(one, one, 48, one, 8, one, 48, 96, one, 48, N.BF16, kw.get("q", 2), kw.get("k", 2), 0, kw.get("heads", 2),
+                                                        kw.get("v_heads", 2), kw.get("maps", 1), 24, 8, 24, 0, kw.get("keep", 0), kw.get("scale", 0.1), None)
     assert win(q=3) == i and win(scale=-1.0) == N.UNSUPPORTED and win(q=0) == N.OK
-    assert lib.tlaloc_b200_latent_gather(one, 56, N.BF16, one, one, 56, 200, 100, 56, 9, 64, 4, None) == i
+    assert win(heads=3) == i and win(maps=4) == i and win(v_heads=0) == i and win(keep=-1) == i
+    gather = lambda first, keep, count: lib.tlaloc_b200_latent_gather(one, 56, N.BF16, one, one, 56, first, keep, count, 56, 9, 64, 4, None)
+    assert gather(200, 0, 100) == i and gather(5, 6, 20) == i and gather(200, 50, 40) == i and gather(200, 50, 107) == i and gather(256, 0, 0) == N.OK
+
+
+def test_refusals_of_the_mixers_need_no_gpu():
+    lib = N.lib()
+    one, i = ctypes.c_void_p(16), N.INVALID_ARGUMENT
+    assert lib.tlaloc_b200_residual_norm(None, None, 0, None, None, None, 0, one, one, one, one, N.BF16, 1, 8, 1e-5, None) == i
+    assert lib.tlaloc_b200_residual_norm(one, None, 0, None, None, None, 2, one, one, one, one, N.BF16, 1, 8, 1e-5, None) == i
+    part = N.RotatePart(out=16, out_ld=16, out_head_ld=8, first=0, heads=2, dim=8, padded=8, rotate=1, by_slot=0, scale=1.0)
+    rotate = lambda ld=16, dims=8, slots=None: lib.tlaloc_b200_rotate_rows(one, ld, ctypes.byref(part), 1, N.BF16, one, one, one, slots, 0, dims, 4, 4, None)
+    assert rotate() == N.OK and rotate(ld=15) == i and rotate(dims=10) == i and rotate(dims=7) == i
+    part.by_slot = 1
+    assert rotate() == i
+    att = lambda **kw: lib.tlaloc_b200_grouped_attention(one, one, kw.get("ld", 96), N.BF16, one, None, one, one, kw.get("slices", 1), kw.get("rows", 0), kw.get("heads", 8),
+                                                         2, 2, 16, 16, kw.get("v_first", 64), 9, 64, 4, 1, kw.get("window", 0), kw.get("keep", 0), 0.1, None)
+    assert att() == N.OK and att(ld=95) == i and att(heads=6) == i and att(v_first=63) == i and att(window=-1) == i and att(keep=-1) == i and att(slices=0) == i
+    assert lib.tlaloc_b200_grouped_attention_slices(4, 8, 2, 2, 24, 16, N.BF16, 4096) == 1  # not the tensor-core kernel's sizes
+    assert lib.tlaloc_b200_map_difference(one, -1, None, 0, one, 16, N.BF16, 1, 2, 8, 8, 0.1, 0.5, 1e-5, None) == i
+    assert lib.tlaloc_b200_map_difference(one, 0, None, 0, one, 15, N.BF16, 1, 2, 8, 8, 0.1, 0.5, 1e-5, None) == i
+    assert lib.tlaloc_b200_head_norm_gate(one, one, 16, one, 15, N.BF16, 1, 2, 8, 1e-5, None) == i
+    step = lambda **kw: lib.tlaloc_b200_retention_step(one, kw.get("ld", 64), one, one, one, one, one, one, one, 16, N.BF16, kw.get("rows", 0), 2, kw.get("dim", 8), 8,
+                                                       kw.get("rot", 8), 3, 4, 0.3, 1e-5, None)
+    assert step() == N.OK and step(ld=63) == i and step(rot=10) == i and step(rows=-1) == i and step(dim=520, ld=9999) == N.UNSUPPORTED
+    assert lib.tlaloc_b200_retention_scan(one, one, 7, one, 8, N.BF16, one, one, one, one, one, 4, 2, 8, 8, 3, None) == i
+    assert lib.tlaloc_b200_moe_route(one, 4, one, one, one, one, one, 3, 5, 2, None) == i and lib.tlaloc_b200_moe_route(one, 8, one, one, one, one, one, 3, 5, 6, None) == i
+    assert lib.tlaloc_b200_gather_rows(one, one, one, 1, 3, None) == i
+    g = N.DenseProblem(x=16, w=16, y=16, ld_x=8, ld_y=16, k=8, n=32, batch=1, act=N.ACT_SILU_MUL, y_dtype=N.F32)
+    dense = lambda *ps: lib.tlaloc_b200_dense_gemm((N.DenseProblem * len(ps))(*ps), len(ps), N.BF16, 0, 0, None)
+    assert dense(g) == N.OK
+    g.n = 40
+    assert dense(g) == i  # gate and factor come in blocks of 16
+    g.n, g.bias = 32, 16
+    assert dense(g) == i
+    g.bias, g.row_offsets = None, 16
+    assert dense(g) == N.OK and dense(g, g) == i  # a grouped projection is the last of a call
 
 
 def test_argument_refusals_need_no_gpu():

@@ -14,7 +14,7 @@ F32, BF16, S8, S32, F8E4M3FN = 11, 16, 2, 4, 20
 OK, INVALID_ARGUMENT, UNSUPPORTED, INTERNAL = 0, -1, -2, -3
 GEMM_EXACT, GEMM_X_F32_EXACT, GEMM_WEIGHTS_CONST, GEMM_I8_MMA, GEMM_X_PLANES = 1, 2, 4, 8, 16
 
-ACT_NONE, ACT_RELU2 = 0, 1
+ACT_NONE, ACT_RELU2, ACT_SILU_MUL, ACT_GELU_TANH_MUL = 0, 1, 2, 3
 
 _lib = None
 _subset: str | None = None
@@ -28,7 +28,13 @@ class DenseProblem(ctypes.Structure):
     """tlaloc_b200_dense_problem"""
     _fields_ = [("x", _vp), ("w", _vp), ("bias", _vp), ("residual", _vp), ("y", _vp),
                 ("ld_x", _i64), ("ld_res", _i64), ("ld_y", _i64), ("batch_x", _i64), ("batch_w", _i64), ("batch_y", _i64),
-                ("k", _i32), ("n", _i32), ("batch", _i32), ("act", _i32), ("y_dtype", _i32)]
+                ("k", _i32), ("n", _i32), ("batch", _i32), ("act", _i32), ("y_dtype", _i32), ("rows", _i32), ("row_offsets", _vp)]
+
+
+class RotatePart(ctypes.Structure):
+    """tlaloc_b200_rotate_part"""
+    _fields_ = [("out", _vp), ("out_ld", _i64), ("out_head_ld", _i64), ("first", _i32), ("heads", _i32), ("dim", _i32), ("padded", _i32),
+                ("rotate", _i32), ("by_slot", _i32), ("scale", _f32)]
 
 
 _SIGNATURES = {
@@ -64,9 +70,19 @@ _SIGNATURES = {
     "tlaloc_b200_rope_interleaved": (ctypes.c_int, [_vp, _i64, _i64, _vp, _i64, _i64, _i32, _vp, _vp, _vp] + [_i32] * 5 + [_vp]),
     "tlaloc_b200_latent_attention_scratch_bytes": (_sz, [_i32] * 5),
     "tlaloc_b200_latent_attention": (ctypes.c_int, [_vp, _vp, _i64, _i32, _vp, _vp, _vp, _vp, _vp, _sz] + [_i32] * 10 + [_f32, _vp]),
-    "tlaloc_b200_latent_gather": (ctypes.c_int, [_vp, _i64, _i32, _vp, _vp, _i64] + [_i32] * 6 + [_vp]),
+    "tlaloc_b200_latent_gather": (ctypes.c_int, [_vp, _i64, _i32, _vp, _vp, _i64] + [_i32] * 7 + [_vp]),
     "tlaloc_b200_window_attention_applies": (ctypes.c_int, [_i32] * 3),
-    "tlaloc_b200_window_attention": (ctypes.c_int, [_vp, _vp, _vp, _i64, _vp, _i64, _i64, _vp, _i64] + [_i32] * 8 + [_f32, _vp]),
+    "tlaloc_b200_window_attention": (ctypes.c_int, [_vp, _vp, _i64, _vp, _i64, _vp, _i64, _i64, _vp, _i64] + [_i32] * 12 + [_f32, _vp]),
+    "tlaloc_b200_residual_norm": (ctypes.c_int, [_vp, _vp, _i64, _vp, _vp, _vp, _i32, _vp, _vp, _vp, _vp, _i32, _i32, _i32, _f32, _vp]),
+    "tlaloc_b200_rotate_rows": (ctypes.c_int, [_vp, _i64, ctypes.POINTER(RotatePart), _i32, _i32, _vp, _vp, _vp, _vp] + [_i32] * 4 + [_vp]),
+    "tlaloc_b200_grouped_attention_slices": (ctypes.c_int, [_i32] * 8),
+    "tlaloc_b200_grouped_attention": (ctypes.c_int, [_vp, _vp, _i64, _i32, _vp, _vp, _vp, _vp] + [_i32] * 14 + [_f32, _vp]),
+    "tlaloc_b200_map_difference": (ctypes.c_int, [_vp, _i32, _vp, _i64, _vp, _i64] + [_i32] * 5 + [_f32, _f32, _f32, _vp]),
+    "tlaloc_b200_head_norm_gate": (ctypes.c_int, [_vp, _vp, _i64, _vp, _i64] + [_i32] * 4 + [_f32, _vp]),
+    "tlaloc_b200_retention_step": (ctypes.c_int, [_vp, _i64] + [_vp] * 7 + [_i64] + [_i32] * 8 + [_f32, _f32, _vp]),
+    "tlaloc_b200_retention_scan": (ctypes.c_int, [_vp, _vp, _i32, _vp, _i32, _i32] + [_vp] * 5 + [_i32] * 5 + [_vp]),
+    "tlaloc_b200_moe_route": (ctypes.c_int, [_vp, _i64] + [_vp] * 5 + [_i32] * 3 + [_vp]),
+    "tlaloc_b200_gather_rows": (ctypes.c_int, [_vp, _vp, _vp, _i32, _i64, _vp]),
     "tlaloc_b200_peer_alloc": (ctypes.c_int, [_sz, ctypes.POINTER(_vp), ctypes.c_char_p]),
     "tlaloc_b200_peer_open": (ctypes.c_int, [ctypes.c_char_p, ctypes.POINTER(_vp)]),
     "tlaloc_b200_peer_close": (ctypes.c_int, [_vp]),

@@ -16,11 +16,17 @@ template <typename T, typename YT>
 __global__ void __launch_bounds__(256) DenseGemmTiled(tlaloc_b200_dense_problem p, int M)
 {
   GridDependencySync();
+  int first = 0;
+  if (p.row_offsets != nullptr) {  // this weight's rows of the matrix
+    first = __ldg(p.row_offsets + blockIdx.z);
+    M = min(__ldg(p.row_offsets + blockIdx.z + 1), M);
+    if (first + static_cast<int>(blockIdx.y) * kTile >= M) return;
+  }
   __shared__ float xs[kStepK][kTile + 4], ws[kStepK][kTile + 4];
-  const int tid = threadIdx.x, n0 = blockIdx.x * kTile, m0 = blockIdx.y * kTile;
-  const T* x = static_cast<const T*>(p.x) + p.batch_x * blockIdx.z;
+  const int tid = threadIdx.x, n0 = blockIdx.x * kTile, m0 = first + blockIdx.y * kTile;
+  const T* x = static_cast<const T*>(p.x) + (p.row_offsets != nullptr ? 0 : p.batch_x * blockIdx.z);
   const T* w = static_cast<const T*>(p.w) + p.batch_w * blockIdx.z;
-  YT* y = static_cast<YT*>(p.y) + p.batch_y * blockIdx.z;
+  YT* y = static_cast<YT*>(p.y) + (p.row_offsets != nullptr ? 0 : p.batch_y * blockIdx.z);
   const int tn = (tid & 15) * 4, tm = (tid >> 4) * 4;
   float acc[4][4] = {};
   for (int k0 = 0; k0 < p.k; k0 += kStepK) {
@@ -41,6 +47,21 @@ __global__ void __launch_bounds__(256) DenseGemmTiled(tlaloc_b200_dense_problem 
     }
     __syncthreads();
   }
+  if (IsGated(p.act)) {  // columns n and n + 16 of a block of 32 are four threads apart
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      const int m = m0 + tm + i;
+#pragma unroll
+      for (int j = 0; j < 4; ++j) {
+        const float other = __shfl_xor_sync(0xffffffffu, acc[i][j], 4);
+        const int n = n0 + tn + j;
+        if (n < p.n && m < M && (n & kGateBlock) == 0) {
+          y[static_cast<size_t>(m) * p.ld_y + (n >> 5) * kGateBlock + (n & 15)] = FromF32<YT>(GatedValue(p.act, acc[i][j], other));
+        }
+      }
+    }
+    return;
+  }
 #pragma unroll
   for (int i = 0; i < 4; ++i) {
     const int m = m0 + tm + i;
@@ -56,6 +77,7 @@ __global__ void __launch_bounds__(256) DenseGemmTiled(tlaloc_b200_dense_problem 
 template <typename T>
 cudaError_t LaunchTiled(const tlaloc_b200_dense_problem& p, int m, cudaStream_t st)
 {
+  if (p.rows > 0) m = p.rows;
   const dim3 grid((p.n + kTile - 1) / kTile, (m + kTile - 1) / kTile, p.batch);
   return p.y_dtype == TLALOC_B200_F32 ? LaunchChained(DenseGemmTiled<T, float>, grid, 256, 0, st, p, m)
                                       : LaunchChained(DenseGemmTiled<T, __nv_bfloat16>, grid, 256, 0, st, p, m);
@@ -78,12 +100,17 @@ extern "C" int tlaloc_b200_dense_gemm(const tlaloc_b200_dense_problem* problems,
     if (!p.x || !p.w || !p.y) return Fail(kInvalid, "%s: a required device pointer is null", op);
     if (p.k < 1 || p.n < 1 || p.batch < 1 || p.batch > 65535) return Fail(kInvalid, "%s: bad sizes", op);
     if (!IsFloatType(p.y_dtype)) return Fail(kInvalid, "%s: y must be f32 or bf16", op);
-    if (p.act != TLALOC_B200_ACT_NONE && p.act != TLALOC_B200_ACT_RELU2) return Fail(kInvalid, "%s: unknown activation %d", op, p.act);
-    if (p.ld_x < p.k || p.ld_y < p.n || (p.residual && p.ld_res < p.n)) return Fail(kInvalid, "%s: a row stride is shorter than its row", op);
+    if (p.act != TLALOC_B200_ACT_NONE && p.act != TLALOC_B200_ACT_RELU2 && !IsGated(p.act)) return Fail(kInvalid, "%s: unknown activation %d", op, p.act);
+    if (IsGated(p.act) && (p.n % (2 * kGateBlock) != 0 || p.bias || p.residual)) {
+      return Fail(kInvalid, "%s: a gated projection has a multiple of %d rows, no bias and no residual", op, 2 * kGateBlock);
+    }
+    if (p.row_offsets && i + 1 < count) return Fail(kInvalid, "%s: a grouped projection is the last of a call", op);
+    if (p.rows < 0 || (p.row_offsets && (p.residual || p.bias || p.batch > kMaxGroups))) return Fail(kInvalid, "%s: bad groups", op);
+    if (((p.rows > 0 ? p.rows : m) + kTile - 1) / kTile > 65535) return Fail(kInvalid, "%s: too many rows", op);
+    if (p.ld_x < p.k || p.ld_y < (IsGated(p.act) ? p.n / 2 : p.n) || (p.residual && p.ld_res < p.n)) return Fail(kInvalid, "%s: a row stride is shorter than its row", op);
     if (p.batch > 1 && (p.residual || p.bias)) return Fail(kInvalid, "%s: a batched projection takes no bias and no residual", op);
   }
   if (m == 0) return kOk;
-  if ((m + kTile - 1) / kTile > 65535) return Fail(kInvalid, "%s: too many rows", op);
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   int launches = 0;
   cudaError_t e = cudaSuccess;

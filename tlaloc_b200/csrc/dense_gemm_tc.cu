@@ -12,6 +12,11 @@
 //   K slices (few tiles)     the slices of one tile are a cluster; each leaves its partial tile in shared memory and the ranks
 //                            finish every ks-th activation row, summing in rank order through distributed shared memory.
 // Rows, columns and k past the ends are outside the tensor maps and arrive as zeros.  Every mbarrier wait is bounded.
+//
+// Grouped problems (experts): the weights are a batch, the activations one matrix whose rows are sorted by weight.  How many tiles
+// a weight has is known on the device alone: each CTA counts them from the row offsets, and a tile that passes the end of its
+// weight's rows computes rows of the next one too and leaves them out.  Gated activations: gate and other factor are sixteen
+// lanes apart; two activation rows at a time, the half warps exchange one value each and both evaluate one output.
 #include <cuda.h>
 
 #include "common.cuh"
@@ -46,13 +51,15 @@ struct Layout {
 struct TcProblem {
   const float* bias;
   const float* residual;
+  const int* offsets;  // grouped: [groups + 1]
   void* y;
   int64_t ld_res, ld_y, batch_y;
-  int k, n, act, y_f32, rows_bf16, tiles_n, swap_x;  // rows_bf16: y takes whole 16-byte words; swap_x: the activations' map has the batch before the rows
+  int M, tiles_m;
+  int k, n, act, y_f32, rows_bf16, tiles_n, swap_x, gated, groups;  // rows_bf16: y takes whole 16-byte words; swap_x: the activations' map has the batch before the rows
 };
 struct TcArgs {
   TcProblem p[2];
-  int M, tiles_m, tiles0, tiles, ks, weights_const;
+  int tiles0, tiles, ks, weights_const;  // a grouped problem's tiles are not counted here
 };
 
 __device__ int g_dense_status = 0;  // nonzero after an mbarrier wait timed out (sticky until read)
@@ -70,18 +77,65 @@ __device__ __forceinline__ void TmaBox3d(uint32_t dst, const CUtensorMap* map, i
       : "memory");
 }
 struct Tile {
-  int pr, n0, m0, b;
+  int pr, n0, m0, b, M;  // M: first row that is not the tile's to write
 };
-__device__ __forceinline__ Tile TileAt(const TcArgs& a, int id, int BT)
+// start: of a grouped problem (the last one), the first tile of every group, counted from the problem's own first tile.
+template <bool GROUPED>
+__device__ __forceinline__ Tile TileAt(const TcArgs& a, int id, int BT, const int* start)
 {
   Tile t;
   t.pr = id >= a.tiles0 ? 1 : 0;
   if (t.pr) id -= a.tiles0;
-  t.m0 = (id % a.tiles_m) * BT;  // activation tiles of one weight tile run side by side: the weights leave HBM once
-  id /= a.tiles_m;
-  t.n0 = (id % a.p[t.pr].tiles_n) * kBN;
-  t.b = id / a.p[t.pr].tiles_n;
+  const TcProblem& p = a.p[t.pr];
+  if (GROUPED && p.offsets != nullptr) {
+    int lo = 0, hi = p.groups;  // start[lo] <= id < start[hi]
+    while (hi - lo > 1) {
+      const int mid = (lo + hi) >> 1;
+      if (start[mid] <= id) lo = mid;
+      else hi = mid;
+    }
+    id -= start[lo];
+    t.b = lo;
+    const int first = p.offsets[lo], tiles_m = (start[lo + 1] - start[lo]) / p.tiles_n;
+    t.M = p.offsets[lo + 1];
+    t.m0 = first + (id % tiles_m) * BT;
+    t.n0 = (id / tiles_m) * kBN;
+    return t;
+  }
+  t.M = p.M;
+  t.m0 = (id % p.tiles_m) * BT;  // activation tiles of one weight tile run side by side: the weights leave HBM once
+  id /= p.tiles_m;
+  t.n0 = (id % p.tiles_n) * kBN;
+  t.b = id / p.tiles_n;
   return t;
+}
+
+// v: CH rows of the warp's 32 columns, gate in the lower sixteen lanes -> CH / 2 outputs of column 16 quad + (lane & 15), of rows
+// 2 i + (lane >> 4).
+template <int CH>
+__device__ __forceinline__ void Gate(int act, float* v, int lane)
+{
+  const bool upper = lane >= kGateBlock;
+#pragma unroll
+  for (int i = 0; i < CH / 2; ++i) {
+    const float a = v[2 * i], b = v[2 * i + 1];
+    const float got = __shfl_xor_sync(0xffffffffu, upper ? a : b, kGateBlock);
+    v[i] = GatedValue(act, upper ? got : a, upper ? b : got);
+  }
+}
+template <int CH>
+__device__ __forceinline__ void StoreGated(const TcProblem& p, const Tile& t, int quad, int lane, int m, int M, const float* v)
+{
+  const int n = (t.n0 >> 1) + quad * kGateBlock + (lane & 15);
+  if (n >= p.n / 2) return;
+#pragma unroll
+  for (int i = 0; i < CH / 2; ++i) {
+    const int r = m + 2 * i + (lane >> 4);
+    if (r >= M) return;
+    const size_t at = t.b * p.batch_y + static_cast<size_t>(r) * p.ld_y + n;
+    if (p.y_f32) static_cast<float*>(p.y)[at] = v[i];
+    else static_cast<__nv_bfloat16*>(p.y)[at] = __float2bfloat16_rn(v[i]);
+  }
 }
 
 // One output column n of CH consecutive rows from m: bias, activation, residual, store.
@@ -141,7 +195,28 @@ __device__ __forceinline__ void StoreRowsBf16(const TcProblem& p, const Tile& t,
   asm volatile("bar.sync %0, 128;\n" ::"r"(1 + group) : "memory");
 }
 
-template <int BT, bool SPLIT>
+// The same for the 64 outputs a row of a gated tile has.
+template <int CH>
+__device__ __forceinline__ void StoreRowsGatedBf16(const TcProblem& p, const Tile& t, int m, int M, const float* v, __nv_bfloat16* stage, int tid,
+                                                   int group)
+{
+  const int col = tid & 127, lane = tid & 31, quad = col >> 5;
+  constexpr int kW = kBN / 2;
+#pragma unroll
+  for (int i = 0; i < CH / 2; ++i) stage[(2 * i + (lane >> 4)) * kW + quad * kGateBlock + (lane & 15)] = __float2bfloat16_rn(v[i]);
+  asm volatile("bar.sync %0, 128;\n" ::"r"(1 + group) : "memory");
+  const int64_t ld = p.ld_y;
+  __nv_bfloat16* y = static_cast<__nv_bfloat16*>(p.y) + t.b * p.batch_y + static_cast<size_t>(m) * ld + (t.n0 >> 1) + (col & 7) * 8;
+  const uint4* src = reinterpret_cast<const uint4*>(stage) + (col & 7);
+#pragma unroll
+  for (int i = 0; i < CH / 16; ++i) {
+    const int r = i * 16 + (col >> 3);
+    if (m + r < M) *reinterpret_cast<uint4*>(y + r * ld) = src[r * 8];
+  }
+  asm volatile("bar.sync %0, 128;\n" ::"r"(1 + group) : "memory");
+}
+
+template <int BT, bool SPLIT, bool GROUPED = false>
 __global__ void __launch_bounds__(kThreads, 1)
     DenseGemmTcKernel(const __grid_constant__ CUtensorMap w0, const __grid_constant__ CUtensorMap x0,
                       const __grid_constant__ CUtensorMap w1, const __grid_constant__ CUtensorMap x1, const __grid_constant__ TcArgs a)
@@ -176,6 +251,30 @@ __global__ void __launch_bounds__(kThreads, 1)
   __syncthreads();
   asm volatile("tcgen05.fence::after_thread_sync;\n" ::: "memory");
   const uint32_t tmem = *slot;
+  __shared__ int s_start[GROUPED ? kMaxGroups + 1 : 1];
+  int tiles = a.tiles;
+  if constexpr (GROUPED) {
+    GridDependencySync();
+    const TcProblem& g = a.p[1].offsets != nullptr ? a.p[1] : a.p[0];
+    if (warp == 0) {
+      int total = 0;
+      for (int e0 = 0; e0 < g.groups; e0 += 32) {
+        const int e = e0 + lane;
+        int v = e < g.groups ? (g.offsets[e + 1] - g.offsets[e] + BT - 1) / BT * g.tiles_n : 0;
+        const int own = v;
+#pragma unroll
+        for (int o = 1; o < 32; o <<= 1) {
+          const int u = __shfl_up_sync(0xffffffffu, v, o);
+          if (lane >= o) v += u;
+        }
+        if (e < g.groups) s_start[e] = total + v - own;
+        total += __shfl_sync(0xffffffffu, v, 31);
+      }
+      if (lane == 0) s_start[g.groups] = total;
+    }
+    __syncthreads();
+    tiles += s_start[g.groups];
+  }
   // The blocks of k of a tile this CTA sums: all of them, or the slice of its cluster rank.
   auto blocks = [&](const Tile& t, int& first) {
     const int nb = (a.p[t.pr].k + kBK - 1) / kBK;
@@ -192,7 +291,7 @@ __global__ void __launch_bounds__(kThreads, 1)
   if (warp == kEpiWarps) {
     if (ElectOne()) {
       uint64_t w_policy, x_policy;
-      if (a.tiles_m == 1) asm volatile("createpolicy.fractional.L2::evict_first.b64 %0, 1.0;\n" : "=l"(w_policy));
+      if (a.p[0].tiles_m == 1) asm volatile("createpolicy.fractional.L2::evict_first.b64 %0, 1.0;\n" : "=l"(w_policy));
       else asm volatile("createpolicy.fractional.L2::evict_normal.b64 %0, 1.0;\n" : "=l"(w_policy));
       asm volatile("createpolicy.fractional.L2::evict_last.b64 %0, 1.0;\n" : "=l"(x_policy));
       auto load_w = [&](const Tile& t, int kb, int s) {
@@ -200,22 +299,27 @@ __global__ void __launch_bounds__(kThreads, 1)
       };
       auto load_x = [&](const Tile& t, int kb, int s) {
         const bool swap = a.p[t.pr].swap_x != 0;
-        TmaBox3d(base + s * L::kStage + kWBytes, t.pr ? &x1 : &x0, kb * kBK, swap ? t.b : t.m0, swap ? t.m0 : t.b, full + 8 * s, x_policy);
+        const int z = GROUPED && a.p[t.pr].offsets != nullptr ? 0 : t.b;
+        TmaBox3d(base + s * L::kStage + kWBytes, t.pr ? &x1 : &x0, kb * kBK, swap ? z : t.m0, swap ? t.m0 : z, full + 8 * s, x_policy);
       };
       // Constant weights of the first stages travel before the dependency wait; activations only after it.
-      Tile t = TileAt(a, blockIdx.x, BT);
-      int first, nb = blocks(t, first);
-      const int ahead = a.weights_const ? min(nb, S) : 0;
+      Tile t;
+      int first = 0, nb = 0;
+      if (!GROUPED) {
+        t = TileAt<GROUPED>(a, blockIdx.x, BT, s_start);
+        nb = blocks(t, first);
+      }
+      const int ahead = !GROUPED && a.weights_const ? min(nb, S) : 0;
       for (int b = 0; b < ahead; ++b) {
         MbarExpectTx(full + 8 * b, L::kStage);
         load_w(t, first + b, b);
       }
-      GridDependencySync();
+      if (!GROUPED) GridDependencySync();
       for (int b = 0; b < ahead; ++b) load_x(t, first + b, b);
       int it = ahead, b = ahead;
-      for (int id = blockIdx.x; id < a.tiles; id += gridDim.x) {
-        if (id != static_cast<int>(blockIdx.x)) {
-          t = TileAt(a, id, BT);
+      for (int id = blockIdx.x; id < tiles; id += gridDim.x) {
+        if (GROUPED || id != static_cast<int>(blockIdx.x)) {
+          t = TileAt<GROUPED>(a, id, BT, s_start);
           nb = blocks(t, first);
           b = 0;
         }
@@ -236,13 +340,13 @@ __global__ void __launch_bounds__(kThreads, 1)
     }
     __syncwarp();
   } else if (warp == kEpiWarps + 1) {
-    GridDependencySync();  // nothing to read, but the time limit of its waits then starts with the work
+    if (!GROUPED) GridDependencySync();  // nothing to read, but the time limit of its waits then starts with the work
     if (ElectOne()) {
       constexpr uint32_t idesc = InstrDescBf16(BT);
       const uint64_t wd0 = SmemDesc(base, 16, 1024), xd0 = SmemDesc(base + kWBytes, 16, 1024);
       int it = 0, lt = 0;
-      for (int id = blockIdx.x; id < a.tiles; id += gridDim.x, ++lt) {
-        const Tile t = TileAt(a, id, BT);
+      for (int id = blockIdx.x; id < tiles; id += gridDim.x, ++lt) {
+        const Tile t = TileAt<GROUPED>(a, id, BT, s_start);
         int first;
         const int nb = blocks(t, first);
         const uint32_t acc = tmem + (lt & 1) * BT;
@@ -264,12 +368,12 @@ __global__ void __launch_bounds__(kThreads, 1)
     }
     __syncwarp();
   } else {
-    GridDependencySync();
+    if (!GROUPED) GridDependencySync();
     const int quad = warp & 3, half = warp >> 2;
     constexpr int kHalf = BT / 2, CH = kHalf < 32 ? kHalf : 32;
     int lt = 0;
-    for (int id = blockIdx.x; id < a.tiles; id += gridDim.x, ++lt) {
-      const Tile t = TileAt(a, id, BT);
+    for (int id = blockIdx.x; id < tiles; id += gridDim.x, ++lt) {
+      const Tile t = TileAt<GROUPED>(a, id, BT, s_start);
       int first;
       const int nb = blocks(t, first);
       const TcProblem& p = a.p[t.pr];
@@ -279,7 +383,7 @@ __global__ void __launch_bounds__(kThreads, 1)
       asm volatile("tcgen05.fence::after_thread_sync;\n" ::: "memory");
 #pragma unroll 1
       for (int c = half * kHalf; c < (half + 1) * kHalf; c += CH) {
-        if (!SPLIT && t.m0 + c >= a.M) break;
+        if (!SPLIT && t.m0 + c >= t.M) break;
         uint32_t r[CH];
         const uint32_t taddr = tmem + (static_cast<uint32_t>(quad * 32) << 16) + (lt & 1) * BT + c;
         if constexpr (CH == 32) TcLd32(taddr, r);
@@ -293,10 +397,15 @@ __global__ void __launch_bounds__(kThreads, 1)
           float v[CH];
 #pragma unroll
           for (int e = 0; e < CH; ++e) v[e] = __uint_as_float(r[e]);
-          if (p.rows_bf16 && t.n0 + kBN <= p.n) {
-            StoreRowsBf16<CH>(p, t, t.m0 + c, a.M, v, bias, reinterpret_cast<__nv_bfloat16*>(smem + L::kOut) + half * CH * kBN, tid, half);
+          __nv_bfloat16* stage = reinterpret_cast<__nv_bfloat16*>(smem + L::kOut) + half * CH * kBN;
+          if (p.gated) {
+            Gate<CH>(p.act, v, lane);
+            if (p.rows_bf16 && t.n0 + kBN <= p.n) StoreRowsGatedBf16<CH>(p, t, t.m0 + c, t.M, v, stage, tid, half);
+            else StoreGated<CH>(p, t, quad, lane, t.m0 + c, t.M, v);
+          } else if (p.rows_bf16 && t.n0 + kBN <= p.n) {
+            StoreRowsBf16<CH>(p, t, t.m0 + c, t.M, v, bias, stage, tid, half);
           } else {
-            StoreColumn<CH>(p, t, n, t.m0 + c, a.M, v, bias);
+            StoreColumn<CH>(p, t, n, t.m0 + c, t.M, v, bias);
           }
         }
       }
@@ -310,12 +419,12 @@ __global__ void __launch_bounds__(kThreads, 1)
     cg::cluster_group cluster = cg::this_cluster();
     cluster.sync();  // every slice's tile is in its CTA's shared memory
     if (warp < kEpiWarps) {
-      const Tile t = TileAt(a, blockIdx.x, BT);
+      const Tile t = TileAt<false>(a, blockIdx.x, BT, s_start);
       const TcProblem& p = a.p[t.pr];
       const int nl = tid & 127, n = t.n0 + nl, nr = static_cast<int>(cluster.num_blocks());
       const float bias = p.bias != nullptr && n < p.n ? __ldg(p.bias + n) : 0.f;
       float* tile = reinterpret_cast<float*>(smem);
-      const int rows = min(BT, a.M - t.m0), step = 2 * nr;
+      const int rows = min(BT, t.M - t.m0), step = 2 * nr;
       constexpr int kU = 4;
       for (int c0 = static_cast<int>(cluster.block_rank()) + nr * (tid >> 7); c0 < rows; c0 += kU * step) {
         float v[kU] = {};
@@ -327,9 +436,23 @@ __global__ void __launch_bounds__(kThreads, 1)
 #pragma unroll
           for (int e = 0; e < kU; ++e) v[e] += u[e];
         }
+        if (p.gated) {
+          // rows c0 + 2 i step of the lower lanes' results, + step of the upper ones'
+          Gate<kU>(p.act, v, lane);
+          const int col = (t.n0 >> 1) + (nl >> 5) * kGateBlock + (lane & 15);
+#pragma unroll
+          for (int i = 0; i < kU / 2; ++i) {
+            const int r = c0 + (2 * i + (lane >> 4)) * step;
+            if (r >= rows || col >= p.n / 2) continue;
+            const size_t at = t.b * p.batch_y + static_cast<size_t>(t.m0 + r) * p.ld_y + col;
+            if (p.y_f32) static_cast<float*>(p.y)[at] = v[i];
+            else static_cast<__nv_bfloat16*>(p.y)[at] = __float2bfloat16_rn(v[i]);
+          }
+          continue;
+        }
 #pragma unroll
         for (int e = 0; e < kU; ++e)
-          if (c0 + e * step < rows) StoreColumn<1>(p, t, n, t.m0 + c0 + e * step, a.M, v + e, bias);
+          if (c0 + e * step < rows) StoreColumn<1>(p, t, n, t.m0 + c0 + e * step, t.M, v + e, bias);
       }
     }
     cluster.sync();  // no CTA leaves while a peer may still read its tile
@@ -383,6 +506,13 @@ cudaError_t PrepareDenseTc()
     TLALOC_OPT_IN(32, true);
     TLALOC_OPT_IN(64, true);
     TLALOC_OPT_IN(128, true);
+#define TLALOC_OPT_IN_GROUPED(BT) \
+  if (e == cudaSuccess) e = cudaFuncSetAttribute(DenseGemmTcKernel<BT, false, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, Layout<BT>::kBytes)
+    TLALOC_OPT_IN_GROUPED(32);
+    TLALOC_OPT_IN_GROUPED(64);
+    TLALOC_OPT_IN_GROUPED(128);
+    TLALOC_OPT_IN_GROUPED(256);
+#undef TLALOC_OPT_IN_GROUPED
 #undef TLALOC_OPT_IN
     if (e != cudaSuccess) return e;
     for (int ks = 1; ks <= 8; ++ks) {
@@ -440,7 +570,7 @@ int ChooseSlices(int tiles, int nb)
   return best;
 }
 
-template <int BT, bool SPLIT>
+template <int BT, bool SPLIT, bool GROUPED = false>
 cudaError_t Launch(const CUtensorMap* maps, const TcArgs& a, int ctas, cudaStream_t st)
 {
   cudaLaunchConfig_t cfg = {};
@@ -451,7 +581,7 @@ cudaError_t Launch(const CUtensorMap* maps, const TcArgs& a, int ctas, cudaStrea
   cudaLaunchAttribute attr[2];
   cfg.numAttrs = ChainAttributes(attr, SPLIT ? a.ks : 0);
   cfg.attrs = attr;
-  return cudaLaunchKernelEx(&cfg, DenseGemmTcKernel<BT, SPLIT>, maps[0], maps[1], maps[2], maps[3], a);
+  return cudaLaunchKernelEx(&cfg, DenseGemmTcKernel<BT, SPLIT, GROUPED>, maps[0], maps[1], maps[2], maps[3], a);
 }
 
 }  // namespace
@@ -466,25 +596,38 @@ cudaError_t LaunchDenseGemmTc(const tlaloc_b200_dense_problem* problems, int cou
 {
   cudaError_t e = PrepareDenseTc();
   if (e != cudaSuccess) return e;
-  int bt = m <= 32 ? 32 : m <= 64 ? 64 : m <= 128 ? 128 : 256;
-  if (bt == 256) {  // half the rows a tile where that fills the last wave of CTAs better by more than its own loss (about a seventh)
+  // Rows of a tile: what the problem has, or what a group has on average (one that has more takes several tiles).
+  int typical = 1;
+  bool grouped = false;
+  for (int i = 0; i < count; ++i) {
+    const tlaloc_b200_dense_problem& s = problems[i];
+    const int rows = s.rows > 0 ? s.rows : m;
+    typical = max(typical, s.row_offsets != nullptr ? (rows + s.batch - 1) / s.batch : rows);
+    grouped = grouped || s.row_offsets != nullptr;
+  }
+  int bt = typical <= 32 ? 32 : typical <= 64 ? 64 : typical <= 128 ? 128 : 256;
+  if (bt == 256 && !grouped) {  // half the rows a tile where that fills the last wave of CTAs better by more than its own loss (about a seventh)
     int columns = 0;
     for (int i = 0; i < count; ++i) columns += (problems[i].n + kBN - 1) / kBN * problems[i].batch;
-    auto waves = [&](int rows) { return (columns * ((m + rows - 1) / rows) + 147) / 148; };
+    auto waves = [&](int rows) { return (columns * ((typical + rows - 1) / rows) + 147) / 148; };
     if (waves(128) * 128 * 1.15 < waves(256) * 256) bt = 128;
   }
   CUtensorMap maps[4];
   TcArgs a = {};
-  a.M = m;
-  a.tiles_m = (m + bt - 1) / bt;
   a.weights_const = weights_const ? 1 : 0;
   int nb = 1 << 30;
   for (int i = 0; i < count; ++i) {
     const tlaloc_b200_dense_problem& s = problems[i];
     TcProblem& p = a.p[i];
     int swap_w = 0;
+    const bool groups = s.row_offsets != nullptr;
+    p.M = s.rows > 0 ? s.rows : m;
+    p.tiles_m = (p.M + bt - 1) / bt;
+    p.offsets = s.row_offsets;
+    p.groups = s.batch;
+    p.gated = IsGated(s.act) ? 1 : 0;
     if (!EncodeMatrix(&maps[2 * i], s.w, s.k, s.n, s.batch, s.k, s.batch_w, kBN, &swap_w) || swap_w ||
-        !EncodeMatrix(&maps[2 * i + 1], s.x, s.k, m, s.batch, s.ld_x, s.batch_x, bt, &p.swap_x)) {
+        !EncodeMatrix(&maps[2 * i + 1], s.x, s.k, p.M, groups ? 1 : s.batch, s.ld_x, s.batch_x, bt, &p.swap_x)) {
       return cudaErrorInvalidValue;
     }
     p.bias = s.bias;
@@ -492,22 +635,31 @@ cudaError_t LaunchDenseGemmTc(const tlaloc_b200_dense_problem* problems, int cou
     p.y = s.y;
     p.ld_res = s.ld_res;
     p.ld_y = s.ld_y;
-    p.batch_y = s.batch_y;
+    p.batch_y = groups ? 0 : s.batch_y;
     p.k = s.k;
     p.n = s.n;
     p.act = s.act;
     p.y_f32 = s.y_dtype == TLALOC_B200_F32 ? 1 : 0;
     p.rows_bf16 = !p.y_f32 && !s.residual && s.ld_y % 8 == 0 && (s.batch == 1 || s.batch_y % 8 == 0) && Aligned16(s.y) ? 1 : 0;
     p.tiles_n = (s.n + kBN - 1) / kBN;
-    a.tiles += p.tiles_n * a.tiles_m * s.batch;
-    if (i == 0) a.tiles0 = a.tiles;
+    if (!groups) a.tiles += p.tiles_n * p.tiles_m * s.batch;
+    if (i == 0) a.tiles0 = groups ? 1 << 30 : a.tiles;
     nb = min(nb, (s.k + kBK - 1) / kBK);
   }
   if (count == 1) {
     maps[2] = maps[0];
     maps[3] = maps[1];
   }
-  a.ks = bt <= 128 && a.tiles_m == 1 ? ChooseSlices(a.tiles, nb) : 1;
+  if (grouped) {
+    a.ks = 1;
+    switch (bt) {
+      case 32: return Launch<32, false, true>(maps, a, 148, st);
+      case 64: return Launch<64, false, true>(maps, a, 148, st);
+      case 128: return Launch<128, false, true>(maps, a, 148, st);
+      default: return Launch<256, false, true>(maps, a, 148, st);
+    }
+  }
+  a.ks = bt <= 128 && a.p[0].tiles_m == 1 && (count == 1 || a.p[1].tiles_m == 1) ? ChooseSlices(a.tiles, nb) : 1;
   if (a.ks > 1) {
     switch (bt) {
       case 32: return Launch<32, true>(maps, a, a.tiles, st);

@@ -12,6 +12,9 @@
 //   MMA lane        S(0); then S(j + 1), O += P(j) V(j)
 //   eight warps     softmax and, at the end, the output rows: warps w and w + 4 share 32 queries
 // Channels past a part's end are outside its tensor map and arrive as zeros.  Every mbarrier wait is bounded.
+//
+// Grouped heads and several maps: a query head is (value head, place in its group, map) and takes the keys of (value head, map).  The
+// first keep_first keys stay visible: their tiles come ahead of the window's.
 #include <cuda.h>
 
 #include "common.cuh"
@@ -29,9 +32,10 @@ constexpr int kThreads = kSoftmaxWarps * 32 + 64;
 constexpr int kMaxSmem = 227 * 1024;
 
 struct WindowArgs {
-  __nv_bfloat16* out;
+  void* out;
   int64_t out_ld;
   int T, L, q0, window;         // query i is key q0 + i; window 0: everything up to itself
+  int keep, group, maps, out_f32;  // keys visible whatever the window; query heads of a value head; key heads of a value head
   int dim, rot, vdim;
   int qk_atoms, dim_atoms, v_atoms, k_stages, v_stages;
   float scale_log2;
@@ -84,8 +88,12 @@ __global__ void __launch_bounds__(kThreads, 1)
   const int v_tile = v_atoms * kAtom, k_tile = qk_atoms * kAtom;
   const int m0 = blockIdx.x * kQ, head = blockIdx.y;
   const int q_last = min(m0 + kQ, a.T) - 1;
+  const int v_head = head / a.group, k_head = v_head * a.maps + head % a.maps;
+  // The tiles of kept keys, then those from the first one the window of any query reaches.
+  const int tile_hi = min(a.q0 + q_last, a.L - 1) / kKeys;
   const int tile_lo = a.window > 0 ? max(0, a.q0 + m0 - a.window + 1) / kKeys : 0;
-  const int tiles = min(a.q0 + q_last, a.L - 1) / kKeys - tile_lo + 1;
+  const int kept = min((a.keep + kKeys - 1) / kKeys, tile_lo), tiles = tile_hi - tile_lo + 1 + kept;
+  auto first_key = [&](int j) { return (j < kept ? j : tile_lo + j - kept) * kKeys; };
   if (tid == 0) {
     *abort_word = 0u;
     for (int i = 0; i < 2; ++i) {
@@ -113,12 +121,12 @@ __global__ void __launch_bounds__(kThreads, 1)
     if (ElectOne()) {
       // Stages are one or two per ring; everything is counted along (a division per box would take longer than the box).
       auto load_k = [&](int j) {
-        const int key = (tile_lo + j) * kKeys, stage = k_stages == 2 ? j & 1 : 0, before = j - k_stages;
+        const int key = first_key(j), stage = k_stages == 2 ? j & 1 : 0, before = j - k_stages;
         const uint32_t bar = kfull + 8 * stage;
         uint32_t dst = base + sk + stage * k_tile;
         if (before >= 0) ok = MbarWait(sfull + 8 * (before & 1), (before >> 1) & 1, abort_word) && ok;
         MbarExpectTx(bar, k_tile);
-        for (int c = 0; c < dim_atoms; ++c, dst += kAtom) TmaBox(dst, &map_k, c * 64, head, key, bar);
+        for (int c = 0; c < dim_atoms; ++c, dst += kAtom) TmaBox(dst, &map_k, c * 64, k_head, key, bar);
         for (int c = dim_atoms; c < qk_atoms; ++c, dst += kAtom) TmaBox(dst, &map_rot, (c - dim_atoms) * 64, 0, key, bar);
       };
       MbarExpectTx(qfull, qk_atoms * kAtom);
@@ -132,7 +140,7 @@ __global__ void __launch_bounds__(kThreads, 1)
         const uint32_t bar = vfull + 8 * stage;
         if (before >= 0) ok = MbarWait(odone + 8 * (before & 1), (before >> 1) & 1, abort_word) && ok;
         MbarExpectTx(bar, v_tile);
-        for (int c = 0; c < v_atoms; ++c) TmaBox(base + sv + stage * v_tile + c * kAtom, &map_v, c * 64, head, (tile_lo + j) * kKeys, bar);
+        for (int c = 0; c < v_atoms; ++c) TmaBox(base + sv + stage * v_tile + c * kAtom, &map_v, c * 64, v_head, first_key(j), bar);
       }
       if (!ok) {  // given up: let the copies in flight land before the CTA's shared memory goes away
         volatile uint32_t never = 0;
@@ -201,7 +209,7 @@ __global__ void __launch_bounds__(kThreads, 1)
     const int o_lo = half * 32;  // O's columns in blocks of 32, every second one
     float top = -INFINITY, sum = 0.f;
     for (int j = 0; j < tiles; ++j) {
-      const int key0 = (tile_lo + j) * kKeys + half * kHalf, b = j & 1;
+      const int key0 = first_key(j) + half * kHalf, b = j & 1;
       ok = MbarWaitWarp(sfull + 8 * b, (j >> 1) & 1, lane, abort_word) && ok;
       asm volatile("tcgen05.fence::after_thread_sync;\n" ::: "memory");
       uint32_t s[kHalf];
@@ -209,11 +217,11 @@ __global__ void __launch_bounds__(kThreads, 1)
       TcLd32(tmem + lanes + b * 128 + half * kHalf + 32, s + 32);
       asm volatile("tcgen05.wait::ld.sync.aligned;\n" ::: "memory");
       float t4[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
-      if (key0 + kHalf - 1 > safe_hi || key0 < safe_lo) {
+      if (key0 + kHalf - 1 > safe_hi || (key0 < safe_lo && key0 + kHalf > a.keep)) {
 #pragma unroll
         for (int e = 0; e < kHalf; ++e) {
           const int key = key0 + e;
-          if (key > qpos || key < first) s[e] = __float_as_uint(-INFINITY);
+          if (key > qpos || (key < first && key >= a.keep)) s[e] = __float_as_uint(-INFINITY);
         }
       }
 #pragma unroll
@@ -262,7 +270,9 @@ __global__ void __launch_bounds__(kThreads, 1)
     ok = MbarWaitWarp(odone + 8 * ((tiles - 1) & 1), ((tiles - 1) >> 1) & 1, lane, abort_word) && ok;
     asm volatile("tcgen05.fence::after_thread_sync;\n" ::: "memory");
     const float inv = sum > 0.f ? 1.f / sum : 0.f;
-    __nv_bfloat16* out = a.out + static_cast<size_t>(m0 + row) * a.out_ld + static_cast<size_t>(head) * a.vdim;
+    const size_t out_at = static_cast<size_t>(m0 + row) * a.out_ld + static_cast<size_t>(head) * a.vdim;
+    __nv_bfloat16* out = static_cast<__nv_bfloat16*>(a.out) + out_at;
+    float* out32 = static_cast<float*>(a.out) + out_at;
     const bool live = m0 + row < a.T;
     for (int c = o_lo; c < a.vdim; c += 64) {
       uint32_t o[32];
@@ -270,7 +280,13 @@ __global__ void __launch_bounds__(kThreads, 1)
       asm volatile("tcgen05.wait::ld.sync.aligned;\n" ::: "memory");
 #pragma unroll
       for (int e = 0; e < 32; e += 8) {
-        if (live && c + e < a.vdim) {  // vdim is a multiple of 8
+        if (live && c + e < a.vdim && a.out_f32) {
+#pragma unroll
+          for (int i = 0; i < 8; i += 4) {
+            *reinterpret_cast<float4*>(out32 + c + e + i) = make_float4(__uint_as_float(o[e + i]) * inv, __uint_as_float(o[e + i + 1]) * inv,
+                                                                        __uint_as_float(o[e + i + 2]) * inv, __uint_as_float(o[e + i + 3]) * inv);
+          }
+        } else if (live && c + e < a.vdim) {  // vdim is a multiple of 8
           uint32_t w[4];
 #pragma unroll
           for (int i = 0; i < 4; ++i) w[i] = Pack(__uint_as_float(o[e + 2 * i]) * inv, __uint_as_float(o[e + 2 * i + 1]) * inv);
@@ -288,14 +304,15 @@ __global__ void __launch_bounds__(kThreads, 1)
   }
 }
 
-// The rows [first, first + count) of one sequence out of its pages, 16 bytes a thread.
+// The rows [0, keep) and [first, first + count - keep) of one sequence out of its pages, 16 bytes a thread.
 __global__ void __launch_bounds__(256) LatentGatherKernel(const uint4* pool, int64_t pool_ld16, const int* table, uint4* out, int64_t out_ld16,
-                                                          int first, int count, int words, int block_size, int num_blocks, int max_blocks)
+                                                          int first, int keep, int count, int words, int block_size, int num_blocks,
+                                                          int max_blocks)
 {
   GridDependencySync();
   const long long i = static_cast<long long>(blockIdx.x) * 256 + threadIdx.x;
   if (i >= static_cast<long long>(count) * words) return;
-  const int r = static_cast<int>(i / words), w = static_cast<int>(i % words), pos = first + r;
+  const int r = static_cast<int>(i / words), w = static_cast<int>(i % words), pos = r < keep ? r : first + r - keep;
   const int page = min(max(__ldg(table + min(pos / block_size, max_blocks - 1)), 0), num_blocks - 1);
   out[r * out_ld16 + w] = pool[(static_cast<size_t>(page) * block_size + pos % block_size) * pool_ld16 + w];
 }
@@ -355,14 +372,14 @@ bool Rings(int dim, int rot, int vdim, WindowArgs* a)
 using namespace tlaloc_b200;
 
 extern "C" int tlaloc_b200_latent_gather(const void* pool, int64_t pool_ld, int32_t dtype, const int32_t* table, void* out, int64_t out_ld,
-                                         int32_t first, int32_t count, int32_t row, int32_t num_blocks, int32_t block_size,
+                                         int32_t first, int32_t keep, int32_t count, int32_t row, int32_t num_blocks, int32_t block_size,
                                          int32_t max_blocks, void* stream)
 {
   const char* op = "LATENT_GATHER";
   if (!pool || !table || !out) return Fail(kInvalid, "%s: a required device pointer is null", op);
   if (!IsFloatType(dtype)) return Fail(kInvalid, "%s: f32 or bf16", op);
-  if (first < 0 || count < 0 || row < 1 || num_blocks < 1 || block_size < 1 || max_blocks < 1) return Fail(kInvalid, "%s: bad sizes", op);
-  if (first + count > static_cast<int64_t>(max_blocks) * block_size) return Fail(kInvalid, "%s: the rows pass the end of the table", op);
+  if (first < keep || keep < 0 || keep > count || count < 0 || row < 1 || num_blocks < 1 || block_size < 1 || max_blocks < 1) return Fail(kInvalid, "%s: bad sizes", op);
+  if (static_cast<int64_t>(first) + count - keep > static_cast<int64_t>(max_blocks) * block_size) return Fail(kInvalid, "%s: the rows pass the end of the table", op);
   const int per = 16 / static_cast<int>(DtypeBytes(dtype));
   const int words = (row + per - 1) / per;
   if (pool_ld % per || out_ld % per || pool_ld < words * per || out_ld < words * per || !Aligned16(pool) || !Aligned16(out)) {
@@ -371,7 +388,7 @@ extern "C" int tlaloc_b200_latent_gather(const void* pool, int64_t pool_ld, int3
   if (count == 0) return kOk;
   const unsigned blocks = static_cast<unsigned>((static_cast<long long>(count) * words + 255) / 256);
   const cudaError_t e = LaunchChained(LatentGatherKernel, blocks, 256, 0, static_cast<cudaStream_t>(stream), static_cast<const uint4*>(pool),
-                                      pool_ld / per, table, static_cast<uint4*>(out), out_ld / per, first, count, words, block_size,
+                                      pool_ld / per, table, static_cast<uint4*>(out), out_ld / per, first, keep, count, words, block_size,
                                       num_blocks, max_blocks);
   if (e != cudaSuccess) return CudaFail("LATENT_GATHER launch", e);
   CountLaunches(1);
@@ -384,20 +401,21 @@ extern "C" int tlaloc_b200_window_attention_applies(int32_t dim, int32_t rot_dim
   return dim >= 8 && dim % 8 == 0 && rot_dim % 8 == 0 && rot_dim >= 0 && vdim >= 8 && vdim % 8 == 0 && Rings(dim, rot_dim, vdim, &a) ? 1 : 0;
 }
 
-extern "C" int tlaloc_b200_window_attention(const void* q, const void* k, const void* k_rot, int64_t rot_ld, const void* v, int64_t kv_ld,
-                                            int64_t kv_head_ld, void* out, int64_t out_ld, int32_t num_queries, int32_t num_keys,
-                                            int32_t first_query, int32_t num_heads, int32_t dim, int32_t rot_dim, int32_t vdim,
-                                            int32_t window, float scale, void* stream)
+extern "C" int tlaloc_b200_window_attention(const void* q, const void* k, int64_t k_head_ld, const void* k_rot, int64_t rot_ld, const void* v,
+                                            int64_t v_head_ld, int64_t kv_ld, void* out, int64_t out_ld, int32_t out_dtype, int32_t num_queries,
+                                            int32_t num_keys, int32_t first_query, int32_t num_heads, int32_t v_heads, int32_t maps, int32_t dim,
+                                            int32_t rot_dim, int32_t vdim, int32_t window, int32_t keep_first, float scale, void* stream)
 {
   const char* op = "WINDOW_ATTENTION";
   if (!q || !k || !v || !out || (rot_dim > 0 && !k_rot)) return Fail(kInvalid, "%s: a required device pointer is null", op);
   if (num_queries < 0 || num_keys < 1 || first_query < 0 || num_heads < 1 || window < 0 || num_heads > 65535) return Fail(kInvalid, "%s: bad sizes", op);
+  if (v_heads < 1 || maps < 1 || num_heads % (v_heads * maps) || keep_first < 0 || !IsFloatType(out_dtype)) return Fail(kInvalid, "%s: bad heads", op);
   if (!(scale > 0.f)) return Fail(kUnsupported, "%s: the scale must be positive", op);
   if (first_query + num_queries > num_keys) return Fail(kInvalid, "%s: query %d has no key of its own", op, first_query + num_queries - 1);
   if (!tlaloc_b200_window_attention_applies(dim, rot_dim, vdim)) {
     return Fail(kUnsupported, "%s: dim, rot_dim and vdim are multiples of 8, vdim up to 256, and the tiles must fit shared memory", op);
   }
-  if (rot_ld % 8 || kv_ld % 8 || kv_head_ld % 8 || out_ld % 8 || !Aligned16(q) || !Aligned16(k) || !Aligned16(k_rot) || !Aligned16(v) || !Aligned16(out)) {
+  if (rot_ld % 8 || kv_ld % 8 || k_head_ld % 8 || v_head_ld % 8 || out_ld % 8 || !Aligned16(q) || !Aligned16(k) || !Aligned16(k_rot) || !Aligned16(v) || !Aligned16(out)) {
     return Fail(kInvalid, "%s: addresses and strides must be multiples of 16 bytes", op);
   }
   if (num_queries == 0) return kOk;
@@ -405,7 +423,11 @@ extern "C" int tlaloc_b200_window_attention(const void* q, const void* k, const 
   if (e != cudaSuccess) return CudaFail("WINDOW_ATTENTION set-up", e);
   WindowArgs a = {};
   Rings(dim, rot_dim, vdim, &a);
-  a.out = static_cast<__nv_bfloat16*>(out);
+  a.out = out;
+  a.out_f32 = out_dtype == TLALOC_B200_F32 ? 1 : 0;
+  a.keep = window > 0 ? keep_first : 0;
+  a.maps = maps;
+  a.group = num_heads / v_heads;
   a.out_ld = out_ld;
   a.T = num_queries;
   a.L = num_keys;
@@ -417,8 +439,8 @@ extern "C" int tlaloc_b200_window_attention(const void* q, const void* k, const 
   a.scale_log2 = scale * 1.4426950408889634f;
   CUtensorMap mq, mk, mr, mv;
   const int64_t q_row = dim + rot_dim;
-  if (!Encode(&mq, q, dim + rot_dim, num_heads, num_queries, q_row, q_row * num_heads) || !Encode(&mk, k, dim, num_heads, num_keys, kv_head_ld, kv_ld) ||
-      !Encode(&mv, v, vdim, num_heads, num_keys, kv_head_ld, kv_ld) || (rot_dim > 0 && !Encode(&mr, k_rot, rot_dim, 1, num_keys, rot_ld, rot_ld))) {
+  if (!Encode(&mq, q, dim + rot_dim, num_heads, num_queries, q_row, q_row * num_heads) || !Encode(&mk, k, dim, v_heads * maps, num_keys, k_head_ld, kv_ld) ||
+      !Encode(&mv, v, vdim, v_heads, num_keys, v_head_ld, kv_ld) || (rot_dim > 0 && !Encode(&mr, k_rot, rot_dim, 1, num_keys, rot_ld, rot_ld))) {
     return Fail(kInternal, "%s: the tensor maps could not be encoded", op);
   }
   if (rot_dim == 0) mr = mk;

@@ -248,10 +248,13 @@ def argmax(logits, out=None):
 # ---------------------------------------------------------------------- unquantized projections, latent attention
 
 
+GATED = (N.ACT_SILU_MUL, N.ACT_GELU_TANH_MUL)
+
+
 def dense(x, w, out, *, bias=None, residual=None, act=N.ACT_NONE) -> N.DenseProblem:
     """One projection out = act(x @ w.T + bias) + residual for `dense_gemm`.  x [M, K], w [N, K], out [M, N]; or a batch
     of them (the heads of a layer): x [B, M, K], w [B, N, K], out [B, M, N].  x, out and residual may be strided views whose
-    last dimension is dense; w is contiguous."""
+    last dimension is dense; w is contiguous.  A gated act (see interleave_gate) leaves out [M, N / 2]."""
     batched = w.dim() == 3
     for name, t in (("x", x), ("out", out)) + ((("residual", residual),) if residual is not None else ()):
         if not t.is_cuda or t.stride(-1) != 1 or t.dim() != w.dim():
@@ -259,7 +262,7 @@ def dense(x, w, out, *, bias=None, residual=None, act=N.ACT_NONE) -> N.DenseProb
     _dev(w, bias)
     b, n, k = w.shape if batched else (1, *w.shape)
     m = x.shape[-2]
-    if x.shape[-1] != k or tuple(out.shape[-2:]) != (m, n) or (batched and (x.shape[0] != b or out.shape[0] != b)) or x.dtype != w.dtype:
+    if x.shape[-1] != k or tuple(out.shape[-2:]) != (m, n // 2 if act in GATED else n) or (batched and (x.shape[0] != b or out.shape[0] != b)) or x.dtype != w.dtype:
         raise ValueError(f"DENSE_PROJ: x {tuple(x.shape)} {x.dtype}, w {tuple(w.shape)} {w.dtype}, out {tuple(out.shape)} do not fit")
     if (bias is not None and (bias.dtype != torch.float32 or tuple(bias.shape) != (n,))) or (
             residual is not None and (residual.dtype != torch.float32 or tuple(residual.shape) != (m, n))):
@@ -272,11 +275,41 @@ def dense(x, w, out, *, bias=None, residual=None, act=N.ACT_NONE) -> N.DenseProb
     return p
 
 
+def grouped_dense(x, w, out, row_offsets, *, act=N.ACT_NONE) -> N.DenseProblem:
+    """The projections of a batch of weights w [B, N, K], each applied to its own rows [row_offsets[b], row_offsets[b + 1]) of x [M, K]
+    -> out [M, N] (N / 2 for a gated act): the last problem of a `dense_gemm` call."""
+    _dev(w, row_offsets)
+    b, n, k = w.shape
+    m = x.shape[0]
+    for name, t in (("x", x), ("out", out)):
+        if not t.is_cuda or t.dim() != 2 or t.stride(1) != 1:
+            raise ValueError(f"GROUPED_PROJ {name}: a CUDA matrix with dense rows is needed")
+    if (x.shape[1] != k or tuple(out.shape) != (m, n // 2 if act in GATED else n) or x.dtype != w.dtype or row_offsets.dtype != torch.int32
+            or row_offsets.shape[0] != b + 1):
+        raise ValueError(f"GROUPED_PROJ: x {tuple(x.shape)} {x.dtype}, w {tuple(w.shape)} {w.dtype}, out {tuple(out.shape)} do not fit")
+    p = N.DenseProblem(x=_ptr(x), w=_ptr(w), y=_ptr(out), ld_x=x.stride(0), ld_y=out.stride(0), batch_w=n * k, k=k, n=n, batch=b, act=act,
+                       y_dtype=_dt(out), row_offsets=_ptr(row_offsets))
+    p.rows, p.like = m, x
+    return p
+
+
+def interleave_gate(gate, up):
+    """Gate and up projections [..., F, K] as a gated `dense` takes them: blocks of 16 rows of each in turn, F padded to a multiple of
+    16 with zeros (whose outputs are zero)."""
+    f, k = gate.shape[-2:]
+    pad = -f % 16
+    if pad:
+        gate, up = (torch.nn.functional.pad(t, (0, 0, 0, pad)) for t in (gate, up))
+    lead = gate.shape[:-2]
+    both = torch.stack([gate.reshape(*lead, -1, 16, k), up.reshape(*lead, -1, 16, k)], dim=-3)
+    return both.reshape(*lead, 2 * (f + pad), k).contiguous()
+
+
 def dense_gemm(*problems, weights_const=False) -> None:
-    """Runs one or two `dense` problems of the same rows and type."""
+    """Runs one or two `dense` problems of the same type (a `grouped_dense` one last)."""
     like, m = problems[0].like, problems[0].rows
-    if any(p.rows != m or p.like.dtype != like.dtype for p in problems):
-        raise ValueError("DENSE_PROJ: the problems of one call have the same rows and type")
+    if any(p.like.dtype != like.dtype for p in problems):
+        raise ValueError("DENSE_PROJ: the problems of one call have the same type")
     N.check(N.lib().tlaloc_b200_dense_gemm((N.DenseProblem * len(problems))(*problems), len(problems), _dt(like), m,
                                            N.GEMM_WEIGHTS_CONST if weights_const else 0, _stream(like)))
 
@@ -339,13 +372,13 @@ def latent_attention(query, pool, block_tables, seq_lens, out, *, kv_rank, scale
         block_tables.shape[0], int(window), int(max_live), float(scale), _stream(query)))
 
 
-def latent_gather(pool, table, out, *, first) -> None:
-    """out [count, row] = the pool rows of positions first .. of the sequence whose block table is `table` [max_blocks]."""
+def latent_gather(pool, table, out, *, first, keep=0) -> None:
+    """out [count, row] = the pool rows of positions 0 .. keep - 1 and first .. of the sequence whose block table is `table` [max_blocks]."""
     _dev(pool, table, out)
     if table.dtype != torch.int32 or table.dim() != 1 or pool.dim() != 3 or out.dtype != pool.dtype:
         raise ValueError("LATENT_GATHER: pool [P, block, row], table i32 [max_blocks], out [count, row] of the pool's type")
     P, bs, ld = pool.shape
-    N.check(N.lib().tlaloc_b200_latent_gather(_ptr(pool), ld, _dt(pool), _ptr(table), _ptr(out), out.shape[1], int(first), out.shape[0],
+    N.check(N.lib().tlaloc_b200_latent_gather(_ptr(pool), ld, _dt(pool), _ptr(table), _ptr(out), out.shape[1], int(first), int(keep), out.shape[0],
                                               out.shape[1], P, bs, table.shape[0], _stream(pool)))
 
 
@@ -353,17 +386,155 @@ def window_attention_applies(dim, rot_dim, vdim) -> bool:
     return bool(N.lib().tlaloc_b200_window_attention_applies(dim, rot_dim, vdim))
 
 
-def window_attention(q, k, k_rot, v, out, *, first_query, scale, window=0) -> None:
-    """q bf16 [T, H, dim + rot] (contiguous, rotated) over k [L, H, dim], k_rot [L, rot] and v [L, H, vdim] (strided views) -> out
-    [T, H * vdim] (a strided view); query i is key first_query + i.  See include/tlaloc_b200.h."""
+def window_attention(q, k, k_rot, v, out, *, first_query, scale, window=0, keep_first=0, maps=1) -> None:
+    """q bf16 [T, H, dim + rot] (contiguous, rotated) over k [L, groups * maps, dim], k_rot [L, rot] (or None) and v [L, groups, vdim]
+    (strided views) -> out [T, H * vdim] (a strided view); query i is key first_query + i.  See include/tlaloc_b200.h."""
     _dev(q)
     T, H, qd = q.shape
-    L, _, dim = k.shape
-    vdim = v.shape[2]
+    L, kh, dim = k.shape
+    vh, vdim = v.shape[1:]
     rot = qd - dim
-    if any(t.dtype != torch.bfloat16 or not t.is_cuda or t.stride(-1) != 1 for t in (q, k, k_rot, v, out)):
+    k_rot = k_rot if rot else None
+    if any(t is not None and (t.dtype != torch.bfloat16 or not t.is_cuda or t.stride(-1) != 1) for t in (q, k, k_rot, v)):
         raise ValueError("WINDOW_ATTENTION: bf16 CUDA tensors with dense rows")
-    if k.shape[1] != H or v.shape[:2] != k.shape[:2] or tuple(k_rot.shape) != (L, rot) or tuple(out.shape) != (T, H * vdim) or v.stride()[:2] != k.stride()[:2]:
-        raise ValueError(f"WINDOW_ATTENTION: q {tuple(q.shape)}, k {tuple(k.shape)}, k_rot {tuple(k_rot.shape)}, v {tuple(v.shape)}, out {tuple(out.shape)} do not fit")
-    N.check(N.lib().tlaloc_b200_window_attention(_ptr(q), _ptr(k), _ptr(k_rot), k_rot.stride(0), _ptr(v), k.stride(0), k.stride(1), _ptr(out),
-                                                 out.stride(0), T, L, int(first_query), H, dim, rot, vdim, int(window), float(scale), _stream(q)))
+    if not out.is_cuda or out.stride(-1) != 1 or out.dtype not in (torch.float32, torch.bfloat16):
+        raise ValueError("WINDOW_ATTENTION: out is an f32 or bf16 CUDA matrix with dense rows")
+    if (kh != vh * maps or H % kh or v.shape[0] != L or rot < 0 or (rot and tuple(k_rot.shape) != (L, rot))
+            or tuple(out.shape) != (T, H * vdim) or v.stride(0) != k.stride(0)):
+        raise ValueError(f"WINDOW_ATTENTION: q {tuple(q.shape)}, k {tuple(k.shape)}, v {tuple(v.shape)}, out {tuple(out.shape)} do not fit")
+    N.check(N.lib().tlaloc_b200_window_attention(_ptr(q), _ptr(k), k.stride(1), _ptr(k_rot), k_rot.stride(0) if rot else 8, _ptr(v), v.stride(1), k.stride(0),
+                                                 _ptr(out), out.stride(0), _dt(out), T, L, int(first_query), H, vh, int(maps), dim, rot, vdim, int(window),
+                                                 int(keep_first), float(scale), _stream(q)))
+
+
+# ---------------------------------------------------------------------- norms on both sides, grouped attention, retention, experts
+
+
+def residual_norm(y, x, gain_post, eps, *, gain_next=None, out=None, gate=None, parts=None, part_rows=None, part_weights=None) -> None:
+    """x += rms_norm(branch) * gain_post with branch = sigmoid(gate) * y + the weighted expert outputs; out = rms_norm(x) * gain_next.
+    y f32 [rows, n] or None; gate f32 [rows] (strided); parts [rows * top, n], part_rows i32 and part_weights f32 [rows, top]."""
+    _dev(x, gain_post, gain_next, y, parts, part_rows, part_weights)
+    rows, n = x.shape
+    if (y is not None and (tuple(y.shape) != (rows, n) or y.dtype != torch.float32)) or (gate is not None and gate.shape[0] != rows):
+        raise ValueError("RESIDUAL_NORM: y is f32 [rows, n], gate f32 [rows]")
+    if out is not None:
+        _out("RESIDUAL_NORM out", out, (rows, n), (torch.float32, torch.bfloat16), x)
+    kind = _dt(parts if parts is not None else out if out is not None else x)
+    if parts is not None and (out is not None and out.dtype != parts.dtype or parts.shape[-1] != n or tuple(part_rows.shape) != tuple(part_weights.shape)
+                              or part_rows.dtype != torch.int32):
+        raise ValueError("RESIDUAL_NORM: parts [.., n] of the result's type, part_rows i32 and part_weights [rows, top]")
+    N.check(N.lib().tlaloc_b200_residual_norm(_ptr(y), _ptr(gate), gate.stride(0) if gate is not None else 0, _ptr(parts), _ptr(part_rows),
+                                              _ptr(part_weights), part_rows.shape[1] if parts is not None else 0, _ptr(x), _ptr(gain_post),
+                                              _ptr(gain_next), _ptr(out), kind, rows, n, float(eps), _stream(x)))
+
+
+def rotate_part(out, first, heads, dim, *, padded=None, row_ld, head_ld=None, rotate=True, scale=1.0, by_slot=False) -> N.RotatePart:
+    """Where one part of a projected row goes (`rotate_rows`): out is the address's tensor, its rows row_ld apart."""
+    padded = dim if padded is None else padded
+    p = N.RotatePart(out=_ptr(out), out_ld=row_ld, out_head_ld=padded if head_ld is None else head_ld, first=first, heads=heads, dim=dim,
+                     padded=padded, rotate=int(rotate), by_slot=int(by_slot), scale=scale)
+    p.like = out
+    return p
+
+
+def rotate_rows(rows, parts, positions, cos, sin, *, rot_dims, slots=None, num_slots=0) -> None:
+    """rows f32 [T, ld] (dense rows): each part rotated, scaled, narrowed and written to its place."""
+    _dev(positions, cos, sin, slots)
+    T = rows.shape[0]
+    if rows.dtype != torch.float32 or not rows.is_cuda or rows.stride(1) != 1 or positions.shape[0] < T or (slots is not None and slots.shape[0] < T):
+        raise ValueError("ROTATE_ROWS: rows f32 [T, ld], positions and slots [T]")
+    if any(p.like.dtype != parts[0].like.dtype for p in parts) or tuple(cos.shape) != (cos.shape[0], rot_dims // 2) or cos.shape != sin.shape:
+        raise ValueError("ROTATE_ROWS: outputs of one type; cos and sin [positions, rot_dims / 2]")
+    N.check(N.lib().tlaloc_b200_rotate_rows(_ptr(rows), rows.stride(0), (N.RotatePart * len(parts))(*parts), len(parts), _dt(parts[0].like),
+                                            _ptr(positions), _ptr(cos), _ptr(sin), _ptr(slots), T, rot_dims, num_slots, max(cos.shape[0], 1), _stream(rows)))
+
+
+def grouped_attention_slices(rows, heads, v_heads, maps, dim, vdim, dtype, max_live) -> int:
+    return int(N.lib().tlaloc_b200_grouped_attention_slices(rows, heads, v_heads, maps, dim, vdim, _DT[dtype], max_live))
+
+
+def grouped_attention(q, pool, block_tables, seq_lens, records, *, v_heads, maps, vdim, v_first, scale, slices, window=0, keep_first=0,
+                      row_tables=None) -> None:
+    """q [T, H, dim] over pool [P, block, row] of rows [v_heads * maps * dim keys | .. | v_heads * vdim values from v_first] -> records f32
+    of at least slices * T * H * (vdim + 2) values; see include/tlaloc_b200.h."""
+    _dev(q, pool, block_tables, seq_lens, records, row_tables)
+    T, H, dim = q.shape
+    P, bs, ld = pool.shape
+    if q.dtype != pool.dtype or records.dtype != torch.float32 or records.numel() < slices * T * H * (vdim + 2):
+        raise ValueError("GROUPED_ATTENTION: q and pool have one type; records are f32 [slices, T, H, vdim + 2]")
+    if any(t is not None and t.dtype != torch.int32 for t in (block_tables, seq_lens, row_tables)):
+        raise TypeError("GROUPED_ATTENTION: tables and lengths are int32")
+    if seq_lens.shape[0] < T or (row_tables is not None and row_tables.shape[0] < T):
+        raise ValueError("GROUPED_ATTENTION: one length and one table per row")
+    N.check(N.lib().tlaloc_b200_grouped_attention(_ptr(q), _ptr(pool), ld, _dt(q), _ptr(block_tables), _ptr(row_tables), _ptr(seq_lens), _ptr(records),
+                                                  slices, T, H, v_heads, maps, dim, vdim, v_first, P, bs, block_tables.shape[1], block_tables.shape[0],
+                                                  int(window), int(keep_first), float(scale), _stream(q)))
+
+
+def map_difference(maps, out, *, rows, heads, vdim, in_ld, lam, keep, eps, slices=0, gate=None) -> None:
+    """The difference of two attention maps, normed and gated: maps f32 (records of `slices` slices, or the maps' outputs), gate f32
+    [rows, heads] (strided), out [rows, heads * vdim] (strided)."""
+    _dev(maps)
+    need = max(slices, 1) * rows * heads * 2 * (in_ld + 2 if slices else in_ld)
+    if maps.dtype != torch.float32 or maps.numel() < need or tuple(out.shape) != (rows, heads * vdim) or out.stride(1) != 1 or not out.is_cuda:
+        raise ValueError("MAP_DIFFERENCE: maps f32 of every head, out [rows, heads * vdim]")
+    N.check(N.lib().tlaloc_b200_map_difference(_ptr(maps), slices, _ptr(gate), gate.stride(0) if gate is not None else 0, _ptr(out), out.stride(0), _dt(out),
+                                               rows, heads, vdim, in_ld, float(lam), float(keep), float(eps), _stream(maps)))
+
+
+def head_norm_gate(o, gate, out, eps) -> None:
+    """o f32 [rows, heads, vdim], gate f32 [rows, heads * vdim] (strided) -> out = o / rms(o) * silu(gate), [rows, heads * vdim]."""
+    _dev(o)
+    rows, heads, vdim = o.shape
+    if o.dtype != torch.float32 or gate.dtype != torch.float32 or gate.stride(1) != 1 or tuple(out.shape) != (rows, heads * vdim) or out.stride(1) != 1:
+        raise ValueError("HEAD_NORM_GATE: o and gate f32, out [rows, heads * vdim]")
+    N.check(N.lib().tlaloc_b200_head_norm_gate(_ptr(o), _ptr(gate), gate.stride(0), _ptr(out), out.stride(0), _dt(out), rows, heads, vdim, float(eps), _stream(o)))
+
+
+def _state_shape(state, heads, dim, vdim):
+    if state.dtype != torch.float32 or tuple(state.shape[1:]) != (heads, dim, -(-vdim // 4) * 4):
+        raise ValueError(f"RETENTION: state {tuple(state.shape)} is not f32 [slots, {heads}, {dim}, vdim rounded up to 4]")
+
+
+def retention_step(rows, positions, cos, sin, decay, row_states, state, out, *, heads, dim, vdim, rot_dims, k_scale, eps) -> None:
+    """One token per row: rows f32 [T, heads * (2 dim + 2 vdim)] = [q | k | v | gate] -> out [T, heads * vdim] and the new states."""
+    _dev(positions, cos, sin, decay, row_states, state)
+    T = rows.shape[0]
+    _state_shape(state, heads, dim, vdim)
+    if rows.dtype != torch.float32 or rows.stride(1) != 1 or tuple(out.shape) != (T, heads * vdim) or out.stride(1) != 1 or decay.numel() != heads:
+        raise ValueError("RETENTION_STEP: rows f32 [T, ..], out [T, heads * vdim], decay f32 [heads]")
+    N.check(N.lib().tlaloc_b200_retention_step(_ptr(rows), rows.stride(0), _ptr(positions), _ptr(cos), _ptr(sin), _ptr(decay), _ptr(row_states), _ptr(state),
+                                               _ptr(out), out.stride(0), _dt(out), T, heads, dim, vdim, rot_dims, state.shape[0], max(cos.shape[0], 1),
+                                               float(k_scale), float(eps), _stream(state)))
+
+
+def retention_scan(q, k, v, positions, decay, row_states, state, o) -> None:
+    """The tokens of one sequence in order: q, k [T, heads, dim] and v [T, heads, vdim] (heads side by side, each padded to a row of its
+    own length) -> o f32 [T, heads, vdim] and the new state."""
+    T, heads, vdim = o.shape
+    _dev(decay, state, o)
+    dim = state.shape[2]
+    _state_shape(state, heads, dim, vdim)
+    for t in (q, k, v):
+        if not t.is_cuda or not t.is_contiguous() or t.shape[:2] != (T, heads) or t.dtype != q.dtype:
+            raise ValueError("RETENTION_SCAN: q, k, v are contiguous [T, heads, ..] of one type")
+    N.check(N.lib().tlaloc_b200_retention_scan(_ptr(q), _ptr(k), q.shape[2], _ptr(v), v.shape[2], _dt(q), _ptr(positions), _ptr(decay), _ptr(row_states),
+                                               _ptr(state), _ptr(o), T, heads, dim, vdim, state.shape[0], _stream(state)))
+
+
+def moe_route(logits, ids, weights, offsets, entry_rows, row_tokens, *, experts) -> None:
+    """logits f32 [T, >= experts] (strided) -> the chosen experts and their weights [T, top], and the entries sorted by expert."""
+    _dev(ids, weights, offsets, entry_rows, row_tokens)
+    T, top = ids.shape
+    if logits.dtype != torch.float32 or logits.stride(1) != 1 or logits.shape[0] != T or offsets.shape[0] != experts + 1:
+        raise ValueError("MOE_ROUTE: logits f32 [T, ..], offsets [experts + 1]")
+    N.check(N.lib().tlaloc_b200_moe_route(_ptr(logits), logits.stride(0), _ptr(ids), _ptr(weights), _ptr(offsets), _ptr(entry_rows), _ptr(row_tokens), T,
+                                          experts, top, _stream(ids)))
+
+
+def gather_rows(x, rows, out) -> None:
+    """out[r] = x[rows[r]]."""
+    _dev(x, rows, out)
+    if rows.dtype != torch.int32 or out.dtype != x.dtype or out.shape != (rows.shape[0], x.shape[1]):
+        raise ValueError("GATHER_ROWS: rows i32 [count], out [count, n] of x's type")
+    N.check(N.lib().tlaloc_b200_gather_rows(_ptr(x), _ptr(rows), _ptr(out), rows.shape[0], x.shape[1] * x.element_size(), _stream(x)))

@@ -110,3 +110,15 @@ def _marotar(config: dict, model_dir: str, sizes: Sizes, dtype: torch.dtype, dev
                           max_sequences=sizes.max_sequences, dtype=dtype, device=device)
     model.load_tensors(read_tensors(model_dir))
     return model
+
+
+@register("Videdra", dtypes=(torch.bfloat16, torch.float32), kernels="mixed")
+def _videdra(config: dict, model_dir: str, sizes: Sizes, dtype: torch.dtype, device: str) -> StepModel:
+    """Differential attention and retention in any order, dense and expert feed-forwards, norms on both sides of every branch."""
+    from .mixed_decoder import MixedDecoder, MixedDecoderConfig
+
+    cfg = MixedDecoderConfig.from_config(config)
+    model = MixedDecoder(cfg, num_blocks=num_blocks(sizes, cfg.block_size), max_len=sizes.max_len, max_tokens=sizes.max_tokens,
+                         max_sequences=sizes.max_sequences, dtype=dtype, device=device)
+    model.load_tensors(read_tensors(model_dir))
+    return model
