@@ -473,6 +473,8 @@ int tlaloc_b200_head_norm_gate(const float* in, const float* gate, int64_t gate_
  * out = o / rms(o) * silu(gate) as `dtype`.  row_states i32 [rows]; decay f32 [heads].
  * _scan: the `tokens` tokens of ONE sequence in order, q and k [tokens][heads][dim_ld] (rotated, scaled) and v [tokens][heads][v_ld] of
  * `dtype`; o f32 [tokens][heads][vdim].  row_states and positions are those of its first token.
+ * _chunks: the same on the tensor cores, bf16, dim up to 256: dim_ld is dim rounded up to a multiple of 16, v_ld a multiple of 8, and
+ * what pads the rows of q, k and v is zero.  scratch: _chunks_scratch_bytes (may be 0); _chunks_applies: 1 if it takes these sizes.
  */
 int tlaloc_b200_retention_step(const float* in, int64_t ld, const int32_t* positions, const float* cos_table, const float* sin_table,
                                const float* decay, const int32_t* row_states, float* state, void* out, int64_t out_ld, int32_t dtype,
@@ -481,6 +483,12 @@ int tlaloc_b200_retention_step(const float* in, int64_t ld, const int32_t* posit
 int tlaloc_b200_retention_scan(const void* q, const void* k, int32_t dim_ld, const void* v, int32_t v_ld, int32_t dtype,
                                const int32_t* positions, const float* decay, const int32_t* row_states, float* state, float* o, int32_t tokens,
                                int32_t heads, int32_t dim, int32_t vdim, int32_t num_slots, void* stream);
+
+int tlaloc_b200_retention_chunks_applies(int32_t dim, int32_t vdim);
+size_t tlaloc_b200_retention_chunks_scratch_bytes(int32_t tokens, int32_t heads, int32_t dim, int32_t vdim);
+int tlaloc_b200_retention_chunks(const void* q, const void* k, int32_t dim_ld, const void* v, int32_t v_ld, const int32_t* positions,
+                                 const float* decay, const int32_t* row_states, float* state, float* o, void* scratch, size_t scratch_bytes,
+                                 int32_t tokens, int32_t heads, int32_t dim, int32_t vdim, int32_t num_slots, void* stream);
 
 /* ------------------------------------------------------------------ mixture of experts */
 

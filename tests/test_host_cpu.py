@@ -41,7 +41,7 @@ def test_a_subset_of_the_kernels_is_a_library_of_its_own():
     assert not hasattr(lib, "tlaloc_b200_int8_gemm")
     lib = ctypes.CDLL(B.build(subset="mixed", own=True))
     for name in ("init", "device_status", "embedding", "argmax", "dense_gemm", "rmsnorm_pair", "latent_gather", "window_attention", "residual_norm", "rotate_rows",
-                 "grouped_attention", "map_difference", "retention_step", "retention_scan", "head_norm_gate", "moe_route", "gather_rows"):
+                 "grouped_attention", "map_difference", "retention_step", "retention_scan", "retention_chunks", "head_norm_gate", "moe_route", "gather_rows"):
         assert hasattr(lib, "tlaloc_b200_" + name), name
 
 
@@ -89,6 +89,8 @@ def test_refusals_of_the_mixers_need_no_gpu():
                                                        kw.get("rot", 8), 3, 4, 0.3, 1e-5, None)
     assert step() == N.OK and step(ld=63) == i and step(rot=10) == i and step(rows=-1) == i and step(dim=520, ld=9999) == N.UNSUPPORTED
     assert lib.tlaloc_b200_retention_scan(one, one, 7, one, 8, N.BF16, one, one, one, one, one, 4, 2, 8, 8, 3, None) == i
+    chunks = lambda dim=24, dim_ld=32, tokens=4: lib.tlaloc_b200_retention_chunks(one, one, dim_ld, one, 16, one, one, one, one, one, None, 0, tokens, 2, dim, 8, 3, None)
+    assert chunks(dim_ld=24) == i and chunks(dim=257, dim_ld=272) == N.UNSUPPORTED and chunks(tokens=0) == N.OK and chunks(tokens=2048) == i  # no scratch
     assert lib.tlaloc_b200_moe_route(one, 4, one, one, one, one, one, 3, 5, 2, None) == i and lib.tlaloc_b200_moe_route(one, 8, one, one, one, one, one, 3, 5, 6, None) == i
     assert lib.tlaloc_b200_gather_rows(one, one, one, 1, 3, None) == i
     g = N.DenseProblem(x=16, w=16, y=16, ld_x=8, ld_y=16, k=8, n=32, batch=1, act=N.ACT_SILU_MUL, y_dtype=N.F32)

@@ -151,3 +151,80 @@ def greedy(config, weights, prompt, n):
     for _ in range(n):
         out.append(int(forward(config, weights, out)[-1].argmax()))
     return out[len(prompt):]
+
+
+# ---------------------------------------------------------------------------------------------- small models
+
+def attention_layer(heads=6, kv_heads=2, dim=24, vdim=40, diff=0.4, window=21, keep=5, rot_dims=16, base=3000.0, scale=None, kv_from=None, mlp=None):
+    m = {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "diff": diff, "rot": {"base": base, "dims": rot_dims},
+         "scale": dim ** -0.5 if scale is None else scale}
+    if window:
+        m["mask"] = {"size": window, "keep_first": keep}
+    if kv_from is not None:
+        m["kv_from"] = kv_from
+    return {"type": "attention", "mixer": m, "mlp": mlp}
+
+
+def retention_layer(heads=3, dim=20, vdim=28, decay=None, rot_dims=12, base=800.0, mlp=None):
+    decay = [1 - 0.5 ** (i + 2.5) for i in range(heads)] if decay is None else decay
+    return {"type": "retention", "mixer": {"heads": heads, "dim": dim, "vdim": vdim, "decay": decay, "rot": {"base": base, "dims": rot_dims}}, "mlp": mlp}
+
+
+def dense_mlp(ff=72):
+    return {"kind": "dense", "ff": ff}
+
+
+def moe_mlp(ff=24, experts=7, top=2, shared=40):
+    out = {"kind": "moe", "expert": {"ff": ff}, "router": {"experts": experts, "top": top}}
+    if shared:
+        out["shared"] = {"ff": shared}
+    return out
+
+
+def model(*layers, width=56, vocab=131, eps=1e-5):
+    return {"architecture": "Videdra", "width": width, "vocab": vocab, "norm": {"eps": eps}, "layers": list(layers)}
+
+
+def make_weights(config, seed=0, q_gain=1.0, router_gain=3.0):
+    """Random tensors with values bf16 can hold.  q_gain scales the queries: larger makes single keys stand out in the softmax;
+    router_gain the router, so that no choice of experts is close."""
+    g = torch.Generator().manual_seed(seed)
+    width, out = config["width"], {}
+
+    def put(name, *shape, std, mean=0.0):
+        out[name] = (mean + std * torch.randn(shape, generator=g)).to(torch.bfloat16).float()
+
+    def gated(p, ff):
+        put(p + "gate", ff, width, std=1.5 * width ** -0.5)
+        put(p + "up", ff, width, std=width ** -0.5)
+        put(p + "down", width, ff, std=ff ** -0.5)
+
+    put("embed", config["vocab"], width, std=1.0)
+    put("head", config["vocab"], width, std=width ** -0.5)
+    put("final.norm", width, std=0.2, mean=1.0)
+    for i, l in enumerate(config["layers"]):
+        m, mlp, p = l["mixer"], l["mlp"], f"l{i}."
+        for n in ("norm1", "norm1b", "ls1") + (("norm2", "norm2b", "ls2") if mlp else ()):
+            put(p + n, width, std=0.2, mean=0.7 if n.startswith("ls") else 1.0)
+        if l["type"] == "attention":
+            put(p + "mix.q", m["heads"] * 2 * m["dim"], width, std=q_gain * width ** -0.5)
+            if m.get("kv_from") is None:
+                put(p + "mix.k", m["kv_heads"] * 2 * m["dim"], width, std=width ** -0.5)
+                put(p + "mix.v", m["kv_heads"] * m["vdim"], width, std=width ** -0.5)
+            for n in ("lq1", "lk1", "lq2", "lk2"):
+                put(p + "mix." + n, m["dim"], std=0.3)
+            put(p + "mix.g", m["heads"], width, std=width ** -0.5)
+        else:
+            for n, d in (("q", "dim"), ("k", "dim"), ("v", "vdim"), ("g", "vdim")):
+                put(p + "mix." + n, m["heads"] * m[d], width, std=width ** -0.5)
+        put(p + "mix.o", width, m["heads"] * m["vdim"], std=(m["heads"] * m["vdim"]) ** -0.5)
+        if mlp and mlp["kind"] == "dense":
+            gated(p + "mlp.", mlp["ff"])
+        elif mlp:
+            put(p + "mlp.router", mlp["router"]["experts"], width, std=router_gain * width ** -0.5)
+            for e in range(mlp["router"]["experts"]):
+                gated(f"{p}mlp.e{e}.", mlp["expert"]["ff"])
+            if mlp.get("shared"):
+                gated(p + "mlp.shared.", mlp["shared"]["ff"])
+                put(p + "mlp.shared.sg", 1, width, std=width ** -0.5)
+    return out

@@ -81,6 +81,9 @@ _SIGNATURES = {
     "tlaloc_b200_head_norm_gate": (ctypes.c_int, [_vp, _vp, _i64, _vp, _i64] + [_i32] * 4 + [_f32, _vp]),
     "tlaloc_b200_retention_step": (ctypes.c_int, [_vp, _i64] + [_vp] * 7 + [_i64] + [_i32] * 8 + [_f32, _f32, _vp]),
     "tlaloc_b200_retention_scan": (ctypes.c_int, [_vp, _vp, _i32, _vp, _i32, _i32] + [_vp] * 5 + [_i32] * 5 + [_vp]),
+    "tlaloc_b200_retention_chunks_applies": (ctypes.c_int, [_i32] * 2),
+    "tlaloc_b200_retention_chunks_scratch_bytes": (_sz, [_i32] * 4),
+    "tlaloc_b200_retention_chunks": (ctypes.c_int, [_vp, _vp, _i32, _vp, _i32] + [_vp] * 6 + [_sz] + [_i32] * 5 + [_vp]),
     "tlaloc_b200_moe_route": (ctypes.c_int, [_vp, _i64] + [_vp] * 5 + [_i32] * 3 + [_vp]),
     "tlaloc_b200_gather_rows": (ctypes.c_int, [_vp, _vp, _vp, _i32, _i64, _vp]),
     "tlaloc_b200_peer_alloc": (ctypes.c_int, [_sz, ctypes.POINTER(_vp), ctypes.c_char_p]),

@@ -25,7 +25,7 @@ LIB_DIR = os.path.join(HERE, "lib")
 LIB = os.path.join(LIB_DIR, "libtlaloc_kernels.so")
 SUBSETS = {"latent": ("runtime", "token_ops", "dense_gemm", "dense_gemm_tc", "latent_ops", "latent_attention", "latent_prefill"),
            "mixed": ("runtime", "token_ops", "dense_gemm", "dense_gemm_tc", "latent_ops", "latent_prefill", "mixer_ops", "grouped_attention",
-                     "retention", "moe")}
+                     "retention", "retention_chunks", "moe")}
 INCLUDE = os.path.join(os.path.dirname(HERE), "include")
 
 NVCC_FLAGS = [

@@ -258,6 +258,8 @@ class MixedDecoder(RaggedModel):
         self._k = flat(R, big(ret, lambda m: m.heads * m.kdim), ty)
         self._v = flat(R, big(ret, lambda m: m.heads * m.vpad), ty)
         self._maps = torch.empty((max([self._map_values(m, R) for m in att] + [R * m.heads * m.vdim for m in ret]),), **f32)
+        sums = max((ops.retention_chunks_scratch_bytes(n, m.heads, m.dim, m.vdim) for m in ret for n in range(64, R + 64, 64)), default=0)
+        self._state_sums = torch.empty((sums // 4,), **f32) if dtype == torch.bfloat16 else None
         self._mixed = flat(R, big(mixers, lambda m: m.heads * m.vdim), ty)
         self.y = torch.empty((R, cfg.width), **f32)
         pad = lambda ff: -(-ff // 16) * 16
@@ -415,7 +417,11 @@ class MixedDecoder(RaggedModel):
                                                ops.rotate_part(v, vcol, m.heads, m.vdim, padded=m.vpad, row_ld=m.heads * m.vpad, rotate=False)],
                             self.positions[first:stop], cos, sin, rot_dims=m.rot.dims)
             o = self._view(self._maps, rows, m.heads, m.vdim)
-            ops.retention_scan(q, k, v, self.positions[first:stop], decay, self.row_states[first:stop], state, o)
+            operands = (q, k, v, self.positions[first:stop], decay, self.row_states[first:stop], state, o)
+            if self.dtype == torch.bfloat16 and ops.retention_chunks_applies(m.dim, m.vdim):
+                ops.retention_chunks(*operands, self._state_sums)
+            else:
+                ops.retention_scan(*operands)
             ops.head_norm_gate(o, proj[first:stop, vcol + m.heads * m.vdim:], out[first:stop], self.cfg.eps)
             lo = stop
         if lo < n:

@@ -522,6 +522,29 @@ def retention_scan(q, k, v, positions, decay, row_states, state, o) -> None:
                                                _ptr(state), _ptr(o), T, heads, dim, vdim, state.shape[0], _stream(state)))
 
 
+def retention_chunks_scratch_bytes(tokens, heads, dim, vdim) -> int:
+    return int(N.lib().tlaloc_b200_retention_chunks_scratch_bytes(tokens, heads, dim, vdim))
+
+
+def retention_chunks_applies(dim, vdim) -> bool:
+    return bool(N.lib().tlaloc_b200_retention_chunks_applies(dim, vdim))
+
+
+def retention_chunks(q, k, v, positions, decay, row_states, state, o, scratch=None) -> None:
+    """`retention_scan` on the tensor cores, bf16: what pads the rows of q, k and v must be zero; scratch f32 of
+    retention_chunks_scratch_bytes."""
+    T, heads, vdim = o.shape
+    _dev(decay, state, o, scratch)
+    dim = state.shape[2]
+    _state_shape(state, heads, dim, vdim)
+    for t in (q, k, v):
+        if not t.is_cuda or not t.is_contiguous() or t.shape[:2] != (T, heads) or t.dtype != torch.bfloat16:
+            raise ValueError("RETENTION_CHUNKS: q, k, v are contiguous bf16 [T, heads, ..]")
+    N.check(N.lib().tlaloc_b200_retention_chunks(_ptr(q), _ptr(k), q.shape[2], _ptr(v), v.shape[2], _ptr(positions), _ptr(decay), _ptr(row_states),
+                                                 _ptr(state), _ptr(o), _ptr(scratch), 0 if scratch is None else scratch.numel() * scratch.element_size(),
+                                                 T, heads, dim, vdim, state.shape[0], _stream(state)))
+
+
 def moe_route(logits, ids, weights, offsets, entry_rows, row_tokens, *, experts) -> None:
     """logits f32 [T, >= experts] (strided) -> the chosen experts and their weights [T, top], and the entries sorted by expert."""
     _dev(ids, weights, offsets, entry_rows, row_tokens)
