@@ -6,6 +6,7 @@ cache, on N B200s of one box (tensor parallel), plus the HBM roofline of its ker
     python bench.py --impl reference --gpus 1 --steps 3 --warmup 1                  # the CPU restatement of the reference
     python bench.py --workload llama8b | paged_attn | int8_proj | peer_sum          # one configuration / operator alone
     python bench.py --workload marotar                                              # the latent-attention decoder beside Llama
+    python bench.py --workload videdra                                              # differential attention and retention beside the latter
     python bench.py --timeline                                                      # per-kernel times inside one step
 
 One JSON line on stdout (rank 0).  A step is one decode step: one new token for every sequence of the batch.
@@ -57,6 +58,19 @@ MAROTAR = {
                    dict(d_model=2048, num_heads=16, num_kv_heads=4, head_dim=128, ffn=5504)),
 }
 MAROTAR_LAYERS, MAROTAR_VOCAB, MAROTAR_WINDOW, MAROTAR_BATCH, MAROTAR_PROMPT = 8, 32768, 4096, 64, 8192
+# The decoder of differential attention and retention at sizes of real models' layers, eight layers (three of retention and one of
+# attention, twice; the second attention layer uses the first one's keys and values), each beside a latent-attention decoder of the same
+# width, heads and (active) feed-forward parameters.
+VIDEDRA = {
+    "width 4096": (dict(width=4096, attention=dict(heads=16, kv_heads=4, dim=128, vdim=256), retention=dict(heads=16, dim=128, vdim=256), mlp=dict(ff=14336)),
+                   dict(width=4096, heads=32, dim=128, rot_dim=64, vdim=128, q_rank=1536, kv_rank=512, ff=21504)),
+    "width 2560": (dict(width=2560, attention=dict(heads=20, kv_heads=5, dim=64, vdim=128), retention=dict(heads=20, dim=64, vdim=128), mlp=dict(ff=6400)),
+                   dict(width=2560, heads=40, dim=64, rot_dim=32, vdim=64, q_rank=768, kv_rank=256, ff=9600)),
+    "width 2048": (dict(width=2048, attention=dict(heads=16, kv_heads=4, dim=64, vdim=128), retention=dict(heads=8, dim=256, vdim=512),
+                        mlp=dict(ff=1408, experts=64, top=6, shared=2816)),
+                   dict(width=2048, heads=16, dim=128, rot_dim=64, vdim=128, q_rank=768, kv_rank=512, ff=16896)),
+}
+VIDEDRA_KEEP = 64
 METRIC, UNIT = "decode_tokens_per_s", "tokens/s"
 BS = 16  # KV block size
 
@@ -817,29 +831,50 @@ def _prefill(torch, model, tokens, portion):
     return best
 
 
-def marotar_case(torch, dev, pk, sizes, llama, steps, local) -> dict:
-    """Decode (batch 64, contexts U[1024, 8192], window 4096) and prefill (one prompt of 8192) of both models, and the kernels of each
+def bench_lens(rng):
+    """Contexts of the decode batch."""
+    return rng.integers(1024, 8193, size=MAROTAR_BATCH).astype(np.int64)
+
+
+def bench_tables(block, max_len, batch=None):
+    """(block tables of the decode batch, pages of any order; blocks of the pool)"""
+    batch, M = MAROTAR_BATCH if batch is None else batch, -(-max_len // block)
+    return (1 + np.random.default_rng(3).permutation(batch * M)).reshape(batch, M).astype(np.int32), 1 + batch * M
+
+
+class KernelTimes:
+    """Kernels alone against their rooflines: HBM or the bf16 rate."""
+
+    def __init__(self, torch, pk):
+        self.torch, self.pk, self.rows = torch, pk, []
+
+    def time(self, name, calls, bytes_, flops, bound):
+        """calls: the same work over sets of operands that together are past L2."""
+        _, med = _time_graph(self.torch, lambda: [c() for c in calls], 10)
+        us = med / len(calls) * 1e3
+        frac = bytes_ / us / 1e3 / self.pk["hbm_gbs"] if bound == "hbm" else flops / us / 1e6 / self.pk["bf16_tflops"]
+        self.rows.append({"kernel": name, "us": us, "bound": bound, "gbs": bytes_ / us / 1e3, "tflops": flops / us / 1e6, "frac": frac})
+
+    def take(self):
+        out, self.rows = self.rows, []
+        return out
+
+
+def latent_case(torch, dev, pk, sizes, steps, local) -> dict:
+    """The latent-attention decoder: decode (batch 64, contexts U[1024, 8192], window 4096), prefill (one prompt of 8192), and its kernels
     alone against their rooflines: HBM for a decode step's kernels, the bf16 rate for a portion's products and attention."""
     from tlaloc_b200 import _native as N
-    from tlaloc_b200 import decoder as D
     from tlaloc_b200 import ops, sharding
-    from tlaloc_b200.attrs import parse_paged_attention
     from tlaloc_b200.latent_decoder import LatentDecoder, LatentDecoderConfig
 
     rng = np.random.default_rng(11)
     B, L = MAROTAR_BATCH, MAROTAR_LAYERS
-    lens = rng.integers(1024, 8193, size=B).astype(np.int64)
+    lens = bench_lens(rng)
     tokens = rng.integers(0, MAROTAR_VOCAB, size=MAROTAR_PROMPT).tolist()
     max_len = 8192 + 64
-    out = {"sizes": dict(sizes, layers=L, vocab=MAROTAR_VOCAB, window=MAROTAR_WINDOW), "llama_sizes": dict(llama, layers=L, vocab=MAROTAR_VOCAB)}
-
-    def tables(block):
-        M = -(-max_len // block)
-        return (1 + np.random.default_rng(3).permutation(B * M)).reshape(B, M).astype(np.int32), 1 + B * M
-
-    # ---- the latent-attention decoder
+    out = {"sizes": dict(sizes, layers=L, vocab=MAROTAR_VOCAB, window=MAROTAR_WINDOW)}
     cfg = LatentDecoderConfig.from_config(marotar_config(sizes))
-    tab, blocks = tables(cfg.block_size)
+    tab, blocks = bench_tables(cfg.block_size, max_len)
     m = LatentDecoder(cfg, num_blocks=blocks, max_len=max_len, max_tokens=2048, max_sequences=B, device=dev)
     m.init_random_weights(0)
     for p in m.pools:
@@ -853,13 +888,8 @@ def marotar_case(torch, dev, pk, sizes, llama, steps, local) -> dict:
     live = int(np.minimum(lens + 1, MAROTAR_WINDOW).sum())
     step_bytes = m.weight_bytes() + 2 * live * x.row * L
     out["decode"] = {"tokens_per_s": B / ms * 1e3, "ms_per_step": ms, "step_hbm_frac": step_bytes / ms / 1e6 / pk["hbm_gbs"], "clocks": clocks.summary()}
-    kernels = []
-
-    def time_kernel(name, calls, bytes_, flops, bound):
-        _, med = _time_graph(torch, lambda: [c() for c in calls], 10)
-        us = med / len(calls) * 1e3
-        frac = bytes_ / us / 1e3 / pk["hbm_gbs"] if bound == "hbm" else flops / us / 1e6 / pk["bf16_tflops"]
-        kernels.append({"kernel": name, "us": us, "bound": bound, "gbs": bytes_ / us / 1e3, "tflops": flops / us / 1e6, "frac": frac})
+    kt = KernelTimes(torch, pk)
+    time_kernel = kt.time
 
     def copies(lws, key):
         """That weight of every layer, repeated until the set is well past L2."""
@@ -905,20 +935,37 @@ def marotar_case(torch, dev, pk, sizes, llama, steps, local) -> dict:
                         2 * (q.numel() + kv.numel() + o.numel()), 2.0 * rows * MAROTAR_WINDOW * x.heads * (x.q_dim + x.vdim), bound)
 
     kernels_at(B, "hbm")
-    out["decode"]["kernels"], kernels = kernels, []
+    out["decode"]["kernels"] = kt.take()
     whole, last = _prefill(torch, m, tokens, 2048)
     out["prefill"] = {"tokens_per_s": MAROTAR_PROMPT / whole * 1e3, "ms": whole, "portion": 2048, "ms_last_portion": last,
                       "tokens_per_s_last_portion": 2048 / last * 1e3}
     kernels_at(2048, "tensor")
-    out["prefill"]["kernels"], kernels = kernels, []
+    out["prefill"]["kernels"] = kt.take()
     out["device_status"] = N.lib().tlaloc_b200_device_status()
     del m
     gc.collect()
     torch.cuda.empty_cache()
 
+    return out
+
+
+def marotar_case(torch, dev, pk, sizes, llama, steps, local) -> dict:
+    """Decode and prefill of the latent-attention decoder and of a Llama of equal size, and the kernels of each."""
+    from tlaloc_b200 import decoder as D
+    from tlaloc_b200 import ops, sharding
+
+    rng = np.random.default_rng(11)
+    B, L = MAROTAR_BATCH, MAROTAR_LAYERS
+    lens = bench_lens(rng)
+    tokens = rng.integers(0, MAROTAR_VOCAB, size=MAROTAR_PROMPT).tolist()
+    pos, max_len = lens.astype(np.int32), 8192 + 64
+    out = dict(latent_case(torch, dev, pk, sizes, steps, local), llama_sizes=dict(llama, layers=L, vocab=MAROTAR_VOCAB))
+    kt = KernelTimes(torch, pk)
+    time_kernel = kt.time
+
     # ---- the closest model the framework had
     lc = D.DecoderConfig(**llama, num_layers=L, vocab=MAROTAR_VOCAB, head_quant=True, max_positions=max_len)
-    tab, blocks = tables(lc.block_size)
+    tab, blocks = bench_tables(lc.block_size, max_len)
     d = D.Decoder(lc, B, blocks, tab.shape[1], device=dev)
     d.init_random_weights(0)
     for p in d.key_pools + d.value_pools:
@@ -939,7 +986,7 @@ def marotar_case(torch, dev, pk, sizes, llama, steps, local) -> dict:
     time_kernel("paged attention", [lambda l=l: ops.paged_attention(d.q_rot, d.key_pools[l], d.value_pools[l], d.block_tables, d.seq_lens, scale=lc.scale, out=d.att,
                                                                      scratch=d.att_scratch) for l in range(L)],
                 sb["kv"] // L, 4.0 * int(lens.sum()) * lc.num_heads * lc.head_dim, "hbm")
-    out["llama_decode"]["kernels"], kernels = kernels, []
+    out["llama_decode"]["kernels"] = kt.take()
     del d
     gc.collect()
     torch.cuda.empty_cache()
@@ -953,6 +1000,180 @@ def marotar_case(torch, dev, pk, sizes, llama, steps, local) -> dict:
     gc.collect()
     torch.cuda.empty_cache()
     return out
+
+
+def videdra_config(sizes: dict) -> dict:
+    """A config.json of the design at one of the bench's sizes."""
+    a, r, f = sizes["attention"], sizes["retention"], sizes["mlp"]
+    rot = lambda d: {"base": 10000.0, "dims": d}
+    attention = dict(a, rot=rot(a["dim"]), scale=a["dim"] ** -0.5, diff=0.3, mask={"size": MAROTAR_WINDOW, "keep_first": VIDEDRA_KEEP})
+    retention = dict(r, rot=rot(r["dim"]), decay=[1 - 0.5 ** (5 + 4 * h / r["heads"]) for h in range(r["heads"])])
+    dense = {"kind": "dense", "ff": f["ff"]}
+    if "experts" in f:
+        dense = {"kind": "moe", "expert": {"ff": f["ff"]}, "router": {"experts": f["experts"], "top": f["top"]}, "shared": {"ff": f["shared"]}}
+    layer = lambda kind, mixer: {"type": kind, "mixer": mixer, "mlp": dense}
+    layers = [layer("retention", retention)] * 3 + [layer("attention", attention)] + [layer("retention", retention)] * 3 + [layer("attention", dict(attention, kv_from=3))]
+    return {"architecture": "Videdra", "width": sizes["width"], "vocab": MAROTAR_VOCAB, "norm": {"eps": 1e-5}, "layers": layers}
+
+
+def videdra_case(torch, dev, pk, sizes, latent, steps, local) -> dict:
+    """Decode and prefill as `latent_case` has them, and every kernel of a step alone."""
+    from tlaloc_b200 import _native as N
+    from tlaloc_b200 import ops, sharding
+    from tlaloc_b200.mixed_decoder import DifferentialAttention, Dense, MixedDecoder, MixedDecoderConfig
+
+    rng = np.random.default_rng(11)
+    B, lens, max_len = MAROTAR_BATCH, bench_lens(rng), 8192 + 64
+    tokens = rng.integers(0, MAROTAR_VOCAB, size=MAROTAR_PROMPT).tolist()
+    cfg = MixedDecoderConfig.from_config(videdra_config(sizes))
+    out = {"sizes": dict(sizes, layers=len(cfg.layers), vocab=MAROTAR_VOCAB, window=MAROTAR_WINDOW, keep_first=VIDEDRA_KEEP)}
+    tab, blocks = bench_tables(cfg.block_size, max_len)
+    m = MixedDecoder(cfg, num_blocks=blocks, max_len=max_len, max_tokens=2048, max_sequences=B, device=dev)
+    m.init_random_weights(0)
+    for p in [p for p, l in zip(m.pools, cfg.layers) if p is not None and l.mixer.kv_from is None] + [s for s in m.states if s is not None]:
+        p.normal_()
+    pos = lens.astype(np.int32)
+    m.set_decode_inputs(rng.integers(0, MAROTAR_VOCAB, size=B).astype(np.int32), pos, tab, pos + 1, sharding.slot_mapping(tab, pos, cfg.block_size),
+                        np.arange(1, B + 1, dtype=np.int32))
+    m.capture(B)
+    with ClockSampler(local) as clocks:
+        ms = _stepped(torch, m, B, steps)
+    att, ret = cfg.layers[3].mixer, cfg.layers[0].mixer
+    live = int(np.where(lens + 1 > MAROTAR_WINDOW, MAROTAR_WINDOW + np.minimum(VIDEDRA_KEEP, lens + 1 - MAROTAR_WINDOW), lens + 1).sum())
+    state_bytes = 8 * B * ret.heads * ret.dim * ret.vdim  # read and written
+    elem = lambda t: t.numel() * t.element_size()
+    moe = not isinstance(cfg.layers[0].mlp, Dense)
+    hit = 1.0
+    if moe:  # the share of the experts a decode step reads
+        f = cfg.layers[0].mlp
+        hit = 1 - (1 - f.top / f.experts) ** B
+    weights = sum(elem(v) * (hit if k.startswith("e_") else 1.0) for lw in m.layers for k, v in lw.items() if k != "lambda") + elem(m.head)
+    step_bytes = weights + 2 * 2 * live * att.row + 6 * state_bytes
+    out["decode"] = {"tokens_per_s": B / ms * 1e3, "ms_per_step": ms, "step_hbm_frac": step_bytes / ms / 1e6 / pk["hbm_gbs"], "clocks": clocks.summary()}
+    kt = KernelTimes(torch, pk)
+    bf = lambda *s: torch.randn(s, device=dev, dtype=torch.bfloat16)
+    f32 = lambda *s: torch.randn(s, device=dev)
+
+    def copies(ws):
+        """Those weights, repeated until the set is well past L2."""
+        n = len(ws)
+        while sum(elem(w) for w in ws) < 4e8:
+            ws = ws + [w.clone() for w in ws[:n]]
+        return ws
+
+    def project(name, ws, x_, y_, bound, **kw):
+        ws, n = copies(ws), ws[0].numel()
+        kt.time(name, [lambda w=w: ops.dense_gemm(ops.dense(x_, w, y_, **kw), weights_const=True) for w in ws], 2 * n + elem(x_) + elem(y_), 2.0 * x_.shape[0] * n, bound)
+
+    def kernels_at(n, bound):
+        W = cfg.width
+        attl, retl = m.layers[3], m.layers[0]
+        h, y = bf(n, W), f32(n, W)
+        ap, rp = f32(n, attl["proj"].shape[0]), f32(n, retl["proj"].shape[0])
+        ao, ro = bf(n, att.heads * att.vdim), bf(n, ret.heads * ret.vdim)
+        project("attention: q|k|v|gate", [m.layers[3]["proj"]], h, ap, bound)
+        project("attention: output", [m.layers[3]["o"]], ao, y, bound)
+        project("retention: q|k|v|gate", [lw["proj"] for lw in m.layers if lw["proj"].shape == retl["proj"].shape], h, rp, bound)
+        project("retention: output", [lw["o"] for lw in m.layers if lw["o"].shape == retl["o"].shape], ro, y, bound)
+        cos, sin = m._rot[3]
+        q = bf(n, att.heads * 2, att.kdim)
+        slots = torch.arange(64, 64 + n, dtype=torch.int32, device=dev)
+        positions = torch.arange(n, dtype=torch.int32, device=dev)
+        pool = m.pools[3]
+        parts = [ops.rotate_part(q, 0, att.heads * 2, att.dim, padded=att.kdim, row_ld=att.heads * 2 * att.kdim),
+                 ops.rotate_part(pool, att.heads * 2 * att.dim, att.kv_heads * 2, att.dim, padded=att.kdim, row_ld=att.row, by_slot=True),
+                 ops.rotate_part(pool[0, 0, att.v_first:], (att.heads + att.kv_heads) * 2 * att.dim, att.kv_heads, att.vdim, padded=att.vpad, row_ld=att.row,
+                                 rotate=False, by_slot=True)]
+        kt.time("attention: rotation and cache rows", [lambda: ops.rotate_rows(ap, parts, positions, cos, sin, rot_dims=att.rot.dims, slots=slots, num_slots=blocks * 64)] * 4,
+                elem(ap) + elem(q) + 2 * n * att.row, 0.0, "hbm")
+        end = lambda maps, slices: ops.map_difference(maps, ao, rows=n, heads=att.heads, vdim=att.vdim, in_ld=att.vpad, lam=0.4, keep=0.7, eps=1e-5, slices=slices, gate=ap[:, -att.heads:])
+        if bound == "hbm":
+            slices = m._slices(att, n)
+            records = slices * n * att.heads * 2 * (att.vpad + 2) * 4
+            sl = torch.from_numpy((lens + 1).astype(np.int32)).to(dev)
+            kt.time("attention over pages", [lambda p=p: ops.grouped_attention(q, p, m.block_tables[:n], sl, m._maps, v_heads=att.kv_heads, maps=2, vdim=att.vpad, v_first=att.v_first,
+                                                                               scale=att.scale, slices=slices, window=MAROTAR_WINDOW, keep_first=VIDEDRA_KEEP)
+                                             for p in (pool, pool)], 2 * live * att.row + elem(q) + records, 2.0 * live * att.heads * 2 * (att.dim + att.vdim), bound)
+            kt.time("attention: merge, difference, norm, gate", [lambda: end(m._maps, slices)] * 4, records + elem(ao), 0.0, "hbm")
+            states, where = [s for s in m.states if s is not None], torch.arange(1, n + 1, dtype=torch.int32, device=dev)
+            cos, sin = m._rot[0]
+            later = positions + 7  # no row starts from nothing
+            kt.time("retention step", [lambda s=s: ops.retention_step(rp, later, cos, sin, m._decay[0], where, s, ro, heads=ret.heads,
+                                                                      dim=ret.dim, vdim=ret.vdim, rot_dims=ret.rot.dims, k_scale=0.1, eps=1e-5) for s in states],
+                    state_bytes + elem(rp) + elem(ro), 0.0, bound)
+        else:
+            keys = n + MAROTAR_WINDOW - 1 + VIDEDRA_KEEP
+            rows, maps = bf(keys, att.row), f32(n, att.heads * 2 * att.vpad)
+            kt.time("attention: gather of the window", [lambda: ops.latent_gather(pool, m.block_tables[0], rows, first=VIDEDRA_KEEP, keep=VIDEDRA_KEEP)] * 4, 4 * elem(rows) // 2, 0.0, "hbm")
+            k_, v_ = rows[:, :att.v_first].view(keys, att.kv_heads * 2, att.kdim), rows[:, att.v_first:].view(keys, att.kv_heads, att.vpad)
+            kt.time("attention of the portion", [lambda: ops.window_attention(q, k_, None, v_, maps, first_query=keys - n, scale=att.scale, window=MAROTAR_WINDOW,
+                                                                              keep_first=VIDEDRA_KEEP, maps=2)] * 4,
+                    elem(q) + elem(rows) + elem(maps), 2.0 * n * (MAROTAR_WINDOW + VIDEDRA_KEEP) * att.heads * 2 * (att.dim + att.vdim), bound)
+            kt.time("attention: difference, norm, gate", [lambda: end(maps, 0)] * 4, elem(maps) + elem(ao), 0.0, "hbm")
+            cos, sin = m._rot[0]
+            rq, rk, rv, o = bf(n, ret.heads, ret.kdim), bf(n, ret.heads, ret.kdim), bf(n, ret.heads, ret.vpad), f32(n, ret.heads, ret.vdim)
+            hd = ret.heads * ret.dim
+            rparts = [ops.rotate_part(rq, 0, ret.heads, ret.dim, padded=ret.kdim, row_ld=ret.heads * ret.kdim), ops.rotate_part(rk, hd, ret.heads, ret.dim, padded=ret.kdim, row_ld=ret.heads * ret.kdim),
+                      ops.rotate_part(rv, 2 * hd, ret.heads, ret.vdim, padded=ret.vpad, row_ld=ret.heads * ret.vpad, rotate=False)]
+            kt.time("retention: rotation", [lambda: ops.rotate_rows(rp, rparts, positions, cos, sin, rot_dims=ret.rot.dims)] * 4, 6 * hd * n * 2 + 6 * n * ret.heads * ret.vdim, 0.0, "hbm")
+            where = torch.ones((n,), dtype=torch.int32, device=dev)
+            states = [s for s in m.states if s is not None]
+            kt.time("retention over the portion", [lambda s=s: ops.retention_chunks(rq, rk, rv, positions, m._decay[0], where, s, o, m._state_sums) for s in states],
+                    elem(rq) + elem(rk) + elem(rv) + elem(o) + 8 * hd * ret.vdim, 2.0 * n * ret.heads * (64 * (ret.dim + ret.vdim) + 2 * ret.dim * ret.vdim), "hbm")
+            kt.time("retention: norm and gate", [lambda: ops.head_norm_gate(o, rp[:, 2 * hd + ret.heads * ret.vdim:], ro, 1e-5)] * 4, 2 * elem(o) + elem(ro), 0.0, "hbm")
+        gain = torch.ones((W,), device=dev)
+        kt.time("norm, residual, norm", [lambda: ops.residual_norm(y, m.x[:n], gain, 1e-5, gain_next=gain, out=h)] * 4, 3 * elem(y) + elem(h), 0.0, "hbm")
+        lw = m.layers[0]
+        act = bf(n, lw["down"].shape[1])
+        project("feed-forward gate|up" + (" (shared expert)" if moe else ""), [l["up"] for l in m.layers], h, act, bound, act=N.ACT_SILU_MUL if moe else N.ACT_GELU_TANH_MUL)
+        project("feed-forward down" + (" (shared expert)" if moe else ""), [l["down"] for l in m.layers], act, y, bound)
+        if not moe:
+            return
+        f = cfg.layers[0].mlp
+        logits = f32(n, f.experts + 1)
+        project("router", [l["router"] for l in m.layers], h, logits, "hbm")
+        ids, wts, rows_of = (m._view(b, n, f.top) for b in (m._ids, m._weights, m._rows_of))
+        tokens_of, offsets = m._tokens_of[:n * f.top], m._offsets
+        kt.time("routing", [lambda: ops.moe_route(logits, ids, wts, offsets, rows_of, tokens_of, experts=f.experts)] * 4, elem(logits) + 16 * n * f.top, 0.0, "hbm")
+        xs, acts, outs = m._view(m._sorted, n * f.top, W), m._view(m._act_sorted, n * f.top, lw["e_down"].shape[2]), m._view(m._out_sorted, n * f.top, W)
+        kt.time("tokens by expert", [lambda: ops.gather_rows(h, tokens_of, xs)] * 4, 2 * elem(xs), 0.0, "hbm")
+        read = int((torch.diff(offsets) > 0).sum()) / f.experts
+        for name, key, a_, b_, act_ in (("experts gate|up", "e_up", xs, acts, N.ACT_SILU_MUL), ("experts down", "e_down", acts, outs, N.ACT_NONE)):
+            w0 = lw[key]
+            kt.time(name, [lambda w=l[key]: ops.dense_gemm(ops.grouped_dense(a_, w, b_, offsets, act=act_)) for l in m.layers], elem(w0) * read + elem(a_) + elem(b_),
+                    2.0 * n * f.top * w0.shape[1] * w0.shape[2], bound)
+        kt.time("experts' sum, norm, residual, norm", [lambda: ops.residual_norm(y, m.x[:n], gain, 1e-5, gain_next=gain, out=h, gate=logits[:, f.experts], parts=outs, part_rows=rows_of,
+                                                                                part_weights=wts)] * 4, 3 * elem(y) + elem(h) + elem(outs), 0.0, "hbm")
+
+    kernels_at(B, "hbm")
+    out["decode"]["kernels"] = kt.take()
+    whole, last = _prefill(torch, m, tokens, 2048)
+    out["prefill"] = {"tokens_per_s": MAROTAR_PROMPT / whole * 1e3, "ms": whole, "portion": 2048, "ms_last_portion": last, "tokens_per_s_last_portion": 2048 / last * 1e3}
+    kernels_at(2048, "tensor")
+    out["prefill"]["kernels"] = kt.take()
+    out["device_status"] = N.lib().tlaloc_b200_device_status()
+    del m
+    gc.collect()
+    torch.cuda.empty_cache()
+    out["latent"] = latent_case(torch, dev, pk, latent, steps, local)
+    return out
+
+
+def run_videdra(args) -> dict:
+    import torch
+
+    local = int(os.environ.get("LOCAL_RANK", "0"))
+    dev = torch.device("cuda", local)
+    torch.cuda.set_device(dev)
+    pk = peaks()
+    names = [n for n in VIDEDRA if not args.only or args.only in n]
+    cases = {n: videdra_case(torch, dev, pk, *VIDEDRA[n], max(args.steps, 5), local) for n in names}
+    head = cases[names[0]]
+    return {"metric": "videdra_decode_tokens_per_s", "value": head["decode"]["tokens_per_s"], "unit": UNIT, "n_gpus": 1, "steps": max(args.steps, 5),
+            "warmup": 3, "ms_per_step": head["decode"]["ms_per_step"], "higher_is_better": True, "data": "synthetic", "dtype": "bf16",
+            "config": {"workload": f"8 layers of the decoder of differential attention and retention at real models' layer sizes (random weights), batch {MAROTAR_BATCH}, "
+                                   f"contexts U[1024,8192], window {MAROTAR_WINDOW} and {VIDEDRA_KEEP} kept tokens; prefill of {MAROTAR_PROMPT} tokens; beside a "
+                                   "latent-attention decoder of equal size; weights, states and pools of a timed set exceed L2", "peaks": pk, "cases": cases}}
 
 
 def run_marotar(args) -> dict:
@@ -1174,9 +1395,9 @@ def main() -> None:
     ap.add_argument("--steps", type=int, default=20)
     ap.add_argument("--warmup", type=int, default=3)
     ap.add_argument("--impl", default="ours", choices=["ours", "reference"])
-    ap.add_argument("--workload", default="llama70b", choices=sorted(WORKLOADS) + ["paged_attn", "int8_proj", "peer_sum", "marotar"])
+    ap.add_argument("--workload", default="llama70b", choices=sorted(WORKLOADS) + ["paged_attn", "int8_proj", "peer_sum", "marotar", "videdra"])
     ap.add_argument("--layers", type=int, default=0, help="override the layer count (debugging only; not a bench value)")
-    ap.add_argument("--only", default="", help="int8_proj: a single shape NxKxM; marotar: a single size, e.g. 4096")
+    ap.add_argument("--only", default="", help="int8_proj: a single shape NxKxM; marotar, videdra: a single size, e.g. 4096")
     ap.add_argument("--no-cpu", action="store_true", help="skip the CPU baseline leg")
     ap.add_argument("--lean", action="store_true", help="skip the projection roofline, the operator sweeps and the 8B-shape block")
     ap.add_argument("--timeline", action="store_true", help="per-kernel durations inside one graph replay of the step")
@@ -1193,6 +1414,8 @@ def main() -> None:
         line = run_peer_sum(args)
     elif args.workload == "marotar":
         line = run_marotar(args)
+    elif args.workload == "videdra":
+        line = run_videdra(args)
     else:
         line = run_ours(args)
     if line:

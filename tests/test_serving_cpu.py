@@ -7,9 +7,11 @@ import pytest
 import torch
 
 import latent_oracle as oracle
+import videdra_oracle as videdra
 from tlaloc_b200 import registry
 from tlaloc_b200.engine import Engine
 from tlaloc_b200.latent_decoder import LatentDecoderConfig
+from tlaloc_b200.mixed_decoder import MixedDecoderConfig
 from tlaloc_b200.paging import PADDING_PAGE, PagePool, Sequence, stage_ragged
 from tlaloc_b200.rotary import Rotation, YarnScaling, pair_tables
 from tlaloc_b200.scheduler import Request, Scheduler
@@ -55,6 +57,54 @@ class HistoryModel(StepModel):
         return self.status
 
 
+class RecurrentModel(HistoryModel):
+    """Also keeps a number per state slot that every token changes, and answers with it: a wrong slot, a lost or a repeated token, or a slot
+    that does not start over with its next sequence shows in every later token.  Attends to the first `keep` tokens and the window."""
+
+    def __init__(self, states=4, keep=0, **kw):
+        super().__init__(sequences=kw.pop("sequences", states), **kw)
+        self.num_states, self.keep_first = states, keep
+        self.numbers = np.full((states + 1,), 12345, np.int64)
+
+    @staticmethod
+    def answer_of(number, seen, vocab):
+        return int((number + sum((i + 1) * (t + 3) for i, t in enumerate(seen))) % vocab)
+
+    @staticmethod
+    def visible(h, window, keep):
+        lo = max(0, len(h) - window) if window else 0
+        return h[:min(keep, lo)] + h[lo:]
+
+    def run(self, step, want):
+        n = len(step.token_ids)
+        assert n <= self.max_tokens and len(step.starts) - 1 <= self.max_sequences
+        self.slots[step.slot_mapping] = step.token_ids
+        out, numbers = torch.full((len(want), self.vocab), -1.0), []
+        for r in range(n):
+            s = step.row_states[r]
+            assert 1 <= s <= self.num_states
+            before = 0 if step.positions[r] == 0 else self.numbers[s]
+            self.numbers[s] = (before * 31 + int(step.token_ids[r]) + 1) % 1000003
+            numbers.append(int(self.numbers[s]))
+        for k, r in enumerate(want):
+            end, table = int(step.seq_lens[r]), step.block_tables[step.row_tables[r]]
+            lo = max(0, end - self.window) if self.window else 0
+            places = [*range(min(self.keep_first, lo)), *range(lo, end)]
+            seen = [int(self.slots[table[p // self.block_size] * self.block_size + p % self.block_size]) for p in places]
+            out[k, self.answer_of(numbers[r], seen, self.vocab)] = 1.0
+        return out
+
+
+def expected_recurrent(prompt, n, vocab=97, window=None, keep=0):
+    h, number = [], 0
+    for t in prompt:
+        h, number = h + [t], (number * 31 + t + 1) % 1000003
+    for _ in range(n):
+        t = RecurrentModel.answer_of(number, RecurrentModel.visible(h, window, keep), vocab)
+        h, number = h + [t], (number * 31 + t + 1) % 1000003
+    return h[len(prompt):]
+
+
 def expected(prompt, n, vocab=97, window=None, stop=()):
     h = list(prompt)
     for _ in range(n):
@@ -74,6 +124,48 @@ def test_generation_under_page_pressure(window, blocks):
     assert eng.generate(prompts, 9) == [expected(p, 9, window=window) for p in prompts]
     assert eng.pool.free_count == eng.pool.capacity
     assert max(len(s) for s in model.steps) <= 4 and max(sum(s) for s in model.steps) <= 16
+
+
+@pytest.mark.parametrize("window,keep", [(None, 0), (5, 0), (4, 1), (6, 9), (1, 4)])
+@pytest.mark.parametrize("blocks,states", [(9, 4), (12, 2), (40, 1)])
+def test_states_and_kept_tokens_under_pressure(window, keep, blocks, states):
+    """Sequences that are sent back lose their state and build it up again; kept first tokens stay in their pages."""
+    rng = np.random.default_rng(blocks)
+    prompts = [rng.integers(0, 97, size=n).tolist() for n in (1, 3, 17, 4, 9, 20, 2)]
+    model = RecurrentModel(states=states, keep=keep, blocks=blocks, window=window)
+    eng = Engine(model)
+    assert eng.generate(prompts, 9) == [expected_recurrent(p, 9, window=window, keep=keep) for p in prompts]
+    assert eng.pool.free_count == eng.pool.capacity and eng.pool._free_states == set(range(1, states + 1))
+
+
+def test_state_slots_that_run_out_and_come_back():
+    eng = Engine(RecurrentModel(states=2, blocks=40))
+    for k in "ab":
+        eng.feed([(k, [1, 2, 3], [])])
+    with pytest.raises(RuntimeError, match="state slot"):
+        eng.feed([("c", [4], [])])
+    eng.sequences.pop("c")
+    eng.close("a")
+    got, = eng.feed([("c", [7, 9], [1])])
+    assert got.argmax(-1).tolist() == expected_recurrent([7, 9], 1)
+    pool = PagePool(4, num_states=1)
+    s = pool.take_state()
+    assert s == 1 and not pool.has_state and pool.take_state() is None
+    pool.give_state(s)
+    for bad in (0, 1, 2):
+        with pytest.raises(ValueError):
+            pool.give_state(bad)
+
+
+def test_pages_between_kept_tokens_and_window_go_back():
+    pool, seq = PagePool(10), Sequence()
+    assert seq.reserve(pool, 30, 4)  # eight pages
+    pages = list(seq.pages)
+    assert seq.drop_before(pool, 21, 4, keep_first=5) == 3  # positions 8 .. 19: two pages stay in front
+    assert seq.pages == pages[:2] + [PADDING_PAGE] * 3 + pages[5:] and pool.free_count == 4
+    assert seq.drop_before(pool, 21, 4, keep_first=5) == 0 and seq.drop_before(pool, 3, 4, keep_first=5) == 0
+    seq.release(pool)
+    assert pool.free_count == pool.capacity
 
 
 def test_prompt_portions_and_decoding_share_a_step():
@@ -209,8 +301,41 @@ def test_configuration_is_read_whole():
             LatentDecoderConfig.from_config(bad)
 
 
+def test_configuration_of_mixed_layers_is_read_whole():
+    A, R = videdra.attention_layer, videdra.retention_layer
+    c = videdra.model(R(mlp=videdra.dense_mlp(30)), A(mlp=videdra.moe_mlp(), window=12, keep=7), A(kv_from=1, window=40, keep=2), R(mlp=videdra.moe_mlp(shared=0, top=1)))
+    cfg = MixedDecoderConfig.from_config(json.loads(json.dumps(c)))
+    assert {k: tuple(v.shape) for k, v in videdra.make_weights(c).items()} == cfg.tensor_shapes()
+    assert cfg.window == 40 and cfg.keep_first == 7 and cfg.recurrent and cfg.layers[2].mlp is None and cfg.layers[3].mlp.shared_ff is None
+    assert cfg.layers[1].mixer.row == 2 * 2 * 32 + 2 * 48 and cfg.layers[2].mixer.kv_from == 1 and cfg.layers[0].mixer.decay == tuple(c["layers"][0]["mixer"]["decay"])
+    assert MixedDecoderConfig.from_config(videdra.model(A(window=0), A(window=3))).window is None
+    alone = MixedDecoderConfig.from_config(videdra.model(R()))
+    assert alone.window == 1 and alone.keep_first == 0
+    assert not MixedDecoderConfig.from_config(videdra.model(A())).recurrent
+    for change in (lambda d: d["layers"][0].update(type="other"), lambda d: d["layers"][0]["mlp"].update(kind="other"), lambda d: d["layers"][2]["mixer"].update(kv_from=2),
+                   lambda d: d["layers"][2]["mixer"].update(kv_from=0), lambda d: d["layers"][2]["mixer"].update(kv_heads=3), lambda d: d["layers"][0]["mixer"]["decay"].pop(),
+                   lambda d: d["layers"][1]["mixer"]["rot"].update(dims=64), lambda d: d["layers"][1]["mixer"].update(kv_heads=4),
+                   lambda d: d["layers"][1]["mlp"]["router"].update(top=8)):
+        bad = json.loads(json.dumps(c))
+        change(bad)
+        with pytest.raises(ValueError):
+            MixedDecoderConfig.from_config(bad)
+
+
+def test_gate_and_factor_are_interleaved_by_sixteen():
+    from tlaloc_b200.ops import interleave_gate
+
+    gate, up = torch.arange(2 * 20 * 3.0).reshape(2, 20, 3) + 1, -torch.arange(2 * 20 * 3.0).reshape(2, 20, 3) - 1
+    w = interleave_gate(gate, up)
+    assert w.shape == (2, 64, 3) and torch.equal(w[1], interleave_gate(gate[1], up[1]))
+    for f in range(20):
+        r = f // 16 * 32 + f % 16
+        assert torch.equal(w[:, r], gate[:, f]) and torch.equal(w[:, r + 16], up[:, f])
+    assert torch.all(w[:, 36:48] == 0) and torch.all(w[:, 52:] == 0)
+
+
 def test_registry_names(tmp_path):
-    assert registry.architecture_of({"architecture": "Marotar"}) == "Marotar"
+    assert registry.architecture_of({"architecture": "Marotar"}) == "Marotar" and registry.architecture_of({"architecture": "Videdra"}) == "Videdra"
     assert registry.architecture_of({"architectures": ["LlamaForCausalLM"]}) == "LlamaForCausalLM"
     with pytest.raises(ValueError):
         registry.architecture_of({"architecture": "unheard of"})
@@ -226,5 +351,6 @@ def test_command_line_lists_models(capsys):
     from tlaloc_b200.__main__ import main
 
     assert main(["models"]) == 0
-    assert "Marotar bfloat16 float32" in capsys.readouterr().out
+    out = capsys.readouterr().out
+    assert "Marotar bfloat16 float32" in out and "Videdra bfloat16 float32" in out
     assert main(["nothing"]) == 2
