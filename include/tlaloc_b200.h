@@ -445,7 +445,7 @@ int tlaloc_b200_rotate_rows(const float* in, int64_t ld, const tlaloc_b200_rotat
  * elements; in bf16 dim and vdim are multiples of 16 and the pool's strides multiples of 8.
  */
 int tlaloc_b200_grouped_attention_slices(int32_t num_tokens, int32_t num_heads, int32_t v_heads, int32_t maps, int32_t dim, int32_t vdim,
-                                         int32_t dtype, int32_t max_live);
+                                         int32_t block_size, int32_t dtype, int32_t max_live);
 int tlaloc_b200_grouped_attention(const void* q, const void* pool, int64_t pool_ld, int32_t dtype, const int32_t* block_tables,
                                   const int32_t* row_tables, const int32_t* seq_lens, float* records, int32_t slices, int32_t num_tokens,
                                   int32_t num_heads, int32_t v_heads, int32_t maps, int32_t dim, int32_t vdim, int32_t v_first,

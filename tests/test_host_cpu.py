@@ -81,7 +81,7 @@ def test_refusals_of_the_mixers_need_no_gpu():
     att = lambda **kw: lib.tlaloc_b200_grouped_attention(one, one, kw.get("ld", 96), N.BF16, one, None, one, one, kw.get("slices", 1), kw.get("rows", 0), kw.get("heads", 8),
                                                          2, 2, 16, 16, kw.get("v_first", 64), 9, 64, 4, 1, kw.get("window", 0), kw.get("keep", 0), 0.1, None)
     assert att() == N.OK and att(ld=95) == i and att(heads=6) == i and att(v_first=63) == i and att(window=-1) == i and att(keep=-1) == i and att(slices=0) == i
-    assert lib.tlaloc_b200_grouped_attention_slices(4, 8, 2, 2, 24, 16, N.BF16, 4096) == 1  # not the tensor-core kernel's sizes
+    assert lib.tlaloc_b200_grouped_attention_slices(4, 8, 2, 2, 24, 16, 64, N.BF16, 4096) == 1  # not the tensor-core kernel's sizes
     assert lib.tlaloc_b200_map_difference(one, -1, None, 0, one, 16, N.BF16, 1, 2, 8, 8, 0.1, 0.5, 1e-5, None) == i
     assert lib.tlaloc_b200_map_difference(one, 0, None, 0, one, 15, N.BF16, 1, 2, 8, 8, 0.1, 0.5, 1e-5, None) == i
     assert lib.tlaloc_b200_head_norm_gate(one, one, 16, one, 15, N.BF16, 1, 2, 8, 1e-5, None) == i

@@ -75,7 +75,7 @@ _SIGNATURES = {
     "tlaloc_b200_window_attention": (ctypes.c_int, [_vp, _vp, _i64, _vp, _i64, _vp, _i64, _i64, _vp, _i64] + [_i32] * 12 + [_f32, _vp]),
     "tlaloc_b200_residual_norm": (ctypes.c_int, [_vp, _vp, _i64, _vp, _vp, _vp, _i32, _vp, _vp, _vp, _vp, _i32, _i32, _i32, _f32, _vp]),
     "tlaloc_b200_rotate_rows": (ctypes.c_int, [_vp, _i64, ctypes.POINTER(RotatePart), _i32, _i32, _vp, _vp, _vp, _vp] + [_i32] * 4 + [_vp]),
-    "tlaloc_b200_grouped_attention_slices": (ctypes.c_int, [_i32] * 8),
+    "tlaloc_b200_grouped_attention_slices": (ctypes.c_int, [_i32] * 9),
     "tlaloc_b200_grouped_attention": (ctypes.c_int, [_vp, _vp, _i64, _i32, _vp, _vp, _vp, _vp] + [_i32] * 14 + [_f32, _vp]),
     "tlaloc_b200_map_difference": (ctypes.c_int, [_vp, _i32, _vp, _i64, _vp, _i64] + [_i32] * 5 + [_f32, _f32, _f32, _vp]),
     "tlaloc_b200_head_norm_gate": (ctypes.c_int, [_vp, _vp, _i64, _vp, _i64] + [_i32] * 4 + [_f32, _vp]),

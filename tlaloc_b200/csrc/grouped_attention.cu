@@ -1,23 +1,36 @@
 // Attention of single tokens over a paged pool of grouped key and value heads, with a sliding window and kept first tokens, one or two
 // maps of scores per query head over the same values (include/tlaloc_b200.h, tlaloc_b200_grouped_attention).
 //
-// The positions a row sees are counted through: the kept ones, then those of the window.  They are cut into groups of 16 and, when there
-// are few rows, into slices; each slice leaves a record per query head ({largest score (log2), sum, weighted values}), and the operator
-// that consumes the result merges them.
-//   GroupedAttentionMma      bf16.  A CTA has one value head, up to 16 of its query heads (8 of two maps each) and one slice, so every cached
-//                            byte of the slice is read once for all of them.  Four warps, each with groups and a three-stage ring of its own,
-//                            fed by 16-byte cp.async copies through the block table: no barrier in the loop.  Query heads are the rows of
-//                            mma.m16n8k16; with two maps the rows 0-7 are the heads' first map and 8-15 the second, each multiplied with its
-//                            own keys, so that one product with the values serves both.  The weights enter that product as two bf16
-//                            parts (f32 up to rounding).
+// The positions are taken in groups of 16, aligned, so that a group lies in one page: those of the kept tokens, then those of the window; what a
+// row does not see of a group is masked.  With few rows the groups are cut into slices; each slice leaves a record per query head
+// ({largest score (log2), sum, weighted values}), and the operator that consumes the result merges them.
+//   GroupedAttentionMma      bf16, pages of a multiple of 16.  A CTA has one value head, up to 16 of its query heads (8 of two maps each) and one
+//                            slice, so every cached byte of the slice is read once for all of them.  Four warps, each with groups and a
+//                            ring of its own: one lane looks up the page and requests the group's boxes (64 channels x 16 rows, 128-byte
+//                            swizzle) by TMA; no CTA-wide barrier in the loop.  Query heads are the rows of mma.m16n8k16; with two maps the
+//                            rows 0-7 are the heads' first map and 8-15 the second, each multiplied with its own keys, so that one
+//                            product with the values serves both.  The weights enter that product as two bf16 parts (f32 up to rounding).
 //   GroupedAttentionGeneric  any size and type, plain FMA: the f32 path.
+#include <cuda.h>
+
 #include "common.cuh"
+#include "tc_common.cuh"
 
 namespace tlaloc_b200 {
 namespace {
 
-constexpr int kGroup = 16, kWarps = 4, kStages = 3;
+using tc::ElectOne;
+using tc::MbarExpectTx;
+using tc::MbarInit;
+using tc::MbarWait;
+using tc::MbarWaitWarp;
+using tc::SmemAddr;
+
+constexpr int kGroup = 16, kWarps = 4, kMaxStages = 4;
+constexpr int kAtom = kGroup * 128;  // 16 rows x 64 channels
 constexpr int kMaxSmem = 227 * 1024;
+
+__device__ int g_grouped_status = 0;
 
 struct GroupedArgs {
   const void* q;
@@ -25,7 +38,7 @@ struct GroupedArgs {
   const int *tables, *row_tables, *lens;
   float* records;
   int64_t pool_ld;
-  int T, heads, v_heads, maps, dim, vdim, v_first, num_blocks, block_size, max_blocks, num_tables, window, keep, slices, qtiles;
+  int T, heads, v_heads, maps, dim, vdim, v_first, num_blocks, block_size, max_blocks, num_tables, window, keep, slices, qtiles, stages;
   float scale_log2;
 };
 
@@ -85,24 +98,43 @@ __device__ __forceinline__ void Split(float a, float b, uint32_t& hi, uint32_t& 
   lo = *reinterpret_cast<const uint32_t*>(&l);
 }
 
-// DK: 16-channel steps of a key head at most, NV: 16-channel steps of a value head at most.
+// DK, NV: 16-channel steps of a key and a value head, in whole atoms of four.  What an atom holds past its head is multiplied with zero
+// queries (keys) or left out of the result (values).
 template <int DK, int NV>
-__global__ void __launch_bounds__(kWarps * 32) GroupedAttentionMma(const __grid_constant__ GroupedArgs a)
+__global__ void __launch_bounds__(kWarps * 32) GroupedAttentionMma(const __grid_constant__ CUtensorMap map, const __grid_constant__ GroupedArgs a)
 {
-  GridDependencySync();
-  extern __shared__ __align__(16) unsigned char smem[];
+  extern __shared__ unsigned char smem_raw[];
+  __shared__ alignas(8) uint64_t bars[kWarps * kMaxStages];
+  __shared__ uint32_t abort_store;
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+  const uint32_t base = (SmemAddr(smem_raw) + 1023u) & ~1023u;
+  unsigned char* smem = smem_raw + (base - SmemAddr(smem_raw));
+  const uint32_t bar = SmemAddr(bars + warp * kMaxStages);
+  volatile uint32_t* abort_word = &abort_store;
+  if (tid == 0) {
+    abort_store = 0u;
+    for (int i = 0; i < kWarps * kMaxStages; ++i) MbarInit(SmemAddr(bars + i), 1);
+    asm volatile("fence.mbarrier_init.release.cluster;\n" ::: "memory");
+  }
+  __syncthreads();
+  GridDependencySync();
   const int slice = blockIdx.x, vh = blockIdx.y / a.qtiles, qt = blockIdx.y % a.qtiles, t = blockIdx.z;
   const int group = a.heads / a.v_heads, per_map = group / a.maps;  // query heads (with maps counted) and without
   const int rows_per_map = 16 / a.maps;
-  const int dk = a.dim >> 4, nv = a.vdim >> 4;
-  const Seen seen = SeenBy(a, t);
-  const int groups = (seen.count + kGroup - 1) / kGroup, share = (groups + a.slices - 1) / a.slices;
+  const int dk = a.dim >> 4;
+  const int len = min(max(__ldg(a.lens + t), 0), a.max_blocks * a.block_size);
+  const int tab = a.row_tables != nullptr ? __ldg(a.row_tables + t) : t;
+  const int* table = a.tables + static_cast<size_t>(min(max(tab, 0), a.num_tables - 1)) * a.max_blocks;
+  // Visible: lo <= position < len, or position < keep.  Groups [0, kept) and [first, ..).
+  const int lo = a.window > 0 ? max(0, len - a.window) : 0, keep = min(a.keep, lo);
+  const int kept = (keep + kGroup - 1) / kGroup, first = max(lo / kGroup, kept);
+  const int groups = kept + (len + kGroup - 1) / kGroup - first, share = (groups + a.slices - 1) / a.slices;
   const int g0 = slice * share, g1 = min(groups, g0 + share);
+  auto position = [&](int g) { return (g < kept ? g : first + g - kept) * kGroup; };
   // The query head of MMA row r: (place in the group, map).
   auto query_head = [&](int r) {
-    const int place = qt * rows_per_map + r % rows_per_map, map = r / rows_per_map;
-    return place < per_map ? (vh * per_map + place) * a.maps + map : -1;
+    const int place = qt * rows_per_map + r % rows_per_map, m = r / rows_per_map;
+    return place < per_map ? (vh * per_map + place) * a.maps + m : -1;
   };
   const int rec = a.vdim + 2;
   float* records = a.records + (static_cast<size_t>(slice) * a.T + t) * a.heads * rec;
@@ -116,6 +148,41 @@ __global__ void __launch_bounds__(kWarps * 32) GroupedAttentionMma(const __grid_
     }
     return;
   }
+
+  // A stage: the atoms of every map's keys, then those of the values.  x is a multiple of 16 channels: a 16-byte boundary.
+  constexpr int k_atoms = DK / 4, v_atoms = NV / 4;
+  const int stage_bytes = (a.maps * k_atoms + v_atoms) * kAtom, stages = a.stages;
+  const uint32_t ring = base + warp * stages * stage_bytes;
+  const int k_col = vh * a.maps * a.dim, v_col = a.v_first + vh * a.vdim;
+  const int steps = (g1 - g0 - warp + kWarps - 1) / kWarps;  // this warp's groups: g0 + warp, + kWarps, ..
+  auto pool_row = [&](int i) {  // of the i-th group
+    const int pos = position(g0 + warp + min(i, steps - 1) * kWarps), b = pos / a.block_size;
+    return min(max(__ldg(table + b), 0), a.num_blocks - 1) * a.block_size + (pos - b * a.block_size);
+  };
+  auto load = [&](int row, int stage) {
+    const uint32_t bar_s = bar + 8 * stage;
+    uint32_t dst = ring + stage * stage_bytes;
+    MbarExpectTx(bar_s, stage_bytes);
+    auto box = [&](int x) {
+      asm volatile("cp.async.bulk.tensor.2d.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1, {%2, %3}], [%4];\n" ::"r"(dst),
+                   "l"(reinterpret_cast<uint64_t>(&map)), "r"(x), "r"(row), "r"(bar_s)
+                   : "memory");
+      dst += kAtom;
+    };
+    for (int m = 0; m < a.maps; ++m)
+#pragma unroll
+      for (int c = 0; c < k_atoms; ++c) box(k_col + m * a.dim + c * 64);
+#pragma unroll
+    for (int c = 0; c < v_atoms; ++c) box(v_col + c * 64);
+  };
+  if (steps > 0) {
+    for (int i = 0; i < min(steps, stages); ++i) {
+      const int row = pool_row(i);
+      if (lane == 0) load(row, i);
+      __syncwarp();
+    }
+  }
+  int next_row = steps > 0 ? pool_row(stages) : 0;  // looked up ahead of its request
 
   // Queries as A fragments: rows lane / 4 and lane / 4 + 8.
   uint32_t qa[DK][2], qb[DK][2];
@@ -139,83 +206,74 @@ __global__ void __launch_bounds__(kWarps * 32) GroupedAttentionMma(const __grid_
     }
   }
 
-  // A stage: 16 rows of [maps x dim] keys, then 16 rows of values; rows 16 bytes longer than their content (ldmatrix without conflicts).
-  const int k_bytes = a.maps * a.dim * 2, k_ld = k_bytes + 16, v_ld = a.vdim * 2 + 16, stage_bytes = kGroup * (k_ld + v_ld);
-  const uint32_t ring = static_cast<uint32_t>(__cvta_generic_to_shared(smem)) + warp * kStages * stage_bytes;
-  const int k_chunks = k_bytes >> 4, chunks = k_chunks + (a.vdim >> 3);
-  int span = 2;  // lanes of a row of chunks: a power of two
-  while (span < chunks && span < 32) span <<= 1;
-  const int c_lane = lane & (span - 1), r_lane = lane / span, r_step = 32 / span;
-  const __nv_bfloat16* pool = static_cast<const __nv_bfloat16*>(a.pool);
-  const int k_col = vh * a.maps * a.dim, v_col = a.v_first + vh * a.vdim;
-  auto load = [&](int g, int stage) {
-    if (g < g1) {
-      const int i = g * kGroup + (lane & 15);
-      long long off = -1;
-      if (i < seen.count) off = PoolRow(a, seen, i) * a.pool_ld;
-      const uint32_t base = ring + stage * stage_bytes;
-      for (int r = r_lane; r < kGroup; r += r_step) {
-        const long long o = __shfl_sync(0xffffffffu, off, r);
-        for (int c = c_lane; c < chunks; c += span) {
-          const bool key = c < k_chunks;
-          const __nv_bfloat16* src = pool + (o < 0 ? 0 : o) + (key ? k_col + c * 8 : v_col + (c - k_chunks) * 8);
-          const uint32_t dst = base + (key ? r * k_ld + c * 16 : kGroup * k_ld + r * v_ld + (c - k_chunks) * 16);
-          asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;\n" ::"r"(dst), "l"(src), "r"(o < 0 ? 0 : 16) : "memory");  // dead rows: zeros
-        }
-      }
-    }
-    asm volatile("cp.async.commit_group;\n" ::: "memory");
-  };
-
+  bool ok = true;
   float o[2 * NV][4], top[2] = {-INFINITY, -INFINITY}, sum[2] = {0.f, 0.f};
 #pragma unroll
   for (int i = 0; i < 2 * NV; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
-  for (int s = 0; s < kStages - 1; ++s) load(g0 + warp + s * kWarps, s);
-  int stage = 0;
-  for (int g = g0 + warp; g < g1; g += kWarps) {
-    {
-      int ahead = stage + kStages - 1;
-      if (ahead >= kStages) ahead -= kStages;
-      load(g + (kStages - 1) * kWarps, ahead);
+  const int mat = lane >> 3, r8 = lane & 7;
+  // Offset of 16-byte word c of row r of a tile of atoms; of the words 2 k + mat this lane reads, those of k = 0..3 (an atom has eight).
+  auto word = [](int r, int c) { return static_cast<uint32_t>((c >> 3) * kAtom + r * 128 + (((c & 7) ^ (r & 7)) << 4)); };
+  uint32_t k_off[4], v_off[4];
+#pragma unroll
+  for (int k = 0; k < 4; ++k) {
+    k_off[k] = word((mat >> 1) * 8 + r8, 2 * k + (mat & 1));
+    v_off[k] = word((mat & 1) * 8 + r8, 2 * k + (mat >> 1));
+  }
+  int stage = 0, phase = 0;
+  for (int i = 0; i < steps; ++i) {
+    const int pos = position(g0 + warp + i * kWarps);
+    const uint32_t kt = ring + stage * stage_bytes, vt = kt + a.maps * k_atoms * kAtom;
+    ok = MbarWaitWarp(bar + 8 * stage, phase, lane, abort_word) && ok;
+    if (pos + kGroup > len) {  // rows past the end hold whatever the page did: 0 times it must stay 0
+      for (int r = len - pos; r < kGroup; ++r)
+        for (int c = lane; c < v_atoms * 8; c += 32) {
+          asm volatile("st.shared.v4.b32 [%0], {%1, %1, %1, %1};\n" ::"r"(vt + word(r, c)), "r"(0u) : "memory");
+        }
+      asm volatile("fence.proxy.async.shared::cta;\n" ::: "memory");
+      __syncwarp();
     }
-    asm volatile("cp.async.wait_group %0;\n" ::"n"(kStages - 1) : "memory");
-    __syncwarp();
-    const uint32_t kt = ring + stage * stage_bytes, vt = kt + kGroup * k_ld;
-    float s[2][4] = {};
+    float s[2][4] = {}, u[2][4] = {};
     {
-      const int m = lane >> 3;
-      const uint32_t at = kt + ((m >> 1) * 8 + (lane & 7)) * k_ld + (m & 1) * 16;
+      uint32_t at[4];
+#pragma unroll
+      for (int k = 0; k < 4; ++k) at[k] = kt + k_off[k];
       if (a.maps == 2) {
-        const uint32_t at2 = at + a.dim * 2;
 #pragma unroll
         for (int k = 0; k < DK; ++k) {
-          if (k < dk) {
-            uint32_t b[4];
-            Ldm4(b, at + k * 32);
-            Mma(s[0], qa[k][0], 0u, qa[k][1], 0u, b[0], b[1]);
-            Mma(s[1], qa[k][0], 0u, qa[k][1], 0u, b[2], b[3]);
-            Ldm4(b, at2 + k * 32);
-            Mma(s[0], 0u, qb[k][0], 0u, qb[k][1], b[0], b[1]);
-            Mma(s[1], 0u, qb[k][0], 0u, qb[k][1], b[2], b[3]);
-          }
+          uint32_t b[4], d[4];
+          Ldm4(b, at[k & 3] + (k >> 2) * kAtom);
+          Ldm4(d, at[k & 3] + (k_atoms + (k >> 2)) * kAtom);
+          Mma(s[0], qa[k][0], 0u, qa[k][1], 0u, b[0], b[1]);
+          Mma(s[1], qa[k][0], 0u, qa[k][1], 0u, b[2], b[3]);
+          Mma(u[0], 0u, qb[k][0], 0u, qb[k][1], d[0], d[1]);
+          Mma(u[1], 0u, qb[k][0], 0u, qb[k][1], d[2], d[3]);
         }
       } else {
 #pragma unroll
         for (int k = 0; k < DK; ++k) {
-          if (k < dk) {
-            uint32_t b[4];
-            Ldm4(b, at + k * 32);
-            Mma(s[0], qa[k][0], qb[k][0], qa[k][1], qb[k][1], b[0], b[1]);
-            Mma(s[1], qa[k][0], qb[k][0], qa[k][1], qb[k][1], b[2], b[3]);
-          }
+          uint32_t b[4];
+          Ldm4(b, at[k & 3] + (k >> 2) * kAtom);
+          float(*acc)[4] = (k & 1) ? u : s;
+          Mma(acc[0], qa[k][0], qb[k][0], qa[k][1], qb[k][1], b[0], b[1]);
+          Mma(acc[1], qa[k][0], qb[k][0], qa[k][1], qb[k][1], b[2], b[3]);
         }
       }
     }
-    const int i0 = g * kGroup + (lane & 3) * 2;
+    const int p0 = pos + (lane & 3) * 2;
+    if (pos + kGroup > len || (pos < lo && pos + kGroup > keep)) {
 #pragma unroll
-    for (int n = 0; n < 2; ++n)
+      for (int n = 0; n < 2; ++n)
 #pragma unroll
-      for (int e = 0; e < 4; ++e) s[n][e] = i0 + n * 8 + (e & 1) < seen.count ? s[n][e] * a.scale_log2 : -INFINITY;
+        for (int e = 0; e < 4; ++e) {
+          const int p = p0 + n * 8 + (e & 1);
+          s[n][e] = p < len && (p >= lo || p < keep) ? (s[n][e] + u[n][e]) * a.scale_log2 : -INFINITY;
+        }
+    } else {
+#pragma unroll
+      for (int n = 0; n < 2; ++n)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) s[n][e] = (s[n][e] + u[n][e]) * a.scale_log2;
+    }
     float p[2][4];
     bool raise = false;
     float next[2];
@@ -224,19 +282,19 @@ __global__ void __launch_bounds__(kWarps * 32) GroupedAttentionMma(const __grid_
       float m = fmaxf(fmaxf(s[0][2 * r], s[0][2 * r + 1]), fmaxf(s[1][2 * r], s[1][2 * r + 1]));
       m = fmaxf(m, __shfl_xor_sync(0xffffffffu, m, 1));
       m = fmaxf(m, __shfl_xor_sync(0xffffffffu, m, 2));
-      next[r] = fmaxf(top[r], m);  // the group's first position is live: finite from here on
+      next[r] = fmaxf(top[r], m);  // some position of every group is visible: finite from here on
       raise = raise || next[r] > top[r];
     }
     if (__any_sync(0xffffffffu, raise)) {
 #pragma unroll
       for (int r = 0; r < 2; ++r) {
-        const float keep = Exp2(top[r] - next[r]);
+        const float f = Exp2(top[r] - next[r]);
         top[r] = next[r];
-        sum[r] *= keep;
+        sum[r] *= f;
 #pragma unroll
-        for (int i = 0; i < 2 * NV; ++i) {
-          o[i][2 * r] *= keep;
-          o[i][2 * r + 1] *= keep;
+        for (int n = 0; n < 2 * NV; ++n) {
+          o[n][2 * r] *= f;
+          o[n][2 * r + 1] *= f;
         }
       }
     }
@@ -247,28 +305,48 @@ __global__ void __launch_bounds__(kWarps * 32) GroupedAttentionMma(const __grid_
         p[n][e] = Exp2(s[n][e] - top[e >> 1]);
         sum[e >> 1] += p[n][e];
       }
-    uint32_t hi[4], lo[4];  // as A: (row, k 0-7), (row + 8, k 0-7), (row, k 8-15), (row + 8, k 8-15)
-    Split(p[0][0], p[0][1], hi[0], lo[0]);
-    Split(p[0][2], p[0][3], hi[1], lo[1]);
-    Split(p[1][0], p[1][1], hi[2], lo[2]);
-    Split(p[1][2], p[1][3], hi[3], lo[3]);
-    const int m = lane >> 3;
-    const uint32_t at = vt + ((m & 1) * 8 + (lane & 7)) * v_ld + (m >> 1) * 16;
+    uint32_t hi[4], low[4];  // as A: (row, k 0-7), (row + 8, k 0-7), (row, k 8-15), (row + 8, k 8-15)
+    Split(p[0][0], p[0][1], hi[0], low[0]);
+    Split(p[0][2], p[0][3], hi[1], low[1]);
+    Split(p[1][0], p[1][1], hi[2], low[2]);
+    Split(p[1][2], p[1][3], hi[3], low[3]);
+    uint32_t at[4];
 #pragma unroll
-    for (int j = 0; j < NV; ++j) {
-      if (j < nv) {
-        uint32_t b[4];
-        Ldm4T(b, at + j * 32);
-        Mma(o[2 * j], hi[0], hi[1], hi[2], hi[3], b[0], b[1]);
-        Mma(o[2 * j + 1], hi[0], hi[1], hi[2], hi[3], b[2], b[3]);
-        Mma(o[2 * j], lo[0], lo[1], lo[2], lo[3], b[0], b[1]);
-        Mma(o[2 * j + 1], lo[0], lo[1], lo[2], lo[3], b[2], b[3]);
-      }
+    for (int k = 0; k < 4; ++k) at[k] = vt + v_off[k];
+#pragma unroll
+    for (int j = 0; j < NV; j += 2) {
+      uint32_t b[4], d[4];
+      Ldm4T(b, at[j & 3] + (j >> 2) * kAtom);
+      Ldm4T(d, at[(j + 1) & 3] + (j >> 2) * kAtom);
+      Mma(o[2 * j], hi[0], hi[1], hi[2], hi[3], b[0], b[1]);
+      Mma(o[2 * j + 1], hi[0], hi[1], hi[2], hi[3], b[2], b[3]);
+      Mma(o[2 * j + 2], hi[0], hi[1], hi[2], hi[3], d[0], d[1]);
+      Mma(o[2 * j + 3], hi[0], hi[1], hi[2], hi[3], d[2], d[3]);
+      Mma(o[2 * j], low[0], low[1], low[2], low[3], b[0], b[1]);
+      Mma(o[2 * j + 1], low[0], low[1], low[2], low[3], b[2], b[3]);
+      Mma(o[2 * j + 2], low[0], low[1], low[2], low[3], d[0], d[1]);
+      Mma(o[2 * j + 3], low[0], low[1], low[2], low[3], d[2], d[3]);
     }
     __syncwarp();  // the stage is read before it is filled again
-    if (++stage == kStages) stage = 0;
+    if (i + stages < steps) {
+      if (lane == 0) load(next_row, stage);
+      next_row = pool_row(i + stages + 1);
+    }
+    if (++stage == stages) {
+      stage = 0;
+      phase ^= 1;
+    }
   }
-  asm volatile("cp.async.wait_group 0;\n" ::: "memory");
+  if (!ok) {
+    // Given up: let the copies in flight land before the CTA's shared memory goes away.
+    if (lane == 0) {
+      volatile uint32_t never = 0;
+      for (int s = 0; s < stages; ++s)
+        if (steps > s) MbarWait(bar + 8 * s, ((steps - 1 - s) / stages) & 1, &never);
+      atomicExch(&g_grouped_status, 1);
+    }
+    __syncwarp();
+  }
 #pragma unroll
   for (int r = 0; r < 2; ++r) {
     sum[r] += __shfl_xor_sync(0xffffffffu, sum[r], 1);
@@ -289,7 +367,7 @@ __global__ void __launch_bounds__(kWarps * 32) GroupedAttentionMma(const __grid_
     }
 #pragma unroll
     for (int i = 0; i < 2 * NV; ++i) {
-      if (i < 2 * nv) {
+      if (i * 8 < a.vdim) {
         float* d = acc + static_cast<size_t>(warp * 16 + row) * acc_ld + i * 8 + (lane & 3) * 2;
         d[0] = o[i][2 * r];
         d[1] = o[i][2 * r + 1];
@@ -392,16 +470,34 @@ __global__ void __launch_bounds__(kGenericThreads) GroupedAttentionGeneric(const
   }
 }
 
-size_t MmaSmem(int maps, int dim, int vdim)
+// Stages of a warp's ring that fit beside the alignment slack; 0: none.
+int Stages(int maps, int dim, int vdim, size_t* smem)
 {
-  const size_t ring = static_cast<size_t>(kWarps) * kStages * kGroup * (maps * dim * 2 + 16 + vdim * 2 + 16);
+  const size_t stage = static_cast<size_t>(maps * ((dim + 63) / 64) + (vdim + 63) / 64) * kAtom;
   const size_t merge = sizeof(float) * (kWarps * 32 + static_cast<size_t>(kWarps) * 16 * (vdim + 4));
-  return ring > merge ? ring : merge;
+  int n = stage <= 8192 ? 3 : kMaxStages;  // small stages: two CTAs per SM
+  while (n > 0 && kWarps * n * stage + 1024 > kMaxSmem - 1024) --n;
+  if (smem != nullptr) *smem = (kWarps * n * stage > merge ? kWarps * n * stage : merge) + 1024;
+  return n;
 }
-bool MmaApplies(int maps, int dim, int vdim, int dtype)
+bool MmaApplies(int maps, int dim, int vdim, int block_size, int dtype)
 {
-  return dtype == TLALOC_B200_BF16 && (maps == 1 || maps == 2) && dim % 16 == 0 && vdim % 16 == 0 && dim <= 128 && vdim <= 256 &&
-         MmaSmem(maps, dim, vdim) <= kMaxSmem && !OrderFaithful();
+  return dtype == TLALOC_B200_BF16 && (maps == 1 || maps == 2) && dim % 16 == 0 && vdim % 16 == 0 && dim <= 128 && vdim <= 256 && block_size % kGroup == 0 &&
+         Stages(maps, dim, vdim, nullptr) >= 2 && !OrderFaithful() && TensorMapEncoder() != nullptr;
+}
+using EncodeTiledFn = CUresult (*)(CUtensorMap*, CUtensorMapDataType, cuuint32_t, void*, const cuuint64_t*, const cuuint64_t*,
+                                   const cuuint32_t*, const cuuint32_t*, CUtensorMapInterleave, CUtensorMapSwizzle,
+                                   CUtensorMapL2promotion, CUtensorMapFloatOOBfill);
+// The pool as rows of pool_ld channels, boxes of 64 channels x 16 rows.
+bool EncodePool(CUtensorMap* map, const void* pool, int64_t pool_ld, int64_t rows)
+{
+  auto encode = reinterpret_cast<EncodeTiledFn>(TensorMapEncoder());
+  const cuuint64_t dims[2] = {static_cast<cuuint64_t>(pool_ld), static_cast<cuuint64_t>(rows)};
+  const cuuint64_t strides[1] = {static_cast<cuuint64_t>(pool_ld) * 2};
+  const cuuint32_t box[2] = {64, kGroup}, elem[2] = {1, 1};
+  return encode != nullptr &&
+         encode(map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, const_cast<void*>(pool), dims, strides, box, elem, CU_TENSOR_MAP_INTERLEAVE_NONE,
+                CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE) == CUDA_SUCCESS;
 }
 int QueryTiles(int heads, int v_heads, int maps)
 {
@@ -409,21 +505,33 @@ int QueryTiles(int heads, int v_heads, int maps)
   return (per_map + rows - 1) / rows;
 }
 
-#define TLALOC_GROUPED_SIZES(F) F(4, 4) F(4, 8) F(4, 16) F(8, 4) F(8, 8) F(8, 16)
+// (channels of a key head, of a value head) / 16, in whole atoms
+#define TLALOC_GROUPED_SIZES(F) F(4, 4) F(4, 8) F(4, 12) F(4, 16) F(8, 4) F(8, 8) F(8, 12) F(8, 16)
 
 cudaError_t PrepareGrouped()
 {
   static OncePerDevice once;
   return once.Run([](int) {
+    TensorMapEncoder();
     cudaError_t e = cudaSuccess;
 #define TLALOC_OPT_IN(DK, NV) \
-  if (e == cudaSuccess) e = cudaFuncSetAttribute(GroupedAttentionMma<DK, NV>, cudaFuncAttributeMaxDynamicSharedMemorySize, kMaxSmem);
+  if (e == cudaSuccess) e = cudaFuncSetAttribute(GroupedAttentionMma<DK, NV>, cudaFuncAttributeMaxDynamicSharedMemorySize, kMaxSmem - 1024);
     TLALOC_GROUPED_SIZES(TLALOC_OPT_IN)
 #undef TLALOC_OPT_IN
     return e;
   });
 }
-KernelSetup g_setup(PrepareGrouped, nullptr);
+int ReadGroupedStatus()
+{
+  int v = 0;
+  if (cudaMemcpyFromSymbol(&v, g_grouped_status, sizeof(int)) != cudaSuccess) return -1;
+  if (v != 0) {
+    const int zero = 0;
+    cudaMemcpyToSymbol(g_grouped_status, &zero, sizeof(int));
+  }
+  return v;
+}
+KernelSetup g_setup(PrepareGrouped, ReadGroupedStatus);
 
 }  // namespace
 }  // namespace tlaloc_b200
@@ -431,12 +539,12 @@ KernelSetup g_setup(PrepareGrouped, nullptr);
 using namespace tlaloc_b200;
 
 extern "C" int tlaloc_b200_grouped_attention_slices(int32_t num_tokens, int32_t num_heads, int32_t v_heads, int32_t maps, int32_t dim, int32_t vdim,
-                                                    int32_t dtype, int32_t max_live)
+                                                    int32_t block_size, int32_t dtype, int32_t max_live)
 {
-  if (num_tokens < 1 || v_heads < 1 || maps < 1 || num_heads < 1 || !MmaApplies(maps, dim, vdim, dtype)) return 1;
+  if (num_tokens < 1 || v_heads < 1 || maps < 1 || num_heads < 1 || block_size < 1 || !MmaApplies(maps, dim, vdim, block_size, dtype)) return 1;
   // Enough CTAs for several waves, but no slice under 256 positions: each warp should have a few groups.
   const long long ctas = static_cast<long long>(num_tokens) * v_heads * QueryTiles(num_heads, v_heads, maps);
-  long long s = (2048 + ctas - 1) / ctas;
+  long long s = (768 + ctas - 1) / ctas;
   const long long most = (max_live + 255) / 256;
   if (s > most) s = most;
   return s < 1 ? 1 : s > 512 ? 512 : static_cast<int>(s);
@@ -485,17 +593,22 @@ extern "C" int tlaloc_b200_grouped_attention(const void* q, const void* pool, in
   a.scale_log2 = scale * 1.4426950408889634f;
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   cudaError_t e;
-  if (MmaApplies(maps, dim, vdim, dtype)) {
+  if (MmaApplies(maps, dim, vdim, block_size, dtype)) {
     if (pool_ld % 8 || v_first % 8 || !Aligned16(q) || !Aligned16(pool)) return Fail(kInvalid, "%s: addresses and strides must be multiples of 16 bytes", op);
     if (static_cast<long long>(v_heads) * a.qtiles > 65535) return Fail(kInvalid, "%s: too many heads", op);
     e = PrepareGrouped();
     if (e != cudaSuccess) return CudaFail("GROUPED_ATTENTION set-up", e);
+    CUtensorMap map;
+    if (static_cast<int64_t>(num_blocks) * block_size > INT32_MAX || !EncodePool(&map, pool, pool_ld, static_cast<int64_t>(num_blocks) * block_size)) {
+      return Fail(kInternal, "%s: the tensor map could not be encoded", op);
+    }
+    size_t smem = 0;
+    a.stages = Stages(maps, dim, vdim, &smem);
     const dim3 grid(slices, v_heads * a.qtiles, num_tokens);
-    const size_t smem = MmaSmem(maps, dim, vdim);
-    const int dk = dim <= 64 ? 4 : 8, nv = vdim <= 64 ? 4 : vdim <= 128 ? 8 : 16;
+    const int dk = (dim + 63) / 64 * 4, nv = (vdim + 63) / 64 * 4;
     e = cudaErrorInvalidValue;
 #define TLALOC_LAUNCH(DK, NV) \
-  if (dk == DK && nv == NV) e = LaunchChained(GroupedAttentionMma<DK, NV>, grid, kWarps * 32, smem, st, a);
+  if (dk == DK && nv == NV) e = LaunchChained(GroupedAttentionMma<DK, NV>, grid, kWarps * 32, smem, st, map, a);
     TLALOC_GROUPED_SIZES(TLALOC_LAUNCH)
 #undef TLALOC_LAUNCH
   } else {

@@ -278,7 +278,7 @@ class MixedDecoder(RaggedModel):
         return self.max_positions if m.window is None else min(self.max_positions, m.window + m.keep_first)
 
     def _slices(self, m: DifferentialAttention, rows: int) -> int:
-        return ops.grouped_attention_slices(rows, m.heads * 2, m.kv_heads, 2, m.kdim, m.vpad, self.dtype, self._max_live(m))
+        return ops.grouped_attention_slices(rows, m.heads * 2, m.kv_heads, 2, m.kdim, m.vpad, self.block_size, self.dtype, self._max_live(m))
 
     def _map_values(self, m: DifferentialAttention, rows: int) -> int:
         """f32 values of the most records a step of up to `rows` rows leaves (few rows have several slices each)."""

@@ -449,8 +449,8 @@ def rotate_rows(rows, parts, positions, cos, sin, *, rot_dims, slots=None, num_s
                                             _ptr(positions), _ptr(cos), _ptr(sin), _ptr(slots), T, rot_dims, num_slots, max(cos.shape[0], 1), _stream(rows)))
 
 
-def grouped_attention_slices(rows, heads, v_heads, maps, dim, vdim, dtype, max_live) -> int:
-    return int(N.lib().tlaloc_b200_grouped_attention_slices(rows, heads, v_heads, maps, dim, vdim, _DT[dtype], max_live))
+def grouped_attention_slices(rows, heads, v_heads, maps, dim, vdim, block_size, dtype, max_live) -> int:
+    return int(N.lib().tlaloc_b200_grouped_attention_slices(rows, heads, v_heads, maps, dim, vdim, block_size, _DT[dtype], max_live))
 
 
 def grouped_attention(q, pool, block_tables, seq_lens, records, *, v_heads, maps, vdim, v_first, scale, slices, window=0, keep_first=0,
