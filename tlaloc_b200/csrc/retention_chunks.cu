@@ -1,44 +1,51 @@
-// Retention over a prompt portion on the tensor cores, bf16 operands (include/tlaloc_b200.h, tlaloc_b200_retention_chunks).
+// Retention over a prompt portion on the tensor cores (include/tlaloc_b200.h, tlaloc_b200_retention_chunks): bf16 operands by TMA,
+// tcgen05.mma kind::f16 with f32 accumulators in TMEM.
 //
-// The portion is cut into chunks of 64 tokens and, for parallelism, into segments of whole chunks.  Within a chunk, with S the state ahead
+// The portion is cut into chunks of 128 tokens and, for parallelism, into segments of whole chunks.  Within a chunk, with S the state ahead
 // of it and w = decay:
 //   o_i = w^(i+1) S^T q_i + sum_{j <= i} w^(i-j) (q_i . k_j) v_j        S <- w^n S + sum_j w^(n-1-j) k_j v_j^T
-// A CTA has one head, a slice of its value columns and one segment; S stays in its registers as f32 accumulators of the transposed product
-// (value columns as the rows of mma.m16n8k16, so that an accumulator is also the operand layout of S^T q).  What was computed in f32 and
-// enters a product as an operand (S, the decayed scores, the decayed values) enters as two bf16 parts, which is f32 up to rounding.
+// A CTA has one head, 64 value columns and one segment; S stays in TMEM (rows: the key's channels, 128 at a time).  What was computed in f32
+// and enters a product as an operand (S, the decayed scores, the decayed values) enters as two bf16 parts, which is f32 up to rounding.
+//   producer lane   Q, K and V of the next chunk
+//   MMA lane        scores Q K^T; O = Q S; O = P V (its first part is in registers by then); S += K^T V'
+//   eight warps     S as an operand (shared memory) and decayed; scores times decay, in their place in TMEM as the A operand P; the
+//                   decayed values V' (in the place of Q); the output rows
 // Two launches where there are several segments: the first computes what each segment adds to the state, the second starts every
-// segment from the sum of those before it, writes the outputs and, in the last segment, the new state.
+// segment from the sum of those before it, writes the outputs and, in the last segment, the new state.  Every mbarrier wait is bounded.
+#include <cuda.h>
+
 #include "common.cuh"
+#include "tc_common.cuh"
 
 namespace tlaloc_b200 {
 namespace {
 
-constexpr int kChunk = 64, kWarps = 4, kThreads = kWarps * 32;
+using namespace tc;
+
+constexpr int kChunk = 128, kVS = 64;
+constexpr int kAtom = kChunk * 128;  // 128 tokens x 64 channels
+constexpr int kWorkers = 8, kWorkerThreads = kWorkers * 32, kThreads = kWorkerThreads + 64;
 constexpr int kMaxSmem = 227 * 1024;
 
 struct ChunkArgs {
-  const __nv_bfloat16 *q, *k, *v;
   const int *positions, *row_states;
   const float* decay;
   float *state, *o, *sums;  // sums [segments][heads][slices][..]: what a segment adds; the last one's place holds the state before the portion
-  int tokens, heads, dim, vdim, dim_ld, v_ld, num_slots, segment, segments;
+  int tokens, heads, dim, vdim, dp, num_slots, segment, segments;
 };
 
-__device__ __forceinline__ void Mma(float* c, const uint32_t* a, uint32_t b0, uint32_t b1)
+__device__ int g_retention_status = 0;
+
+// f32 accumulator, bf16 operands, M = 128.
+__host__ __device__ constexpr uint32_t InstrDesc(int n, bool a_mn, bool b_mn)
 {
-  asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};\n"
-               : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
-               : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
+  return (1u << 4) | (1u << 7) | (1u << 10) | (a_mn ? 1u << 15 : 0u) | (b_mn ? 1u << 16 : 0u) | (static_cast<uint32_t>(n >> 3) << 17) | (8u << 24);
 }
-__device__ __forceinline__ void Ldm4(uint32_t* r, uint32_t addr)
+// x is a multiple of 64 channels: a 16-byte boundary.
+__device__ __forceinline__ void TmaBox(uint32_t dst, const CUtensorMap* map, int x, int y, int z, uint32_t bar)
 {
-  asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];\n" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr) : "memory");
-}
-__device__ __forceinline__ void Ldm4T(uint32_t* r, uint32_t addr)
-{
-  asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];\n"
-               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3])
-               : "r"(addr)
+  asm volatile("cp.async.bulk.tensor.3d.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1, {%2, %3, %4}], [%5];\n" ::"r"(dst),
+               "l"(reinterpret_cast<uint64_t>(map)), "r"(x), "r"(y), "r"(z), "r"(bar)
                : "memory");
 }
 __device__ __forceinline__ void Split(float a, float b, uint32_t& hi, uint32_t& lo)
@@ -50,299 +57,448 @@ __device__ __forceinline__ void Split(float a, float b, uint32_t& hi, uint32_t& 
 }
 __device__ __forceinline__ float Low(uint32_t u) { return __uint_as_float(u << 16); }
 __device__ __forceinline__ float High(uint32_t u) { return __uint_as_float(u & 0xffff0000u); }
-
-// DK: 16-channel steps of a key at most; VS: value columns of a slice.  The warps share S as VS / 16 groups of value columns by
-// 64 / VS parts of the channels.
-template <int DK, int VS, bool OUT>
-__global__ void __launch_bounds__(kThreads) RetentionChunkKernel(const __grid_constant__ ChunkArgs a)
+__device__ __forceinline__ void StoreShared16(uint32_t at, const uint32_t* v)
 {
-  GridDependencySync();
-  constexpr int kParts = 64 / VS, kTiles = 2 * DK / kParts;  // 8-channel tiles of S a warp holds
-  extern __shared__ __align__(16) unsigned char smem[];
+  asm volatile("st.shared.v4.b32 [%0], {%1, %2, %3, %4};\n" ::"r"(at), "r"(v[0]), "r"(v[1]), "r"(v[2]), "r"(v[3]) : "memory");
+}
+
+// Shared memory: Q | K | V | S (two parts) and, where Q is a single atom, the second part of V'; the first (two) atoms of Q hold V' when
+// Q has been used.
+struct Places {
+  uint32_t q, k, v, s_hi, s_lo, vd_hi, vd_lo;
+};
+__host__ __device__ inline uint32_t PlaceAll(int dp, uint32_t base, Places* p)
+{
+  const uint32_t atoms = (dp + 63) / 64;
+  p->q = base;
+  p->k = p->q + atoms * kAtom;
+  p->v = p->k + atoms * kAtom;
+  p->s_hi = p->v + kAtom;
+  p->s_lo = p->s_hi + dp * 128;
+  p->vd_hi = p->q;
+  uint32_t end = p->s_lo + dp * 128;
+  if (atoms >= 2) {
+    p->vd_lo = p->q + kAtom;
+  } else {
+    p->vd_lo = end;
+    end += kAtom;
+  }
+  return end - base;
+}
+
+// BLOCKS: 128-channel blocks of S.
+template <int BLOCKS, bool OUT>
+__global__ void __launch_bounds__(kThreads) RetentionChunkTc(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
+                                                             const __grid_constant__ CUtensorMap map_v, const __grid_constant__ ChunkArgs a)
+{
+  constexpr uint32_t kCols = BLOCKS == 1 ? 256u : 512u;  // scores 128, O 64, S 64 per block
+  extern __shared__ __align__(1024) unsigned char smem_raw[];
+  __shared__ alignas(8) uint64_t bars[8];
+  __shared__ uint32_t slot_store[2];
   __shared__ float pw[kChunk + 1];
+  const uint32_t base = SmemAddr(smem_raw);  // two CTAs of 128 channels fill an SM to the byte: no slack to align within
+  if ((base & 1023u) != 0u) {
+    if (threadIdx.x == 0) atomicExch(&g_retention_status, 1);
+    return;
+  }
+  Places at;
+  PlaceAll(a.dp, base, &at);
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+  const uint32_t full = SmemAddr(bars), sc_done = full + 8, s_ready = full + 16, o_done = full + 24, p_ready = full + 32, pv_done = full + 40, vd_ready = full + 48,
+                 st_done = full + 56;
+  volatile uint32_t* abort_word = slot_store + 1;
+  if (tid == 0) {
+    slot_store[1] = 0u;
+    MbarInit(full, 1);
+    MbarInit(sc_done, 1);
+    MbarInit(s_ready, kWorkers);
+    MbarInit(o_done, 1);
+    MbarInit(p_ready, kWorkers);
+    MbarInit(pv_done, 1);
+    MbarInit(vd_ready, kWorkers);
+    MbarInit(st_done, 1);
+    asm volatile("fence.mbarrier_init.release.cluster;\n" ::: "memory");
+  }
+  if (warp == 0) {
+    asm volatile("tcgen05.alloc.cta_group::1.sync.aligned.shared::cta.b32 [%0], %1;\n" ::"r"(SmemAddr(slot_store)), "r"(kCols) : "memory");
+    asm volatile("tcgen05.relinquish_alloc_permit.cta_group::1.sync.aligned;\n" ::: "memory");
+  }
+  asm volatile("tcgen05.fence::before_thread_sync;\n" ::: "memory");
+  __syncthreads();
+  asm volatile("tcgen05.fence::after_thread_sync;\n" ::: "memory");
+  const uint32_t tmem = *reinterpret_cast<volatile uint32_t*>(slot_store), t_p = tmem, t_o = tmem + 128, t_s = tmem + 192;
+  GridDependencySync();
+
   const int head = blockIdx.x, slice = blockIdx.y, seg = blockIdx.z, slices = gridDim.y;
-  const int dk = a.dim_ld >> 4, k_ld = a.dim_ld * 2 + 16, v_ld = VS * 2 + 16;
-  const uint32_t base = static_cast<uint32_t>(__cvta_generic_to_shared(smem));
-  const int q_bytes = OUT ? kChunk * k_ld : 0, k_bytes = kChunk * k_ld, buf_bytes = q_bytes + k_bytes + kChunk * v_ld;
-  const uint32_t s_hi = base + 2 * buf_bytes, s_lo = s_hi + VS * k_ld;
-  const float w = __ldg(a.decay + head);
-  for (int i = tid; i <= kChunk; i += kThreads) pw[i] = powf(w, static_cast<float>(i));
+  const int t_begin = seg * a.segment, t_end = min(a.tokens, t_begin + a.segment), chunks = (t_end - t_begin + kChunk - 1) / kChunk;
+  const bool last = seg + 1 == a.segments;
+  // Whether the state behind chunk c is wanted.
+  auto carries = [&](int c) { return !OUT || last || c + 1 < chunks; };
+  const int atoms = (a.dp + 63) / 64, steps = a.dp / 16;
+  bool ok = true;
 
-  const int t_begin = seg * a.segment, t_end = min(a.tokens, t_begin + a.segment);
-  auto load = [&](int t0, int buf) {
-    const uint32_t dst = base + buf * buf_bytes;
-    const int kc = a.dim_ld >> 3, rows = t_end - t0;
-    for (int i = tid; i < kChunk * kc; i += kThreads) {
-      const int r = i / kc, c = i - r * kc;
-      const size_t at = (static_cast<size_t>(t0 + min(r, rows - 1)) * a.heads + head) * a.dim_ld + c * 8;
-      const int bytes = r < rows ? 16 : 0;
-      if (OUT) asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;\n" ::"r"(dst + r * k_ld + c * 16), "l"(a.q + at), "r"(bytes) : "memory");
-      asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;\n" ::"r"(dst + q_bytes + r * k_ld + c * 16), "l"(a.k + at), "r"(bytes) : "memory");
+  if (warp == kWorkers) {
+    if (ElectOne()) {
+      for (int c = 0; c < chunks; ++c) {
+        // Everything of the chunk before has been used when its last product is done.
+        if (c > 0) ok = MbarWait(st_done, (c - 1) & 1, abort_word) && ok;
+        const int t0 = t_begin + c * kChunk;
+        MbarExpectTx(full, ((OUT ? 2 : 1) * atoms + 1) * kAtom);
+        if (OUT)
+          for (int x = 0; x < atoms; ++x) TmaBox(at.q + x * kAtom, &map_q, x * 64, head, t0, full);
+        for (int x = 0; x < atoms; ++x) TmaBox(at.k + x * kAtom, &map_k, x * 64, head, t0, full);
+        TmaBox(at.v, &map_v, slice * kVS, head, t0, full);
+      }
+      if (!ok) {  // given up: let the copies in flight land before the CTA's shared memory goes away
+        volatile uint32_t never = 0;
+        MbarWait(full, (chunks - 1) & 1, &never);
+      }
     }
-    for (int i = tid; i < kChunk * (VS / 8); i += kThreads) {
-      const int r = i / (VS / 8), c = i % (VS / 8), col = slice * VS + c * 8;
-      const size_t at = (static_cast<size_t>(t0 + min(r, rows - 1)) * a.heads + head) * a.v_ld + min(col, a.v_ld - 8);
-      const int bytes = r < rows && col < a.v_ld ? 16 : 0;
-      asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;\n" ::"r"(dst + q_bytes + k_bytes + r * v_ld + c * 16), "l"(a.v + at), "r"(bytes) : "memory");
-    }
-    asm volatile("cp.async.commit_group;\n" ::: "memory");
-  };
-  load(t_begin, 0);
-
-  // S: rows v0 + lane / 4 (+ 8), channels d0 + 8 n + 2 (lane % 4) (+ 1).
-  const int v0 = (warp / kParts) * 16, d0 = (warp % kParts) * (kTiles * 8);
-  float s[kTiles][4];
-  const int vp = (a.vdim + 3) & ~3;
-  const int slot = min(max(__ldg(a.row_states), 0), a.num_slots - 1);
-  float* state = a.state + (static_cast<size_t>(slot) * a.heads + head) * a.dim * vp;
-  const size_t frag = static_cast<size_t>(kTiles) * 4 * kThreads;
-  auto sums = [&](int g) { return a.sums + ((static_cast<size_t>(g) * a.heads + head) * slices + slice) * frag + tid; };
-#pragma unroll
-  for (int n = 0; n < kTiles; ++n) s[n][0] = s[n][1] = s[n][2] = s[n][3] = 0.f;
-  if (seg == 0 && !(OUT && a.segments > 1)) {
-    if (__ldg(a.positions) != 0) {
-#pragma unroll
-      for (int n = 0; n < kTiles; ++n)
-#pragma unroll
-        for (int e = 0; e < 4; ++e) {
-          const int d = d0 + n * 8 + (lane & 3) * 2 + (e & 1), v = slice * VS + v0 + (lane >> 2) + (e >> 1) * 8;
-          if (d < a.dim && v < vp) s[n][e] = state[static_cast<size_t>(d) * vp + v];
+    __syncwarp();
+  } else if (warp == kWorkers + 1) {
+    if (ElectOne()) {
+      constexpr uint32_t scores_desc = InstrDesc(kChunk, false, false), out_desc = InstrDesc(kVS, false, true), state_desc = InstrDesc(kVS, true, true);
+      const uint64_t qd = SmemDesc(at.q, 16, 1024), kd = SmemDesc(at.k, 16, 1024), kt = SmemDesc(at.k, kAtom, 1024), vd = SmemDesc(at.v, kAtom, 1024);
+      const uint64_t sh = SmemDesc(at.s_hi, kAtom, 1024), sl = SmemDesc(at.s_lo, kAtom, 1024);
+      const uint64_t dh = SmemDesc(at.vd_hi, kAtom, 1024), dl = SmemDesc(at.vd_lo, kAtom, 1024);
+      constexpr uint64_t kRows = (16 * 128) >> 4;  // sixteen rows of a tile further
+      for (int c = 0; c < chunks; ++c) {
+        const uint32_t par = c & 1;
+        ok = MbarWait(full, par, abort_word) && ok;
+        asm volatile("tcgen05.fence::after_thread_sync;\n" ::: "memory");
+        if (OUT) {
+          for (int k = 0; k < steps; ++k) {
+            const uint64_t off = static_cast<uint64_t>((k >> 2) * (kAtom >> 4) + 2 * (k & 3));
+            TcMmaBf16(t_p, qd + off, kd + off, scores_desc, k > 0 ? 1u : 0u);
+          }
+          TcCommit(sc_done);
+          ok = MbarWait(s_ready, par, abort_word) && ok;
+          asm volatile("tcgen05.fence::after_thread_sync;\n" ::: "memory");
+          for (int k = 0; k < steps; ++k) {
+            const uint64_t off = static_cast<uint64_t>((k >> 2) * (kAtom >> 4) + 2 * (k & 3));
+            TcMmaBf16(t_o, qd + off, sh + k * kRows, out_desc, k > 0 ? 1u : 0u);
+            TcMmaBf16(t_o, qd + off, sl + k * kRows, out_desc, 1u);
+          }
+          TcCommit(o_done);
+          ok = MbarWait(p_ready, par, abort_word) && ok;
+          asm volatile("tcgen05.fence::after_thread_sync;\n" ::: "memory");
+          for (int k = 0; k < kChunk / 16; ++k) {
+            TcMmaTmemA(t_o, t_p + 8 * k, vd + k * kRows, out_desc, k > 0 ? 1u : 0u);
+            TcMmaTmemA(t_o, t_p + 64 + 8 * k, vd + k * kRows, out_desc, 1u);
+          }
+          TcCommit(pv_done);
         }
-    }
-    if (!OUT) {
-      float* p = sums(a.segments - 1);
+        if (carries(c)) {
+          ok = MbarWait(vd_ready, par, abort_word) && ok;
+          asm volatile("tcgen05.fence::after_thread_sync;\n" ::: "memory");
 #pragma unroll
-      for (int n = 0; n < kTiles; ++n)
-#pragma unroll
-        for (int e = 0; e < 4; ++e) p[(n * 4 + e) * kThreads] = s[n][e];
+          for (int b = 0; b < BLOCKS; ++b) {
+            const uint64_t kb = kt + static_cast<uint64_t>(b * 2 * (kAtom >> 4));
+            for (int k = 0; k < kChunk / 16; ++k) {
+              TcMmaBf16(t_s + b * 64, kb + k * kRows, dh + k * kRows, state_desc, 1u);
+              TcMmaBf16(t_s + b * 64, kb + k * kRows, dl + k * kRows, state_desc, 1u);
+            }
+          }
+          TcCommit(st_done);
+        }
+      }
     }
-  } else if (OUT) {
+    __syncwarp();
+  } else {
+    const int quad = warp & 3, half = warp >> 2, row = quad * 32 + lane;  // TMEM lane; columns [32 half, 32 half + 32) of O and S
+    const uint32_t lanes = static_cast<uint32_t>(quad * 32) << 16;
+    const float w = __ldg(a.decay + head);
+    for (int i = tid; i <= kChunk; i += kWorkerThreads) pw[i] = powf(w, static_cast<float>(i));
+    asm volatile("bar.sync 5, 256;\n" ::: "memory");
+
+    // The state ahead of the segment.
+    const int vp = (a.vdim + 3) & ~3, v0 = slice * kVS + half * 32;
+    const int slot = min(max(__ldg(a.row_states), 0), a.num_slots - 1);
+    float* state = a.state + (static_cast<size_t>(slot) * a.heads + head) * a.dim * vp;
+    auto sums = [&](int g) {
+      return a.sums + ((static_cast<size_t>(g) * a.heads + head) * slices + slice) * (static_cast<size_t>(BLOCKS) * 32 * kWorkerThreads) + tid;
+    };
+    const bool own = seg == 0 && !(OUT && a.segments > 1);
+    const bool fresh = __ldg(a.positions) == 0;
     const float ws = powf(w, static_cast<float>(a.segment));
-    for (int g = seg == 0 ? a.segments - 1 : 0; g < (seg == 0 ? a.segments : seg); ++g) {
-      const float* p = sums(g);
-#pragma unroll
-      for (int n = 0; n < kTiles; ++n)
-#pragma unroll
-        for (int e = 0; e < 4; ++e) s[n][e] = fmaf(ws, s[n][e], p[(n * 4 + e) * kThreads]);
-    }
-  }
-
-  int buf = 0;
-  for (int t0 = t_begin; t0 < t_end; t0 += kChunk, buf ^= 1) {
-    const int count = min(kChunk, t_end - t0);
-    const uint32_t qt = base + buf * buf_bytes, kt = qt + q_bytes, vt = kt + k_bytes;
-    if (OUT) {  // the state ahead of the chunk, for all warps
-#pragma unroll
-      for (int n = 0; n < kTiles; ++n) {
-        if (d0 + n * 8 < a.dim_ld) {
-#pragma unroll
-          for (int r = 0; r < 2; ++r) {
-            uint32_t hi, lo;
-            Split(s[n][2 * r], s[n][2 * r + 1], hi, lo);
-            const uint32_t at = (v0 + (lane >> 2) + 8 * r) * k_ld + (d0 + n * 8 + (lane & 3) * 2) * 2;
-            asm volatile("st.shared.b32 [%0], %1;\n" ::"r"(s_hi + at), "r"(hi) : "memory");
-            asm volatile("st.shared.b32 [%0], %1;\n" ::"r"(s_lo + at), "r"(lo) : "memory");
-          }
-        }
-      }
-    }
-    asm volatile("cp.async.wait_group 0;\n" ::: "memory");
-    __syncthreads();
-    if (t0 + kChunk < t_end) load(t0 + kChunk, buf ^ 1);  // its last readers are behind the barrier at the end of the chunk before
-
-    const int m = lane >> 3, r8 = lane & 7;
-    if (OUT) {
-      const int i0 = warp * 16 + (lane >> 2);
-      uint32_t qa[DK][4];
-#pragma unroll
-      for (int k = 0; k < DK; ++k)
-        if (k < dk) Ldm4(qa[k], qt + (warp * 16 + (m & 1) * 8 + r8) * k_ld + k * 32 + (m >> 1) * 16);
-      float o[VS / 8][4];
-#pragma unroll
-      for (int n = 0; n < VS / 8; ++n) o[n][0] = o[n][1] = o[n][2] = o[n][3] = 0.f;
-#pragma unroll
-      for (int k = 0; k < DK; ++k) {
-        if (k < dk) {
-#pragma unroll
-          for (int n = 0; n < VS / 16; ++n) {
-            uint32_t b[4];
-            const uint32_t at = (n * 16 + (m >> 1) * 8 + r8) * k_ld + k * 32 + (m & 1) * 16;
-            Ldm4(b, s_hi + at);
-            Mma(o[2 * n], qa[k], b[0], b[1]);
-            Mma(o[2 * n + 1], qa[k], b[2], b[3]);
-            Ldm4(b, s_lo + at);
-            Mma(o[2 * n], qa[k], b[0], b[1]);
-            Mma(o[2 * n + 1], qa[k], b[2], b[3]);
-          }
-        }
-      }
-      const float w0 = pw[i0 + 1], w1 = pw[i0 + 9];
-#pragma unroll
-      for (int n = 0; n < VS / 8; ++n) {
-        o[n][0] *= w0;
-        o[n][1] *= w0;
-        o[n][2] *= w1;
-        o[n][3] *= w1;
-      }
+    const int g_lo = seg == 0 ? a.segments - 1 : 0, g_hi = seg == 0 ? a.segments : seg;
 #pragma unroll 1
-      for (int j = 0; j <= warp; ++j) {  // 16 keys at a time, none past the queries
-        float c[2][4] = {};
+    for (int b = 0; b < BLOCKS; ++b) {
+      const int d = b * 128 + row;
+      float s[32];
 #pragma unroll
-        for (int k = 0; k < DK; ++k) {
-          if (k < dk) {
-            uint32_t b[4];
-            Ldm4(b, kt + (j * 16 + (m >> 1) * 8 + r8) * k_ld + k * 32 + (m & 1) * 16);
-            Mma(c[0], qa[k], b[0], b[1]);
-            Mma(c[1], qa[k], b[2], b[3]);
+      for (int e = 0; e < 32; ++e) s[e] = 0.f;
+      if (own) {
+        if (!fresh && d < a.dim) {
+          const float* p = state + static_cast<size_t>(d) * vp + v0;
+#pragma unroll
+          for (int e = 0; e < 32; e += 4) {
+            if (v0 + e < vp) {
+              const float4 x = *reinterpret_cast<const float4*>(p + e);
+              s[e] = x.x; s[e + 1] = x.y; s[e + 2] = x.z; s[e + 3] = x.w;
+            }
           }
         }
+        if (!OUT) {
+          float* p = sums(a.segments - 1) + b * 32 * kWorkerThreads;
 #pragma unroll
-        for (int n = 0; n < 2; ++n)
+          for (int e = 0; e < 32; ++e) p[e * kWorkerThreads] = s[e];
+        }
+      } else if (OUT) {
+        for (int g = g_lo; g < g_hi; ++g) {
+          const float* p = sums(g) + b * 32 * kWorkerThreads;
 #pragma unroll
-          for (int e = 0; e < 4; ++e) {
-            const int back = i0 + (e >> 1) * 8 - (j * 16 + n * 8 + (lane & 3) * 2 + (e & 1));
-            c[n][e] = back >= 0 ? c[n][e] * pw[max(back, 0)] : 0.f;
-          }
-        uint32_t hi[4], lo[4];
-        Split(c[0][0], c[0][1], hi[0], lo[0]);
-        Split(c[0][2], c[0][3], hi[1], lo[1]);
-        Split(c[1][0], c[1][1], hi[2], lo[2]);
-        Split(c[1][2], c[1][3], hi[3], lo[3]);
-#pragma unroll
-        for (int n = 0; n < VS / 16; ++n) {
-          uint32_t b[4];
-          Ldm4T(b, vt + (j * 16 + (m & 1) * 8 + r8) * v_ld + n * 32 + (m >> 1) * 16);
-          Mma(o[2 * n], hi, b[0], b[1]);
-          Mma(o[2 * n + 1], hi, b[2], b[3]);
-          Mma(o[2 * n], lo, b[0], b[1]);
-          Mma(o[2 * n + 1], lo, b[2], b[3]);
+          for (int e = 0; e < 32; ++e) s[e] = fmaf(ws, s[e], p[e * kWorkerThreads]);
         }
       }
-      float* out = a.o + (static_cast<size_t>(t0) * a.heads + head) * a.vdim;
-      const bool pairs = a.vdim % 2 == 0;
-#pragma unroll
-      for (int n = 0; n < VS / 8; ++n)
-#pragma unroll
-        for (int r = 0; r < 2; ++r) {
-          const int i = i0 + 8 * r, col = slice * VS + n * 8 + (lane & 3) * 2;
-          float* p = out + static_cast<size_t>(i) * a.heads * a.vdim + col;
-          if (i < count && col + 1 < a.vdim && pairs) {
-            *reinterpret_cast<float2*>(p) = make_float2(o[n][2 * r], o[n][2 * r + 1]);
-          } else if (i < count) {
-            if (col < a.vdim) p[0] = o[n][2 * r];
-            if (col + 1 < a.vdim) p[1] = o[n][2 * r + 1];
-          }
-        }
+      TcSt32(t_s + lanes + b * 64 + half * 32, reinterpret_cast<const uint32_t*>(s));
     }
+    asm volatile("tcgen05.wait::st.sync.aligned;\n" ::: "memory");
 
-    // the state behind the chunk
-    if (!OUT || seg + 1 == a.segments || t0 + kChunk < t_end) {
-      const float wn = pw[count];
-#pragma unroll
-      for (int n = 0; n < kTiles; ++n) {
-        s[n][0] *= wn;
-        s[n][1] *= wn;
-        s[n][2] *= wn;
-        s[n][3] *= wn;
+    for (int c = 0; c < chunks; ++c) {
+      const uint32_t par = c & 1;
+      const int t0 = t_begin + c * kChunk, n = min(kChunk, t_end - t0);
+      // S as an operand, and decayed for what the chunk adds.
+      if (c > 0) {
+        ok = MbarWaitWarp(st_done, (c - 1) & 1, lane, abort_word) && ok;
+        asm volatile("tcgen05.fence::after_thread_sync;\n" ::: "memory");
       }
+      const float wn = pw[n];
 #pragma unroll 1
-      for (int j = 0; j < kChunk / 16; ++j) {
-        uint32_t va[4], hi[4], lo[4];
-        Ldm4T(va, vt + (j * 16 + (m >> 1) * 8 + r8) * v_ld + (v0 + (m & 1) * 8) * 2);
+      for (int b = 0; b < BLOCKS; ++b) {
+        const int d = b * 128 + row;
+        if (b * 128 + quad * 32 >= a.dp) break;  // nothing but padding in this warp's rows
+        uint32_t s[32];
+        TcLd32(t_s + lanes + b * 64 + half * 32, s);
+        asm volatile("tcgen05.wait::ld.sync.aligned;\n" ::: "memory");
+        if (OUT && d < a.dp) {
 #pragma unroll
-        for (int h = 0; h < 2; ++h) {
-          const int tok = count - 1 - (j * 16 + h * 8 + (lane & 3) * 2);
-          const float wa = tok >= 0 ? pw[max(tok, 0)] : 0.f, wb = tok >= 1 ? pw[max(tok - 1, 0)] : 0.f;
-          Split(Low(va[2 * h]) * wa, High(va[2 * h]) * wb, hi[2 * h], lo[2 * h]);
-          Split(Low(va[2 * h + 1]) * wa, High(va[2 * h + 1]) * wb, hi[2 * h + 1], lo[2 * h + 1]);
+          for (int i = 0; i < 4; ++i) {
+            uint32_t hi[4], lo[4];
+#pragma unroll
+            for (int e = 0; e < 4; ++e) Split(__uint_as_float(s[8 * i + 2 * e]), __uint_as_float(s[8 * i + 2 * e + 1]), hi[e], lo[e]);
+            const uint32_t off = d * 128 + (((half * 4 + i) ^ (d & 7)) << 4);
+            StoreShared16(at.s_hi + off, hi);
+            StoreShared16(at.s_lo + off, lo);
+          }
         }
 #pragma unroll
-        for (int n = 0; n < kTiles / 2; ++n) {
-          if (d0 + n * 16 < a.dim_ld) {
-            uint32_t b[4];
-            Ldm4T(b, kt + (j * 16 + (m & 1) * 8 + r8) * k_ld + (d0 + n * 16 + (m >> 1) * 8) * 2);
-            Mma(s[2 * n], hi, b[0], b[1]);
-            Mma(s[2 * n + 1], hi, b[2], b[3]);
-            Mma(s[2 * n], lo, b[0], b[1]);
-            Mma(s[2 * n + 1], lo, b[2], b[3]);
+        for (int e = 0; e < 32; ++e) s[e] = __float_as_uint(__uint_as_float(s[e]) * wn);
+        TcSt32(t_s + lanes + b * 64 + half * 32, s);
+      }
+      asm volatile("tcgen05.wait::st.sync.aligned;\n" ::: "memory");
+      float o[32];
+      if (OUT) {
+        asm volatile("fence.proxy.async.shared::cta;\n" ::: "memory");
+        asm volatile("tcgen05.fence::before_thread_sync;\n" ::: "memory");
+        __syncwarp();
+        if (lane == 0) MbarArrive(s_ready);
+
+        // Scores times decay: columns [64 half, 64 half + 64), 32 at a time; the parts go to columns 32 half and 64 + 32 half.
+        ok = MbarWaitWarp(sc_done, par, lane, abort_word) && ok;
+        asm volatile("tcgen05.fence::after_thread_sync;\n" ::: "memory");
+        uint32_t hi[32], lo[32];
+#pragma unroll
+        for (int g = 0; g < 2; ++g) {
+          const int j0 = half * 64 + g * 32;
+          if (j0 > quad * 32 + 31) {  // all of it in the future
+#pragma unroll
+            for (int e = 0; e < 16; ++e) hi[g * 16 + e] = lo[g * 16 + e] = 0u;
+          } else {
+            uint32_t s[32];
+            TcLd32(t_p + lanes + j0, s);
+            asm volatile("tcgen05.wait::ld.sync.aligned;\n" ::: "memory");
+#pragma unroll
+            for (int e = 0; e < 32; e += 2) {
+              const int back = row - j0 - e;
+              const float x = back >= 0 ? __uint_as_float(s[e]) * pw[max(back, 0)] : 0.f;
+              const float y = back >= 1 ? __uint_as_float(s[e + 1]) * pw[max(back - 1, 0)] : 0.f;
+              Split(x, y, hi[g * 16 + e / 2], lo[g * 16 + e / 2]);
+            }
+          }
+        }
+        asm volatile("bar.sync %0, 64;\n" ::"r"(1 + quad) : "memory");  // both warps of the quad have their scores
+        TcSt32(t_p + lanes + half * 32, hi);
+        TcSt32(t_p + lanes + 64 + half * 32, lo);
+        asm volatile("tcgen05.wait::st.sync.aligned;\n" ::: "memory");
+        ok = MbarWaitWarp(o_done, par, lane, abort_word) && ok;
+        asm volatile("tcgen05.fence::after_thread_sync;\n" ::: "memory");
+        TcLd32(t_o + lanes + half * 32, reinterpret_cast<uint32_t*>(o));
+        asm volatile("tcgen05.wait::ld.sync.aligned;\n" ::: "memory");
+        asm volatile("tcgen05.fence::before_thread_sync;\n" ::: "memory");
+        __syncwarp();
+        if (lane == 0) MbarArrive(p_ready);
+        const float wi = pw[row + 1];
+#pragma unroll
+        for (int e = 0; e < 32; ++e) o[e] *= wi;
+      }
+
+      // Decayed values, in the place of Q (its products are done).
+      if (carries(c)) {
+        ok = MbarWaitWarp(full, par, lane, abort_word) && ok;
+#pragma unroll
+        for (int i = 0; i < kAtom / 16 / kWorkerThreads; ++i) {
+          const int idx = i * kWorkerThreads + tid, j = idx >> 3;
+          uint32_t v[4], hi[4], lo[4];
+          asm volatile("ld.shared.v4.b32 {%0, %1, %2, %3}, [%4];\n" : "=r"(v[0]), "=r"(v[1]), "=r"(v[2]), "=r"(v[3]) : "r"(at.v + idx * 16) : "memory");
+          const float wj = j < n ? pw[max(n - 1 - j, 0)] : 0.f;
+#pragma unroll
+          for (int e = 0; e < 4; ++e) Split(Low(v[e]) * wj, High(v[e]) * wj, hi[e], lo[e]);
+          StoreShared16(at.vd_hi + idx * 16, hi);
+          StoreShared16(at.vd_lo + idx * 16, lo);
+        }
+        asm volatile("fence.proxy.async.shared::cta;\n" ::: "memory");
+        asm volatile("tcgen05.fence::before_thread_sync;\n" ::: "memory");
+        __syncwarp();
+        if (lane == 0) MbarArrive(vd_ready);
+      }
+
+      if (OUT) {
+        ok = MbarWaitWarp(pv_done, par, lane, abort_word) && ok;
+        asm volatile("tcgen05.fence::after_thread_sync;\n" ::: "memory");
+        uint32_t x[32];
+        TcLd32(t_o + lanes + half * 32, x);
+        asm volatile("tcgen05.wait::ld.sync.aligned;\n" ::: "memory");
+        if (row < n) {
+          float* p = a.o + (static_cast<size_t>(t0 + row) * a.heads + head) * a.vdim + v0;
+          if (a.vdim % 4 == 0) {
+#pragma unroll
+            for (int e = 0; e < 32; e += 4) {
+              if (v0 + e < a.vdim) {
+                *reinterpret_cast<float4*>(p + e) = make_float4(o[e] + __uint_as_float(x[e]), o[e + 1] + __uint_as_float(x[e + 1]),
+                                                                o[e + 2] + __uint_as_float(x[e + 2]), o[e + 3] + __uint_as_float(x[e + 3]));
+              }
+            }
+          } else {
+#pragma unroll
+            for (int e = 0; e < 32; ++e)
+              if (v0 + e < a.vdim) p[e] = o[e] + __uint_as_float(x[e]);
           }
         }
       }
     }
-    __syncthreads();
-  }
 
-  if (!OUT) {
-    float* p = sums(seg);
+    if (!OUT || last) {
+      ok = MbarWaitWarp(st_done, (chunks - 1) & 1, lane, abort_word) && ok;
+      asm volatile("tcgen05.fence::after_thread_sync;\n" ::: "memory");
+#pragma unroll 1
+      for (int b = 0; b < BLOCKS; ++b) {
+        const int d = b * 128 + row;
+        uint32_t s[32];
+        TcLd32(t_s + lanes + b * 64 + half * 32, s);
+        asm volatile("tcgen05.wait::ld.sync.aligned;\n" ::: "memory");
+        if (!OUT) {
+          float* p = sums(seg) + b * 32 * kWorkerThreads;
 #pragma unroll
-    for (int n = 0; n < kTiles; ++n)
+          for (int e = 0; e < 32; ++e) p[e * kWorkerThreads] = d < a.dp ? __uint_as_float(s[e]) : 0.f;
+        } else if (d < a.dim) {
+          float* p = state + static_cast<size_t>(d) * vp + v0;
 #pragma unroll
-      for (int e = 0; e < 4; ++e) p[(n * 4 + e) * kThreads] = s[n][e];
-  } else if (seg + 1 == a.segments) {
-#pragma unroll
-    for (int n = 0; n < kTiles; ++n)
-#pragma unroll
-      for (int e = 0; e < 4; ++e) {
-        const int d = d0 + n * 8 + (lane & 3) * 2 + (e & 1), v = slice * VS + v0 + (lane >> 2) + (e >> 1) * 8;
-        if (d < a.dim && v < vp) state[static_cast<size_t>(d) * vp + v] = s[n][e];
+          for (int e = 0; e < 32; e += 4) {
+            if (v0 + e < vp) {
+              *reinterpret_cast<float4*>(p + e) = make_float4(__uint_as_float(s[e]), __uint_as_float(s[e + 1]), __uint_as_float(s[e + 2]), __uint_as_float(s[e + 3]));
+            }
+          }
+        }
       }
+    }
+    asm volatile("tcgen05.fence::before_thread_sync;\n" ::: "memory");
   }
+  if (!ok) atomicExch(&g_retention_status, 1);
+  __syncthreads();
+  if (warp == 0) {
+    asm volatile("tcgen05.fence::after_thread_sync;\n" ::: "memory");
+    asm volatile("tcgen05.dealloc.cta_group::1.sync.aligned.b32 %0, %1;\n" ::"r"(tmem), "r"(kCols) : "memory");
+  }
+}
+
+size_t SmemBytes(int dp)
+{
+  Places p;
+  return PlaceAll(dp, 0, &p);
 }
 
 // What a call is cut into.
 struct Plan {
-  int dk, vs, slices, segment, segments;
+  int dp, blocks, slices, segment, segments;
   size_t sums_bytes;
 };
 Plan PlanFor(int tokens, int heads, int dim, int vdim)
 {
   Plan p;
-  const int dp = (dim + 15) / 16 * 16;
-  p.dk = dp <= 64 ? 4 : dp <= 128 ? 8 : 16;
-  p.vs = p.dk == 16 ? 32 : 64;
-  p.slices = (vdim + p.vs - 1) / p.vs;
-  const int chunks = (tokens + kChunk - 1) / kChunk;
-  int want = (3 * 148 + heads * p.slices - 1) / (heads * p.slices);  // a few CTAs per SM
-  want = want < 1 ? 1 : want > 32 ? 32 : want;
-  const int per = (chunks + want - 1) / want;
+  p.dp = (dim + 15) / 16 * 16;
+  p.blocks = (p.dp + 127) / 128;
+  p.slices = (vdim + kVS - 1) / kVS;
+  const int chunks = (tokens + kChunk - 1) / kChunk, ctas = heads * p.slices, slots = 148 * (2 * (SmemBytes(p.dp) + 2048) <= 228 * 1024 && p.blocks == 1 ? 2 : 1);
+  // Rounds of CTAs times chunks of a segment, the state-only launch at two fifths of the other, a launch at one chunk.
+  double best = 1e30;
+  p.segments = 1;
+  int per = chunks;
+  for (int n = 1; n <= chunks && n <= 32; ++n) {
+    const int len = (chunks + n - 1) / n, used = (chunks + len - 1) / len;
+    double cost = static_cast<double>((ctas * used + slots - 1) / slots) * len;
+    if (used > 1) cost += 0.4 * ((ctas * (used - 1) + slots - 1) / slots) * len + 1.0;
+    if (cost < best * 0.97) {
+      best = cost;
+      p.segments = used;
+      per = len;
+    }
+  }
   p.segment = per * kChunk;
-  p.segments = (chunks + per - 1) / per;
-  p.sums_bytes = p.segments > 1 ? static_cast<size_t>(p.segments) * heads * p.slices * p.vs * p.dk * 16 * sizeof(float) : 0;
+  p.sums_bytes = p.segments > 1 ? static_cast<size_t>(p.segments) * ctas * p.blocks * 32 * kWorkerThreads * sizeof(float) : 0;
   return p;
 }
-size_t SmemBytes(int dk, int vs, int dim_ld, bool out)
+
+using EncodeTiledFn = CUresult (*)(CUtensorMap*, CUtensorMapDataType, cuuint32_t, void*, const cuuint64_t*, const cuuint64_t*,
+                                   const cuuint32_t*, const cuuint32_t*, CUtensorMapInterleave, CUtensorMapSwizzle,
+                                   CUtensorMapL2promotion, CUtensorMapFloatOOBfill);
+// bf16 [tokens][heads][ld], boxes of 64 channels of one head x 128 tokens.
+bool Encode(CUtensorMap* map, const void* ptr, int ld, int heads, int tokens)
 {
-  const size_t k_ld = dim_ld * 2 + 16, v_ld = vs * 2 + 16;
-  (void)dk;
-  return 2 * ((out ? 2 : 1) * kChunk * k_ld + kChunk * v_ld) + (out ? 2 * vs * k_ld : 0);
+  auto encode = reinterpret_cast<EncodeTiledFn>(TensorMapEncoder());
+  const cuuint64_t dims[3] = {static_cast<cuuint64_t>(ld), static_cast<cuuint64_t>(heads), static_cast<cuuint64_t>(tokens)};
+  const cuuint64_t strides[2] = {static_cast<cuuint64_t>(ld) * 2, static_cast<cuuint64_t>(ld) * 2 * heads};
+  const cuuint32_t box[3] = {64, 1, kChunk}, elem[3] = {1, 1, 1};
+  return encode != nullptr &&
+         encode(map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 3, const_cast<void*>(ptr), dims, strides, box, elem, CU_TENSOR_MAP_INTERLEAVE_NONE,
+                CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE) == CUDA_SUCCESS;
 }
 
 cudaError_t PrepareChunks()
 {
   static OncePerDevice once;
   return once.Run([](int) {
+    TensorMapEncoder();
     cudaError_t e = cudaSuccess;
-#define TLALOC_OPT_IN(DK, VS)                                                                                                                    \
-  if (e == cudaSuccess) e = cudaFuncSetAttribute(RetentionChunkKernel<DK, VS, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, kMaxSmem - 1024); \
-  if (e == cudaSuccess) e = cudaFuncSetAttribute(RetentionChunkKernel<DK, VS, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, kMaxSmem - 1024);
-    TLALOC_OPT_IN(4, 64)
-    TLALOC_OPT_IN(8, 64)
-    TLALOC_OPT_IN(16, 32)
+#define TLALOC_OPT_IN(BLOCKS, OUT) \
+  if (e == cudaSuccess) e = cudaFuncSetAttribute(RetentionChunkTc<BLOCKS, OUT>, cudaFuncAttributeMaxDynamicSharedMemorySize, kMaxSmem - 1024);
+    TLALOC_OPT_IN(1, true)
+    TLALOC_OPT_IN(1, false)
+    TLALOC_OPT_IN(2, true)
+    TLALOC_OPT_IN(2, false)
 #undef TLALOC_OPT_IN
     return e;
   });
 }
-KernelSetup g_setup(PrepareChunks, nullptr);
+int ReadRetentionStatus()
+{
+  int v = 0;
+  if (cudaMemcpyFromSymbol(&v, g_retention_status, sizeof(int)) != cudaSuccess) return -1;
+  if (v != 0) {
+    const int zero = 0;
+    cudaMemcpyToSymbol(g_retention_status, &zero, sizeof(int));
+  }
+  return v;
+}
+KernelSetup g_setup(PrepareChunks, ReadRetentionStatus);
 
 template <bool OUT>
-cudaError_t Launch(const Plan& p, const ChunkArgs& a, int segments, cudaStream_t st)
+cudaError_t Launch(const Plan& p, const CUtensorMap* maps, const ChunkArgs& a, int segments, cudaStream_t st)
 {
   const dim3 grid(a.heads, p.slices, segments);
-  const size_t smem = SmemBytes(p.dk, p.vs, a.dim_ld, OUT);
-  if (p.dk == 4) return LaunchChained(RetentionChunkKernel<4, 64, OUT>, grid, kThreads, smem, st, a);
-  if (p.dk == 8) return LaunchChained(RetentionChunkKernel<8, 64, OUT>, grid, kThreads, smem, st, a);
-  return LaunchChained(RetentionChunkKernel<16, 32, OUT>, grid, kThreads, smem, st, a);
+  const size_t smem = SmemBytes(a.dp);
+  return p.blocks == 1 ? LaunchChained(RetentionChunkTc<1, OUT>, grid, kThreads, smem, st, maps[0], maps[1], maps[2], a)
+                       : LaunchChained(RetentionChunkTc<2, OUT>, grid, kThreads, smem, st, maps[0], maps[1], maps[2], a);
 }
 
 }  // namespace
@@ -366,18 +522,20 @@ extern "C" int tlaloc_b200_retention_chunks(const void* q, const void* k, int32_
   if (!q || !k || !v || !positions || !decay || !row_states || !state || !o) return Fail(kInvalid, "%s: a required device pointer is null", op);
   if (tokens < 0 || heads < 1 || heads > 65535 || dim < 1 || vdim < 1 || num_slots < 1) return Fail(kInvalid, "%s: bad sizes", op);
   if (!tlaloc_b200_retention_chunks_applies(dim, vdim)) return Fail(kUnsupported, "%s: dim up to 256", op);
-  if (dim_ld != (dim + 15) / 16 * 16 || v_ld < vdim || v_ld % 8 || !Aligned16(q) || !Aligned16(k) || !Aligned16(v) || !Aligned16(state)) {
+  if (dim_ld != (dim + 15) / 16 * 16 || v_ld < vdim || v_ld % 8 || !Aligned16(q) || !Aligned16(k) || !Aligned16(v) || !Aligned16(state) || !Aligned16(o)) {
     return Fail(kInvalid, "%s: rows of dim rounded up to 16 and of a multiple of 8 values, 16-byte aligned", op);
   }
   if (tokens == 0) return kOk;
   const Plan p = PlanFor(tokens, heads, dim, vdim);
+  if (p.slices > 65535) return Fail(kInvalid, "%s: bad sizes", op);
   if (p.sums_bytes > 0 && (!scratch || scratch_bytes < p.sums_bytes)) return Fail(kInvalid, "%s: %zu bytes of scratch are needed", op, p.sums_bytes);
   cudaError_t e = PrepareChunks();
   if (e != cudaSuccess) return CudaFail("RETENTION_CHUNKS set-up", e);
+  CUtensorMap maps[3];
+  if (!Encode(&maps[0], q, dim_ld, heads, tokens) || !Encode(&maps[1], k, dim_ld, heads, tokens) || !Encode(&maps[2], v, v_ld, heads, tokens)) {
+    return Fail(kInternal, "%s: the tensor maps could not be encoded", op);
+  }
   ChunkArgs a = {};
-  a.q = static_cast<const __nv_bfloat16*>(q);
-  a.k = static_cast<const __nv_bfloat16*>(k);
-  a.v = static_cast<const __nv_bfloat16*>(v);
   a.positions = positions;
   a.row_states = row_states;
   a.decay = decay;
@@ -388,17 +546,16 @@ extern "C" int tlaloc_b200_retention_chunks(const void* q, const void* k, int32_
   a.heads = heads;
   a.dim = dim;
   a.vdim = vdim;
-  a.dim_ld = dim_ld;
-  a.v_ld = v_ld;
+  a.dp = p.dp;
   a.num_slots = num_slots;
   a.segment = p.segment;
   a.segments = p.segments;
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   if (p.segments > 1) {
-    e = Launch<false>(p, a, p.segments - 1, st);
+    e = Launch<false>(p, maps, a, p.segments - 1, st);
     if (e == cudaSuccess) CountLaunches(1);
   }
-  if (e == cudaSuccess) e = Launch<true>(p, a, p.segments, st);
+  if (e == cudaSuccess) e = Launch<true>(p, maps, a, p.segments, st);
   if (e != cudaSuccess) return CudaFail("RETENTION_CHUNKS launch", e);
   CountLaunches(1);
   return kOk;
