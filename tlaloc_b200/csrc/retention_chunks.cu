@@ -8,8 +8,8 @@
 // and enters a product as an operand (S, the decayed scores, the decayed values) enters as two bf16 parts, which is f32 up to rounding.
 //   producer lane   Q, K and V of the next chunk
 //   MMA lane        scores Q K^T; O = Q S; O = P V (its first part is in registers by then); S += K^T V'
-//   eight warps     S as an operand (shared memory) and decayed; scores times decay, in their place in TMEM as the A operand P; the
-//                   decayed values V' (in the place of Q); the output rows
+//   worker warps    S as an operand (shared memory) and decayed; scores times decay, in their place in TMEM as the A operand P; the
+//                   decayed values V' (in the place of Q); the output rows.  Eight, and two CTAs per SM, up to 128 channels; else sixteen
 // Two launches where there are several segments: the first computes what each segment adds to the state, the second starts every
 // segment from the sum of those before it, writes the outputs and, in the last segment, the new state.  Every mbarrier wait is bounded.
 #include <cuda.h>
@@ -24,7 +24,6 @@ using namespace tc;
 
 constexpr int kChunk = 128, kVS = 64;
 constexpr int kAtom = kChunk * 128;  // 128 tokens x 64 channels
-constexpr int kWorkers = 8, kWorkerThreads = kWorkers * 32, kThreads = kWorkerThreads + 64;
 constexpr int kMaxSmem = 227 * 1024;
 
 struct ChunkArgs {
@@ -86,16 +85,34 @@ __host__ __device__ inline uint32_t PlaceAll(int dp, uint32_t base, Places* p)
   return end - base;
 }
 
+template <int N>
+__device__ __forceinline__ void LoadTmem(uint32_t taddr, uint32_t* r)
+{
+  if constexpr (N == 32) TcLd32(taddr, r);
+  else TcLd16(taddr, r);
+}
+template <int N>
+__device__ __forceinline__ void StoreTmem(uint32_t taddr, const uint32_t* r)
+{
+  if constexpr (N == 32) TcSt32(taddr, r);
+  else TcSt16(taddr, r);
+}
+
+constexpr int WorkersFor(int blocks) { return blocks == 1 ? 8 : 16; }
+
 // BLOCKS: 128-channel blocks of S.
 template <int BLOCKS, bool OUT>
-__global__ void __launch_bounds__(kThreads) RetentionChunkTc(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
+__global__ void __launch_bounds__(WorkersFor(BLOCKS) * 32 + 64, BLOCKS == 1 ? 2 : 1) RetentionChunkTc(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
                                                              const __grid_constant__ CUtensorMap map_v, const __grid_constant__ ChunkArgs a)
 {
+  constexpr int kWorkers = WorkersFor(BLOCKS), kWorkerThreads = kWorkers * 32, kParts = kWorkers / 4;
+  constexpr int VC = kVS / kParts, PC = kChunk / kParts;  // columns of O and S, and of the scores, of a worker warp
   constexpr uint32_t kCols = BLOCKS == 1 ? 256u : 512u;  // scores 128, O 64, S 64 per block
   extern __shared__ __align__(1024) unsigned char smem_raw[];
   __shared__ alignas(8) uint64_t bars[8];
   __shared__ uint32_t slot_store[2];
   __shared__ float pw[kChunk + 1];
+  __shared__ __align__(16) float pw_down[32];  // w^31 .. w^0
   const uint32_t base = SmemAddr(smem_raw);  // two CTAs of 128 channels fill an SM to the byte: no slack to align within
   if ((base & 1023u) != 0u) {
     if (threadIdx.x == 0) atomicExch(&g_retention_status, 1);
@@ -183,8 +200,9 @@ __global__ void __launch_bounds__(kThreads) RetentionChunkTc(const __grid_consta
           ok = MbarWait(p_ready, par, abort_word) && ok;
           asm volatile("tcgen05.fence::after_thread_sync;\n" ::: "memory");
           for (int k = 0; k < kChunk / 16; ++k) {
-            TcMmaTmemA(t_o, t_p + 8 * k, vd + k * kRows, out_desc, k > 0 ? 1u : 0u);
-            TcMmaTmemA(t_o, t_p + 64 + 8 * k, vd + k * kRows, out_desc, 1u);
+            const uint32_t pa = t_p + 32 * (k >> 1) + 8 * (k & 1);
+            TcMmaTmemA(t_o, pa, vd + k * kRows, out_desc, k > 0 ? 1u : 0u);
+            TcMmaTmemA(t_o, pa + 16, vd + k * kRows, out_desc, 1u);
           }
           TcCommit(pv_done);
         }
@@ -205,18 +223,19 @@ __global__ void __launch_bounds__(kThreads) RetentionChunkTc(const __grid_consta
     }
     __syncwarp();
   } else {
-    const int quad = warp & 3, half = warp >> 2, row = quad * 32 + lane;  // TMEM lane; columns [32 half, 32 half + 32) of O and S
+    const int quad = warp & 3, part = warp >> 2, row = quad * 32 + lane;  // row: TMEM lane
     const uint32_t lanes = static_cast<uint32_t>(quad * 32) << 16;
     const float w = __ldg(a.decay + head);
     for (int i = tid; i <= kChunk; i += kWorkerThreads) pw[i] = powf(w, static_cast<float>(i));
-    asm volatile("bar.sync 5, 256;\n" ::: "memory");
+    if (tid < 32) pw_down[tid] = powf(w, static_cast<float>(31 - tid));
+    asm volatile("bar.sync 5, %0;\n" ::"n"(kWorkerThreads) : "memory");
 
     // The state ahead of the segment.
-    const int vp = (a.vdim + 3) & ~3, v0 = slice * kVS + half * 32;
+    const int vp = (a.vdim + 3) & ~3, v0 = slice * kVS + part * VC;
     const int slot = min(max(__ldg(a.row_states), 0), a.num_slots - 1);
     float* state = a.state + (static_cast<size_t>(slot) * a.heads + head) * a.dim * vp;
     auto sums = [&](int g) {
-      return a.sums + ((static_cast<size_t>(g) * a.heads + head) * slices + slice) * (static_cast<size_t>(BLOCKS) * 32 * kWorkerThreads) + tid;
+      return a.sums + ((static_cast<size_t>(g) * a.heads + head) * slices + slice) * (static_cast<size_t>(BLOCKS) * VC * kWorkerThreads) + tid;
     };
     const bool own = seg == 0 && !(OUT && a.segments > 1);
     const bool fresh = __ldg(a.positions) == 0;
@@ -225,14 +244,14 @@ __global__ void __launch_bounds__(kThreads) RetentionChunkTc(const __grid_consta
 #pragma unroll 1
     for (int b = 0; b < BLOCKS; ++b) {
       const int d = b * 128 + row;
-      float s[32];
+      float s[VC];
 #pragma unroll
-      for (int e = 0; e < 32; ++e) s[e] = 0.f;
+      for (int e = 0; e < VC; ++e) s[e] = 0.f;
       if (own) {
         if (!fresh && d < a.dim) {
           const float* p = state + static_cast<size_t>(d) * vp + v0;
 #pragma unroll
-          for (int e = 0; e < 32; e += 4) {
+          for (int e = 0; e < VC; e += 4) {
             if (v0 + e < vp) {
               const float4 x = *reinterpret_cast<const float4*>(p + e);
               s[e] = x.x; s[e + 1] = x.y; s[e + 2] = x.z; s[e + 3] = x.w;
@@ -240,18 +259,18 @@ __global__ void __launch_bounds__(kThreads) RetentionChunkTc(const __grid_consta
           }
         }
         if (!OUT) {
-          float* p = sums(a.segments - 1) + b * 32 * kWorkerThreads;
+          float* p = sums(a.segments - 1) + b * VC * kWorkerThreads;
 #pragma unroll
-          for (int e = 0; e < 32; ++e) p[e * kWorkerThreads] = s[e];
+          for (int e = 0; e < VC; ++e) p[e * kWorkerThreads] = s[e];
         }
       } else if (OUT) {
         for (int g = g_lo; g < g_hi; ++g) {
-          const float* p = sums(g) + b * 32 * kWorkerThreads;
+          const float* p = sums(g) + b * VC * kWorkerThreads;
 #pragma unroll
-          for (int e = 0; e < 32; ++e) s[e] = fmaf(ws, s[e], p[e * kWorkerThreads]);
+          for (int e = 0; e < VC; ++e) s[e] = fmaf(ws, s[e], p[e * kWorkerThreads]);
         }
       }
-      TcSt32(t_s + lanes + b * 64 + half * 32, reinterpret_cast<const uint32_t*>(s));
+      StoreTmem<VC>(t_s + lanes + b * 64 + part * VC, reinterpret_cast<const uint32_t*>(s));
     }
     asm volatile("tcgen05.wait::st.sync.aligned;\n" ::: "memory");
 
@@ -268,69 +287,78 @@ __global__ void __launch_bounds__(kThreads) RetentionChunkTc(const __grid_consta
       for (int b = 0; b < BLOCKS; ++b) {
         const int d = b * 128 + row;
         if (b * 128 + quad * 32 >= a.dp) break;  // nothing but padding in this warp's rows
-        uint32_t s[32];
-        TcLd32(t_s + lanes + b * 64 + half * 32, s);
+        uint32_t s[VC];
+        LoadTmem<VC>(t_s + lanes + b * 64 + part * VC, s);
         asm volatile("tcgen05.wait::ld.sync.aligned;\n" ::: "memory");
         if (OUT && d < a.dp) {
 #pragma unroll
-          for (int i = 0; i < 4; ++i) {
+          for (int i = 0; i < VC / 8; ++i) {
             uint32_t hi[4], lo[4];
 #pragma unroll
             for (int e = 0; e < 4; ++e) Split(__uint_as_float(s[8 * i + 2 * e]), __uint_as_float(s[8 * i + 2 * e + 1]), hi[e], lo[e]);
-            const uint32_t off = d * 128 + (((half * 4 + i) ^ (d & 7)) << 4);
+            const uint32_t off = d * 128 + (((part * (VC / 8) + i) ^ (d & 7)) << 4);
             StoreShared16(at.s_hi + off, hi);
             StoreShared16(at.s_lo + off, lo);
           }
         }
 #pragma unroll
-        for (int e = 0; e < 32; ++e) s[e] = __float_as_uint(__uint_as_float(s[e]) * wn);
-        TcSt32(t_s + lanes + b * 64 + half * 32, s);
+        for (int e = 0; e < VC; ++e) s[e] = __float_as_uint(__uint_as_float(s[e]) * wn);
+        StoreTmem<VC>(t_s + lanes + b * 64 + part * VC, s);
       }
       asm volatile("tcgen05.wait::st.sync.aligned;\n" ::: "memory");
-      float o[32];
+      float o[VC];
       if (OUT) {
         asm volatile("fence.proxy.async.shared::cta;\n" ::: "memory");
         asm volatile("tcgen05.fence::before_thread_sync;\n" ::: "memory");
         __syncwarp();
         if (lane == 0) MbarArrive(s_ready);
 
-        // Scores times decay: columns [64 half, 64 half + 64), 32 at a time; the parts go to columns 32 half and 64 + 32 half.
+        // Scores times decay, 32 columns at a time: their first parts go to the first 16 of the columns, the second parts to the others.
         ok = MbarWaitWarp(sc_done, par, lane, abort_word) && ok;
         asm volatile("tcgen05.fence::after_thread_sync;\n" ::: "memory");
-        uint32_t hi[32], lo[32];
 #pragma unroll
-        for (int g = 0; g < 2; ++g) {
-          const int j0 = half * 64 + g * 32;
+        for (int g = 0; g < PC / 32; ++g) {
+          const int j0 = part * PC + g * 32;
+          uint32_t hi[16], lo[16];
           if (j0 > quad * 32 + 31) {  // all of it in the future
 #pragma unroll
-            for (int e = 0; e < 16; ++e) hi[g * 16 + e] = lo[g * 16 + e] = 0u;
+            for (int e = 0; e < 16; ++e) hi[e] = lo[e] = 0u;
           } else {
             uint32_t s[32];
             TcLd32(t_p + lanes + j0, s);
             asm volatile("tcgen05.wait::ld.sync.aligned;\n" ::: "memory");
+            if (j0 < quad * 32) {  // all of it in the past: w^(row - j) = w^(row - j0 - 31) w^(31 - e), both exponents from 0 up
+              const float wr = pw[row - j0 - 31];
 #pragma unroll
-            for (int e = 0; e < 32; e += 2) {
-              const int back = row - j0 - e;
-              const float x = back >= 0 ? __uint_as_float(s[e]) * pw[max(back, 0)] : 0.f;
-              const float y = back >= 1 ? __uint_as_float(s[e + 1]) * pw[max(back - 1, 0)] : 0.f;
-              Split(x, y, hi[g * 16 + e / 2], lo[g * 16 + e / 2]);
+              for (int e = 0; e < 32; e += 4) {
+                const float4 we = *reinterpret_cast<const float4*>(pw_down + e);
+                Split(__uint_as_float(s[e]) * we.x * wr, __uint_as_float(s[e + 1]) * we.y * wr, hi[e / 2], lo[e / 2]);
+                Split(__uint_as_float(s[e + 2]) * we.z * wr, __uint_as_float(s[e + 3]) * we.w * wr, hi[e / 2 + 1], lo[e / 2 + 1]);
+              }
+            } else {
+#pragma unroll
+              for (int e = 0; e < 32; e += 2) {
+                const int back = lane - e;
+                const float x = back >= 0 ? __uint_as_float(s[e]) * pw[max(back, 0)] : 0.f;
+                const float y = back >= 1 ? __uint_as_float(s[e + 1]) * pw[max(back - 1, 0)] : 0.f;
+                Split(x, y, hi[e / 2], lo[e / 2]);
+              }
             }
           }
+          TcSt16(t_p + lanes + j0, hi);
+          TcSt16(t_p + lanes + j0 + 16, lo);
         }
-        asm volatile("bar.sync %0, 64;\n" ::"r"(1 + quad) : "memory");  // both warps of the quad have their scores
-        TcSt32(t_p + lanes + half * 32, hi);
-        TcSt32(t_p + lanes + 64 + half * 32, lo);
         asm volatile("tcgen05.wait::st.sync.aligned;\n" ::: "memory");
         ok = MbarWaitWarp(o_done, par, lane, abort_word) && ok;
         asm volatile("tcgen05.fence::after_thread_sync;\n" ::: "memory");
-        TcLd32(t_o + lanes + half * 32, reinterpret_cast<uint32_t*>(o));
+        LoadTmem<VC>(t_o + lanes + part * VC, reinterpret_cast<uint32_t*>(o));
         asm volatile("tcgen05.wait::ld.sync.aligned;\n" ::: "memory");
         asm volatile("tcgen05.fence::before_thread_sync;\n" ::: "memory");
         __syncwarp();
         if (lane == 0) MbarArrive(p_ready);
         const float wi = pw[row + 1];
 #pragma unroll
-        for (int e = 0; e < 32; ++e) o[e] *= wi;
+        for (int e = 0; e < VC; ++e) o[e] *= wi;
       }
 
       // Decayed values, in the place of Q (its products are done).
@@ -356,14 +384,14 @@ __global__ void __launch_bounds__(kThreads) RetentionChunkTc(const __grid_consta
       if (OUT) {
         ok = MbarWaitWarp(pv_done, par, lane, abort_word) && ok;
         asm volatile("tcgen05.fence::after_thread_sync;\n" ::: "memory");
-        uint32_t x[32];
-        TcLd32(t_o + lanes + half * 32, x);
+        uint32_t x[VC];
+        LoadTmem<VC>(t_o + lanes + part * VC, x);
         asm volatile("tcgen05.wait::ld.sync.aligned;\n" ::: "memory");
         if (row < n) {
           float* p = a.o + (static_cast<size_t>(t0 + row) * a.heads + head) * a.vdim + v0;
           if (a.vdim % 4 == 0) {
 #pragma unroll
-            for (int e = 0; e < 32; e += 4) {
+            for (int e = 0; e < VC; e += 4) {
               if (v0 + e < a.vdim) {
                 *reinterpret_cast<float4*>(p + e) = make_float4(o[e] + __uint_as_float(x[e]), o[e + 1] + __uint_as_float(x[e + 1]),
                                                                 o[e + 2] + __uint_as_float(x[e + 2]), o[e + 3] + __uint_as_float(x[e + 3]));
@@ -371,7 +399,7 @@ __global__ void __launch_bounds__(kThreads) RetentionChunkTc(const __grid_consta
             }
           } else {
 #pragma unroll
-            for (int e = 0; e < 32; ++e)
+            for (int e = 0; e < VC; ++e)
               if (v0 + e < a.vdim) p[e] = o[e] + __uint_as_float(x[e]);
           }
         }
@@ -384,17 +412,17 @@ __global__ void __launch_bounds__(kThreads) RetentionChunkTc(const __grid_consta
 #pragma unroll 1
       for (int b = 0; b < BLOCKS; ++b) {
         const int d = b * 128 + row;
-        uint32_t s[32];
-        TcLd32(t_s + lanes + b * 64 + half * 32, s);
+        uint32_t s[VC];
+        LoadTmem<VC>(t_s + lanes + b * 64 + part * VC, s);
         asm volatile("tcgen05.wait::ld.sync.aligned;\n" ::: "memory");
         if (!OUT) {
-          float* p = sums(seg) + b * 32 * kWorkerThreads;
+          float* p = sums(seg) + b * VC * kWorkerThreads;
 #pragma unroll
-          for (int e = 0; e < 32; ++e) p[e * kWorkerThreads] = d < a.dp ? __uint_as_float(s[e]) : 0.f;
+          for (int e = 0; e < VC; ++e) p[e * kWorkerThreads] = d < a.dp ? __uint_as_float(s[e]) : 0.f;
         } else if (d < a.dim) {
           float* p = state + static_cast<size_t>(d) * vp + v0;
 #pragma unroll
-          for (int e = 0; e < 32; e += 4) {
+          for (int e = 0; e < VC; e += 4) {
             if (v0 + e < vp) {
               *reinterpret_cast<float4*>(p + e) = make_float4(__uint_as_float(s[e]), __uint_as_float(s[e + 1]), __uint_as_float(s[e + 2]), __uint_as_float(s[e + 3]));
             }
@@ -430,14 +458,17 @@ Plan PlanFor(int tokens, int heads, int dim, int vdim)
   p.blocks = (p.dp + 127) / 128;
   p.slices = (vdim + kVS - 1) / kVS;
   const int chunks = (tokens + kChunk - 1) / kChunk, ctas = heads * p.slices, slots = 148 * (2 * (SmemBytes(p.dp) + 2048) <= 228 * 1024 && p.blocks == 1 ? 2 : 1);
-  // Rounds of CTAs times chunks of a segment, the state-only launch at two fifths of the other, a launch at one chunk.
+  // Rounds of CTAs times chunks of a segment, in chunks of the second launch: the state alone at two fifths, a launch at one half, the sums of
+  // an earlier segment at a sixteenth per block of S.
   double best = 1e30;
   p.segments = 1;
   int per = chunks;
   for (int n = 1; n <= chunks && n <= 32; ++n) {
     const int len = (chunks + n - 1) / n, used = (chunks + len - 1) / len;
     double cost = static_cast<double>((ctas * used + slots - 1) / slots) * len;
-    if (used > 1) cost += 0.4 * ((ctas * (used - 1) + slots - 1) / slots) * len + 1.0;
+    if (used > 1) {
+      cost += 0.4 * ((ctas * (used - 1) + slots - 1) / slots) * len + 0.5 + 0.0625 * p.blocks * (used - 1) * ((ctas * used + slots - 1) / slots);
+    }
     if (cost < best * 0.97) {
       best = cost;
       p.segments = used;
@@ -445,7 +476,7 @@ Plan PlanFor(int tokens, int heads, int dim, int vdim)
     }
   }
   p.segment = per * kChunk;
-  p.sums_bytes = p.segments > 1 ? static_cast<size_t>(p.segments) * ctas * p.blocks * 32 * kWorkerThreads * sizeof(float) : 0;
+  p.sums_bytes = p.segments > 1 ? static_cast<size_t>(p.segments) * ctas * p.blocks * kChunk * kVS * sizeof(float) : 0;
   return p;
 }
 
@@ -497,8 +528,9 @@ cudaError_t Launch(const Plan& p, const CUtensorMap* maps, const ChunkArgs& a, i
 {
   const dim3 grid(a.heads, p.slices, segments);
   const size_t smem = SmemBytes(a.dp);
-  return p.blocks == 1 ? LaunchChained(RetentionChunkTc<1, OUT>, grid, kThreads, smem, st, maps[0], maps[1], maps[2], a)
-                       : LaunchChained(RetentionChunkTc<2, OUT>, grid, kThreads, smem, st, maps[0], maps[1], maps[2], a);
+  const int threads = WorkersFor(p.blocks) * 32 + 64;
+  return p.blocks == 1 ? LaunchChained(RetentionChunkTc<1, OUT>, grid, threads, smem, st, maps[0], maps[1], maps[2], a)
+                       : LaunchChained(RetentionChunkTc<2, OUT>, grid, threads, smem, st, maps[0], maps[1], maps[2], a);
 }
 
 }  // namespace
