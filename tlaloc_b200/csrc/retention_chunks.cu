@@ -65,10 +65,11 @@ __device__ __forceinline__ void StoreShared16(uint32_t at, const uint32_t* v)
   asm volatile("st.shared.v4.b32 [%0], {%1, %2, %3, %4};\n" ::"r"(at), "r"(v[0]), "r"(v[1]), "r"(v[2]), "r"(v[3]) : "memory");
 }
 
-// Shared memory: Q | K (one or two buffers) | V, later the output rows | S as an operand, later V'.
+// Shared memory: Q | K (one or two buffers) | V, later the output rows | S as an operand, later V'.  For the state alone: two buffers of
+// K from Q's place on, two of V, and V' (one or two).
 struct Places {
   uint32_t q, k, v, s, bytes;
-  int k_buffers;
+  int k_buffers, vd_buffers;
 };
 __host__ __device__ inline Places PlaceAll(int dp, int vs)
 {
@@ -80,6 +81,7 @@ __host__ __device__ inline Places PlaceAll(int dp, int vs)
   p.k = tile;
   p.v = p.k + p.k_buffers * tile;
   p.s = p.v + o_bytes;
+  p.vd_buffers = s_bytes >= 2 * vd_bytes ? 2 : 1;
   p.bytes = p.v + rest;
   return p;
 }
@@ -107,7 +109,7 @@ __global__ void __launch_bounds__(kThreads, 1) RetentionChunkTc(const __grid_con
   constexpr int VC = VS / kParts, kVAtoms = VS / 64;  // value columns of a worker thread
   constexpr uint32_t kCols = 512;                     // scores, O and each block of S: 128 columns
   extern __shared__ __align__(1024) unsigned char smem_raw[];
-  __shared__ alignas(8) uint64_t bars[13];
+  __shared__ alignas(8) uint64_t bars[15];
   __shared__ uint32_t slot_store[2];
   __shared__ float pw_store[31 + kChunk + 1];  // 31 zeros, then w^0 .. w^128
   float* pw = pw_store + 31;
@@ -117,16 +119,16 @@ __global__ void __launch_bounds__(kThreads, 1) RetentionChunkTc(const __grid_con
     return;
   }
   const Places at = PlaceAll(a.dp, VS);
-  const uint32_t at_q = base + at.q, at_k = base + at.k, at_v = base + at.v, at_s = base + at.s;
+  const uint32_t at_q = base + at.q, at_k = base + (OUT ? at.k : at.q), at_v = base + at.v, at_s = base + at.s;
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
-  const uint32_t full_q = SmemAddr(bars), full_k = full_q + 8, full_v = full_k + 16, sc_done = full_v + 8, s_ready = sc_done + 8, o_done = s_ready + 8,
-                 p_ready = o_done + 8, pv_done = p_ready + 8, vd_ready = pv_done + 8, st_done = vd_ready + 8, o_ready = st_done + 16;
+  const uint32_t full_q = SmemAddr(bars), full_k = full_q + 8, full_v = full_k + 16, sc_done = full_v + 16, s_ready = sc_done + 8, o_done = s_ready + 8,
+                 p_ready = o_done + 8, pv_done = p_ready + 8, vd_ready = pv_done + 8, st_done = vd_ready + 16, o_ready = st_done + 16;
   volatile uint32_t* abort_word = slot_store + 1;
   if (tid == 0) {
     slot_store[1] = 0u;
-    for (int i = 0; i < 13; ++i) {
+    for (int i = 0; i < 15; ++i) {
       const uint32_t bar = SmemAddr(bars + i);
-      MbarInit(bar, bar == s_ready || bar == p_ready || bar == vd_ready || bar == o_ready ? kWorkers : 1);
+      MbarInit(bar, bar == s_ready || bar == p_ready || bar == vd_ready || bar == vd_ready + 8 || bar == o_ready ? kWorkers : 1);
     }
     asm volatile("fence.mbarrier_init.release.cluster;\n" ::: "memory");
   }
@@ -145,12 +147,19 @@ __global__ void __launch_bounds__(kThreads, 1) RetentionChunkTc(const __grid_con
   const bool last = seg + 1 == a.segments;
   // Whether the state behind chunk c is wanted.
   auto carries = [&](int c) { return !OUT || last || c + 1 < chunks; };
-  const int atoms = (a.dp + 63) / 64, steps = a.dp / 16, kb = at.k_buffers;
+  const int atoms = (a.dp + 63) / 64, steps = a.dp / 16, kb = OUT ? at.k_buffers : 2;
   const uint32_t k_tile = atoms * kAtom;
-  // Barriers of K's buffers and of the state's products alternate with the chunk.
+  // Barriers of K's buffers, of V' and of the state's products alternate with the chunk (one that is two phases ahead of a wait looks like one
+  // that has not come).
   auto k_buf = [&](int c) { return kb == 2 ? c & 1 : 0; };
   auto k_par = [&](int c) { return static_cast<uint32_t>((kb == 2 ? c >> 1 : c) & 1); };
   auto st_bar = [&](int c) { return st_done + 8 * (c & 1); };
+  auto vd_bar = [&](int c) { return vd_ready + 8 * (c & 1); };
+  // The state alone: buffers of V alternate too, and those of V' if there are two.
+  auto v_buf = [&](int c) { return OUT ? 0 : c & 1; };
+  auto v_par = [&](int c) { return static_cast<uint32_t>((OUT ? c : c >> 1) & 1); };
+  const int vdb = OUT ? 1 : at.vd_buffers;
+  auto vd_at = [&](int c) { return static_cast<uint32_t>(vdb == 2 && (c & 1) ? 2 * kVAtoms * kAtom : 0); };
   bool ok = true;
 
   if (warp == kWorkers) {
@@ -179,12 +188,10 @@ __global__ void __launch_bounds__(kThreads, 1) RetentionChunkTc(const __grid_con
           MbarExpectTx(full_q, k_tile);
           for (int x = 0; x < atoms; ++x) TmaBox(at_q + x * kAtom, &map_q, x * 64, head, t0, full_q);
         }
-        if (c > 0) {  // V has been multiplied with and read, and the output rows in its place have left
-          if (OUT) store_rows(c - 1);
-          else ok = MbarWait(vd_ready, (c - 1) & 1, abort_word) && ok;
-        }
-        MbarExpectTx(full_v, kVAtoms * kAtom);
-        for (int x = 0; x < kVAtoms; ++x) TmaBox(at_v + x * kAtom, &map_v, slice * VS + x * 64, head, t0, full_v);
+        if (OUT && c > 0) store_rows(c - 1);  // V has been multiplied with and read, and the output rows in its place have left
+        const uint32_t bar_v = full_v + 8 * v_buf(c), v_dst = at_v + v_buf(c) * kVAtoms * kAtom;
+        MbarExpectTx(bar_v, kVAtoms * kAtom);
+        for (int x = 0; x < kVAtoms; ++x) TmaBox(v_dst + x * kAtom, &map_v, slice * VS + x * 64, head, t0, bar_v);
       }
       if (OUT) {
         store_rows(chunks - 1);
@@ -194,7 +201,7 @@ __global__ void __launch_bounds__(kThreads, 1) RetentionChunkTc(const __grid_con
         volatile uint32_t never = 0;
         for (int c = max(0, chunks - kb); c < chunks; ++c) MbarWait(full_k + 8 * k_buf(c), k_par(c), &never);
         if (OUT) MbarWait(full_q, (chunks - 1) & 1, &never);
-        MbarWait(full_v, (chunks - 1) & 1, &never);
+        for (int c = max(0, chunks - (OUT ? 1 : 2)); c < chunks; ++c) MbarWait(full_v + 8 * v_buf(c), v_par(c), &never);
       }
     }
     __syncwarp();
@@ -244,14 +251,15 @@ __global__ void __launch_bounds__(kThreads, 1) RetentionChunkTc(const __grid_con
           ok = MbarWait(full_k + 8 * k_buf(c), k_par(c), abort_word) && ok;
         }
         if (carries(c)) {
-          ok = MbarWait(vd_ready, par, abort_word) && ok;
+          ok = MbarWait(vd_bar(c), (c >> 1) & 1, abort_word) && ok;
           asm volatile("tcgen05.fence::after_thread_sync;\n" ::: "memory");
 #pragma unroll
           for (int b = 0; b < BLOCKS; ++b) {
             const uint64_t ka = kt + static_cast<uint64_t>((k_buf(c) * k_tile + b * 2 * kAtom) >> 4);
+            const uint64_t off = vd_at(c) >> 4;
             for (int k = 0; k < kChunk / 16; ++k) {
-              TcMmaBf16(t_s + b * 128, ka + k * kRows, dh + k * kRows, state_desc, 1u);
-              if (!kSideBySide) TcMmaBf16(t_s + b * 128, ka + k * kRows, dl + k * kRows, state_desc, 1u);
+              TcMmaBf16(t_s + b * 128, ka + k * kRows, dh + off + k * kRows, state_desc, 1u);
+              if (!kSideBySide) TcMmaBf16(t_s + b * 128, ka + k * kRows, dl + off + k * kRows, state_desc, 1u);
             }
           }
           TcCommit(st_bar(c));
@@ -340,8 +348,8 @@ __global__ void __launch_bounds__(kThreads, 1) RetentionChunkTc(const __grid_con
     for (int c = 0; c < chunks; ++c) {
       const uint32_t par = c & 1;
       const int t0 = t_begin + c * kChunk, n = min(kChunk, t_end - t0);
-      if (c > 0) {
-        ok = MbarWaitWarp(st_bar(c - 1), ((c - 1) >> 1) & 1, lane, abort_word) && ok;
+      if (c >= vdb) {
+        ok = MbarWaitWarp(st_bar(c - vdb), ((c - vdb) >> 1) & 1, lane, abort_word) && ok;
         asm volatile("tcgen05.fence::after_thread_sync;\n" ::: "memory");
       }
       float o[VC];
@@ -410,28 +418,29 @@ __global__ void __launch_bounds__(kThreads, 1) RetentionChunkTc(const __grid_con
 
       // Decayed values, in the place of S's operand (its products, or those with the values before, are done).
       if (carries(c)) {
-        ok = MbarWaitWarp(full_v, par, lane, abort_word) && ok;
+        ok = MbarWaitWarp(full_v + 8 * v_buf(c), v_par(c), lane, abort_word) && ok;
+        const uint32_t v_src = at_v + v_buf(c) * kVAtoms * kAtom, vd_dst = at_s + vd_at(c);
         const float wc = OUT ? 1.f : powf(w, static_cast<float>((chunks - 1 - c) * kChunk));  // from the chunk's end to the segment's
 #pragma unroll
         for (int i = 0; i < kVAtoms * kAtom / 16 / kWorkerThreads; ++i) {
           const int idx = i * kWorkerThreads + tid, j = (idx & (kAtom / 16 - 1)) >> 3;
           uint32_t v[4], hi[4], lo[4];
-          asm volatile("ld.shared.v4.b32 {%0, %1, %2, %3}, [%4];\n" : "=r"(v[0]), "=r"(v[1]), "=r"(v[2]), "=r"(v[3]) : "r"(at_v + idx * 16) : "memory");
+          asm volatile("ld.shared.v4.b32 {%0, %1, %2, %3}, [%4];\n" : "=r"(v[0]), "=r"(v[1]), "=r"(v[2]), "=r"(v[3]) : "r"(v_src + idx * 16) : "memory");
           const float wj = j < n ? pw[max(n - 1 - j, 0)] * wc : 0.f;
 #pragma unroll
           for (int e = 0; e < 4; ++e) Split(Low(v[e]) * wj, High(v[e]) * wj, hi[e], lo[e]);
-          StoreShared16(at_s + idx * 16, hi);
-          StoreShared16(at_s + kVAtoms * kAtom + idx * 16, lo);
+          StoreShared16(vd_dst + idx * 16, hi);
+          StoreShared16(vd_dst + kVAtoms * kAtom + idx * 16, lo);
         }
         asm volatile("fence.proxy.async.shared::cta;\n" ::: "memory");
         asm volatile("tcgen05.fence::before_thread_sync;\n" ::: "memory");
         __syncwarp();
-        if (lane == 0) MbarArrive(vd_ready);
+        if (lane == 0) MbarArrive(vd_bar(c));
       }
 
       if (OUT) {
         ok = MbarWaitWarp(pv_done, par, lane, abort_word) && ok;
-        if (carries(c)) ok = MbarWaitWarp(vd_ready, par, lane, abort_word) && ok;  // all warps have read V
+        if (carries(c)) ok = MbarWaitWarp(vd_bar(c), (c >> 1) & 1, lane, abort_word) && ok;  // all warps have read V
         asm volatile("tcgen05.fence::after_thread_sync;\n" ::: "memory");
         uint32_t x[VC];
         LoadTmem<VC>(t_o + lanes + part * VC, x);
