@@ -843,7 +843,7 @@ def bench_tables(block, max_len, batch=None):
 
 
 class KernelTimes:
-    """Kernels alone against their rooflines: HBM or the bf16 rate."""
+    """Kernels alone against their rooflines: HBM or the bf16 rate (`slower`: whichever takes longer)."""
 
     def __init__(self, torch, pk):
         self.torch, self.pk, self.rows = torch, pk, []
@@ -852,7 +852,10 @@ class KernelTimes:
         """calls: the same work over sets of operands that together are past L2."""
         _, med = _time_graph(self.torch, lambda: [c() for c in calls], 10)
         us = med / len(calls) * 1e3
-        frac = bytes_ / us / 1e3 / self.pk["hbm_gbs"] if bound == "hbm" else flops / us / 1e6 / self.pk["bf16_tflops"]
+        hbm, tensor = bytes_ / us / 1e3 / self.pk["hbm_gbs"], flops / us / 1e6 / self.pk["bf16_tflops"]
+        if bound == "slower":
+            bound = "hbm" if hbm > tensor else "tensor"
+        frac = hbm if bound == "hbm" else tensor
         self.rows.append({"kernel": name, "us": us, "bound": bound, "gbs": bytes_ / us / 1e3, "tflops": flops / us / 1e6, "frac": frac})
 
     def take(self):
@@ -1119,7 +1122,7 @@ def videdra_case(torch, dev, pk, sizes, latent, steps, local) -> dict:
             where = torch.ones((n,), dtype=torch.int32, device=dev)
             states = [s for s in m.states if s is not None]
             kt.time("retention over the portion", [lambda s=s: ops.retention_chunks(rq, rk, rv, positions, m._decay[0], where, s, o, m._state_sums) for s in states],
-                    elem(rq) + elem(rk) + elem(rv) + elem(o) + 8 * hd * ret.vdim, 2.0 * n * ret.heads * (64 * (ret.dim + ret.vdim) + 2 * ret.dim * ret.vdim), "hbm")
+                    elem(rq) + elem(rk) + elem(rv) + elem(o) + 8 * hd * ret.vdim, 2.0 * n * ret.heads * (64 * (ret.dim + ret.vdim) + 2 * ret.dim * ret.vdim), "slower")
             kt.time("retention: norm and gate", [lambda: ops.head_norm_gate(o, rp[:, 2 * hd + ret.heads * ret.vdim:], ro, 1e-5)] * 4, 2 * elem(o) + elem(ro), 0.0, "hbm")
         gain = torch.ones((W,), device=dev)
         kt.time("norm, residual, norm", [lambda: ops.residual_norm(y, m.x[:n], gain, 1e-5, gain_next=gain, out=h)] * 4, 3 * elem(y) + elem(h), 0.0, "hbm")
@@ -1141,7 +1144,7 @@ def videdra_case(torch, dev, pk, sizes, latent, steps, local) -> dict:
         for name, key, a_, b_, act_ in (("experts gate|up", "e_up", xs, acts, N.ACT_SILU_MUL), ("experts down", "e_down", acts, outs, N.ACT_NONE)):
             w0 = lw[key]
             kt.time(name, [lambda w=l[key]: ops.dense_gemm(ops.grouped_dense(a_, w, b_, offsets, act=act_)) for l in m.layers], elem(w0) * read + elem(a_) + elem(b_),
-                    2.0 * n * f.top * w0.shape[1] * w0.shape[2], bound)
+                    2.0 * n * f.top * w0.shape[1] * w0.shape[2], "slower")
         kt.time("experts' sum, norm, residual, norm", [lambda: ops.residual_norm(y, m.x[:n], gain, 1e-5, gain_next=gain, out=h, gate=logits[:, f.experts], parts=outs, part_rows=rows_of,
                                                                                 part_weights=wts)] * 4, 3 * elem(y) + elem(h) + elem(outs), 0.0, "hbm")
 

@@ -45,6 +45,8 @@ __device__ __forceinline__ void Store4(__nv_bfloat16* o, float4 v)
   u.y = *reinterpret_cast<const uint32_t*>(&hi);
   *reinterpret_cast<uint2*>(o) = u;
 }
+__device__ __forceinline__ void StorePair(float* o, float a, float b) { *reinterpret_cast<float2*>(o) = make_float2(a, b); }
+__device__ __forceinline__ void StorePair(__nv_bfloat16* o, float a, float b) { *reinterpret_cast<__nv_bfloat162*>(o) = __floats2bfloat162_rn(a, b); }
 __device__ __forceinline__ float4 Fma4(float a, float4 v, float4 c)
 {
   return make_float4(fmaf(a, v.x, c.x), fmaf(a, v.y, c.y), fmaf(a, v.z, c.z), fmaf(a, v.w, c.w));
@@ -201,8 +203,9 @@ __global__ void __launch_bounds__(256) RotateRowsKernel(const float* in, int64_t
 }
 
 // One warp per (token, head): the two maps' outputs out of the slices' records ({maximum (log2), sum, acc[in_ld]}; slices > 0) or as
-// they are (slices 0); their difference, its norm, the head's gate.
-template <typename T>
+// they are (slices 0); their difference, its norm, the head's gate.  PAIRS: even sizes up to 512 values, two a lane at a time, kept in
+// registers; else the values are computed twice.
+template <typename T, bool PAIRS>
 __global__ void __launch_bounds__(128) MapDifferenceKernel(const float* in, int slices, const float* gate, int64_t gate_ld, T* out, int64_t out_ld, int rows,
                                                            int heads, int vdim, int in_ld, float lambda, float keep, float eps)
 {
@@ -213,7 +216,7 @@ __global__ void __launch_bounds__(128) MapDifferenceKernel(const float* in, int 
   const int rec = slices > 0 ? in_ld + 2 : in_ld;
   const float* a = in + (static_cast<size_t>(t) * heads + h) * 2 * rec;
   const size_t slice_ld = static_cast<size_t>(rows) * heads * 2 * rec;
-  float top[2] = {0.f, 0.f}, inv_sum[2] = {1.f, 1.f};
+  float top[2] = {0.f, 0.f}, scale[2] = {1.f, -lambda};  // of each map's values in the difference
   if (slices > 0) {
 #pragma unroll
     for (int p = 0; p < 2; ++p) {
@@ -225,46 +228,70 @@ __global__ void __launch_bounds__(128) MapDifferenceKernel(const float* in, int 
         if (ms > -INFINITY) sum += a[s * slice_ld + p * rec + 1] * exp2f(ms - m);
       }
       top[p] = m;
-      inv_sum[p] = sum > 0.f ? 1.f / sum : 0.f;
+      scale[p] = sum > 0.f ? scale[p] / sum : 0.f;
     }
   }
-  auto value = [&](int c) {
-    float o[2];
+  const float g = keep * (gate != nullptr ? Sigmoid(gate[t * gate_ld + h]) : 1.f);
+  T* dst = out + t * out_ld + static_cast<size_t>(h) * vdim;
+  if constexpr (PAIRS) {
+    const int pairs = vdim >> 1;
+    float2 v[8];
 #pragma unroll
-    for (int p = 0; p < 2; ++p) {
-      if (slices == 0) {
-        o[p] = a[p * rec + c];
-      } else {
-        o[p] = 0.f;
-        for (int s = 0; s < slices; ++s) {
-          const float ms = a[s * slice_ld + p * rec];
-          if (ms > -INFINITY) o[p] = fmaf(a[s * slice_ld + p * rec + 2 + c], exp2f(ms - top[p]), o[p]);
+    for (int i = 0; i < 8; ++i) v[i] = make_float2(0.f, 0.f);
+    for (int s = 0; s < max(slices, 1); ++s) {
+#pragma unroll
+      for (int p = 0; p < 2; ++p) {
+        const float* r = a + s * slice_ld + p * rec;
+        float f = scale[p];
+        if (slices > 0) {
+          if (!(r[0] > -INFINITY)) continue;  // nothing of the row is in this slice
+          f *= exp2f(r[0] - top[p]);
+          r += 2;
         }
-        o[p] *= inv_sum[p];
+        float2 x[8];
+#pragma unroll
+        for (int i = 0; i < 8; ++i) {
+          if (lane + 32 * i < pairs) x[i] = *reinterpret_cast<const float2*>(r + 2 * (lane + 32 * i));
+        }
+#pragma unroll
+        for (int i = 0; i < 8; ++i) {
+          if (lane + 32 * i < pairs) v[i] = make_float2(fmaf(f, x[i].x, v[i].x), fmaf(f, x[i].y, v[i].y));
+        }
       }
     }
-    return o[0] - lambda * o[1];
-  };
-  float v[8], ss = 0.f;  // the first 256 values stay in registers
+    float ss = 0.f;
 #pragma unroll
-  for (int i = 0; i < 8; ++i) {
-    v[i] = lane + 32 * i < vdim ? value(lane + 32 * i) : 0.f;
-    ss = fmaf(v[i], v[i], ss);
-  }
-  for (int c = lane + 256; c < vdim; c += 32) {
-    const float u = value(c);
-    ss = fmaf(u, u, ss);
-  }
-  const float f = InvRms(WarpSum(ss), vdim, eps) * keep * (gate != nullptr ? Sigmoid(gate[t * gate_ld + h]) : 1.f);
-  T* dst = out + t * out_ld + static_cast<size_t>(h) * vdim;
+    for (int i = 0; i < 8; ++i) ss = fmaf(v[i].x, v[i].x, fmaf(v[i].y, v[i].y, ss));
+    const float f = InvRms(WarpSum(ss), vdim, eps) * g;
 #pragma unroll
-  for (int i = 0; i < 8; ++i)
-    if (lane + 32 * i < vdim) dst[lane + 32 * i] = FromF32<T>(v[i] * f);
-  for (int c = lane + 256; c < vdim; c += 32) dst[c] = FromF32<T>(value(c) * f);
+    for (int i = 0; i < 8; ++i) {
+      if (lane + 32 * i < pairs) StorePair(dst + 2 * (lane + 32 * i), v[i].x * f, v[i].y * f);
+    }
+  } else {
+    auto value = [&](int c) {
+      float v = 0.f;
+      for (int s = 0; s < max(slices, 1); ++s) {
+#pragma unroll
+        for (int p = 0; p < 2; ++p) {
+          const float* r = a + s * slice_ld + p * rec;
+          if (slices == 0) v = fmaf(scale[p], r[c], v);
+          else if (r[0] > -INFINITY) v = fmaf(scale[p] * exp2f(r[0] - top[p]), r[2 + c], v);
+        }
+      }
+      return v;
+    };
+    float ss = 0.f;
+    for (int c = lane; c < vdim; c += 32) {
+      const float u = value(c);
+      ss = fmaf(u, u, ss);
+    }
+    const float f = InvRms(WarpSum(ss), vdim, eps) * g;
+    for (int c = lane; c < vdim; c += 32) dst[c] = FromF32<T>(value(c) * f);
+  }
 }
 
-// One warp per (token, head): a recurrence's output over its root mean square, times silu of the gate.
-template <typename T>
+// One warp per (token, head): a recurrence's output over its root mean square, times silu of the gate.  PAIRS as above.
+template <typename T, bool PAIRS>
 __global__ void __launch_bounds__(128) HeadNormGateKernel(const float* in, const float* gate, int64_t gate_ld, T* out, int64_t out_ld, int rows, int heads,
                                                           int vdim, float eps)
 {
@@ -276,9 +303,29 @@ __global__ void __launch_bounds__(128) HeadNormGateKernel(const float* in, const
   const float* g = gate + t * gate_ld + static_cast<size_t>(h) * vdim;
   T* dst = out + t * out_ld + static_cast<size_t>(h) * vdim;
   float ss = 0.f;
-  for (int c = lane; c < vdim; c += 32) ss = fmaf(a[c], a[c], ss);
-  const float inv = InvRms(WarpSum(ss), vdim, eps);
-  for (int c = lane; c < vdim; c += 32) dst[c] = FromF32<T>(a[c] * inv * Silu(g[c]));
+  if constexpr (PAIRS) {
+    const int pairs = vdim >> 1;
+    float2 v[8], z[8];
+#pragma unroll
+    for (int i = 0; i < 8; ++i) {
+      v[i] = z[i] = make_float2(0.f, 0.f);
+      if (lane + 32 * i < pairs) {
+        v[i] = *reinterpret_cast<const float2*>(a + 2 * (lane + 32 * i));
+        z[i] = *reinterpret_cast<const float2*>(g + 2 * (lane + 32 * i));
+      }
+    }
+#pragma unroll
+    for (int i = 0; i < 8; ++i) ss = fmaf(v[i].x, v[i].x, fmaf(v[i].y, v[i].y, ss));
+    const float inv = InvRms(WarpSum(ss), vdim, eps);
+#pragma unroll
+    for (int i = 0; i < 8; ++i) {
+      if (lane + 32 * i < pairs) StorePair(dst + 2 * (lane + 32 * i), v[i].x * inv * Silu(z[i].x), v[i].y * inv * Silu(z[i].y));
+    }
+  } else {
+    for (int c = lane; c < vdim; c += 32) ss = fmaf(a[c], a[c], ss);
+    const float inv = InvRms(WarpSum(ss), vdim, eps);
+    for (int c = lane; c < vdim; c += 32) dst[c] = FromF32<T>(a[c] * inv * Silu(g[c]));
+  }
 }
 
 }  // namespace
@@ -368,10 +415,17 @@ extern "C" int tlaloc_b200_map_difference(const float* in, int32_t slices, const
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   const unsigned blocks = static_cast<unsigned>((static_cast<long long>(rows) * heads + 3) / 4);
   cudaError_t e;
-#define TLALOC_LAUNCH(T) \
-  e = LaunchChained(MapDifferenceKernel<T>, blocks, 128, 0, st, in, slices, gate, gate_ld, static_cast<T*>(out), out_ld, rows, heads, vdim, in_ld, lambda, keep, eps)
-  if (dtype == TLALOC_B200_F32) TLALOC_LAUNCH(float);
-  else TLALOC_LAUNCH(__nv_bfloat16);
+  const bool pairs = vdim % 2 == 0 && in_ld % 2 == 0 && vdim <= 512 && out_ld % 2 == 0 && reinterpret_cast<uintptr_t>(in) % 8 == 0 &&
+                     reinterpret_cast<uintptr_t>(out) % 8 == 0;
+#define TLALOC_LAUNCH(T, PAIRS) \
+  e = LaunchChained(MapDifferenceKernel<T, PAIRS>, blocks, 128, 0, st, in, slices, gate, gate_ld, static_cast<T*>(out), out_ld, rows, heads, vdim, in_ld, lambda, keep, eps)
+  if (dtype == TLALOC_B200_F32) {
+    if (pairs) TLALOC_LAUNCH(float, true);
+    else TLALOC_LAUNCH(float, false);
+  } else {
+    if (pairs) TLALOC_LAUNCH(__nv_bfloat16, true);
+    else TLALOC_LAUNCH(__nv_bfloat16, false);
+  }
 #undef TLALOC_LAUNCH
   if (e != cudaSuccess) return CudaFail("MAP_DIFFERENCE launch", e);
   CountLaunches(1);
@@ -389,10 +443,17 @@ extern "C" int tlaloc_b200_head_norm_gate(const float* in, const float* gate, in
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   const unsigned blocks = static_cast<unsigned>((static_cast<long long>(rows) * heads + 3) / 4);
   cudaError_t e;
-#define TLALOC_LAUNCH(T) \
-  e = LaunchChained(HeadNormGateKernel<T>, blocks, 128, 0, st, in, gate, gate_ld, static_cast<T*>(out), out_ld, rows, heads, vdim, eps)
-  if (dtype == TLALOC_B200_F32) TLALOC_LAUNCH(float);
-  else TLALOC_LAUNCH(__nv_bfloat16);
+  const bool pairs = vdim % 2 == 0 && vdim <= 512 && out_ld % 2 == 0 && gate_ld % 2 == 0 && reinterpret_cast<uintptr_t>(in) % 8 == 0 &&
+                     reinterpret_cast<uintptr_t>(gate) % 8 == 0 && reinterpret_cast<uintptr_t>(out) % 8 == 0;
+#define TLALOC_LAUNCH(T, PAIRS) \
+  e = LaunchChained(HeadNormGateKernel<T, PAIRS>, blocks, 128, 0, st, in, gate, gate_ld, static_cast<T*>(out), out_ld, rows, heads, vdim, eps)
+  if (dtype == TLALOC_B200_F32) {
+    if (pairs) TLALOC_LAUNCH(float, true);
+    else TLALOC_LAUNCH(float, false);
+  } else {
+    if (pairs) TLALOC_LAUNCH(__nv_bfloat16, true);
+    else TLALOC_LAUNCH(__nv_bfloat16, false);
+  }
 #undef TLALOC_LAUNCH
   if (e != cudaSuccess) return CudaFail("HEAD_NORM_GATE launch", e);
   CountLaunches(1);
