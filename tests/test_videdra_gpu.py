@@ -83,7 +83,7 @@ CONFIGS = {
     "one head, one pair": oracle.model(A(heads=1, kv_heads=1, dim=8, vdim=8, rot_dims=2, window=1, keep=1), R(heads=1, dim=4, vdim=4, rot_dims=2), width=40, vocab=33),
     "odd sizes": oracle.model(A(heads=3, kv_heads=3, dim=10, vdim=14, rot_dims=6, window=30, keep=3, mlp=oracle.dense_mlp(50)), R(heads=3, dim=14, vdim=22, rot_dims=10), width=44, vocab=57),
     "wide": oracle.model(A(heads=20, kv_heads=2, dim=64, vdim=128, rot_dims=64, window=130, keep=70), R(heads=4, dim=128, vdim=128, rot_dims=64, mlp=oracle.dense_mlp(640)),
-                         A(heads=6, kv_heads=2, dim=128, vdim=256, rot_dims=32, window=70, keep=130), width=320, vocab=257),
+                         A(heads=6, kv_heads=2, dim=128, vdim=256, rot_dims=32, window=70, keep=130), width=336, vocab=257),
 }
 # Router choices in 16-bit arithmetic can differ from the exact ones where two logits are close: those models run in f32 on random tokens,
 # and in bf16 on sizes where the least distance was looked at.

@@ -335,6 +335,7 @@ __global__ void __launch_bounds__(kThreads, 1) RetentionChunkTc(const __grid_con
           }
         }
       } else if (OUT) {
+#pragma unroll 2
         for (int g = g_lo; g < g_hi; ++g) {
           const float* p = sums(g) + b * VC * kWorkerThreads;
 #pragma unroll
@@ -345,6 +346,7 @@ __global__ void __launch_bounds__(kThreads, 1) RetentionChunkTc(const __grid_con
     }
     asm volatile("tcgen05.wait::st.sync.aligned;\n" ::: "memory");
 
+    float w_ahead = 1.f;
     for (int c = 0; c < chunks; ++c) {
       const uint32_t par = c & 1;
       const int t0 = t_begin + c * kChunk, n = min(kChunk, t_end - t0);
@@ -420,7 +422,11 @@ __global__ void __launch_bounds__(kThreads, 1) RetentionChunkTc(const __grid_con
       if (carries(c)) {
         ok = MbarWaitWarp(full_v + 8 * v_buf(c), v_par(c), lane, abort_word) && ok;
         const uint32_t v_src = at_v + v_buf(c) * kVAtoms * kAtom, vd_dst = at_s + vd_at(c);
-        const float wc = OUT ? 1.f : powf(w, static_cast<float>((chunks - 1 - c) * kChunk));  // from the chunk's end to the segment's
+        float wc = 1.f;
+        if (!OUT) {  // from the chunk's end to the segment's: one power a lane for 32 chunks
+          if ((c & 31) == 0) w_ahead = powf(w, static_cast<float>(max(chunks - 1 - c - lane, 0) * kChunk));
+          wc = __shfl_sync(0xffffffffu, w_ahead, c & 31);
+        }
 #pragma unroll
         for (int i = 0; i < kVAtoms * kAtom / 16 / kWorkerThreads; ++i) {
           const int idx = i * kWorkerThreads + tid, j = (idx & (kAtom / 16 - 1)) >> 3;
