@@ -338,15 +338,12 @@ def test_retention_step(heads, dim, vdim, dims, dtype):
         assert torch.equal(state[s], old[s])
 
 
-@pytest.mark.parametrize("dtype", [F32, BF16])
-@pytest.mark.parametrize("heads,dim,vdim,dims", RETENTION)
+@pytest.mark.parametrize("heads,dim,vdim,dims,how,dtype", [(*r, how, dtype) for r in RETENTION for how, dtype in (("scan", F32), ("scan", BF16), ("chunks", BF16))
+                                                           if how == "scan" or r[1] <= 256])
 @pytest.mark.parametrize("tokens,fresh", [(2, True), (9, False), (130, True), (67, False), (64, False), (65, True), (700, False)])
-@pytest.mark.parametrize("how", ["scan", "chunks"])
 def test_retention_over_a_portion(heads, dim, vdim, dims, tokens, fresh, how, dtype):
     from tlaloc_b200 import ops
 
-    if how == "chunks" and (dtype == F32 or not ops.retention_chunks_applies(dim, vdim)):
-        pytest.skip("bf16, up to 256 channels")
     decay = [1 - 0.5 ** (3 + h) for h in range(heads)]
     vp, kd, vd = -(-vdim // 4) * 4, -(-dim // 16) * 16, -(-vdim // 16) * 16
     q, k, v = (torch.zeros((tokens, heads, n), device=DEV, dtype=dtype) for n in (kd, kd, vd))
